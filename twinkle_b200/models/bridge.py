@@ -158,8 +158,42 @@ def _nested(cfg: DecoderConfig) -> bool:
     return bool(cfg.vision) or cfg.model_type.startswith('qwen3_5')
 
 
+# Pomelix checkpoints: ``l<i>.mix.*`` / ``l<i>.mlp.*`` with one tensor per projection; here a layer's projections of the
+# same input are one matrix and its convolution filters one tensor
+_LISTED = {'input_layernorm.weight': ('norm1', ), 'conv_weight': ('mix.q.conv', 'mix.k.conv', 'mix.v.conv'), 'v_lambda': ('mix.vmix', ),
+           'o_proj.weight': ('mix.o', ), 'down_proj.weight': ('mlp.down', ), 'mixer_scale': ('ls1', ), 'mlp_scale': ('ls2', )}
+
+
+def _listed_names(name: str, cfg: DecoderConfig) -> List[str]:
+    """Checkpoint tensors that make up one internal tensor of a stack with listed layers, in concatenation order."""
+    if name == 'embed_tokens.weight':
+        return ['embed']
+    if name == 'norm.weight':
+        return ['final.norm']
+    m = _LAYER.match(name)
+    if not m:
+        raise KeyError(f'no checkpoint mapping for {name}')
+    i, rest = int(m.group(1)), m.group(2)
+    if rest == 'in_proj.weight':
+        return [f'l{i}.mix.{p}' for p in 'qkv'] + ([f'l{i}.mlp.gate', f'l{i}.mlp.up'] if cfg.layer_specs[i].ff else [])
+    return [f'l{i}.{p}' for p in _LISTED[rest]]
+
+
+def _listed_split(name: str, tensor: torch.Tensor, cfg: DecoderConfig) -> List[Tuple[str, torch.Tensor]]:
+    names = _listed_names(name, cfg)
+    if name.endswith('.v_lambda'):
+        return [(names[0], tensor.reshape(()))]
+    if len(names) == 1:
+        return [(names[0], tensor)]
+    sp = cfg.layer_specs[int(_LAYER.match(name).group(1))]
+    sizes = list(sp.qkv_sizes) + ([sp.ff, sp.ff] if name.endswith('in_proj.weight') and sp.ff else [])
+    return list(zip(names, tensor.split(sizes, dim=0)))
+
+
 def internal_to_hf(name: str, tensor: torch.Tensor, cfg: DecoderConfig) -> List[Tuple[str, torch.Tensor]]:
     """One internal (full, un-sharded) tensor → one or more HF tensors."""
+    if cfg.layer_specs is not None:
+        return _listed_split(name, tensor, cfg)
     if name.startswith('visual.'):
         return [('model.' + name, tensor)]
     return [(_family(_vl(n, cfg), cfg), t) for n, t in _internal_to_hf_text(name, tensor, cfg)]
@@ -230,6 +264,8 @@ def _internal_to_hf_text(name: str, tensor: torch.Tensor, cfg: DecoderConfig) ->
 
 def hf_names_for(name: str, cfg: DecoderConfig) -> List[str]:
     """HF tensor names that make up one internal tensor (in concat order)."""
+    if cfg.layer_specs is not None:
+        return _listed_names(name, cfg)
     if name.startswith('visual.'):
         return ['model.' + name]
     return [_family(_vl(n, cfg), cfg) for n in _hf_names_for_text(name, cfg)]
@@ -280,6 +316,8 @@ def hf_to_internal(name: str, cfg: DecoderConfig, get: Callable[[str], torch.Ten
                    expert_range: Optional[Tuple[int, int]] = None) -> torch.Tensor:
     """Assemble one internal tensor from HF tensors fetched by ``get``.  An output head that the checkpoint does not carry
     (tied embeddings saved once) is read from the embedding."""
+    if cfg.layer_specs is not None:
+        return torch.cat([get(n).reshape(1) if n.endswith('.vmix') else get(n) for n in _listed_names(name, cfg)], 0)
     m = _LAYER.match(name)
     rest = m.group(2) if m else ''
     i = int(m.group(1)) if m else -1

@@ -11,7 +11,7 @@ import json
 import math
 import os
 from dataclasses import asdict, dataclass, field
-from typing import List, Any, Dict, Optional
+from typing import List, Any, Dict, Optional, Tuple, Union
 
 
 # config.json ``model_type`` values whose layer maths is what ``models/decoder.py`` computes (each checked against transformers)
@@ -37,6 +37,67 @@ def _rope_scaling_of(cfg: Dict[str, Any]) -> Optional[Dict[str, Any]]:
         out.setdefault('max_position_embeddings', cfg.get('max_position_embeddings', 4096))
     out.pop('partial_rotary_factor', None)
     return out
+
+
+def _pomelix_fields(cfg: Dict[str, Any]) -> Dict[str, Any]:
+    """``config.json`` of a Pomelix checkpoint → keyword arguments of :class:`DecoderConfig`."""
+    specs = []
+    for i, layer in enumerate(cfg['layers']):
+        if layer['type'] != 'attention':
+            raise NotImplementedError(f"layer {i}: mixer type {layer['type']!r} is not implemented (attention is)")
+        m, mlp, qt = layer['mixer'], layer.get('mlp'), layer['mixer'].get('q_temp')
+        if mlp is not None and mlp.get('kind', 'dense') != 'dense':
+            raise NotImplementedError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not implemented (dense is)")
+        if qt is not None and (qt['every'] != int(qt['every']) or qt['every'] < 1):
+            raise ValueError(f"layer {i}: q_temp.every must be a positive whole number of positions, not {qt['every']!r}")
+        specs.append(LayerSpec(heads=int(m['heads']), kv_heads=int(m['kv_heads']), dim=int(m['dim']), vdim=int(m['vdim']), scale=float(m['scale']),
+                               conv=int(m.get('conv') or 0), temp_coef=float(qt['coef']) if qt else 0.0, temp_every=int(qt['every']) if qt else 0,
+                               v_mix=bool(m.get('v_mix')), ff=int(mlp['ff']) if mlp else 0))
+    return dict(model_type='pomelix', vocab_size=int(cfg['vocab']), hidden_size=int(cfg['width']), rms_norm_eps=float(cfg['norm']['eps']),
+                residual_multiplier=float(cfg.get('residual_mult', 1.0)), tie_word_embeddings=True, qk_norm=False, layer_specs=specs,
+                eos_token_id=cfg.get('eos_token_id'), pad_token_id=cfg.get('pad_token_id'), torch_dtype=str(cfg.get('torch_dtype', 'bfloat16')))
+
+
+def _pomelix_mapping(c: 'DecoderConfig') -> Dict[str, Any]:
+    """The inverse of :func:`_pomelix_fields`."""
+    layers = []
+    for sp in c.layer_specs:
+        m = {'heads': sp.heads, 'kv_heads': sp.kv_heads, 'dim': sp.dim, 'vdim': sp.vdim, 'scale': sp.scale, 'conv': sp.conv, 'v_mix': sp.v_mix}
+        if sp.temp_every:
+            m['q_temp'] = {'coef': sp.temp_coef, 'every': sp.temp_every}
+        layers.append({'type': 'attention', 'mixer': m, 'mlp': {'kind': 'dense', 'ff': sp.ff} if sp.ff else None})
+    d = {'architecture': 'Pomelix', 'vocab': c.vocab_size, 'width': c.hidden_size, 'norm': {'eps': c.rms_norm_eps},
+         'residual_mult': c.residual_multiplier, 'layers': layers}
+    d.update({k: v for k, v in (('eos_token_id', c.eos_token_id), ('pad_token_id', c.pad_token_id)) if v is not None})
+    return d
+
+
+# checkpoints whose config.json names its ``architecture`` and lists every layer: (reader → DecoderConfig fields, writer)
+NATIVE_ARCHITECTURES = {'Pomelix': (_pomelix_fields, _pomelix_mapping)}
+
+
+@dataclass
+class LayerSpec:
+    """Sizes and constants of one layer of a stack whose layers are listed one by one (``DecoderConfig.layer_specs``): an
+    attention mixer with ``heads`` query and ``kv_heads`` key / value heads, query / key width ``dim`` and value width
+    ``vdim``; ``conv`` taps of causal depth-wise convolution on q, k and v (1 = the newest row only, 0 = none);
+    query temperature ``1 + temp_coef · ln(⌊(p + 1) / temp_every⌋ + 1)`` (``temp_every`` 0 = none); softmax ``scale``;
+    ``v_mix``: values mixed with those of the first layer that has it; ``ff``: width of the gated feed-forward block
+    (0 = the layer has none)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    conv: int = 0
+    temp_coef: float = 0.0
+    temp_every: int = 0
+    v_mix: bool = False
+    ff: int = 0
+
+    @property
+    def qkv_sizes(self) -> Tuple[int, int, int]:
+        return self.heads * self.dim, self.kv_heads * self.dim, self.kv_heads * self.vdim
 
 
 @dataclass
@@ -145,8 +206,24 @@ class DecoderConfig:
     vision_end_token_id: Optional[int] = None
     mrope_section: Optional[List[int]] = None
     mrope_interleaved: bool = False  # Qwen3-VL lays the three position components out t h w t h w … instead of in blocks
+    # stacks whose layers are listed one by one and run mixer and feed-forward side by side on one norm (Pomelix): the
+    # residual stream is 32-bit, each sub-layer's result has a learned per-channel scale, positions enter through a short
+    # convolution and the query temperature only (no rotary embedding)
+    layer_specs: Optional[List[Union[LayerSpec, Dict[str, Any]]]] = None
 
     def __post_init__(self):
+        if self.layer_specs is not None:
+            self.layer_specs = [LayerSpec(**sp) if isinstance(sp, dict) else sp for sp in self.layer_specs]
+            first = self.layer_specs[0]
+            self.num_hidden_layers = len(self.layer_specs)
+            self.num_attention_heads, self.num_key_value_heads, self.head_dim = first.heads, first.kv_heads, first.dim
+            self.intermediate_size = max(sp.ff for sp in self.layer_specs)
+            for i, sp in enumerate(self.layer_specs):
+                if sp.heads % sp.kv_heads:
+                    raise ValueError(f'layer {i}: {sp.heads} query heads do not divide over {sp.kv_heads} key / value heads')
+            mixed = [sp for sp in self.layer_specs if sp.v_mix]
+            if any((sp.kv_heads, sp.vdim) != (mixed[0].kv_heads, mixed[0].vdim) for sp in mixed):
+                raise ValueError('layers that mix values must agree on the number and width of the value heads')
         if self.vision is not None:
             from .vision import VisionConfig
             self.vision = VisionConfig.from_hf(self.vision).to_hf()  # only the fields the tower uses, in the family's spelling
@@ -158,6 +235,22 @@ class DecoderConfig:
     @property
     def is_mla(self) -> bool:
         return self.kv_lora_rank > 0
+
+    @property
+    def first_mixing_layer(self) -> Optional[int]:
+        """Index of the layer whose values the later value-mixing layers take in (None: no layer mixes)."""
+        return next((i for i, sp in enumerate(self.layer_specs or []) if sp.v_mix), None)
+
+    def kv_layout(self) -> List[Tuple[int, int, int]]:
+        """Per layer ``(key / value heads, key row width, value row width)`` of the paged cache.  Layers with widths of their
+        own keep rows of whole 16-byte vectors (widths rounded up to a multiple of 8, the rest zero)."""
+        if self.layer_specs is None:
+            return [(self.num_key_value_heads, self.head_dim, self.head_dim)] * self.num_hidden_layers
+        return [(sp.kv_heads, -(-sp.dim // 8) * 8, -(-sp.vdim // 8) * 8) for sp in self.layer_specs]
+
+    def conv_layout(self) -> List[Optional[Tuple[int, int]]]:
+        """Per layer ``(rows, channels)`` of the convolution history a sequence keeps between steps (None: no history)."""
+        return [(sp.conv - 1, sum(sp.qkv_sizes)) if sp.conv > 1 else None for sp in self.layer_specs or []]
 
     def layer_is_moe(self, layer_idx: int) -> bool:
         return self.num_experts > 0 and layer_idx >= self.first_k_dense_replace
@@ -200,8 +293,15 @@ class DecoderConfig:
             return q + h * (self.kv_lora_rank + self.qk_rope_head_dim) + self.kv_lora_rank * nh * (self.qk_nope_head_dim + self.v_head_dim) + nh * self.v_head_dim * h
         return h * (self.q_size + 2 * self.kv_size) + self.q_size * h + (self.q_size * h if self.attn_output_gate else 0)
 
+    def _listed_matmul_weights(self) -> int:
+        h = self.hidden_size
+        return sum(h * sum(sp.qkv_sizes) + h * sp.heads * sp.vdim + 3 * h * sp.ff for sp in self.layer_specs)
+
     def num_params(self) -> int:
         h, L = self.hidden_size, self.num_hidden_layers
+        if self.layer_specs is not None:
+            small = sum(sp.conv * sum(sp.qkv_sizes) + h * (3 if sp.ff else 2) + int(sp.v_mix) for sp in self.layer_specs)
+            return self._listed_matmul_weights() + small + self.vocab_size * h * (1 if self.tie_word_embeddings else 2) + h
         attn = self._attn_weights() + (2 * self.head_dim if self.qk_norm else 0)
         moe = self.num_experts * 3 * h * self.moe_intermediate_size + h * self.num_experts + 3 * h * self.shared_expert_intermediate_size
         dense = 3 * h * self.intermediate_size
@@ -219,6 +319,9 @@ class DecoderConfig:
     def flops_per_token(self, avg_context: float = 0.0) -> float:
         """Forward+backward matmul FLOPs per token (6·N_active + attention)."""
         h, L = self.hidden_size, self.num_hidden_layers
+        if self.layer_specs is not None:
+            attn = sum((sp.dim + sp.vdim) * sp.heads for sp in self.layer_specs) * avg_context
+            return 6.0 * (self._listed_matmul_weights() + self.vocab_size * h) + 6.0 * attn
         attn_w = self._attn_weights()
         moe_w = self.num_experts_per_tok * 3 * h * self.moe_intermediate_size + h * self.num_experts + 3 * h * self.shared_expert_intermediate_size
         n_moe = sum(self.layer_is_moe(i) for i in range(L))
@@ -231,6 +334,8 @@ class DecoderConfig:
     @classmethod
     def from_hf(cls, cfg: Dict[str, Any]) -> 'DecoderConfig':
         cfg = dict(cfg)
+        if cfg.get('architecture') in NATIVE_ARCHITECTURES:
+            return cls(**NATIVE_ARCHITECTURES[cfg['architecture']][0](cfg))
         top = cfg
         if 'text_config' in cfg:
             cfg = dict(cfg['text_config'])
@@ -327,6 +432,8 @@ class DecoderConfig:
             return cls.from_hf(json.load(f))
 
     def to_hf(self) -> Dict[str, Any]:
+        if self.layer_specs is not None:
+            return NATIVE_ARCHITECTURES['Pomelix'][1](self)
         arch = 'Qwen3MoeForCausalLM' if self.is_moe else ('Qwen3ForCausalLM' if self.qk_norm else 'LlamaForCausalLM')
         arch = {'mixtral': 'MixtralForCausalLM', 'qwen2_moe': 'Qwen2MoeForCausalLM', 'qwen2': 'Qwen2ForCausalLM', 'mistral': 'MistralForCausalLM',
                 'seed_oss': 'SeedOssForCausalLM'}.get(self.model_type, arch)
@@ -526,6 +633,19 @@ PRESETS: Dict[str, Dict[str, Any]] = {
     'tiny-moe-shared': dict(vocab_size=1024, hidden_size=256, num_hidden_layers=2, num_attention_heads=4, num_key_value_heads=2,
                             head_dim=64, rope_theta=1e4, tie_word_embeddings=True, num_experts=8, num_experts_per_tok=2,
                             moe_intermediate_size=128, shared_expert_intermediate_size=192, torch_dtype='float32'),
+    # Pomelix in small: layers of unequal widths and head counts, one without a feed-forward block, one without convolution
+    'tiny-pomelix': dict(vocab_size=1024, hidden_size=192, tie_word_embeddings=True, qk_norm=False, torch_dtype='float32', model_type='pomelix',
+                         rms_norm_eps=1e-5, residual_multiplier=0.5,
+                         layer_specs=[dict(heads=6, kv_heads=2, dim=24, vdim=40, scale=0.3, conv=3, temp_coef=0.2, temp_every=16, v_mix=False, ff=256),
+                                      dict(heads=4, kv_heads=2, dim=32, vdim=32, scale=0.2, conv=4, temp_coef=0.2, temp_every=16, v_mix=True, ff=0),
+                                      dict(heads=8, kv_heads=2, dim=16, vdim=32, scale=0.25, conv=0, v_mix=True, ff=160)]),
+    # Pomelix layers at the sizes of the Qwen3 presets (benchmarks)
+    'pomelix-0.6b': dict(vocab_size=151936, hidden_size=1024, tie_word_embeddings=True, qk_norm=False, model_type='pomelix', rms_norm_eps=1e-5,
+                         residual_multiplier=0.5, layer_specs=[dict(heads=16, kv_heads=8, dim=128, vdim=128, scale=128**-0.5, conv=4, temp_coef=0.1,
+                                                                    temp_every=4096, v_mix=True, ff=3072)] * 28),
+    'pomelix-8b': dict(vocab_size=151936, hidden_size=4096, tie_word_embeddings=True, qk_norm=False, model_type='pomelix', rms_norm_eps=1e-5,
+                       residual_multiplier=0.5, layer_specs=[dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128**-0.5, conv=4, temp_coef=0.1,
+                                                                  temp_every=4096, v_mix=True, ff=12288)] * 36),
     'qwen3-0.6b': dict(hidden_size=1024, intermediate_size=3072, num_hidden_layers=28, num_attention_heads=16,
                        num_key_value_heads=8, head_dim=128, tie_word_embeddings=True),
     'qwen3-8b': dict(hidden_size=4096, intermediate_size=12288, num_hidden_layers=36, num_attention_heads=32,

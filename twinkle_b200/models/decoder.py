@@ -24,6 +24,7 @@ import torch.nn.functional as F
 from .. import ops
 from .config import DecoderConfig
 from .layers import Embedding, Linear, RMSNorm
+from .parallel_layer import CacheView, ParallelLayer, Stream
 
 
 @dataclass
@@ -49,6 +50,8 @@ class PackedBatch:
     image_grid_thw: Optional[torch.Tensor] = None
     # (row indices of the placeholder tokens, features per early layer) — set by ``embed`` for towers with deep-stack outputs
     deepstack: Optional[tuple] = None
+    # stacks with listed layers: where the rows live in the sampler's cache (None: no cache is read or written)
+    cache: Optional[CacheView] = None
     # under sequence / context parallelism: rows of the tower's output that belong to this rank's placeholder tokens
     vision_rows: Optional[torch.Tensor] = None
 
@@ -500,7 +503,7 @@ class DecoderModel(nn.Module):
         lo, hi = layer_range or (0, cfg.num_hidden_layers)
         self.layer_range = (lo, hi)
         self.embed_tokens = Embedding(cfg.vocab_size, cfg.hidden_size) if has_embed else None
-        self.layers = nn.ModuleList([DecoderLayer(cfg, i) for i in range(lo, hi)])
+        self.layers = nn.ModuleList([(ParallelLayer if cfg.layer_specs is not None else DecoderLayer)(cfg, i) for i in range(lo, hi)])
         self.norm = RMSNorm(cfg.hidden_size, cfg.rms_norm_eps, cfg.rms_norm_offset) if has_head else None
         if has_head and not cfg.tie_word_embeddings:
             self.lm_head = Linear(cfg.hidden_size, cfg.vocab_size, name='lm_head')
@@ -527,6 +530,9 @@ class DecoderModel(nn.Module):
         from ..utils.seed import stable_seed
         for name, p in self.named_parameters():
             if 'lora_' in name or name.startswith('lora'):
+                continue
+            if name.endswith('v_lambda'):
+                p.fill_(0.5)
                 continue
             if name.endswith(('bias', 'sinks')):       # also the per-expert bias matrices
                 p.zero_()
@@ -576,7 +582,26 @@ class DecoderModel(nn.Module):
             batch.deepstack = (where.nonzero(as_tuple=True)[0], deep) if deep else None
         return x
 
+    def _forward_listed(self, batch: PackedBatch) -> torch.Tensor:
+        """Stacks with listed layers: fp32 stream, final norm in the compute dtype (see ``models/parallel_layer.py``)."""
+        cfg, run = self.cfg, self.layer_runner
+        x = self.embed(batch)
+        mult = float(cfg.residual_multiplier)
+        if run is None and not torch.is_grad_enabled():
+            x = x.float().clone() if batch.inputs_embeds is not None else x.float()      # updated in place from here on
+            st = Stream(x.contiguous())
+            for layer in self.layers:
+                st = layer.advance(st, batch)
+            return ops.stream_rmsnorm(st.x, self.norm.weight, cfg.rms_norm_eps, st.adds, mult)[0]
+        first = cfg.layer_specs[cfg.first_mixing_layer] if cfg.first_mixing_layer is not None else None
+        x = F.pad(x.float(), (0, first.kv_heads * first.vdim if first is not None else 0))
+        for layer in self.layers:
+            x = run(layer, x, None, None, batch) if run is not None else layer(x, None, None, batch)
+        return ops.stream_rmsnorm(x[:, :cfg.hidden_size].contiguous(), self.norm.weight, cfg.rms_norm_eps)[0]
+
     def forward(self, batch: PackedBatch, hidden: Optional[torch.Tensor] = None, kv_sink=None) -> torch.Tensor:
+        if self.cfg.layer_specs is not None:
+            return self._forward_listed(batch)
         x = self.embed(batch) if hidden is None else hidden
         if batch.position_ids.dim() == 2:  # [3, T] (time, height, width) positions of a vision-language batch
             from .vision import mrope_tables
@@ -607,6 +632,8 @@ class DecoderModel(nn.Module):
         return x
 
     def logits(self, hidden: torch.Tensor) -> torch.Tensor:
+        if self.cfg.layer_specs is not None and not torch.is_grad_enabled():
+            return ops.linear_f32(hidden, self.head_weight())
         z = ops.linear(hidden, self.head_weight())
         if self.cfg.logits_scaling != 1.0:
             z = z / self.cfg.logits_scaling

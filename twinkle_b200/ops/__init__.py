@@ -150,8 +150,23 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] =
            value_unused: bool = False):
     """``value_unused``: the caller never reads the result when the graph is being rebuilt (see ``dead_values``)."""
     if _cuda(x) and x.dtype == torch.bfloat16:
+        n, k = weight.shape
+        if n % 8 or k % 8:      # TMA rows are whole 16-byte vectors: odd sizes are filled up with zero rows / columns
+            y = _Linear.apply(torch.nn.functional.pad(x, (0, -k % 8)), torch.nn.functional.pad(weight, (0, -k % 8, 0, -n % 8)), None, None, False)[..., :n]
+            return y if bias is None else y + bias
         return _Linear.apply(x, weight, bias, wgrad_out, value_unused and _DeadValues.on)
     return torch.nn.functional.linear(x, weight, bias)
+
+
+def linear_f32(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """``x Wᵀ`` of 16-bit operands with the fp32 sums kept (no gradient): an output head whose logits are not rounded."""
+    if not (_cuda(x) and x.dtype == torch.bfloat16):
+        return torch.nn.functional.linear(x, weight).float()
+    n, k = weight.shape
+    if k % 8:
+        x, weight = torch.nn.functional.pad(x, (0, -k % 8)), torch.nn.functional.pad(weight, (0, -k % 8))
+    out = torch.empty(x.shape[0], -(-n // 4) * 4, dtype=torch.float32, device=x.device)[:, :n]
+    return gemm(x.contiguous(), weight, 'nt', out=out)
 
 
 # ------------------------------------------------------------------- norms
@@ -237,14 +252,14 @@ _WARNED_HEAD_DIM = set()
 
 
 def _head_dim_ok(d: int) -> bool:
-    """The attention-side kernels are written for 128-wide heads (every Qwen3 / Llama-3 size). Other widths — the tiny
-    presets used in tests, vision towers — run on the PyTorch restatement; said once per width."""
+    """The training attention and q/k-norm + RoPE kernels are written for 128-wide heads (every Qwen3 / Llama-3 size). Other
+    widths — the tiny presets used in tests, vision towers — run on the PyTorch restatement; said once per width."""
     if d == 128:
         return True
     if d not in _WARNED_HEAD_DIM:
         _WARNED_HEAD_DIM.add(d)
         import logging
-        logging.getLogger('twinkle_b200').warning(f'head_dim {d}: attention, q/k-norm + RoPE and paged decode run on PyTorch ops (the sm_100a kernels are for head_dim 128)')
+        logging.getLogger('twinkle_b200').warning(f'head_dim {d}: training attention and q/k-norm + RoPE run on PyTorch ops (those sm_100a kernels are for head_dim 128)')
     return False
 
 
@@ -263,6 +278,69 @@ def qkv_norm_rope(qkv: torch.Tensor, q_weight, k_weight, cos, sin, hq: int, hkv:
 
 def rope_tables(positions: torch.Tensor, head_dim: int, theta: float = 1e6, scaling: Optional[dict] = None):
     return ref.rope_tables(positions, head_dim, theta, scaling)
+
+
+# ------------------------------------------- layers with a 32-bit residual stream
+def _needs_grad(*ts) -> bool:
+    return torch.is_grad_enabled() and any(t is not None and t.requires_grad for t in ts)
+
+
+def stream_rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, adds=(), mult: float = 1.0):
+    """fp32 residual stream ``x [T, W]``: ``x ← x + mult · Σ y_i ⊙ s_i`` for ``adds = [(y, s), …]`` (at most two) and its RMS
+    norm in ``weight``'s dtype, one kernel on CUDA.  Returns ``(norm, x)``; without gradients ``x`` is updated in place."""
+    if not _cuda(x) or _needs_grad(x, weight, *[t for a in adds for t in a]):
+        return ref.stream_rmsnorm(x, weight, eps, weight.dtype, adds, mult)
+    (y1, s1), (y2, s2) = (list(adds) + [(None, None)] * 2)[:2]
+    return ext().stream_rmsnorm(x, weight, eps, None if y1 is None else y1.contiguous(), s1, None if y2 is None else y2.contiguous(), s2, mult), x
+
+
+def conv_heads(proj, weight, positions, hq: int, hkv: int, d: int, e: int, eps: float, coef: float = 0.0, every: int = 0, v_first=None, lam=None,
+               view=None, layer: int = -1):
+    """Leading ``[q | k | v]`` columns of a fused projection → ``(q [T,hq,d'], k [T,hkv,d'] | None, v [T,hkv,e'])``: causal depth-wise
+    convolution (``weight [C, taps]`` or None), q and k over their root mean square per head, query temperature, value mixing.
+    ``view`` (a ``CacheView``) says where the tokens live in the sampler's cache: keys, values and the convolution history are
+    written there, and single steps take their history from it (then k is None).  Widths ``d'``, ``e'`` are ``d``, ``e`` rounded
+    up to multiples of 8, the rest zero; with gradients (no ``view``) they are ``d`` and ``e``."""
+    step = view is not None and view.stepping
+    cache = view.cache if view is not None else None
+    hist = cache.conv[layer] if cache is not None else None
+    if _cuda(proj) and not _needs_grad(proj, weight, v_first, lam):
+        if v_first is not None:
+            v_first = torch.nn.functional.pad(v_first, (0, -(-e // 8) * 8 - v_first.shape[-1])).contiguous()
+        out = ext().conv_heads(proj, weight, positions, hq, hkv, d, e, eps, coef, every, v_first, lam, step, hist,
+                               *((view.slots, view.left, view.rows, cache.k[layer], cache.v[layer]) if view is not None else (None, ) * 5), not step)
+        return (out[0], None, out[1]) if step else tuple(out)
+    if v_first is not None:
+        v_first = v_first[..., :e]
+    q, k, v = ref.conv_heads(proj, weight, positions, hq, hkv, d, e, eps, coef, every, v_first, lam, hist if step else None, view.slots if step else None)
+    if _needs_grad(proj, weight, v_first, lam):
+        return q, k, v
+    q, k, v = (torch.nn.functional.pad(t, (0, -t.shape[-1] % 8)) for t in (q, k, v))
+    if view is not None:
+        cache.k[layer].view(-1, *k.shape[1:])[view.rows] = k
+        cache.v[layer].view(-1, *v.shape[1:])[view.rows] = v
+        if hist is not None:
+            n, C = hist.shape[1:]
+            keep = (view.left < n).nonzero(as_tuple=True)[0]
+            hist[view.slots[keep].long(), positions[keep] % n] = proj[keep, :C]
+    return q, (None if step else k), v
+
+
+def glu_columns(proj: torch.Tensor, gate: int, up: int, width: int) -> torch.Tensor:
+    """``silu(proj[:, gate : gate+width]) · proj[:, up : up+width]`` without copying the column ranges."""
+    if _cuda(proj) and not _needs_grad(proj):
+        return ext().glu_columns(proj, gate, up, width)
+    return ref.swiglu(torch.cat([proj[:, gate:gate + width], proj[:, up:up + width]], -1))
+
+
+def attention_packed(q, k, v, cu_seqlens, max_seqlen: int, scale: float):
+    """Causal packed attention for any key / value widths up to 256: tensor-core kernel for bf16 heads up to 128 wide, an
+    fp32-arithmetic kernel for wider heads and for 32-bit models."""
+    if not _cuda(q) or _needs_grad(q, k, v):
+        return flash_attn_varlen(q, k, v, cu_seqlens, max_seqlen, True, scale)
+    if _flash_widths(q, k, v):
+        return ext().flash_attn_fwd(q.contiguous(), k.contiguous(), v.contiguous(), cu_seqlens.to(torch.int32), int(max_seqlen), True, scale)[0]
+    return ext().attention_packed(q.contiguous(), k.contiguous(), v.contiguous(), cu_seqlens.to(torch.int32), int(max_seqlen), scale)
 
 
 # ------------------------------------------------------------------ swiglu
@@ -364,6 +442,12 @@ class AttentionStash:
         AttentionStash.current = self._prev
 
 
+def _flash_widths(q, k, v) -> bool:
+    """Whether the forward kernel takes these heads (training also needs the backward kernel, which is for 128-wide heads)."""
+    d, e = q.shape[-1], v.shape[-1]
+    return q.dtype == torch.bfloat16 and v.dtype == torch.bfloat16 and d <= 128 and e <= 128 and d % 8 == 0 and e % 8 == 0
+
+
 def flash_attn_varlen(q, k, v, cu_seqlens, max_seqlen: int, causal: bool = True, scale: Optional[float] = None,
                       cu_seqlens_k=None, max_seqlen_k: int = 0, return_lse: bool = False, window: Optional[int] = None,
                       softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None):
@@ -382,6 +466,8 @@ def flash_attn_varlen(q, k, v, cu_seqlens, max_seqlen: int, causal: bool = True,
         else:
             out, lse = ref.attention_varlen(q, k, v, cu_seqlens, causal, scale, True, cu_seqlens_k)
         return (out, lse) if return_lse else out
+    if _cuda(q) and q.shape[-1] != 128 and _flash_widths(q, k, v) and not _needs_grad(q, k, v) and AttentionStash.current is None:
+        return ext().flash_attn_fwd(q.contiguous(), k.contiguous(), v.contiguous(), cu_seqlens.to(torch.int32), int(max_seqlen), causal, scale)[0]
     if _cuda(q) and q.dtype == torch.bfloat16 and _head_dim_ok(q.shape[-1]):
         q, k, v = q.contiguous(), k.contiguous(), v.contiguous()
         cu = cu_seqlens.to(torch.int32)
@@ -403,7 +489,8 @@ def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, scale: O
     scale = 1.0 / math.sqrt(q.shape[-1]) if scale is None else scale
     if window is not None or softcap or sinks is not None:
         return ref.paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, scale, window, softcap, sinks)
-    if _cuda(q) and q.dtype == torch.bfloat16 and _head_dim_ok(q.shape[-1]):
+    vec = 16 // q.element_size()
+    if (_cuda(q) and q.dtype in (torch.bfloat16, torch.float32) and all(t.shape[-1] % vec == 0 and t.shape[-1] <= 256 for t in (q, v_cache))):
         return ext().paged_attn_decode(q.contiguous(), k_cache, v_cache, block_tables.to(torch.int32),
                                        seq_lens.to(torch.int32), scale)
     return ref.paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, scale)

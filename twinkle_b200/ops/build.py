@@ -5,6 +5,10 @@
 file (nvcc cross-compiles without a GPU).  ``load_extension()`` imports the
 built module; when a GPU is present and the module is missing it is built on
 the spot, and any failure raises — there is no silent fallback on a GPU box.
+
+A process that only generates (``prefer_serving()``, e.g. the trace replayer) and finds no built ``_C.so`` compiles the
+serving subset into ``_C_serving.so`` instead: the kernels behind prefill, decode and sampling of listed-layer stacks.
+Objects are shared between the two builds.
 """
 from __future__ import annotations
 
@@ -21,14 +25,26 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 _CSRC = os.path.join(_HERE, 'csrc')
 _SO = os.path.join(_HERE, '_C.so')
 _STAMP = os.path.join(_HERE, '_C.stamp')
+_SERVING_SO = os.path.join(_HERE, '_C_serving.so')
+_SERVING_STAMP = os.path.join(_HERE, '_C_serving.stamp')
+_SERVING_SOURCES = ('bindings.cpp', 'host.cu', 'gemm.cu', 'gemm2.cu', 'attention_fwd.cu', 'attention_packed.cu', 'decode.cu', 'stream_ops.cu')
 _MOD = None
+_SERVING_ONLY = False
 
 NVCC_FLAGS = ['-gencode', 'arch=compute_100a,code=sm_100a', '-lineinfo', '-O3', '-std=c++17', '--use_fast_math',
               '-Xcompiler', '-fPIC', '--expt-relaxed-constexpr', '--expt-extended-lambda', '-DNDEBUG',
               '-U__CUDA_NO_HALF_OPERATORS__', '-U__CUDA_NO_BFLOAT16_CONVERSIONS__', '-U__CUDA_NO_HALF_CONVERSIONS__']
 
 
-def _sources() -> List[str]:
+def prefer_serving() -> None:
+    """Let the serving subset stand in for the full extension when that is not built (call before the first kernel)."""
+    global _SERVING_ONLY
+    _SERVING_ONLY = True
+
+
+def _sources(serving: bool = False) -> List[str]:
+    if serving:
+        return [os.path.join(_CSRC, f) for f in _SERVING_SOURCES]
     return sorted(glob.glob(os.path.join(_CSRC, '*.cu')) + glob.glob(os.path.join(_CSRC, '*.cpp')))
 
 
@@ -54,31 +70,33 @@ def _digest() -> str:
     return h.hexdigest()
 
 
-def is_built() -> bool:
-    if not os.path.isfile(_SO) or not os.path.isfile(_STAMP):
+def is_built(serving: bool = False) -> bool:
+    so, stamp = (_SERVING_SO, _SERVING_STAMP) if serving else (_SO, _STAMP)
+    if not os.path.isfile(so) or not os.path.isfile(stamp):
         return False
-    with open(_STAMP) as f:
+    with open(stamp) as f:
         return f.read().strip() == _digest()
 
 
-def build_extension(verbose: bool = False, jobs: Optional[int] = None) -> str:
+def build_extension(verbose: bool = False, jobs: Optional[int] = None, serving: bool = False) -> str:
     """Compile each source to an object (in parallel) and link ``_C.so``.  Processes that arrive together (the ranks
     of one job) take a file lock in turn: the first builds, the others find the stamp current and return."""
-    if is_built():
-        return _SO
+    so = _SERVING_SO if serving else _SO
+    if is_built(serving):
+        return so
     import fcntl
     lock = open(os.path.join(_HERE, '.build.lock'), 'w')
     fcntl.flock(lock, fcntl.LOCK_EX)
     try:
-        if is_built():
-            return _SO
-        return _build_locked(verbose, jobs)
+        if is_built(serving):
+            return so
+        return _build_locked(verbose, jobs, serving)
     finally:
         fcntl.flock(lock, fcntl.LOCK_UN)
         lock.close()
 
 
-def _build_locked(verbose: bool, jobs: Optional[int]) -> str:
+def _build_locked(verbose: bool, jobs: Optional[int], serving: bool) -> str:
     import torch
     from torch.utils import cpp_extension as ce
     from concurrent.futures import ThreadPoolExecutor
@@ -92,7 +110,8 @@ def _build_locked(verbose: bool, jobs: Optional[int]) -> str:
     objs = []
 
     def compile_one(src: str) -> str:
-        obj = os.path.join(build_dir, os.path.basename(src) + '.o')
+        own = ['-DTK_SERVING_ONLY'] if serving and src.endswith('bindings.cpp') else []
+        obj = os.path.join(build_dir, os.path.basename(src) + ('.serving' if own else '') + '.o')
         dep_stamp = obj + '.sha'
         h = hashlib.sha1(open(src, 'rb').read())
         for hdr in _local_includes(src):  # only the headers this source pulls in: touching one header rebuilds its users
@@ -100,7 +119,7 @@ def _build_locked(verbose: bool, jobs: Optional[int]) -> str:
         h.update(' '.join(NVCC_FLAGS).encode())
         if os.path.isfile(obj) and os.path.isfile(dep_stamp) and open(dep_stamp).read() == h.hexdigest():
             return obj
-        cmd = [nvcc, '-c', src, '-o', obj] + NVCC_FLAGS + inc + defs
+        cmd = [nvcc, '-c', src, '-o', obj] + NVCC_FLAGS + inc + defs + own
         if verbose:
             cmd += ['-Xptxas', '-v']
             print(' '.join(cmd), file=sys.stderr)
@@ -114,17 +133,18 @@ def _build_locked(verbose: bool, jobs: Optional[int]) -> str:
         return obj
 
     with ThreadPoolExecutor(max_workers=jobs or min(8, os.cpu_count() or 4)) as pool:
-        objs = list(pool.map(compile_one, _sources()))
+        objs = list(pool.map(compile_one, _sources(serving)))
     torch_lib = os.path.join(os.path.dirname(torch.__file__), 'lib')
-    link = ['g++', '-shared', '-o', _SO] + objs + [
+    so, stamp = (_SERVING_SO, _SERVING_STAMP) if serving else (_SO, _STAMP)
+    link = ['g++', '-shared', '-o', so] + objs + [
         '-L' + torch_lib, '-L' + os.path.join(cuda_home, 'lib64'), '-lc10', '-lc10_cuda', '-ltorch_cpu', '-ltorch_cuda',
         '-ltorch', '-ltorch_python', '-lcudart', '-Wl,-rpath,' + torch_lib, '-Wl,-rpath,' + os.path.join(cuda_home, 'lib64')]
     r = subprocess.run(link, capture_output=True, text=True)
     if r.returncode != 0:
         raise RuntimeError(f'link failed:\n{r.stdout}\n{r.stderr}')
-    with open(_STAMP, 'w') as f:
+    with open(stamp, 'w') as f:
         f.write(_digest())
-    return _SO
+    return so
 
 
 def load_extension():
@@ -132,14 +152,17 @@ def load_extension():
     if _MOD is not None:
         return _MOD
     import torch  # noqa: F401  (libtorch must be loaded before the extension)
-    if not is_built():
+    so = _SO
+    if _SERVING_ONLY and not is_built():
+        so = build_extension(serving=True)
+    elif not is_built():
         if not torch.cuda.is_available() and os.environ.get('TWINKLE_B200_BUILD', '0') != '1' and not os.path.isfile(_SO):
             raise ImportError('twinkle_b200.ops._C is not built (run `python -c "import __graft_entry__ as g; g.build()"`)')
         if not os.path.isfile(_SO) or os.environ.get('TWINKLE_B200_BUILD', '0') == '1' or torch.cuda.is_available():
             # a binary whose stamp does not match the sources is never loaded in place of a failed rebuild: the
             # numbers and tests of a run must come from the code in the tree
             build_extension()
-    spec = importlib.util.spec_from_file_location('twinkle_b200.ops._C', _SO)
+    spec = importlib.util.spec_from_file_location('twinkle_b200.ops._C', so)
     mod = importlib.util.module_from_spec(spec)
     spec.loader.exec_module(mod)  # type: ignore[union-attr]
     sys.modules['twinkle_b200.ops._C'] = mod

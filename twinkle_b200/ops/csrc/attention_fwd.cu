@@ -1,4 +1,5 @@
-// Flash-attention forward for sm_100a: causal, GQA, packed variable-length sequences, D = 128.
+// Flash-attention forward for sm_100a: causal, GQA, packed variable-length sequences, query / key and value widths up to 128.
+// A row narrower than its 64- or 128-wide tile is filled up with zeros by the TMA load (the tensor map ends at the row's width).
 //
 // One CTA per (128-row query tile of one sequence, query head).  192 threads:
 //   warps 0-3  softmax: thread = one query row; reads S from tensor memory (tcgen05.ld), keeps the
@@ -10,7 +11,7 @@
 // Tensor memory: S0 [0,128), S1 [128,256), O [256,384) fp32 columns.
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
-#include <torch/extension.h>
+#include <torch/types.h>
 
 #include "common.cuh"
 #include "host.h"
@@ -33,6 +34,7 @@ constexpr float RESCALE_THRESHOLD = 8.f;  // log2 units
 struct FwdParams {
   bf16* out;          // [T, Hq, D]
   float* lse;         // [Hq, T]  natural-log LSE of the scaled scores
+  int e;              // width of a value / output row (a multiple of 8)
   const int* cu;      // [n+1] query boundaries
   const int* cu_k;    // [n+1] key/value boundaries (== cu for self-attention over the same packing)
   int T, hq, hkv;
@@ -41,6 +43,8 @@ struct FwdParams {
   int* err;
 };
 
+// KA / VA: 64-wide chunks of a query / key row and of a value row (1 or 2).
+template <int KA, int VA>
 __global__ void __launch_bounds__(fa::THREADS, 1)
 flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                  const __grid_constant__ CUtensorMap tmV, const FwdParams p) {
@@ -103,31 +107,31 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       tma_prefetch_desc(&tmQ);
       tma_prefetch_desc(&tmK);
       tma_prefetch_desc(&tmV);
-      mbar_expect_tx(q_full, TILE_BYTES);
+      mbar_expect_tx(q_full, KA * ATOM_BYTES);
       tma_load_3d(smem + SMEM_Q, &tmQ, q_full, 0, head, seq_start + q0);
-      tma_load_3d(smem + SMEM_Q + ATOM_BYTES, &tmQ, q_full, 64, head, seq_start + q0);
+      if constexpr (KA > 1) tma_load_3d(smem + SMEM_Q + ATOM_BYTES, &tmQ, q_full, 64, head, seq_start + q0);
       for (int j = 0; j < n_blocks; ++j) {
         const int st = j & 1;
         if (j >= 2 && !mbar_wait(&kv_empty[st], ((j >> 1) - 1) & 1, p.err, ERR_ATTN_WAIT)) break;
         const int row = kv_start + j * BKV;
-        mbar_expect_tx(&k_full[st], TILE_BYTES);
+        mbar_expect_tx(&k_full[st], KA * ATOM_BYTES);
         tma_load_3d(smem + SMEM_K + st * TILE_BYTES, &tmK, &k_full[st], 0, kv_head, row);
-        tma_load_3d(smem + SMEM_K + st * TILE_BYTES + ATOM_BYTES, &tmK, &k_full[st], 64, kv_head, row);
-        mbar_expect_tx(&v_full[st], TILE_BYTES);
+        if constexpr (KA > 1) tma_load_3d(smem + SMEM_K + st * TILE_BYTES + ATOM_BYTES, &tmK, &k_full[st], 64, kv_head, row);
+        mbar_expect_tx(&v_full[st], VA * ATOM_BYTES);
         tma_load_3d(smem + SMEM_V + st * TILE_BYTES, &tmV, &v_full[st], 0, kv_head, row);
-        tma_load_3d(smem + SMEM_V + st * TILE_BYTES + ATOM_BYTES, &tmV, &v_full[st], 64, kv_head, row);
+        if constexpr (VA > 1) tma_load_3d(smem + SMEM_V + st * TILE_BYTES + ATOM_BYTES, &tmV, &v_full[st], 64, kv_head, row);
       }
     }
   } else if (warp == 9) {
     // ----------------------------------------------------------- MMA issuer
     if (lane == 0) {
       constexpr uint32_t idesc_s = umma_idesc_bf16(BQ, BKV, false, false);
-      constexpr uint32_t idesc_o = umma_idesc_bf16(BQ, D, false, true);
+      constexpr uint32_t idesc_o = umma_idesc_bf16(BQ, VA * 64, false, true);
       const uint32_t sq = smem_u32(smem + SMEM_Q), sp = smem_u32(smem + SMEM_P);
       auto issue_s = [&](int j) {
         const uint32_t sk = smem_u32(smem + SMEM_K + (j & 1) * TILE_BYTES);
 #pragma unroll
-        for (int k = 0; k < D / 16; ++k) {
+        for (int k = 0; k < KA * 4; ++k) {
           const uint32_t off = (k >> 2) * ATOM_BYTES + (k & 3) * 32;
           umma_bf16(tmem_base + (j & 1) * 128, umma_desc(sq + off, 16, 1024), umma_desc(sk + off, 16, 1024), idesc_s, k ? 1u : 0u);
         }
@@ -218,7 +222,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       if (!dead && j > 0 && !mbar_wait(o_done, (j - 1) & 1, p.err, ERR_ATTN_WAIT)) dead = true;
       if (dead) continue;
       tc_fence_after();
-      if (__any_sync(0xffffffffu, rescale)) {
+      if (wg < VA && __any_sync(0xffffffffu, rescale)) {
 #pragma unroll 1
         for (int c = 0; c < 2; ++c) {
           uint32_t r[32];
@@ -255,15 +259,16 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       tc_fence_after();
       const float inv_l = (l_sum > 0.f) ? 1.f / l_sum : 0.f;
       const bool valid = q_pos < seq_len;
-      bf16* orow = p.out + (static_cast<size_t>(seq_start + q_pos) * p.hq + head) * D;
+      bf16* orow = p.out + (static_cast<size_t>(seq_start + q_pos) * p.hq + head) * p.e;
 #pragma unroll 1
-      for (int c = 2 * wg; c < 2 * wg + 2; ++c) {
+      for (int c = 2 * wg; c < 2 * wg + 2 && c * 32 < p.e; ++c) {
         uint32_t r[32];
         tmem_ld32(tmem_o + lane_off + c * 32, r);
         tmem_ld_wait();
         if (valid) {
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
+            if (VA == 1 || c >= 2) { if (c * 32 + i >= p.e) break; }
             uint4 v = make_uint4(pack_bf16(__uint_as_float(r[i]) * inv_l, __uint_as_float(r[i + 1]) * inv_l),
                                  pack_bf16(__uint_as_float(r[i + 2]) * inv_l, __uint_as_float(r[i + 3]) * inv_l),
                                  pack_bf16(__uint_as_float(r[i + 4]) * inv_l, __uint_as_float(r[i + 5]) * inv_l),
@@ -290,32 +295,44 @@ CUtensorMap make_head_tmap(const torch::Tensor& t, int rows) {
 
 std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor& q, const torch::Tensor& k, const torch::Tensor& v, const torch::Tensor& cu,
                                           int64_t max_seqlen, bool causal, double scale, const c10::optional<torch::Tensor>& cu_k) {
-  TORCH_CHECK(q.is_cuda() && q.scalar_type() == torch::kBFloat16 && q.dim() == 3 && q.is_contiguous(), "q [T,Hq,128] bf16 contiguous");
-  TORCH_CHECK(k.is_contiguous() && v.is_contiguous() && k.sizes() == v.sizes() && k.scalar_type() == torch::kBFloat16, "k/v [T,Hkv,128]");
-  TORCH_CHECK(q.size(2) == 128 && k.size(2) == 128, "head_dim must be 128");
+  TORCH_CHECK(q.is_cuda() && q.scalar_type() == torch::kBFloat16 && q.dim() == 3 && q.is_contiguous(), "q [T,Hq,D] bf16 contiguous");
+  TORCH_CHECK(k.is_contiguous() && v.is_contiguous() && k.dim() == 3 && v.dim() == 3 && k.size(0) == v.size(0) && k.size(1) == v.size(1) &&
+                  k.scalar_type() == torch::kBFloat16 && v.scalar_type() == torch::kBFloat16, "k [T,Hkv,D], v [T,Hkv,E] bf16 contiguous");
+  TORCH_CHECK(q.size(2) == k.size(2) && k.size(2) % 8 == 0 && v.size(2) % 8 == 0 && k.size(2) > 0 && v.size(2) > 0 && k.size(2) <= 128 && v.size(2) <= 128,
+              "head widths: multiples of 8 up to 128");
   TORCH_CHECK(cu.is_cuda() && cu.scalar_type() == torch::kInt32 && cu.is_contiguous(), "cu_seqlens int32 on device");
   TORCH_CHECK(q.size(1) % k.size(1) == 0, "Hq must be a multiple of Hkv");
   c10::cuda::CUDAGuard guard(q.device());
   const int T = q.size(0), hq = q.size(1), hkv = k.size(1), nseq = cu.numel() - 1;
-  auto out = torch::empty_like(q);
+  auto out = torch::empty({T, hq, v.size(2)}, q.options());
   auto lse = torch::empty({hq, T}, q.options().dtype(torch::kFloat32));
   if (T == 0 || nseq <= 0) return {out, lse};
   CUtensorMap tq = make_head_tmap(q, 128), tk_ = make_head_tmap(k, 128), tv = make_head_tmap(v, 128);
   FwdParams p{};
-  p.out = reinterpret_cast<bf16*>(out.data_ptr()); p.lse = lse.data_ptr<float>(); p.cu = cu.data_ptr<int>();
+  p.out = reinterpret_cast<bf16*>(out.data_ptr()); p.lse = lse.data_ptr<float>(); p.e = v.size(2); p.cu = cu.data_ptr<int>();
   p.cu_k = p.cu;
   if (cu_k.has_value() && cu_k->defined()) {
     TORCH_CHECK(cu_k->is_cuda() && cu_k->scalar_type() == torch::kInt32 && cu_k->is_contiguous() && cu_k->numel() == cu.numel(), "cu_k like cu");
     p.cu_k = cu_k->data_ptr<int>();
   }
   p.T = T; p.hq = hq; p.hkv = hkv; p.scale_log2 = static_cast<float>(scale * 1.4426950408889634); p.causal = causal; p.err = error_word();
-  static bool configured = false;
-  if (!configured) {
-    TK_CUDA_CHECK(cudaFuncSetAttribute(flash_fwd_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, fa::SMEM_TOTAL));
-    configured = true;
-  }
-  dim3 grid(hq, (static_cast<int>(max_seqlen) + fa::BQ - 1) / fa::BQ, nseq);
-  flash_fwd_kernel<<<grid, fa::THREADS, fa::SMEM_TOTAL, at::cuda::getCurrentCUDAStream()>>>(tq, tk_, tv, p);
+  const dim3 grid(hq, (static_cast<int>(max_seqlen) + fa::BQ - 1) / fa::BQ, nseq);
+  auto stream = at::cuda::getCurrentCUDAStream();
+#define TK_FLASH(KA, VA)                                                                                                                \
+  do {                                                                                                                                  \
+    static bool configured = false;                                                                                                     \
+    if (!configured) {                                                                                                                  \
+      TK_CUDA_CHECK(cudaFuncSetAttribute(flash_fwd_kernel<KA, VA>, cudaFuncAttributeMaxDynamicSharedMemorySize, fa::SMEM_TOTAL));       \
+      configured = true;                                                                                                                \
+    }                                                                                                                                   \
+    flash_fwd_kernel<KA, VA><<<grid, fa::THREADS, fa::SMEM_TOTAL, stream>>>(tq, tk_, tv, p);                                            \
+  } while (0)
+  const bool wide_k = q.size(2) > 64, wide_v = v.size(2) > 64;
+  if (wide_k && wide_v) TK_FLASH(2, 2);
+  else if (wide_k) TK_FLASH(2, 1);
+  else if (wide_v) TK_FLASH(1, 2);
+  else TK_FLASH(1, 1);
+#undef TK_FLASH
   count_launch();
   TK_CUDA_CHECK(cudaGetLastError());
   return {out, lse};

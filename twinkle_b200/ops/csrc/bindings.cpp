@@ -1,4 +1,5 @@
-// Python bindings of the sm_100a extension.
+// Python bindings of the sm_100a extension.  With TK_SERVING_ONLY the module holds just what generation with a
+// listed-layer stack launches (see ops/build.py): a box that only serves does not compile the training kernels.
 #include <torch/extension.h>
 
 #include "host.h"
@@ -6,6 +7,21 @@
 namespace tk {
 torch::Tensor gemm(const torch::Tensor&, const torch::Tensor&, const std::string&, const c10::optional<torch::Tensor>&, bool,
                    c10::optional<torch::ScalarType>);
+std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t,
+                                          bool, double, const c10::optional<torch::Tensor>&);
+torch::Tensor attention_packed(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t, double);
+torch::Tensor paged_attn_decode(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, double);
+std::vector<torch::Tensor> sample_tokens(const torch::Tensor&, double, int64_t, double, const torch::Tensor&);
+std::vector<torch::Tensor> conv_heads(const torch::Tensor&, const c10::optional<torch::Tensor>&, const torch::Tensor&, int64_t, int64_t, int64_t, int64_t,
+                                      double, double, int64_t, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, bool,
+                                      const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&,
+                                      const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, bool);
+torch::Tensor stream_rmsnorm(torch::Tensor, const torch::Tensor&, double, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&,
+                             const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, double);
+torch::Tensor glu_columns(const torch::Tensor&, int64_t, int64_t, int64_t);
+void set_gemm_pair(int64_t);
+void set_gemm_staged(int64_t);
+#ifndef TK_SERVING_ONLY
 torch::Tensor grouped_gemm(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const std::string&, const c10::optional<torch::Tensor>&,
                            const c10::optional<torch::Tensor>&, bool, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
 torch::Tensor grouped_gemm_wgrad(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t);
@@ -27,8 +43,6 @@ torch::Tensor sumsq(const torch::Tensor&);
 std::vector<torch::Tensor> logprob_fwd(const torch::Tensor&, const torch::Tensor&, double, bool);
 torch::Tensor logprob_bwd(torch::Tensor, const torch::Tensor&, const torch::Tensor&, const c10::optional<torch::Tensor>&,
                           const torch::Tensor&, const c10::optional<torch::Tensor>&, double);
-std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t,
-                                          bool, double, const c10::optional<torch::Tensor>&);
 std::vector<torch::Tensor> flash_attn_bwd(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&,
                                           const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t, bool, double,
                                           const c10::optional<torch::Tensor>&, int64_t);
@@ -45,11 +59,7 @@ void peer_copy_cast(const torch::Tensor&, const std::vector<int64_t>&, int64_t);
 torch::Tensor causal_conv1d_fwd(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, bool);
 std::vector<torch::Tensor> gdn_recurrent_fwd(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&,
                                              const torch::Tensor&, const torch::Tensor&, const c10::optional<torch::Tensor>&, double, bool);
-torch::Tensor paged_attn_decode(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, double);
-std::vector<torch::Tensor> sample_tokens(const torch::Tensor&, double, int64_t, double, const torch::Tensor&);
 std::vector<torch::Tensor> moe_router(const torch::Tensor&, int64_t, bool);
-void set_gemm_pair(int64_t);
-void set_gemm_staged(int64_t);
 void gemm_rs(const torch::Tensor&, const torch::Tensor&, const std::string&, const std::vector<int64_t>&, int64_t);
 void gemm_head_scatter(const torch::Tensor&, const torch::Tensor&, const std::vector<int64_t>&, int64_t, int64_t, int64_t, int64_t);
 std::vector<torch::Tensor> gemm_ag(const std::vector<int64_t>&, int64_t, const torch::Tensor&, const std::string&, int64_t, const torch::Tensor&, int64_t, int64_t);
@@ -61,11 +71,30 @@ torch::Tensor ep_rows_gather(const std::vector<int64_t>&, const std::vector<int6
                              const torch::Tensor&, int64_t, int64_t);
 torch::Tensor ep_rows_combine(const std::vector<int64_t>&, const torch::Tensor&, const torch::Tensor&, const c10::optional<torch::Tensor>&, int64_t, int64_t);
 torch::Tensor ep_combine_wgrad(const torch::Tensor&, const std::vector<int64_t>&, const torch::Tensor&, const torch::Tensor&, int64_t);
+#endif
 }  // namespace tk
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm", &tk::gemm, py::arg("a"), py::arg("b"), py::arg("layout") = "nt", py::arg("out") = py::none(),
         py::arg("accumulate") = false, py::arg("out_dtype") = py::none());
+  m.def("flash_attn_fwd", &tk::flash_attn_fwd, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("cu"), py::arg("max_seqlen"), py::arg("causal"),
+        py::arg("scale"), py::arg("cu_k") = py::none());
+  m.def("paged_attn_decode", &tk::paged_attn_decode);
+  m.def("sample_tokens", &tk::sample_tokens);
+  m.def("set_gemm_pair", &tk::set_gemm_pair);
+  m.def("set_gemm_staged", &tk::set_gemm_staged);
+  m.def("read_and_clear_error", &tk::read_and_clear_error, "Value of the device error word (0 = healthy); clears it.");
+  m.def("num_sms", &tk::num_sms);
+  m.def("launch_count", &tk::launch_count, "Number of kernels launched by this extension so far.");
+  m.def("attention_packed", &tk::attention_packed);
+  m.def("conv_heads", &tk::conv_heads, py::arg("proj"), py::arg("weight"), py::arg("pos"), py::arg("hq"), py::arg("hkv"), py::arg("d"), py::arg("e"), py::arg("eps"),
+        py::arg("coef") = 0.0, py::arg("every") = 0, py::arg("v_first") = py::none(), py::arg("lam") = py::none(), py::arg("step") = false,
+        py::arg("hist") = py::none(), py::arg("slot") = py::none(), py::arg("left") = py::none(), py::arg("pool_row") = py::none(),
+        py::arg("k_pool") = py::none(), py::arg("v_pool") = py::none(), py::arg("want_k") = true);
+  m.def("stream_rmsnorm", &tk::stream_rmsnorm, py::arg("x"), py::arg("w"), py::arg("eps"), py::arg("y1") = py::none(), py::arg("s1") = py::none(),
+        py::arg("y2") = py::none(), py::arg("s2") = py::none(), py::arg("mult") = 1.0);
+  m.def("glu_columns", &tk::glu_columns);
+#ifndef TK_SERVING_ONLY
   m.def("grouped_gemm", &tk::grouped_gemm, py::arg("x"), py::arg("w"), py::arg("offsets"), py::arg("layout") = "nt", py::arg("group_map") = py::none(),
         py::arg("out") = py::none(), py::arg("accumulate") = false, py::arg("x2") = py::none(), py::arg("w2") = py::none());
   m.def("grouped_gemm_wgrad", &tk::grouped_gemm_wgrad);
@@ -82,8 +111,6 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("sumsq", &tk::sumsq);
   m.def("logprob_fwd", &tk::logprob_fwd);
   m.def("logprob_bwd", &tk::logprob_bwd);
-  m.def("flash_attn_fwd", &tk::flash_attn_fwd, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("cu"), py::arg("max_seqlen"), py::arg("causal"),
-        py::arg("scale"), py::arg("cu_k") = py::none());
   m.def("flash_attn_bwd", &tk::flash_attn_bwd, py::arg("dout"), py::arg("q"), py::arg("k"), py::arg("v"), py::arg("out"), py::arg("lse"), py::arg("cu"),
         py::arg("max_seqlen"), py::arg("causal"), py::arg("scale"), py::arg("cu_k") = py::none(), py::arg("max_seqlen_k") = 0);
   m.def("symm_alloc", &tk::symm_alloc, "cudaMalloc'ed uint8 tensor + its CUDA IPC handle");
@@ -99,11 +126,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("causal_conv1d_fwd", &tk::causal_conv1d_fwd);
   m.def("gdn_recurrent_fwd", &tk::gdn_recurrent_fwd, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("g"), py::arg("beta"), py::arg("cu"),
         py::arg("init_state") = py::none(), py::arg("scale") = 1.0, py::arg("want_state") = false);
-  m.def("paged_attn_decode", &tk::paged_attn_decode);
-  m.def("sample_tokens", &tk::sample_tokens);
   m.def("moe_router", &tk::moe_router);
-  m.def("set_gemm_pair", &tk::set_gemm_pair);
-  m.def("set_gemm_staged", &tk::set_gemm_staged);
   m.def("gemm_rs", &tk::gemm_rs);
   m.def("gemm_head_scatter", &tk::gemm_head_scatter);
   m.def("gemm_ag", &tk::gemm_ag);
@@ -114,7 +137,5 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("ep_rows_gather", &tk::ep_rows_gather);
   m.def("ep_rows_combine", &tk::ep_rows_combine);
   m.def("ep_combine_wgrad", &tk::ep_combine_wgrad);
-  m.def("read_and_clear_error", &tk::read_and_clear_error, "Value of the device error word (0 = healthy); clears it.");
-  m.def("num_sms", &tk::num_sms);
-  m.def("launch_count", &tk::launch_count, "Number of kernels launched by this extension so far.");
+#endif
 }

@@ -4,7 +4,7 @@
 // All three are bandwidth / latency bound; none needs tensor cores.
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
-#include <torch/extension.h>
+#include <torch/types.h>
 
 #include "common.cuh"
 #include "host.h"
@@ -14,76 +14,91 @@ namespace tk {
 using bf16 = __nv_bfloat16;
 
 // ---------------------------------------------------------------- paged decode
-// One CTA per (sequence, kv head, group of GH query heads); 4 warps.  A warp handles 4 context tokens per step —
-// 8 lanes per token, 16 dims (two 16-byte loads of K, two of V) per lane — and two steps are issued back to back, so
-// 32 token rows per CTA are in flight.  Every lane group keeps an online-softmax state per query head; lane groups
-// and warps are merged at the end.
-template <int GH>
-__global__ void __launch_bounds__(128) paged_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const bf16* __restrict__ vc,
-                                                            const int* __restrict__ tables, const int* __restrict__ seq_lens, bf16* __restrict__ out,
-                                                            int hq, int hkv, int block_size, int max_blocks, float scale_log2, int G) {
-  constexpr int D = 128;
-  const int b = blockIdx.x, kvh = blockIdx.y, h0 = kvh * G + blockIdx.z * GH;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, grp = lane >> 3, sub = lane & 7;  // sub owns dims [16·sub, 16·sub+16)
+// One CTA per (sequence, kv head, group of GH query heads); 4 warps.  A warp handles 4 context tokens per step — 8 lanes
+// per token, each lane NC 16-byte vectors of the K row and of the V row — and U steps are issued back to back (two for rows
+// of up to 256 bytes: 32 token rows per CTA in flight).  Every lane group keeps an online-softmax state per query head;
+// lane groups and warps are merged at the end.  Key and value rows are `d` and `e` elements wide, whole 16-byte vectors.
+__device__ __forceinline__ void unpack_vec(const uint4& u, float (&x)[8], const bf16*) {
+  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const float2 a = unpack_bf16(w[k]);
+    x[2 * k] = a.x; x[2 * k + 1] = a.y;
+  }
+}
+__device__ __forceinline__ void unpack_vec(const uint4& u, float (&x)[4], const float*) {
+  x[0] = __uint_as_float(u.x); x[1] = __uint_as_float(u.y); x[2] = __uint_as_float(u.z); x[3] = __uint_as_float(u.w);
+}
+__device__ __forceinline__ float to_float(bf16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float to_float(float v) { return v; }
+__device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ void put(float* p, float v) { *p = v; }
+
+template <typename T, int GH, int NC, int U>
+__global__ void __launch_bounds__(128) paged_decode_kernel(const T* __restrict__ q, const T* __restrict__ kc, const T* __restrict__ vc,
+                                                            const int* __restrict__ tables, const int* __restrict__ seq_lens, T* __restrict__ out,
+                                                            int hq, int hkv, int d, int e, int block_size, int max_blocks, float scale_log2, int G) {
+  constexpr int V = 16 / sizeof(T), D = NC * 8 * V;   // elements per vector, widest row of this instance
+  const int b = blockIdx.x, kvh = blockIdx.y, g0 = blockIdx.z * GH, h0 = kvh * G + g0;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, grp = lane >> 3, sub = lane & 7;  // vector c of a lane: elements [(8c + sub)·V, …+V)
   const int n = seq_lens[b];
   // the query (pre-scaled, fp32) lives in shared memory: registers are kept for two iterations' worth of K/V rows
-  __shared__ float s_q[GH][D];
-  for (int i = threadIdx.x; i < GH * D; i += blockDim.x)
-    s_q[i / D][i % D] = __bfloat162float(q[(static_cast<size_t>(b) * hq + h0 + i / D) * D + i % D]) * scale_log2;
+  __shared__ __align__(16) float s_q[GH][D];
+  for (int i = threadIdx.x; i < GH * D; i += blockDim.x) {
+    const int g = i / D, c = i % D;
+    s_q[g][c] = (g0 + g < G && c < d) ? to_float(q[(static_cast<size_t>(b) * hq + h0 + g) * d + c]) * scale_log2 : 0.f;
+  }
   __syncthreads();
-  float m[GH], l[GH], acc[GH][16];
+  float m[GH], l[GH], acc[GH][NC * V];
 #pragma unroll
   for (int g = 0; g < GH; ++g) {
     m[g] = -INFINITY; l[g] = 0.f;
 #pragma unroll
-    for (int d = 0; d < 16; ++d) acc[g][d] = 0.f;
+    for (int i = 0; i < NC * V; ++i) acc[g][i] = 0.f;
   }
   const int* table = tables + static_cast<size_t>(b) * max_blocks;
-  // token handled by (warp, grp) in half-step u of iteration `base`: t = base + grp + 16·u.  The loop bound depends on
+  // token handled by (warp, grp) in step u of iteration `base`: t = base + grp + 16·u.  The loop bound depends on
   // the warp only, so all 32 lanes stay in the loop together (the shuffles below name the full warp).  The rows of
   // iteration i+1 are requested before iteration i is consumed.
-  uint4 kr[2][2], vr[2][2], kn[2][2], vn[2][2];
-  auto fetch = [&](int base, uint4 (&kk)[2][2], uint4 (&vv)[2][2]) {
+  uint4 kr[U][NC], vr[U][NC], kn[U][NC], vn[U][NC];
+  auto fetch = [&](int base, uint4 (&kk)[U][NC], uint4 (&vv)[U][NC]) {
 #pragma unroll
-    for (int u = 0; u < 2; ++u) {
+    for (int u = 0; u < U; ++u) {
       const int t = base + grp + u * 16;
       if (t < n) {
         const int blk = table[t / block_size], off = t % block_size;
-        // lane `sub` owns dims [8·sub, 8·sub+8) and [64+8·sub, 64+8·sub+8): each load instruction covers 128 contiguous bytes per token
-        const size_t base_off = ((static_cast<size_t>(blk) * block_size + off) * hkv + kvh) * D + sub * 8;
-        kk[u][0] = *reinterpret_cast<const uint4*>(kc + base_off); kk[u][1] = *reinterpret_cast<const uint4*>(kc + base_off + 64);
-        vv[u][0] = *reinterpret_cast<const uint4*>(vc + base_off); vv[u][1] = *reinterpret_cast<const uint4*>(vc + base_off + 64);
+        const size_t row = (static_cast<size_t>(blk) * block_size + off) * hkv + kvh;
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {   // each load instruction covers up to 128 contiguous bytes per token
+          const int el = (8 * c + sub) * V;
+          kk[u][c] = el < d ? *reinterpret_cast<const uint4*>(kc + row * d + el) : make_uint4(0u, 0u, 0u, 0u);
+          vv[u][c] = el < e ? *reinterpret_cast<const uint4*>(vc + row * e + el) : make_uint4(0u, 0u, 0u, 0u);
+        }
       }
     }
   };
   if (warp * 4 < n) fetch(warp * 4, kr, vr);
-  for (int base = warp * 4; base < n; base += 32) {
-    if (base + 32 < n) fetch(base + 32, kn, vn);
+  for (int base = warp * 4; base < n; base += 16 * U) {
+    if (base + 16 * U < n) fetch(base + 16 * U, kn, vn);
 #pragma unroll
-    for (int u = 0; u < 2; ++u) {
+    for (int u = 0; u < U; ++u) {
       const bool live = base + grp + u * 16 < n;
-      float kf[16], vf[16];
+      float kf[NC][V], vf[NC][V];
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const uint32_t* pk = &kr[u][h].x;
-        const uint32_t* pv = &vr[u][h].x;
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          const float2 a = unpack_bf16(pk[k]), c = unpack_bf16(pv[k]);
-          kf[h * 8 + 2 * k] = a.x; kf[h * 8 + 2 * k + 1] = a.y;
-          vf[h * 8 + 2 * k] = c.x; vf[h * 8 + 2 * k + 1] = c.y;
-        }
+      for (int c = 0; c < NC; ++c) {
+        unpack_vec(kr[u][c], kf[c], kc);
+        unpack_vec(vr[u][c], vf[c], vc);
       }
 #pragma unroll
       for (int g = 0; g < GH; ++g) {
         float s = 0.f;
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          const float4* qs = reinterpret_cast<const float4*>(&s_q[g][h * 64 + sub * 8]);
+        for (int c = 0; c < NC; ++c) {
+          const float4* qs = reinterpret_cast<const float4*>(&s_q[g][(8 * c + sub) * V]);
 #pragma unroll
-          for (int d4 = 0; d4 < 2; ++d4) {
+          for (int d4 = 0; d4 < V / 4; ++d4) {
             const float4 qq = qs[d4];
-            s += qq.x * kf[h * 8 + 4 * d4] + qq.y * kf[h * 8 + 4 * d4 + 1] + qq.z * kf[h * 8 + 4 * d4 + 2] + qq.w * kf[h * 8 + 4 * d4 + 3];
+            s += qq.x * kf[c][4 * d4] + qq.y * kf[c][4 * d4 + 1] + qq.z * kf[c][4 * d4 + 2] + qq.w * kf[c][4 * d4 + 3];
           }
         }
         if (!live) s = 0.f;  // rows that were not fetched hold stale registers
@@ -95,16 +110,17 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const bf16* __restric
           const float corr = exp2f(m[g] - mn), p = exp2f(s - mn);
           l[g] = l[g] * corr + p;
 #pragma unroll
-          for (int d = 0; d < 16; ++d) acc[g][d] = acc[g][d] * corr + p * vf[d];
+          for (int c = 0; c < NC; ++c)
+#pragma unroll
+            for (int x = 0; x < V; ++x) acc[g][c * V + x] = acc[g][c * V + x] * corr + p * vf[c][x];
           m[g] = mn;
         }
       }
     }
 #pragma unroll
-    for (int u = 0; u < 2; ++u) {
-      kr[u][0] = kn[u][0]; kr[u][1] = kn[u][1];
-      vr[u][0] = vn[u][0]; vr[u][1] = vn[u][1];
-    }
+    for (int u = 0; u < U; ++u)
+#pragma unroll
+      for (int c = 0; c < NC; ++c) { kr[u][c] = kn[u][c]; vr[u][c] = vn[u][c]; }
   }
   // merge the 4 lane groups of the warp, then the 4 warps
   __shared__ float s_m[4][GH], s_l[4][GH], s_acc[4][GH][D];
@@ -116,57 +132,75 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const bf16* __restric
       const float mn = fmaxf(m[g], mo);
       const float c0 = (m[g] == -INFINITY) ? 0.f : exp2f(m[g] - mn), c1 = (mo == -INFINITY) ? 0.f : exp2f(mo - mn);
 #pragma unroll
-      for (int d = 0; d < 16; ++d) acc[g][d] = acc[g][d] * c0 + __shfl_xor_sync(0xffffffffu, acc[g][d], o) * c1;
+      for (int i = 0; i < NC * V; ++i) acc[g][i] = acc[g][i] * c0 + __shfl_xor_sync(0xffffffffu, acc[g][i], o) * c1;
       l[g] = l[g] * c0 + lo * c1;
       m[g] = mn;
     }
     if (lane == 0) { s_m[warp][g] = m[g]; s_l[warp][g] = l[g]; }
     if (grp == 0) {
 #pragma unroll
-      for (int d = 0; d < 16; ++d) s_acc[warp][g][(d >> 3) * 64 + sub * 8 + (d & 7)] = acc[g][d];
+      for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int x = 0; x < V; ++x) s_acc[warp][g][(8 * c + sub) * V + x] = acc[g][c * V + x];
     }
   }
   __syncthreads();
-  const int d = threadIdx.x;  // thread d (0..127) finishes dimension d of every head of the group
+  for (int i = threadIdx.x; i < e; i += blockDim.x) {  // a thread finishes dimension i of every head of the group
 #pragma unroll
-  for (int g = 0; g < GH; ++g) {
-    const float mm = fmaxf(fmaxf(s_m[0][g], s_m[1][g]), fmaxf(s_m[2][g], s_m[3][g]));
-    float ll = 0.f, o = 0.f;
+    for (int g = 0; g < GH; ++g) {
+      if (g0 + g >= G) break;
+      const float mm = fmaxf(fmaxf(s_m[0][g], s_m[1][g]), fmaxf(s_m[2][g], s_m[3][g]));
+      float ll = 0.f, o = 0.f;
 #pragma unroll
-    for (int w = 0; w < 4; ++w) {
-      const float c = (s_m[w][g] == -INFINITY) ? 0.f : exp2f(s_m[w][g] - mm);
-      ll += s_l[w][g] * c;
-      o += s_acc[w][g][d] * c;
+      for (int w = 0; w < 4; ++w) {
+        const float c = (s_m[w][g] == -INFINITY) ? 0.f : exp2f(s_m[w][g] - mm);
+        ll += s_l[w][g] * c;
+        o += s_acc[w][g][i] * c;
+      }
+      put(out + (static_cast<size_t>(b) * hq + h0 + g) * e + i, ll > 0.f ? o / ll : 0.f);
     }
-    out[(static_cast<size_t>(b) * hq + h0 + g) * D + d] = __float2bfloat16(ll > 0.f ? o / ll : 0.f);
+  }
+}
+
+template <typename T>
+static void launch_paged_decode(const torch::Tensor& q, const torch::Tensor& kc, const torch::Tensor& vc, const torch::Tensor& tables,
+                                const torch::Tensor& seq_lens, torch::Tensor& out, float sl2, cudaStream_t stream) {
+  constexpr int V = 16 / sizeof(T);
+  const int B = q.size(0), hq = q.size(1), hkv = kc.size(2), G = hq / hkv, d = q.size(2), e = vc.size(3);
+  auto go = [&](auto kern, int GH) {
+    // query heads of a group are processed GH at a time (register budget): G = 8 → two CTAs per (sequence, kv head)
+    kern<<<dim3(B, hkv, (G + GH - 1) / GH), 128, 0, stream>>>(reinterpret_cast<const T*>(q.data_ptr()), reinterpret_cast<const T*>(kc.data_ptr()),
+        reinterpret_cast<const T*>(vc.data_ptr()), tables.data_ptr<int>(), seq_lens.data_ptr<int>(), reinterpret_cast<T*>(out.data_ptr()), hq, hkv, d, e,
+        static_cast<int>(kc.size(1)), static_cast<int>(tables.size(1)), sl2, G);
+  };
+  const int vectors = (std::max(d, e) + 8 * V - 1) / (8 * V);   // per lane
+  if (vectors <= 1) {
+    if (G == 1) go(paged_decode_kernel<T, 1, 1, 2>, 1); else if (G == 2) go(paged_decode_kernel<T, 2, 1, 2>, 2); else go(paged_decode_kernel<T, 4, 1, 2>, 4);
+  } else if (vectors <= 2) {
+    if (G == 1) go(paged_decode_kernel<T, 1, 2, 2>, 1); else if (G == 2) go(paged_decode_kernel<T, 2, 2, 2>, 2); else go(paged_decode_kernel<T, 4, 2, 2>, 4);
+  } else if (vectors <= 4) {
+    if (G == 1) go(paged_decode_kernel<T, 1, 4, 1>, 1); else go(paged_decode_kernel<T, 2, 4, 1>, 2);
+  } else if constexpr (sizeof(T) == 4) {   // 16-bit rows of up to 256 elements are four vectors per lane
+    go(paged_decode_kernel<T, 1, 8, 1>, 1);
   }
 }
 
 torch::Tensor paged_attn_decode(const torch::Tensor& q, const torch::Tensor& kc, const torch::Tensor& vc, const torch::Tensor& tables,
                                 const torch::Tensor& seq_lens, double scale) {
-  TORCH_CHECK(q.is_cuda() && q.scalar_type() == torch::kBFloat16 && q.is_contiguous() && q.dim() == 3 && q.size(2) == 128, "q [B,Hq,128] bf16");
-  TORCH_CHECK(kc.is_contiguous() && vc.is_contiguous() && kc.dim() == 4 && kc.size(3) == 128 && kc.scalar_type() == torch::kBFloat16, "cache [blocks,bs,Hkv,128] bf16");
+  const auto st = q.scalar_type();
+  TORCH_CHECK(q.is_cuda() && (st == torch::kBFloat16 || st == torch::kFloat32) && q.is_contiguous() && q.dim() == 3, "q [B,Hq,D] bf16 or fp32");
+  TORCH_CHECK(kc.is_contiguous() && vc.is_contiguous() && kc.dim() == 4 && vc.dim() == 4 && kc.scalar_type() == st && vc.scalar_type() == st, "caches [blocks,bs,Hkv,·] in q's dtype");
+  const int64_t V = 16 / q.element_size();
+  TORCH_CHECK(kc.size(3) == q.size(2) && kc.size(3) % V == 0 && vc.size(3) % V == 0 && kc.size(3) <= 256 && vc.size(3) <= 256, "rows of whole 16-byte vectors, up to 256 wide");
+  TORCH_CHECK(kc.size(0) == vc.size(0) && kc.size(1) == vc.size(1) && kc.size(2) == vc.size(2) && q.size(1) % kc.size(2) == 0, "shapes of the caches");
   TORCH_CHECK(tables.scalar_type() == torch::kInt32 && tables.is_contiguous() && seq_lens.scalar_type() == torch::kInt32, "int32 tables / lens");
   c10::cuda::CUDAGuard guard(q.device());
-  const int B = q.size(0), hq = q.size(1), hkv = kc.size(2), G = hq / hkv;
-  auto out = torch::empty_like(q);
-  if (B == 0) return out;
+  auto out = torch::empty({q.size(0), q.size(1), vc.size(3)}, q.options());
+  if (q.size(0) == 0) return out;
   const float sl2 = static_cast<float>(scale * 1.4426950408889634);
   auto stream = at::cuda::getCurrentCUDAStream();
-  // query heads of a group are processed GH at a time (register budget): G = 8 → two CTAs per (sequence, kv head)
-  const int GH = G >= 4 ? 4 : G;
-  TORCH_CHECK(G == 1 || G == 2 || G == 4 || G == 8, "GQA group size must be 1, 2, 4 or 8");
-  dim3 grid(B, hkv, G / GH);
-#define TK_DEC(GG)                                                                                                                   \
-  paged_decode_kernel<GG><<<grid, 128, 0, stream>>>(reinterpret_cast<const bf16*>(q.data_ptr()), reinterpret_cast<const bf16*>(kc.data_ptr()), \
-      reinterpret_cast<const bf16*>(vc.data_ptr()), tables.data_ptr<int>(), seq_lens.data_ptr<int>(), reinterpret_cast<bf16*>(out.data_ptr()),  \
-      hq, hkv, static_cast<int>(kc.size(1)), static_cast<int>(tables.size(1)), sl2, G)
-  switch (GH) {
-    case 1: TK_DEC(1); break;
-    case 2: TK_DEC(2); break;
-    default: TK_DEC(4); break;
-  }
-#undef TK_DEC
+  if (st == torch::kBFloat16) launch_paged_decode<bf16>(q, kc, vc, tables, seq_lens, out, sl2, stream);
+  else launch_paged_decode<float>(q, kc, vc, tables, seq_lens, out, sl2, stream);
   count_launch();
   TK_CUDA_CHECK(cudaGetLastError());
   return out;

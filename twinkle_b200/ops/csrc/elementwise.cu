@@ -4,7 +4,7 @@
 // algorithmic bytes.
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
-#include <torch/extension.h>
+#include <torch/types.h>
 
 #include "common.cuh"
 #include "host.h"

@@ -14,7 +14,7 @@
 // Rewriting o_t = α·(S_{t-1}ᵀq̂) + δ·(q̂·k̂) lets both dot products run in the single pass over the old state.
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
-#include <torch/extension.h>
+#include <torch/types.h>
 
 #include "common.cuh"
 #include "host.h"

@@ -15,7 +15,7 @@
 // share the same pipeline and differ only in the tile scheduler.
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
-#include <torch/extension.h>
+#include <torch/types.h>
 
 #include <mutex>
 #include <unordered_map>

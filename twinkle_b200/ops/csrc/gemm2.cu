@@ -24,7 +24,7 @@
 // All waits are bounded (common.cuh); both CTAs always meet at a cluster barrier before TMEM is released.
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
-#include <torch/extension.h>
+#include <torch/types.h>
 
 #include "common.cuh"
 #include "host.h"

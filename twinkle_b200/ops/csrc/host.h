@@ -2,7 +2,7 @@
 #pragma once
 #include <cuda.h>
 #include <cuda_runtime.h>
-#include <torch/extension.h>
+#include <torch/types.h>
 
 #define TK_CUDA_CHECK(expr)                                                                              \
   do {                                                                                                   \

@@ -5,7 +5,7 @@
 // logits tensor never exists.
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
-#include <torch/extension.h>
+#include <torch/types.h>
 
 #include "common.cuh"
 #include "host.h"

@@ -7,7 +7,7 @@
 // One warp per destination row; 16-byte accesses; bf16 data, fp32 math.
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
-#include <torch/extension.h>
+#include <torch/types.h>
 
 #include "common.cuh"
 #include "host.h"

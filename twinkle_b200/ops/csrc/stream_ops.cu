@@ -1,0 +1,493 @@
+// Element-wise steps of decoder layers whose residual stream is 32-bit and whose mixer and feed-forward block read one
+// fused projection [q | k | v | gate | up]:
+//   conv_heads      short causal convolution on q, k and v, q / k over their root mean square per head, query temperature,
+//                   value mixing, and the writes into the paged K/V pools and the convolution history — one pass
+//   stream_rmsnorm  x += mult · (y1 ⊙ s1 + y2 ⊙ s2) in fp32 and the RMS norm of the sum in the compute dtype — one pass
+//   glu_columns     silu(gate) · up on two column ranges of the projection
+// All are templated on the compute dtype (bf16 or fp32) and work for any width: vector kernels where rows are made of
+// whole vectors, plain ones otherwise.
+#include <ATen/cuda/CUDAContext.h>
+#include <c10/cuda/CUDAGuard.h>
+#include <torch/types.h>
+
+#include "common.cuh"
+#include "host.h"
+
+namespace tk {
+
+using bf16 = __nv_bfloat16;
+
+template <typename T> __device__ __forceinline__ float to_f(T v);
+template <> __device__ __forceinline__ float to_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ float to_f<bf16>(bf16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f(float v);
+template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ bf16 from_f<bf16>(float v) { return __float2bfloat16(v); }
+
+// four consecutive elements as fp32
+__device__ __forceinline__ float4 load4(const bf16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = unpack_bf16(u.x), b = unpack_bf16(u.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ void store4(bf16* p, const float4& v) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+}
+__device__ __forceinline__ void store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+
+__device__ __forceinline__ float block_sum(float v, float* sh) {
+  v = warp_sum(v);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = (blockDim.x + 31) >> 5;
+  __syncthreads();
+  if (lane == 0) sh[warp] = v;
+  __syncthreads();
+  return warp_sum(lane < nw ? sh[lane] : 0.f);
+}
+
+// ------------------------------------------------------------------ conv_heads
+template <typename T>
+struct ConvHeads {
+  const T* proj; long ld;               // [rows, ld]: q | k | v in the leading columns
+  const T* w;                           // [C, taps] (nullptr: no convolution)
+  int taps;
+  int hq, hkv, d, e;                    // heads and widths
+  int dp, ep;                           // row widths of the outputs and pools (≥ d, e; the rest is written as zero)
+  float eps, coef; int every;           // query temperature (every = 0: none)
+  const int64_t* pos;                   // place of every row in its sequence
+  T *q, *k, *v;                         // [rows, hq, dp], [rows, hkv, dp] (may be null), [rows, hkv, ep]
+  const T* v_first; const T* lam;       // [rows, hkv, ep], [1] (null: values are not mixed)
+  T *k_pool, *v_pool; const int64_t* pool_row;   // [·, hkv, dp], [·, hkv, ep]; row of every token (< 0: not kept)
+  T* hist; const int* slot; const int* left;     // [slots, taps − 1, C]; left[t] = later rows of the same sequence in this call
+  int rows;
+};
+
+template <typename T>
+__device__ __forceinline__ float query_factor(const ConvHeads<T>& p, int64_t pos) {
+  return p.every > 0 ? 1.f + p.coef * log1pf(static_cast<float>((pos + 1) / p.every)) : 1.f;
+}
+
+// One warp per (head, run of `run` rows); a lane owns NV groups of four channels of the head.  Rows of a run are read once
+// and slide through registers as history of the rows behind them (packed rows: the history of row t is t−1, t−2, … as far
+// as its position allows).  STEP: every row is a sequence of its own and takes its history from the pool.
+template <typename T, int TAPS, int NV, bool STEP>
+__global__ void __launch_bounds__(128) conv_heads_kernel(const ConvHeads<T> p, int run) {
+  constexpr int H = TAPS - 1, AHEAD = 4;
+  const int lane = threadIdx.x & 31;
+  const int head = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (head >= p.hq + 2 * p.hkv) return;
+  const bool is_v = head >= p.hq + p.hkv, is_q = head < p.hq;
+  const int width = is_v ? p.e : p.d, padded = is_v ? p.ep : p.dp;
+  const int c0 = is_v ? (p.hq + p.hkv) * p.d + (head - p.hq - p.hkv) * p.e : head * p.d;   // first column of the head
+  const int C = (p.hq + p.hkv) * p.d + p.hkv * p.e;
+  const int gh = is_q ? head : (is_v ? head - p.hq - p.hkv : head - p.hq);                  // head inside its own tensor
+  bool own[NV], out[NV];
+  float w[NV][TAPS][4];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int el = (i * 32 + lane) * 4;
+    own[i] = el < width;
+    out[i] = el < padded;
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) w[i][j][c] = own[i] && p.w != nullptr ? to_f(p.w[static_cast<size_t>(c0 + el + c) * TAPS + j]) : 1.f;
+  }
+  const float lam = (is_v && p.v_first != nullptr) ? to_f(p.lam[0]) : 0.f;
+  const int t0 = blockIdx.x * run, t1 = min(t0 + run, p.rows);
+  float4 h[H > 0 ? H : 1][NV];         // h[j] = row t − 1 − j
+  if constexpr (!STEP) {
+#pragma unroll
+    for (int j = 0; j < H; ++j)
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        h[j][i] = (own[i] && t0 - 1 - j >= 0) ? load4(p.proj + static_cast<size_t>(t0 - 1 - j) * p.ld + c0 + (i * 32 + lane) * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  for (int tb = t0; tb < t1; tb += AHEAD) {
+    float4 cur[AHEAD][NV];
+    int64_t ps[AHEAD];
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) {
+      const int t = min(tb + u, t1 - 1);
+      ps[u] = p.pos[t];
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        cur[u][i] = own[i] ? load4(p.proj + static_cast<size_t>(t) * p.ld + c0 + (i * 32 + lane) * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) {
+      const int t = tb + u;
+      if (t >= t1) break;
+      const int64_t pos = ps[u];
+      float4 y[NV];
+      if constexpr (STEP && H > 0) {
+#pragma unroll
+        for (int j = 0; j < H; ++j)
+#pragma unroll
+          for (int i = 0; i < NV; ++i)
+            h[j][i] = (own[i] && j + 1 <= pos) ? load4(p.hist + (static_cast<size_t>(p.slot[t]) * H + (pos - 1 - j) % H) * C + c0 + (i * 32 + lane) * 4)
+                                               : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const float4 a = cur[u][i];
+        y[i] = make_float4(w[i][H][0] * a.x, w[i][H][1] * a.y, w[i][H][2] * a.z, w[i][H][3] * a.w);
+#pragma unroll
+        for (int j = 0; j < H; ++j) {
+          if (j + 1 <= pos) {
+            const float4 b = h[j][i];
+            y[i].x += w[i][H - 1 - j][0] * b.x; y[i].y += w[i][H - 1 - j][1] * b.y;
+            y[i].z += w[i][H - 1 - j][2] * b.z; y[i].w += w[i][H - 1 - j][3] * b.w;
+          }
+        }
+        if (!own[i]) y[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        ss += y[i].x * y[i].x + y[i].y * y[i].y + y[i].z * y[i].z + y[i].w * y[i].w;
+      }
+      if (!is_v) {
+        ss = warp_sum(ss);
+        float f = rsqrtf(ss / width + p.eps);
+        if (is_q) f *= query_factor(p, pos);
+#pragma unroll
+        for (int i = 0; i < NV; ++i) { y[i].x *= f; y[i].y *= f; y[i].z *= f; y[i].w *= f; }
+      }
+      const int64_t row = p.pool_row != nullptr ? p.pool_row[t] : -1;
+      const bool keep = H > 0 && p.hist != nullptr && p.left[t] < H;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int el = (i * 32 + lane) * 4;
+        if (out[i]) {
+          if (is_q) {
+            store4(p.q + (static_cast<size_t>(t) * p.hq + gh) * p.dp + el, y[i]);
+          } else if (!is_v) {
+            if (p.k != nullptr) store4(p.k + (static_cast<size_t>(t) * p.hkv + gh) * p.dp + el, y[i]);
+            if (row >= 0) store4(p.k_pool + (static_cast<size_t>(row) * p.hkv + gh) * p.dp + el, y[i]);
+          } else {
+            if (p.v_first != nullptr) {
+              const float4 f = load4(p.v_first + (static_cast<size_t>(t) * p.hkv + gh) * p.ep + el);
+              y[i].x += lam * (f.x - y[i].x); y[i].y += lam * (f.y - y[i].y); y[i].z += lam * (f.z - y[i].z); y[i].w += lam * (f.w - y[i].w);
+            }
+            store4(p.v + (static_cast<size_t>(t) * p.hkv + gh) * p.ep + el, y[i]);
+            if (row >= 0) store4(p.v_pool + (static_cast<size_t>(row) * p.hkv + gh) * p.ep + el, y[i]);
+          }
+        }
+        // the newest rows of a sequence are what its next step looks back at (same thread read this place above)
+        if constexpr (H > 0) {
+          if (keep && own[i]) store4(p.hist + (static_cast<size_t>(p.slot[t]) * H + pos % H) * C + c0 + el, cur[u][i]);
+        }
+      }
+      if constexpr (!STEP) {
+#pragma unroll
+        for (int j = H - 1; j > 0; --j)
+#pragma unroll
+          for (int i = 0; i < NV; ++i) h[j][i] = h[j - 1][i];
+        if constexpr (H > 0) {
+#pragma unroll
+          for (int i = 0; i < NV; ++i) h[0][i] = cur[u][i];
+        }
+      }
+    }
+  }
+}
+
+// Any number of taps, any widths: one block per (row, head), element-wise loads.
+template <typename T, bool STEP>
+__global__ void __launch_bounds__(128) conv_heads_plain_kernel(const ConvHeads<T> p) {
+  extern __shared__ float row_buf[];
+  __shared__ float sh[32];
+  const int t = blockIdx.x, head = blockIdx.y, H = p.taps > 0 ? p.taps - 1 : 0;
+  const bool is_v = head >= p.hq + p.hkv, is_q = head < p.hq;
+  const int width = is_v ? p.e : p.d, padded = is_v ? p.ep : p.dp;
+  const int c0 = is_v ? (p.hq + p.hkv) * p.d + (head - p.hq - p.hkv) * p.e : head * p.d;
+  const int C = (p.hq + p.hkv) * p.d + p.hkv * p.e;
+  const int gh = is_q ? head : (is_v ? head - p.hq - p.hkv : head - p.hq);
+  const int64_t pos = p.pos[t];
+  const int64_t row = p.pool_row != nullptr ? p.pool_row[t] : -1;
+  const bool keep = H > 0 && p.hist != nullptr && p.left[t] < H;
+  float ss = 0.f;
+  for (int el = threadIdx.x; el < width; el += blockDim.x) {
+    const int c = c0 + el;
+    const T now = p.proj[static_cast<size_t>(t) * p.ld + c];
+    float y = to_f(now);
+    if (p.w != nullptr) {
+      y *= to_f(p.w[static_cast<size_t>(c) * p.taps + H]);
+      for (int j = 1; j <= H && j <= pos; ++j) {
+        const T b = STEP ? p.hist[(static_cast<size_t>(p.slot[t]) * H + (pos - j) % H) * C + c] : p.proj[static_cast<size_t>(t - j) * p.ld + c];
+        y += to_f(p.w[static_cast<size_t>(c) * p.taps + H - j]) * to_f(b);
+      }
+    }
+    if (keep) p.hist[(static_cast<size_t>(p.slot[t]) * H + pos % H) * C + c] = now;
+    row_buf[el] = y;
+    ss += y * y;
+  }
+  float f = 1.f;
+  if (!is_v) {
+    f = rsqrtf(block_sum(ss, sh) / width + p.eps);
+    if (is_q) f *= query_factor(p, pos);
+  }
+  for (int el = threadIdx.x; el < padded; el += blockDim.x) {   // an element is finished by the thread that computed it
+    float y = el < width ? row_buf[el] * f : 0.f;
+    if (is_q) {
+      p.q[(static_cast<size_t>(t) * p.hq + gh) * p.dp + el] = from_f<T>(y);
+    } else if (!is_v) {
+      if (p.k != nullptr) p.k[(static_cast<size_t>(t) * p.hkv + gh) * p.dp + el] = from_f<T>(y);
+      if (row >= 0) p.k_pool[(static_cast<size_t>(row) * p.hkv + gh) * p.dp + el] = from_f<T>(y);
+    } else {
+      if (p.v_first != nullptr) y += to_f(p.lam[0]) * (to_f(p.v_first[(static_cast<size_t>(t) * p.hkv + gh) * p.ep + el]) - y);
+      p.v[(static_cast<size_t>(t) * p.hkv + gh) * p.ep + el] = from_f<T>(y);
+      if (row >= 0) p.v_pool[(static_cast<size_t>(row) * p.hkv + gh) * p.ep + el] = from_f<T>(y);
+    }
+  }
+}
+
+static bool aligned16(const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; }
+
+template <typename T, int TAPS>
+static void launch_conv_heads(const ConvHeads<T>& p, bool step, bool wide, cudaStream_t stream) {
+  const int heads = p.hq + 2 * p.hkv;
+  // enough warps to fill the device first, then longer runs (fewer history rows read twice)
+  const long target = 16L * num_sms() * 4;
+  int run = step ? 1 : static_cast<int>(std::min<long>(32, std::max<long>(4, static_cast<long>(p.rows) * heads / target)));
+  const dim3 grid((p.rows + run - 1) / run, (heads + 3) / 4);
+  if (step) {
+    if (wide) conv_heads_kernel<T, TAPS, 2, true><<<grid, 128, 0, stream>>>(p, run);
+    else conv_heads_kernel<T, TAPS, 1, true><<<grid, 128, 0, stream>>>(p, run);
+  } else {
+    if (wide) conv_heads_kernel<T, TAPS, 2, false><<<grid, 128, 0, stream>>>(p, run);
+    else conv_heads_kernel<T, TAPS, 1, false><<<grid, 128, 0, stream>>>(p, run);
+  }
+}
+
+using OptT = c10::optional<torch::Tensor>;
+static bool has(const OptT& t) { return t.has_value() && t->defined(); }
+
+template <typename T>
+static void conv_heads_t(ConvHeads<T>& p, bool step) {
+  auto stream = at::cuda::getCurrentCUDAStream();
+  const int wmax = std::max(p.dp, p.ep);
+  const bool vec = p.d % 4 == 0 && p.e % 4 == 0 && p.ld % 4 == 0 && wmax <= 256 && p.taps <= 4 && aligned16(p.proj) &&
+                   (p.hist == nullptr || ((p.hq + p.hkv) * p.d + p.hkv * p.e) % 4 == 0);
+  if (vec) {
+    switch (p.taps) {
+      case 4: launch_conv_heads<T, 4>(p, step, wmax > 128, stream); break;
+      case 3: launch_conv_heads<T, 3>(p, step, wmax > 128, stream); break;
+      case 2: launch_conv_heads<T, 2>(p, step, wmax > 128, stream); break;
+      default: launch_conv_heads<T, 1>(p, step, wmax > 128, stream); break;
+    }
+  } else {
+    const dim3 grid(p.rows, p.hq + 2 * p.hkv);
+    const size_t smem = static_cast<size_t>(wmax) * sizeof(float);
+    TORCH_CHECK(smem <= 48 * 1024, "head width too large");
+    if (step) conv_heads_plain_kernel<T, true><<<grid, 128, smem, stream>>>(p);
+    else conv_heads_plain_kernel<T, false><<<grid, 128, smem, stream>>>(p);
+  }
+  count_launch();
+  TK_CUDA_CHECK(cudaGetLastError());
+}
+
+std::vector<torch::Tensor> conv_heads(const torch::Tensor& proj, const OptT& weight, const torch::Tensor& pos, int64_t hq, int64_t hkv, int64_t d, int64_t e,
+                                      double eps, double coef, int64_t every, const OptT& v_first, const OptT& lam, bool step, const OptT& hist,
+                                      const OptT& slot, const OptT& left, const OptT& pool_row, const OptT& k_pool, const OptT& v_pool, bool want_k) {
+  const auto st = proj.scalar_type();
+  TORCH_CHECK(proj.is_cuda() && proj.dim() == 2 && proj.stride(1) == 1 && (st == torch::kBFloat16 || st == torch::kFloat32), "proj [rows, N] bf16 or fp32");
+  const int64_t rows = proj.size(0), C = (hq + hkv) * d + hkv * e, dp = (d + 7) / 8 * 8, ep = (e + 7) / 8 * 8;
+  TORCH_CHECK(hq > 0 && hkv > 0 && d > 0 && e > 0 && proj.size(1) >= C, "projection narrower than its q | k | v columns");
+  TORCH_CHECK(pos.is_cuda() && pos.scalar_type() == torch::kInt64 && pos.is_contiguous() && pos.numel() == rows, "positions int64 [rows]");
+  int taps = 0;
+  if (has(weight)) {
+    TORCH_CHECK(weight->scalar_type() == st && weight->is_contiguous() && weight->dim() == 2 && weight->size(0) == C && weight->size(1) >= 1, "filters [C, taps]");
+    taps = weight->size(1);
+  }
+  if (has(v_first)) {
+    TORCH_CHECK(v_first->scalar_type() == st && v_first->is_contiguous() && v_first->numel() == rows * hkv * ep, "v_first [rows, hkv, ep]");
+    TORCH_CHECK(has(lam) && lam->scalar_type() == st && lam->numel() == 1, "mixing weight [1]");
+  }
+  TORCH_CHECK(!step || taps <= 1 || has(hist), "single steps of a convolution need its history");
+  if (has(hist) && taps > 1) {
+    TORCH_CHECK(hist->scalar_type() == st && hist->is_contiguous() && hist->dim() == 3 && hist->size(1) == taps - 1 && hist->size(2) == C, "history [slots, taps-1, C]");
+    TORCH_CHECK(has(slot) && has(left) && slot->scalar_type() == torch::kInt32 && left->scalar_type() == torch::kInt32 && slot->is_contiguous() &&
+                    left->is_contiguous() && slot->numel() == rows && left->numel() == rows, "slot / left int32 [rows]");
+  }
+  if (has(pool_row)) {
+    TORCH_CHECK(has(k_pool) && has(v_pool) && k_pool->scalar_type() == st && v_pool->scalar_type() == st && k_pool->is_contiguous() && v_pool->is_contiguous() &&
+                    k_pool->size(-1) == dp && v_pool->size(-1) == ep && k_pool->size(-2) == hkv && v_pool->size(-2) == hkv, "pools [..., hkv, dp] and [..., hkv, ep]");
+    TORCH_CHECK(pool_row->scalar_type() == torch::kInt64 && pool_row->is_contiguous() && pool_row->numel() == rows, "pool rows int64 [rows]");
+  }
+  c10::cuda::CUDAGuard guard(proj.device());
+  auto q = torch::empty({rows, hq, dp}, proj.options());
+  auto k = want_k ? torch::empty({rows, hkv, dp}, proj.options()) : torch::Tensor();
+  auto v = torch::empty({rows, hkv, ep}, proj.options());
+  if (rows > 0) {
+    auto fill = [&](auto tag) {
+      using T = decltype(tag);
+      auto ptr = [](const OptT& t) { return has(t) ? reinterpret_cast<T*>(t->data_ptr()) : static_cast<T*>(nullptr); };
+      ConvHeads<T> p{};
+      p.proj = reinterpret_cast<const T*>(proj.data_ptr()); p.ld = proj.stride(0); p.w = ptr(weight); p.taps = taps;
+      p.hq = hq; p.hkv = hkv; p.d = d; p.e = e; p.dp = dp; p.ep = ep; p.eps = eps; p.coef = coef; p.every = every;
+      p.pos = pos.data_ptr<int64_t>();
+      p.q = reinterpret_cast<T*>(q.data_ptr()); p.k = want_k ? reinterpret_cast<T*>(k.data_ptr()) : nullptr; p.v = reinterpret_cast<T*>(v.data_ptr());
+      p.v_first = ptr(v_first); p.lam = ptr(lam);
+      if (has(pool_row)) { p.pool_row = pool_row->data_ptr<int64_t>(); p.k_pool = ptr(k_pool); p.v_pool = ptr(v_pool); }
+      if (has(hist) && taps > 1) { p.hist = ptr(hist); p.slot = slot->data_ptr<int>(); p.left = left->data_ptr<int>(); }
+      p.rows = rows;
+      conv_heads_t<T>(p, step);
+    };
+    if (st == torch::kBFloat16) fill(bf16{}); else fill(float{});
+  }
+  if (want_k) return {q, k, v};
+  return {q, v};
+}
+
+// -------------------------------------------------------------- stream_rmsnorm
+// One block per row.  VPT > 0: a thread keeps its VPT groups of four sums in registers between the two passes; VPT = 0:
+// rows of any width, element-wise, the second pass re-reads what the thread wrote.
+template <typename T, int VPT>
+__global__ void stream_rmsnorm_kernel(float* __restrict__ x, const T* __restrict__ y1, const T* __restrict__ s1, const T* __restrict__ y2,
+                                      const T* __restrict__ s2, float mult, const T* __restrict__ w, T* __restrict__ h, int W, float eps) {
+  __shared__ float sh[32];
+  const size_t base = static_cast<size_t>(blockIdx.x) * W;
+  float ss = 0.f;
+  if constexpr (VPT > 0) {
+    float4 v[VPT];
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * 4;
+      v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < W) {
+        v[i] = load4(x + base + c);
+        if (y1 != nullptr) {
+          const float4 a = load4(y1 + base + c), b = load4(s1 + c);
+          float4 s = make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w);
+          if (y2 != nullptr) {
+            const float4 e = load4(y2 + base + c), f = load4(s2 + c);
+            s.x += e.x * f.x; s.y += e.y * f.y; s.z += e.z * f.z; s.w += e.w * f.w;
+          }
+          v[i].x += mult * s.x; v[i].y += mult * s.y; v[i].z += mult * s.z; v[i].w += mult * s.w;
+          store4(x + base + c, v[i]);
+        }
+      }
+      ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    }
+    const float r = rsqrtf(block_sum(ss, sh) / W + eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * 4;
+      if (c < W) {
+        const float4 g = load4(w + c);
+        store4(h + base + c, make_float4(v[i].x * r * g.x, v[i].y * r * g.y, v[i].z * r * g.z, v[i].w * r * g.w));
+      }
+    }
+  } else {
+    for (int c = threadIdx.x; c < W; c += blockDim.x) {
+      float v = x[base + c];
+      if (y1 != nullptr) {
+        float s = to_f(y1[base + c]) * to_f(s1[c]);
+        if (y2 != nullptr) s += to_f(y2[base + c]) * to_f(s2[c]);
+        v += mult * s;
+        x[base + c] = v;
+      }
+      ss += v * v;
+    }
+    const float r = rsqrtf(block_sum(ss, sh) / W + eps);
+    for (int c = threadIdx.x; c < W; c += blockDim.x) h[base + c] = from_f<T>(x[base + c] * r * to_f(w[c]));
+  }
+}
+
+// x [rows, W] fp32 is updated in place when y1 is given; returns the norm in w's dtype.
+torch::Tensor stream_rmsnorm(torch::Tensor x, const torch::Tensor& w, double eps, const OptT& y1, const OptT& s1, const OptT& y2, const OptT& s2, double mult) {
+  const auto st = w.scalar_type();
+  TORCH_CHECK(x.is_cuda() && x.scalar_type() == torch::kFloat32 && x.is_contiguous() && x.dim() == 2, "stream [rows, W] fp32 contiguous");
+  TORCH_CHECK((st == torch::kBFloat16 || st == torch::kFloat32) && w.is_contiguous() && w.numel() == x.size(1), "norm weight [W] bf16 or fp32");
+  const int rows = x.size(0), W = x.size(1);
+  bool vec = W % 4 == 0 && W <= 8192 && aligned16(w.data_ptr());
+  auto check = [&](const OptT& y, const OptT& s) {
+    if (!has(y)) return;
+    TORCH_CHECK(y->scalar_type() == st && y->is_contiguous() && y->numel() == x.numel(), "sub-layer result [rows, W] in the norm weight's dtype");
+    TORCH_CHECK(has(s) && s->scalar_type() == st && s->is_contiguous() && s->numel() == W, "channel scale [W]");
+    vec = vec && aligned16(y->data_ptr()) && aligned16(s->data_ptr());
+  };
+  TORCH_CHECK(has(y1) || !has(y2), "the second result comes with a first");
+  check(y1, s1);
+  check(y2, s2);
+  c10::cuda::CUDAGuard guard(x.device());
+  auto h = torch::empty(x.sizes(), w.options());
+  if (rows == 0) return h;
+  auto stream = at::cuda::getCurrentCUDAStream();
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    auto ptr = [](const OptT& t) { return has(t) ? reinterpret_cast<const T*>(t->data_ptr()) : static_cast<const T*>(nullptr); };
+    auto go = [&](auto kern, int threads) {
+      kern<<<rows, threads, 0, stream>>>(x.data_ptr<float>(), ptr(y1), ptr(s1), ptr(y2), ptr(s2), static_cast<float>(mult),
+                                         reinterpret_cast<const T*>(w.data_ptr()), reinterpret_cast<T*>(h.data_ptr()), W, static_cast<float>(eps));
+    };
+    const int nvec = (W + 3) / 4;
+    const int vpt = nvec <= 512 ? 1 : (nvec <= 1024 ? 2 : 4);
+    const int threads = std::min(512, ((nvec + vpt - 1) / vpt + 31) / 32 * 32);
+    if (!vec) go(stream_rmsnorm_kernel<T, 0>, std::min(512, (W + 31) / 32 * 32));
+    else if (vpt == 1) go(stream_rmsnorm_kernel<T, 1>, threads);
+    else if (vpt == 2) go(stream_rmsnorm_kernel<T, 2>, threads);
+    else go(stream_rmsnorm_kernel<T, 4>, threads);
+  };
+  if (st == torch::kBFloat16) run(bf16{}); else run(float{});
+  count_launch();
+  TK_CUDA_CHECK(cudaGetLastError());
+  return h;
+}
+
+// ----------------------------------------------------------------- glu_columns
+template <typename T, int V>
+__global__ void __launch_bounds__(256) glu_columns_kernel(const T* __restrict__ p, long ld, int gate, int up, T* __restrict__ out, long rows, int I) {
+  const int per_row = I / V;
+  const long total = rows * per_row;
+  for (long i = blockIdx.x * static_cast<long>(blockDim.x) + threadIdx.x; i < total; i += static_cast<long>(gridDim.x) * blockDim.x) {
+    const long r = i / per_row;
+    const int c = static_cast<int>(i - r * per_row) * V;
+    const T* g = p + r * ld + gate + c;
+    const T* u = p + r * ld + up + c;
+    T* o = out + r * I + c;
+    if constexpr (V == 8) {        // bf16: 16-byte accesses
+      const uint4 a = *reinterpret_cast<const uint4*>(g), b = *reinterpret_cast<const uint4*>(u);
+      const uint32_t pa[4] = {a.x, a.y, a.z, a.w}, pb[4] = {b.x, b.y, b.z, b.w};
+      uint32_t po[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float2 x = unpack_bf16(pa[k]), y = unpack_bf16(pb[k]);
+        po[k] = pack_bf16(x.x / (1.f + __expf(-x.x)) * y.x, x.y / (1.f + __expf(-x.y)) * y.y);
+      }
+      *reinterpret_cast<uint4*>(o) = make_uint4(po[0], po[1], po[2], po[3]);
+    } else {
+#pragma unroll
+      for (int k = 0; k < V; ++k) {
+        const float x = to_f(g[k]);
+        o[k] = from_f<T>(x / (1.f + __expf(-x)) * to_f(u[k]));
+      }
+    }
+  }
+}
+
+torch::Tensor glu_columns(const torch::Tensor& p, int64_t gate, int64_t up, int64_t I) {
+  const auto st = p.scalar_type();
+  TORCH_CHECK(p.is_cuda() && p.dim() == 2 && p.stride(1) == 1 && (st == torch::kBFloat16 || st == torch::kFloat32), "projection [rows, N] bf16 or fp32");
+  TORCH_CHECK(I > 0 && gate >= 0 && up >= 0 && gate + I <= p.size(1) && up + I <= p.size(1), "gate / up columns outside the projection");
+  const long rows = p.size(0), ld = p.stride(0);
+  c10::cuda::CUDAGuard guard(p.device());
+  auto out = torch::empty({rows, I}, p.options());
+  if (rows == 0) return out;
+  auto stream = at::cuda::getCurrentCUDAStream();
+  const bool vec = st == torch::kBFloat16 && I % 8 == 0 && gate % 8 == 0 && up % 8 == 0 && ld % 8 == 0 && aligned16(p.data_ptr());
+  const long total = rows * (vec ? I / 8 : I);
+  const int blocks = static_cast<int>(std::min<long>((total + 255) / 256, num_sms() * 16L));
+  if (st == torch::kBFloat16) {
+    const bf16* in = reinterpret_cast<const bf16*>(p.data_ptr());
+    bf16* o = reinterpret_cast<bf16*>(out.data_ptr());
+    if (vec) glu_columns_kernel<bf16, 8><<<blocks, 256, 0, stream>>>(in, ld, gate, up, o, rows, I);
+    else glu_columns_kernel<bf16, 1><<<blocks, 256, 0, stream>>>(in, ld, gate, up, o, rows, I);
+  } else {
+    glu_columns_kernel<float, 1><<<blocks, 256, 0, stream>>>(p.data_ptr<float>(), ld, gate, up, out.data_ptr<float>(), rows, I);
+  }
+  count_launch();
+  TK_CUDA_CHECK(cudaGetLastError());
+  return out;
+}
+
+}  // namespace tk

@@ -140,6 +140,60 @@ def qk_norm_rope(q: torch.Tensor, k: torch.Tensor, q_weight: Optional[torch.Tens
     return apply_rope(q, cos, sin), apply_rope(k, cos, sin)
 
 
+# ------------------------------------------- short convolution in front of attention
+def short_conv(u: torch.Tensor, weight: Optional[torch.Tensor], positions: torch.Tensor, history: Optional[torch.Tensor] = None,
+               slots: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal depth-wise convolution without bias, in fp32: row t is ``Σ_j w[:, taps−1−j] · u_{t−j}`` over the rows of its own
+    sequence.  ``u [T, C]``, ``weight [C, taps]`` (None: ``u`` itself), ``positions [T]`` = place of every row in its sequence.
+    Packed rows (``history`` None) find their predecessors in front of them and start at position 0; with ``history
+    [slots, taps−1, C]`` every row stands alone and the row of position p lies in ``history[slots[t], p mod (taps−1)]``."""
+    x = u.float()
+    if weight is None:
+        return x
+    w = weight.float()
+    taps = w.shape[1]
+    y = x * w[:, taps - 1]
+    for j in range(1, taps):
+        if history is None:
+            prev = F.pad(x, (0, 0, j, 0))[:x.shape[0]]
+        else:
+            prev = history[slots.long(), (positions - j) % (taps - 1)].float()
+        y = y + torch.where((positions >= j)[:, None], prev * w[:, taps - 1 - j], torch.zeros((), device=x.device))
+    return y
+
+
+def query_temperature(positions: torch.Tensor, coef: float, every: int) -> torch.Tensor:
+    """``1 + coef · ln(⌊(p + 1) / every⌋ + 1)`` in fp32."""
+    return 1.0 + coef * torch.log(((positions + 1) // every + 1).float())
+
+
+def conv_heads(proj: torch.Tensor, weight: Optional[torch.Tensor], positions: torch.Tensor, hq: int, hkv: int, d: int, e: int, eps: float,
+               coef: float = 0.0, every: int = 0, v_first: Optional[torch.Tensor] = None, lam: Optional[torch.Tensor] = None,
+               history: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None):
+    """Leading ``[q | k | v]`` columns of a projection → ``(q [T,hq,d], k [T,hkv,d], v [T,hkv,e])``: short convolution, q and k
+    over their root mean square per head, query temperature, values mixed as ``(1 − λ) v + λ v_first``.  fp32 inside; the
+    results are rounded to the projection's dtype."""
+    T = proj.shape[0]
+    y = short_conv(proj[:, :hq * d + hkv * (d + e)], weight, positions, history, slots)
+    q, k, v = y[:, :hq * d].reshape(T, hq, d), y[:, hq * d:(hq + hkv) * d].reshape(T, hkv, d), y[:, (hq + hkv) * d:].reshape(T, hkv, e)
+    q = q * torch.rsqrt(q.pow(2).mean(-1, keepdim=True) + eps)
+    k = k * torch.rsqrt(k.pow(2).mean(-1, keepdim=True) + eps)
+    if every:
+        q = q * query_temperature(positions, coef, every)[:, None, None]
+    if v_first is not None:
+        v = v + lam.float() * (v_first.reshape(v.shape).float() - v)
+    return q.to(proj.dtype), k.to(proj.dtype), v.to(proj.dtype)
+
+
+def stream_rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype, adds=(), mult: float = 1.0):
+    """fp32 residual stream: ``x ← x + mult · Σ y_i ⊙ s_i`` over ``adds = [(y, s), …]``, then its RMS norm in ``out_dtype``.
+    Returns ``(norm, x)``."""
+    x = x.float()
+    if adds:
+        x = x + mult * sum(y.float() * sc.float() for y, sc in adds)
+    return (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * weight.float()).to(out_dtype), x
+
+
 # -------------------------------------------------------------------- swiglu
 def swiglu(gate_up: torch.Tensor) -> torch.Tensor:
     """``[T, 2I]`` laid out as ``[gate | up]`` → ``silu(gate) * up`` ``[T, I]``."""
@@ -207,19 +261,22 @@ def paged_attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
                            seq_lens: torch.Tensor, scale: Optional[float] = None, window: Optional[int] = None,
                            softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """One query token per sequence against a paged KV cache.
-    ``q [B,Hq,D]``; caches ``[num_blocks, block_size, Hkv, D]``; ``block_tables
+    ``q [B,Hq,D]``; caches ``[num_blocks, block_size, Hkv, D]`` (values may have a width of their own); ``block_tables
     [B, max_blocks]`` int; ``seq_lens [B]`` (including the current token)."""
     B, Hq, D = q.shape
     bs, Hkv = k_cache.shape[1], k_cache.shape[2]
     rep = Hq // Hkv
     scale = 1.0 / math.sqrt(D) if scale is None else scale
-    out = torch.empty_like(q)
+    E = v_cache.shape[-1]
+    out = q.new_zeros(B, Hq, E)
     for b in range(B):
         n = int(seq_lens[b])
+        if n == 0:
+            continue
         nb = (n + bs - 1) // bs
         blocks = block_tables[b, :nb].long()
         kk = k_cache[blocks].reshape(-1, Hkv, D)[:n].float().repeat_interleave(rep, 1)
-        vv = v_cache[blocks].reshape(-1, Hkv, D)[:n].float().repeat_interleave(rep, 1)
+        vv = v_cache[blocks].reshape(-1, Hkv, E)[:n].float().repeat_interleave(rep, 1)
         s = torch.einsum('hd,nhd->hn', q[b].float(), kk) * scale
         if softcap:
             s = torch.tanh(s / softcap) * softcap

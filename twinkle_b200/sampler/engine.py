@@ -23,18 +23,49 @@ from ..data_format import SampledSequence, SampleResponse, SamplingParams
 from ..models.config import DecoderConfig
 from ..models.decoder import DecoderModel, PackedBatch
 from ..models.layers import LoraBatch, lora_batch
+from ..models.parallel_layer import CacheView
 
 
 class PagedKVCache:
-    """``[layers][num_blocks, block_size, Hkv, D]`` K and V pools + a free list.  Block 0 is never handed
-    out so that an all-zero block table row is harmless."""
+    """Per layer K and V pools ``[num_blocks, block_size, Hkv, width]`` (key and value rows have the layer's own widths) + a
+    free list.  Layers with a short convolution in front of attention also have a history pool ``[num_slots, taps − 1,
+    channels]``; a sequence owns one slot of all of them.  Block 0 and slot 0 are never handed out so that the all-zero
+    rows that fill up a captured batch are harmless."""
 
-    def __init__(self, cfg: DecoderConfig, num_blocks: int, block_size: int, device, dtype):
-        self.cfg, self.block_size, self.num_blocks = cfg, block_size, num_blocks
-        shape = (cfg.num_hidden_layers, num_blocks, block_size, cfg.num_key_value_heads, cfg.head_dim)
-        self.k = torch.zeros(shape, device=device, dtype=dtype)
-        self.v = torch.zeros(shape, device=device, dtype=dtype)
-        self.free: List[int] = list(range(num_blocks - 1, 0, -1))
+    def __init__(self, cfg: DecoderConfig, num_blocks: int, block_size: int, device, dtype, num_slots: int = 0):
+        self.cfg, self.block_size, self.num_blocks, self.device, self.dtype = cfg, block_size, num_blocks, device, dtype
+        self.num_slots = num_slots if any(cfg.conv_layout()) else 0
+        self.build()
+
+    def build(self) -> None:
+        """(Re)create empty pools and free lists."""
+        mk = lambda *shape: torch.zeros(shape, device=self.device, dtype=self.dtype)  # noqa: E731
+        layout = self.cfg.kv_layout()
+        self.k = [mk(self.num_blocks, self.block_size, h, d) for h, d, _ in layout]
+        self.v = [mk(self.num_blocks, self.block_size, h, e) for h, _, e in layout]
+        conv = self.cfg.conv_layout() or [None] * len(layout)
+        self.conv = [mk(self.num_slots, *c) if c else None for c in conv]
+        self.free: List[int] = list(range(self.num_blocks - 1, 0, -1))
+        self.free_slots: List[int] = list(range(self.num_slots - 1, 0, -1))
+
+    def drop(self) -> None:
+        """Give the pools' memory back (``build`` makes new ones)."""
+        self.k = self.v = self.conv = None
+
+    @staticmethod
+    def block_bytes(cfg: DecoderConfig, block_size: int, elem: int) -> int:
+        return elem * block_size * sum(h * (d + e) for h, d, e in cfg.kv_layout())
+
+    def allocate_slot(self) -> int:
+        if not self.num_slots:
+            return 0
+        if not self.free_slots:
+            raise RuntimeError(f'convolution history exhausted: {self.num_slots - 1} sequences are live')
+        return self.free_slots.pop()
+
+    def release_slot(self, slot: int) -> None:
+        if slot:
+            self.free_slots.append(slot)
 
     def allocate(self, n: int) -> List[int]:
         if n > len(self.free):
@@ -53,8 +84,8 @@ class PagedKVCache:
         pos = torch.arange(start, start + n, device=k.device)
         blk = torch.as_tensor(blocks, device=k.device)[pos // self.block_size]
         off = pos % self.block_size
-        self.k[layer, blk, off] = k
-        self.v[layer, blk, off] = v
+        self.k[layer][blk, off] = k
+        self.v[layer][blk, off] = v
 
 
 @dataclass
@@ -67,6 +98,7 @@ class _Seq:
     lora_scale: float = 0.0
     lora_target: Any = None
     blocks: List[int] = field(default_factory=list)
+    state_slot: int = 0     # row of the convolution-history pools
     tokens: List[int] = field(default_factory=list)
     logprobs: List[float] = field(default_factory=list)
     topk: List[List[Tuple[int, float]]] = field(default_factory=list)
@@ -92,13 +124,13 @@ class NativeEngine:
         self.device = device or next(model.parameters()).device
         self.dtype = next(model.parameters()).dtype
         if num_blocks is None:
-            per_block = 2 * cfg.num_hidden_layers * block_size * cfg.num_key_value_heads * cfg.head_dim * (2 if self.dtype != torch.float32 else 4)
+            per_block = PagedKVCache.block_bytes(cfg, block_size, 2 if self.dtype != torch.float32 else 4)
             if self.device.type == 'cuda':
                 free, _ = torch.cuda.mem_get_info(self.device)
                 num_blocks = max(int(free * gpu_memory_utilization * 0.9 // per_block), 64)
             else:
                 num_blocks = 1024
-        self.cache = PagedKVCache(cfg, num_blocks, block_size, self.device, self.dtype)
+        self.cache = PagedKVCache(cfg, num_blocks, block_size, self.device, self.dtype, num_slots=max_batch + 1)
         self.max_batch = max_batch
         self.decode_text = decode
         self.capture_routing = False
@@ -115,6 +147,37 @@ class NativeEngine:
             lo += n
         return LoraBatch(segs, self.device, [s.lora_target for s in seqs])
 
+    # -------------------------------------------------- what a sequence holds
+    def admit(self, seqs: Sequence[_Seq]) -> None:
+        """Blocks for the prompt, the tokens it may generate and one more, and a convolution-history slot."""
+        for s in seqs:
+            s.blocks = self.cache.allocate(self.cache.blocks_for(len(s.prompt) + (s.params.max_tokens or 0) + 1))
+            s.state_slot = self.cache.allocate_slot()
+
+    def grow(self, seqs: Sequence[_Seq]) -> None:
+        """Extend the block list of sequences whose next token crosses a block boundary."""
+        for s in seqs:
+            need = self.cache.blocks_for(s.length + 1) - len(s.blocks)
+            if need > 0:
+                s.blocks += self.cache.allocate(need)
+
+    def release(self, seqs: Sequence[_Seq]) -> None:
+        for s in seqs:
+            self.cache.release(s.blocks)
+            self.cache.release_slot(s.state_slot)
+            s.blocks, s.state_slot, s.linear = [], 0, {}
+
+    def _prompt_view(self, seqs: Sequence[_Seq], lens: Sequence[int]) -> CacheView:
+        """Cache places of packed prompts: one row per token, built on the host and copied once."""
+        bs = self.cache.block_size
+        rows, slots, left = [], [], []
+        for s, n in zip(seqs, lens):
+            rows += [s.blocks[p // bs] * bs + p % bs for p in range(n)]
+            slots += [s.state_slot] * n
+            left += range(n - 1, -1, -1)
+        mk = lambda x, dt: torch.tensor(x, dtype=dt).to(self.device, non_blocking=True)  # noqa: E731
+        return CacheView(self.cache, mk(rows, torch.int64), mk(slots, torch.int32), mk(left, torch.int32))
+
     # ------------------------------------------------------------- prefill
     @torch.no_grad()
     def prefill(self, seqs: List[_Seq]) -> torch.Tensor:
@@ -124,8 +187,7 @@ class NativeEngine:
         ids = torch.tensor([t for s in seqs for t in s.prompt], dtype=torch.long, device=self.device)
         pos = torch.cat([torch.arange(n, device=self.device) for n in lens])
         cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=self.device)
-        for s, n in zip(seqs, lens):
-            s.blocks = self.cache.allocate(self.cache.blocks_for(n + (s.params.max_tokens or 0) + 1))
+        self.admit(seqs)
         bounds = cu.tolist()
 
         def sink(layer: int, k: torch.Tensor, v: torch.Tensor) -> None:
@@ -138,6 +200,8 @@ class NativeEngine:
 
         sink.linear_state = linear_state
         batch = PackedBatch(ids, pos, cu, max(lens))
+        if self.cfg.layer_specs is not None:
+            batch.cache = self._prompt_view(seqs, lens)
         if any(s.vision for s in seqs):  # prompts with images: patches, grids and (time, height, width) positions beside the row
             p3, pix, grids = [], [], []
             for s, n in zip(seqs, lens):
@@ -164,10 +228,16 @@ class NativeEngine:
 
     # --------------------------------------------------------------- decode
     def _decode_body(self, tokens, positions, table, seq_lens, lora: Optional[LoraBatch], seqs: Optional[List[_Seq]] = None,
-                     rope_positions: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     rope_positions: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None) -> torch.Tensor:
         """One decode token per row from device tensors only (what a CUDA graph captures). Linear-attention layers of
         hybrid stacks keep their state on the sequences (``seqs``) and always run eagerly."""
         cfg, B = self.cfg, tokens.shape[0]
+        if cfg.layer_specs is not None:      # one forward serves prompts and steps: the view tells the layers which it is
+            bs = self.cache.block_size
+            rows = table.gather(1, (positions // bs).unsqueeze(1)).squeeze(1).long() * bs + positions % bs
+            batch = PackedBatch(tokens, positions, None, 1, cache=CacheView(self.cache, rows, slots, torch.zeros_like(slots), table, seq_lens))
+            with lora_batch(lora):
+                return self.model.logits(self.model(batch)).float()
         # ``positions`` index the KV cache; the rotary position differs from it after a prompt with images
         cos, sin = ops.rope_tables(positions if rope_positions is None else rope_positions, cfg.rotary_dim, cfg.rope_theta, cfg.rope_scaling)
         local = None
@@ -190,7 +260,7 @@ class NativeEngine:
                     x = x + layer.feed_forward(n)
                     continue
                 q, k, v, gate = at.heads_from(h, *(local if (local is not None and getattr(at, 'local_rope', False)) else (cos, sin)))
-                self.cache.k[li, blk, off], self.cache.v[li, blk, off] = at.cache_entry(k, v)
+                self.cache.k[li][blk, off], self.cache.v[li][blk, off] = at.cache_entry(k, v)
                 o = ops.paged_attention_decode(q, self.cache.k[li], self.cache.v[li], table, seq_lens, at.scale,
                                                window=getattr(at, 'window', None), softcap=getattr(at, 'softcap', None), sinks=getattr(at, 'sinks', None))
                 n, x = layer.after_attention(x, at.project_out(o, gate))
@@ -208,16 +278,17 @@ class NativeEngine:
             return ent
         dev = self.device
         st = {'tokens': torch.zeros(B, dtype=torch.long, device=dev), 'positions': torch.zeros(B, dtype=torch.long, device=dev),
-              'table': torch.zeros(B, max_blocks, dtype=torch.int32, device=dev), 'seq_lens': torch.zeros(B, dtype=torch.int32, device=dev)}
+              'table': torch.zeros(B, max_blocks, dtype=torch.int32, device=dev), 'seq_lens': torch.zeros(B, dtype=torch.int32, device=dev),
+              'slots': torch.zeros(B, dtype=torch.int32, device=dev)}
         side = torch.cuda.Stream(device=dev)
         side.wait_stream(torch.cuda.current_stream(dev))
         with torch.cuda.stream(side):  # warm-up outside the capture: one-time kernel attribute set-up, allocator warm-up
             for _ in range(2):
-                self._decode_body(st['tokens'], st['positions'], st['table'], st['seq_lens'], None)
+                self._decode_body(st['tokens'], st['positions'], st['table'], st['seq_lens'], None, slots=st['slots'])
         torch.cuda.current_stream(dev).wait_stream(side)
         graph = torch.cuda.CUDAGraph()
         with torch.cuda.graph(graph):
-            st['logits'] = self._decode_body(st['tokens'], st['positions'], st['table'], st['seq_lens'], None)
+            st['logits'] = self._decode_body(st['tokens'], st['positions'], st['table'], st['seq_lens'], None, slots=st['slots'])
         st['graph'] = graph
         self._graphs[key] = st
         return st
@@ -251,6 +322,9 @@ class NativeEngine:
                     table[i, :len(s.blocks)] = torch.tensor(s.blocks, dtype=torch.int32)
                 lens = torch.zeros(Bb, dtype=torch.int32)
                 lens[:B] = torch.tensor([s.length for s in seqs], dtype=torch.int32)
+                slots = torch.zeros(Bb, dtype=torch.int32)
+                slots[:B] = torch.tensor([s.state_slot for s in seqs], dtype=torch.int32)
+                st['slots'].copy_(slots, non_blocking=True)
                 st['table'].copy_(table, non_blocking=True)
                 st['seq_lens'].copy_(lens, non_blocking=True)
                 st['tokens'].zero_()
@@ -266,7 +340,8 @@ class NativeEngine:
         self.model.set_record_routing(self.capture_routing)
         deltas = [s.rope_delta for s in seqs]
         rope_pos = positions + torch.tensor(deltas, device=self.device) if any(deltas) else None
-        logits = self._decode_body(last_tokens, positions, table, seq_lens, lora, seqs, rope_pos)
+        slots = torch.tensor([s.state_slot for s in seqs], dtype=torch.int32, device=self.device)
+        logits = self._decode_body(last_tokens, positions, table, seq_lens, lora, seqs, rope_pos, slots)
         if self.capture_routing:
             routed = self.model.collect_routed_experts()  # per layer [B, k]: the experts of the token just fed
             if routed is not None:
@@ -382,15 +457,11 @@ class NativeEngine:
                 if not nxt:
                     break
                 last = torch.tensor([s.tokens[-1] for s in nxt], device=self.device)
-                for s in nxt:  # grow the block list when a sequence crosses a block boundary
-                    need = self.cache.blocks_for(s.length + 1) - len(s.blocks)
-                    if need > 0:
-                        s.blocks += self.cache.allocate(need)
+                self.grow(nxt)
                 logits = self.decode_step(nxt, last)
                 live = nxt
+        self.release(seqs)
         for s in seqs:
-            self.cache.release(s.blocks)
-            s.blocks, s.linear = [], {}
             if not s.params.scoring_only:
                 responses[s.request].sequences.append(SampledSequence(stop_reason=s.stop_reason, tokens=s.tokens, logprobs=s.logprobs,
                                                                       topk_logprobs=s.topk or None, routed_experts=s.routed))

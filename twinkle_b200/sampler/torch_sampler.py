@@ -35,7 +35,7 @@ class TorchSampler(Sampler, CheckpointEngineMixin):
 
     def __init__(self, model_id: Optional[str] = None, config: Union[DecoderConfig, Dict[str, Any], None] = None,
                  device_mesh: DeviceMesh = None, engine_args: Optional[Dict[str, Any]] = None, seed: int = 42, device=None,
-                 max_loras: int = 4, max_r: int = 32, enable_lora: bool = True, **kwargs):
+                 max_loras: int = 4, max_r: int = 32, enable_lora: bool = True, dtype: Optional[str] = None, **kwargs):
         self.device_mesh = device_mesh
         self.device = torch.device(device) if device is not None else Platform.current_device()
         if self.device.type == 'cuda':
@@ -51,7 +51,8 @@ class TorchSampler(Sampler, CheckpointEngineMixin):
             model_id = HubOperation.download_model(model_id)
             self.config = DecoderConfig.from_pretrained(model_id)
         self.model_id = model_id
-        dtype = torch.bfloat16 if self.device.type == 'cuda' else torch.float32
+        # bf16 on a GPU and 32-bit on the CPU unless asked otherwise
+        dtype = getattr(torch, dtype) if dtype else (torch.bfloat16 if self.device.type == 'cuda' else torch.float32)
         load_dir = model_id if model_id and os.path.isdir(str(model_id)) else None
         self.model = build_model(self.config, device=self.device, dtype=dtype, seed=kwargs.get('weight_seed', 0), init=load_dir is None)
         if load_dir:
@@ -243,7 +244,8 @@ class TorchSampler(Sampler, CheckpointEngineMixin):
     @remote_function()
     def sleep(self, level: int = 1) -> None:
         """Level 1 drops the KV pools (they are rebuilt on wake-up); level 2 also moves weights to the host."""
-        self.engine.cache.k = self.engine.cache.v = None
+        self.engine.cache.drop()
+        self.engine._graphs.clear()      # captured steps hold the addresses of the pools (and of the weights)
         if level >= 2:
             self.model.to('cpu')
         if self.device.type == 'cuda':
@@ -255,11 +257,7 @@ class TorchSampler(Sampler, CheckpointEngineMixin):
         if not self._asleep:
             return
         self.model.to(self.device)
-        c = self.engine.cache
-        shape = (self.config.num_hidden_layers, c.num_blocks, c.block_size, self.config.num_key_value_heads, self.config.head_dim)
-        c.k = torch.zeros(shape, device=self.device, dtype=self.engine.dtype)
-        c.v = torch.zeros(shape, device=self.device, dtype=self.engine.dtype)
-        c.free = list(range(c.num_blocks - 1, 0, -1))
+        self.engine.cache.build()
         self._asleep = False
 
     @remote_function()
