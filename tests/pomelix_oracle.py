@@ -90,3 +90,61 @@ def forward(cfg, weights, tokens, dtype=torch.float64):
         x = x + mult * add
         trail.append(x)
     return rms_norm(x, W['final.norm'], eps) @ W['embed'].t(), trail
+
+
+# ---------------------------------------------------------------- models for the tests
+def spec(heads, kv_heads, dim, vdim, conv, scale, v_mix=False, temp=None, ff=0):
+    m = {'heads': heads, 'kv_heads': kv_heads, 'dim': dim, 'vdim': vdim, 'conv': conv, 'scale': scale, 'v_mix': v_mix}
+    if temp:
+        m['q_temp'] = {'coef': temp[0], 'every': temp[1]}
+    return {'type': 'attention', 'mixer': m, 'mlp': {'kind': 'dense', 'ff': ff} if ff else None}
+
+
+CONFIGS = {
+    # layers of unequal sizes; the first does not mix values, the second gives them and has no feed-forward block
+    'mixed': dict(vocab=120, width=96, norm={'eps': 1e-5}, residual_mult=0.6,
+                  layers=[spec(6, 2, 24, 40, 3, 0.31, False, (0.25, 7), 64), spec(4, 4, 32, 16, 4, 0.2, True, (0.4, 20)),
+                          spec(8, 4, 16, 16, 2, 0.35, True, (0.1, 5), 88)]),
+    # widths that are no whole vectors, more taps than the vector kernel takes, groups of three and five, no temperature
+    'odd': dict(vocab=97, width=52, norm={'eps': 1e-3}, residual_mult=0.9,
+                layers=[spec(3, 1, 20, 12, 5, 0.4, True, (0.3, 3), 36), spec(5, 1, 7, 12, 1, 0.5, True, None, 20), spec(10, 2, 9, 11, 3, 0.3, False, (0.2, 1))]),
+    # heads on both sides of 64, 128 and at 256
+    'wide': dict(vocab=64, width=72, norm={'eps': 1e-6}, residual_mult=1.0,
+                 layers=[spec(2, 1, 160, 256, 4, 0.08, False, (0.2, 11), 40), spec(4, 2, 128, 128, 4, 0.09, True, (0.2, 11), 48),
+                         spec(2, 2, 64, 128, 2, 0.12, True), spec(3, 1, 72, 64, 3, 0.12)]),
+}
+for _c in CONFIGS.values():
+    _c['architecture'] = 'Pomelix'
+
+
+def random_weights(cfg, seed=0):
+    """Weights under their checkpoint names, every value representable in bfloat16."""
+    g = torch.Generator().manual_seed(seed)
+    rnd = lambda *s: torch.randn(*s, generator=g)  # noqa: E731
+    mat = lambda o, i: rnd(o, i) / i**0.5  # noqa: E731
+    width = cfg['width']
+    W = {'embed': rnd(cfg['vocab'], width), 'final.norm': 1 + 0.2 * rnd(width)}
+    for i, layer in enumerate(cfg['layers']):
+        p, m = f'l{i}.', layer['mixer']
+        sizes = {'q': m['heads'] * m['dim'], 'k': m['kv_heads'] * m['dim'], 'v': m['kv_heads'] * m['vdim']}
+        W[p + 'norm1'], W[p + 'ls1'] = 1 + 0.2 * rnd(width), 1 + 0.3 * rnd(width)
+        for n, s in sizes.items():
+            W[p + f'mix.{n}'], W[p + f'mix.{n}.conv'] = mat(s, width), 0.6 * rnd(s, m['conv'])
+        W[p + 'mix.o'] = mat(width, m['heads'] * m['vdim'])
+        if m['v_mix']:
+            W[p + 'mix.vmix'] = torch.rand((), generator=g) * 0.6 + 0.2
+        if layer['mlp']:
+            ff = layer['mlp']['ff']
+            W[p + 'mlp.gate'], W[p + 'mlp.up'], W[p + 'mlp.down'], W[p + 'ls2'] = mat(ff, width), mat(ff, width), mat(width, ff), 1 + 0.3 * rnd(width)
+    return {n: t.to(torch.bfloat16) for n, t in W.items()}
+
+
+def write_checkpoint(path, cfg, weights):
+    import json
+    import os
+    from safetensors.torch import save_file
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, 'config.json'), 'w') as f:
+        json.dump(cfg, f)
+    save_file({n: t.contiguous() for n, t in weights.items()}, os.path.join(path, 'model.safetensors'))
+    return str(path)

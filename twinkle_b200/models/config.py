@@ -660,5 +660,8 @@ PRESETS: Dict[str, Dict[str, Any]] = {
 
 def preset(name: str, **overrides) -> DecoderConfig:
     kw = dict(PRESETS[name.lower()])
+    n = overrides.get('num_hidden_layers')
+    if kw.get('layer_specs') and n:      # listed layers: the list repeated or cut to the wanted depth
+        kw['layer_specs'] = (list(kw['layer_specs']) * -(-n // len(kw['layer_specs'])))[:n]
     kw.update(overrides)
     return DecoderConfig(**kw)

@@ -63,128 +63,179 @@ struct ConvHeads {
 };
 
 template <typename T>
-__device__ __forceinline__ float query_factor(const ConvHeads<T>& p, int64_t pos) {
-  return p.every > 0 ? 1.f + p.coef * log1pf(static_cast<float>((pos + 1) / p.every)) : 1.f;
+__device__ __forceinline__ float query_factor(const ConvHeads<T>& p, int pos) {
+  return p.every > 0 ? 1.f + p.coef * log1pf(static_cast<float>(static_cast<uint32_t>(pos + 1) / static_cast<uint32_t>(p.every))) : 1.f;
 }
 
-// One warp per (head, run of `run` rows); a lane owns NV groups of four channels of the head.  Rows of a run are read once
-// and slide through registers as history of the rows behind them (packed rows: the history of row t is t−1, t−2, … as far
-// as its position allows).  STEP: every row is a sequence of its own and takes its history from the pool.
+// Eight consecutive elements as they lie in memory.
+template <typename T> struct Raw8;
+template <> struct Raw8<bf16> {
+  uint4 u;
+  __device__ __forceinline__ void load(const bf16* p) { u = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void store(bf16* p) const { *reinterpret_cast<uint4*>(p) = u; }
+  __device__ __forceinline__ void zero() { u = make_uint4(0u, 0u, 0u, 0u); }
+  __device__ __forceinline__ void get(float (&x)[8]) const {
+    const float2 a = unpack_bf16(u.x), b = unpack_bf16(u.y), c = unpack_bf16(u.z), d = unpack_bf16(u.w);
+    x[0] = a.x; x[1] = a.y; x[2] = b.x; x[3] = b.y; x[4] = c.x; x[5] = c.y; x[6] = d.x; x[7] = d.y;
+  }
+  __device__ __forceinline__ void set(const float (&x)[8]) {
+    u = make_uint4(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]), pack_bf16(x[4], x[5]), pack_bf16(x[6], x[7]));
+  }
+};
+template <> struct Raw8<float> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) { a = reinterpret_cast<const float4*>(p)[0]; b = reinterpret_cast<const float4*>(p)[1]; }
+  __device__ __forceinline__ void store(float* p) const { reinterpret_cast<float4*>(p)[0] = a; reinterpret_cast<float4*>(p)[1] = b; }
+  __device__ __forceinline__ void zero() { a = b = make_float4(0.f, 0.f, 0.f, 0.f); }
+  __device__ __forceinline__ void get(float (&x)[8]) const { x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w; }
+  __device__ __forceinline__ void set(const float (&x)[8]) { a = make_float4(x[0], x[1], x[2], x[3]); b = make_float4(x[4], x[5], x[6], x[7]); }
+};
+
+// Half a warp per (head, run of `run` ≤ 32 rows); a lane owns NV groups of eight channels of the head.  Rows of a run are
+// read once and slide through registers as history of the rows behind them (packed rows: the history of row t is t−1, t−2, …
+// as far as its position allows).  STEP: every row is a sequence of its own and takes its history from the pool.  What
+// depends on the row only (position, temperature, places in the cache) is worked out once per run, one row per lane.
 template <typename T, int TAPS, int NV, bool STEP>
 __global__ void __launch_bounds__(128) conv_heads_kernel(const ConvHeads<T> p, int run) {
-  constexpr int H = TAPS - 1, AHEAD = 4;
-  const int lane = threadIdx.x & 31;
-  const int head = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (head >= p.hq + 2 * p.hkv) return;
+  constexpr int H = TAPS - 1, AHEAD = STEP ? 1 : (NV == 1 ? 4 : 2);
+  const int lane = threadIdx.x & 31, sub = lane & 15;
+  const int heads = p.hq + 2 * p.hkv;
+  int head = (blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5)) * 2 + (lane >> 4);
+  const bool live = head < heads;
+  head = min(head, heads - 1);                       // idle half-warps stay for the shuffles and store nothing
   const bool is_v = head >= p.hq + p.hkv, is_q = head < p.hq;
-  const int width = is_v ? p.e : p.d, padded = is_v ? p.ep : p.dp;
+  const int width = is_v ? p.e : p.d;
   const int c0 = is_v ? (p.hq + p.hkv) * p.d + (head - p.hq - p.hkv) * p.e : head * p.d;   // first column of the head
   const int C = (p.hq + p.hkv) * p.d + p.hkv * p.e;
   const int gh = is_q ? head : (is_v ? head - p.hq - p.hkv : head - p.hq);                  // head inside its own tensor
-  bool own[NV], out[NV];
-  float w[NV][TAPS][4];
+  const int own_heads = is_q ? p.hq : p.hkv;
+  const int t0 = blockIdx.x * run, t1 = min(t0 + run, p.rows);
+  // one row per lane
+  const int mine = min(t0 + lane, p.rows - 1);
+  const int m_pos = static_cast<int>(p.pos[mine]);
+  const float m_temp = query_factor(p, m_pos);
+  const int m_row = p.pool_row != nullptr ? static_cast<int>(p.pool_row[mine]) : -1;
+  int m_hist = -1, m_slot = 0;                       // row of the history pool this row is kept in (< 0: not kept)
+  if constexpr (H > 0) {
+    if (p.hist != nullptr) {
+      m_slot = p.slot[mine];
+      if (p.left[mine] < H) m_hist = m_slot * H + m_pos % H;
+    }
+  }
+  bool own[NV];
+  float w[NV][TAPS][8];
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
-    const int el = (i * 32 + lane) * 4;
-    own[i] = el < width;
-    out[i] = el < padded;
+    const int el = (i * 16 + sub) * 8;
+    own[i] = live && el < width;
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j)
+    for (int c = 0; c < 8; ++c)
 #pragma unroll
-      for (int c = 0; c < 4; ++c) w[i][j][c] = own[i] && p.w != nullptr ? to_f(p.w[static_cast<size_t>(c0 + el + c) * TAPS + j]) : 1.f;
+      for (int j = 0; j < TAPS; ++j) w[i][j][c] = own[i] && p.w != nullptr ? to_f(p.w[static_cast<size_t>(c0 + el + c) * TAPS + j]) : 1.f;
   }
-  const float lam = (is_v && p.v_first != nullptr) ? to_f(p.lam[0]) : 0.f;
-  const int t0 = blockIdx.x * run, t1 = min(t0 + run, p.rows);
-  float4 h[H > 0 ? H : 1][NV];         // h[j] = row t − 1 − j
+  const bool mixes = is_v && p.v_first != nullptr;
+  const float lam = mixes ? to_f(p.lam[0]) : 0.f, inv_width = 1.f / width;
+  const T* src = p.proj + c0 + sub * 8;              // + t · ld
+  T* dst = is_q ? p.q : (is_v ? p.v : p.k);          // + t · own_heads · width (keys of single steps have no copy of their own)
+  const size_t off = static_cast<size_t>(gh) * width + sub * 8, pitch = static_cast<size_t>(own_heads) * width;
+  T* pool = is_v ? p.v_pool : p.k_pool;
+  float h[H > 0 ? H : 1][NV][8];                     // h[j] = row t − 1 − j
   if constexpr (!STEP) {
 #pragma unroll
     for (int j = 0; j < H; ++j)
 #pragma unroll
-      for (int i = 0; i < NV; ++i)
-        h[j][i] = (own[i] && t0 - 1 - j >= 0) ? load4(p.proj + static_cast<size_t>(t0 - 1 - j) * p.ld + c0 + (i * 32 + lane) * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int i = 0; i < NV; ++i) {
+        Raw8<T> r;
+        r.zero();
+        if (own[i] && t0 - 1 - j >= 0) r.load(src + static_cast<size_t>(t0 - 1 - j) * p.ld + i * 128);
+        r.get(h[j][i]);
+      }
   }
   for (int tb = t0; tb < t1; tb += AHEAD) {
-    float4 cur[AHEAD][NV];
-    int64_t ps[AHEAD];
+    Raw8<T> cur[AHEAD][NV], first[AHEAD][NV];
 #pragma unroll
     for (int u = 0; u < AHEAD; ++u) {
       const int t = min(tb + u, t1 - 1);
-      ps[u] = p.pos[t];
 #pragma unroll
-      for (int i = 0; i < NV; ++i)
-        cur[u][i] = own[i] ? load4(p.proj + static_cast<size_t>(t) * p.ld + c0 + (i * 32 + lane) * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int i = 0; i < NV; ++i) {
+        cur[u][i].zero();
+        first[u][i].zero();
+        if (own[i]) {
+          cur[u][i].load(src + static_cast<size_t>(t) * p.ld + i * 128);
+          if (mixes) first[u][i].load(p.v_first + static_cast<size_t>(t) * pitch + off + i * 128);
+        }
+      }
     }
 #pragma unroll
     for (int u = 0; u < AHEAD; ++u) {
       const int t = tb + u;
       if (t >= t1) break;
-      const int64_t pos = ps[u];
-      float4 y[NV];
+      const int pos = __shfl_sync(0xffffffffu, m_pos, t - t0), row = __shfl_sync(0xffffffffu, m_row, t - t0);
+      const float temp = __shfl_sync(0xffffffffu, m_temp, t - t0);
+      const int kept = H > 0 ? __shfl_sync(0xffffffffu, m_hist, t - t0) : -1;
       if constexpr (STEP && H > 0) {
+        const int slot = __shfl_sync(0xffffffffu, m_slot, t - t0);
+        Raw8<T> r[H][NV];
 #pragma unroll
         for (int j = 0; j < H; ++j)
 #pragma unroll
-          for (int i = 0; i < NV; ++i)
-            h[j][i] = (own[i] && j + 1 <= pos) ? load4(p.hist + (static_cast<size_t>(p.slot[t]) * H + (pos - 1 - j) % H) * C + c0 + (i * 32 + lane) * 4)
-                                               : make_float4(0.f, 0.f, 0.f, 0.f);
+          for (int i = 0; i < NV; ++i) {
+            r[j][i].zero();
+            if (own[i] && j + 1 <= pos) r[j][i].load(p.hist + (static_cast<size_t>(slot) * H + (pos - 1 - j) % H) * C + c0 + sub * 8 + i * 128);
+          }
+#pragma unroll
+        for (int j = 0; j < H; ++j)
+#pragma unroll
+          for (int i = 0; i < NV; ++i) r[j][i].get(h[j][i]);
       }
-      float ss = 0.f;
+      float x[NV][8], y[NV][8], ss = 0.f;
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
-        const float4 a = cur[u][i];
-        y[i] = make_float4(w[i][H][0] * a.x, w[i][H][1] * a.y, w[i][H][2] * a.z, w[i][H][3] * a.w);
+        cur[u][i].get(x[i]);
+#pragma unroll
+        for (int c = 0; c < 8; ++c) y[i][c] = w[i][H][c] * x[i][c];
 #pragma unroll
         for (int j = 0; j < H; ++j) {
           if (j + 1 <= pos) {
-            const float4 b = h[j][i];
-            y[i].x += w[i][H - 1 - j][0] * b.x; y[i].y += w[i][H - 1 - j][1] * b.y;
-            y[i].z += w[i][H - 1 - j][2] * b.z; y[i].w += w[i][H - 1 - j][3] * b.w;
+#pragma unroll
+            for (int c = 0; c < 8; ++c) y[i][c] += w[i][H - 1 - j][c] * h[j][i][c];
           }
         }
-        if (!own[i]) y[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-        ss += y[i].x * y[i].x + y[i].y * y[i].y + y[i].z * y[i].z + y[i].w * y[i].w;
-      }
-      if (!is_v) {
-        ss = warp_sum(ss);
-        float f = rsqrtf(ss / width + p.eps);
-        if (is_q) f *= query_factor(p, pos);
 #pragma unroll
-        for (int i = 0; i < NV; ++i) { y[i].x *= f; y[i].y *= f; y[i].z *= f; y[i].w *= f; }
+        for (int c = 0; c < 8; ++c) ss += own[i] ? y[i][c] * y[i][c] : 0.f;
       }
-      const int64_t row = p.pool_row != nullptr ? p.pool_row[t] : -1;
-      const bool keep = H > 0 && p.hist != nullptr && p.left[t] < H;
+#pragma unroll
+      for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);      // inside the half-warp
+      const float f = is_v ? 1.f : rsqrtf(ss * inv_width + p.eps) * (is_q ? temp : 1.f);
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
-        const int el = (i * 32 + lane) * 4;
-        if (out[i]) {
-          if (is_q) {
-            store4(p.q + (static_cast<size_t>(t) * p.hq + gh) * p.dp + el, y[i]);
-          } else if (!is_v) {
-            if (p.k != nullptr) store4(p.k + (static_cast<size_t>(t) * p.hkv + gh) * p.dp + el, y[i]);
-            if (row >= 0) store4(p.k_pool + (static_cast<size_t>(row) * p.hkv + gh) * p.dp + el, y[i]);
+        if (own[i]) {
+          if (mixes) {
+            float v1[8];
+            first[u][i].get(v1);
+#pragma unroll
+            for (int c = 0; c < 8; ++c) y[i][c] += lam * (v1[c] - y[i][c]);
           } else {
-            if (p.v_first != nullptr) {
-              const float4 f = load4(p.v_first + (static_cast<size_t>(t) * p.hkv + gh) * p.ep + el);
-              y[i].x += lam * (f.x - y[i].x); y[i].y += lam * (f.y - y[i].y); y[i].z += lam * (f.z - y[i].z); y[i].w += lam * (f.w - y[i].w);
-            }
-            store4(p.v + (static_cast<size_t>(t) * p.hkv + gh) * p.ep + el, y[i]);
-            if (row >= 0) store4(p.v_pool + (static_cast<size_t>(row) * p.hkv + gh) * p.ep + el, y[i]);
+#pragma unroll
+            for (int c = 0; c < 8; ++c) y[i][c] *= f;
           }
-        }
-        // the newest rows of a sequence are what its next step looks back at (same thread read this place above)
-        if constexpr (H > 0) {
-          if (keep && own[i]) store4(p.hist + (static_cast<size_t>(p.slot[t]) * H + pos % H) * C + c0 + el, cur[u][i]);
+          Raw8<T> r;
+          r.set(y[i]);
+          if (dst != nullptr) r.store(dst + static_cast<size_t>(t) * pitch + off + i * 128);
+          if (!is_q && row >= 0) r.store(pool + static_cast<size_t>(row) * pitch + off + i * 128);
+          // the newest rows of a sequence are what its next step looks back at (the same thread read this place above)
+          if (kept >= 0) cur[u][i].store(p.hist + static_cast<size_t>(kept) * C + c0 + sub * 8 + i * 128);
         }
       }
-      if constexpr (!STEP) {
+      if constexpr (!STEP && H > 0) {
 #pragma unroll
-        for (int j = H - 1; j > 0; --j)
+        for (int i = 0; i < NV; ++i)
 #pragma unroll
-          for (int i = 0; i < NV; ++i) h[j][i] = h[j - 1][i];
-        if constexpr (H > 0) {
+          for (int c = 0; c < 8; ++c) {
 #pragma unroll
-          for (int i = 0; i < NV; ++i) h[0][i] = cur[u][i];
-        }
+            for (int j = H - 1; j > 0; --j) h[j][i][c] = h[j - 1][i][c];
+            h[0][i][c] = x[i][c];
+          }
       }
     }
   }
@@ -201,7 +252,7 @@ __global__ void __launch_bounds__(128) conv_heads_plain_kernel(const ConvHeads<T
   const int c0 = is_v ? (p.hq + p.hkv) * p.d + (head - p.hq - p.hkv) * p.e : head * p.d;
   const int C = (p.hq + p.hkv) * p.d + p.hkv * p.e;
   const int gh = is_q ? head : (is_v ? head - p.hq - p.hkv : head - p.hq);
-  const int64_t pos = p.pos[t];
+  const int pos = static_cast<int>(p.pos[t]);
   const int64_t row = p.pool_row != nullptr ? p.pool_row[t] : -1;
   const bool keep = H > 0 && p.hist != nullptr && p.left[t] < H;
   float ss = 0.f;
@@ -246,9 +297,9 @@ template <typename T, int TAPS>
 static void launch_conv_heads(const ConvHeads<T>& p, bool step, bool wide, cudaStream_t stream) {
   const int heads = p.hq + 2 * p.hkv;
   // enough warps to fill the device first, then longer runs (fewer history rows read twice)
-  const long target = 16L * num_sms() * 4;
-  int run = step ? 1 : static_cast<int>(std::min<long>(32, std::max<long>(4, static_cast<long>(p.rows) * heads / target)));
-  const dim3 grid((p.rows + run - 1) / run, (heads + 3) / 4);
+  const long target = 16L * num_sms();               // warps; two heads each
+  int run = step ? 1 : static_cast<int>(std::min<long>(32, std::max<long>(4, static_cast<long>(p.rows) * heads / 2 / target)));
+  const dim3 grid((p.rows + run - 1) / run, (heads + 7) / 8);
   if (step) {
     if (wide) conv_heads_kernel<T, TAPS, 2, true><<<grid, 128, 0, stream>>>(p, run);
     else conv_heads_kernel<T, TAPS, 1, true><<<grid, 128, 0, stream>>>(p, run);
@@ -265,8 +316,7 @@ template <typename T>
 static void conv_heads_t(ConvHeads<T>& p, bool step) {
   auto stream = at::cuda::getCurrentCUDAStream();
   const int wmax = std::max(p.dp, p.ep);
-  const bool vec = p.d % 4 == 0 && p.e % 4 == 0 && p.ld % 4 == 0 && wmax <= 256 && p.taps <= 4 && aligned16(p.proj) &&
-                   (p.hist == nullptr || ((p.hq + p.hkv) * p.d + p.hkv * p.e) % 4 == 0);
+  const bool vec = p.d % 8 == 0 && p.e % 8 == 0 && p.ld % 8 == 0 && wmax <= 256 && p.taps <= 4 && aligned16(p.proj);
   if (vec) {
     switch (p.taps) {
       case 4: launch_conv_heads<T, 4>(p, step, wmax > 128, stream); break;
@@ -317,6 +367,8 @@ std::vector<torch::Tensor> conv_heads(const torch::Tensor& proj, const OptT& wei
   auto q = torch::empty({rows, hq, dp}, proj.options());
   auto k = want_k ? torch::empty({rows, hkv, dp}, proj.options()) : torch::Tensor();
   auto v = torch::empty({rows, hkv, ep}, proj.options());
+  TORCH_CHECK(every >= 0 && every < (int64_t(1) << 31) && (!has(pool_row) || k_pool->numel() / (hkv * dp) < (int64_t(1) << 31)) &&
+                  (!has(hist) || hist->size(0) * std::max(taps - 1, 1) < (int64_t(1) << 31)), "32-bit row numbers");
   if (rows > 0) {
     auto fill = [&](auto tag) {
       using T = decltype(tag);

@@ -87,6 +87,43 @@ def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
         q, k, v, rstd = E.qk_norm_rope_fwd(qkv, qw, kw, cos, sin, hq, hkv, 128, 1e-6)
         gq, gk, gv = torch.randn_like(q), torch.randn_like(k), torch.randn_like(v)
         return (lambda: E.qk_norm_rope_bwd(gq, gk, gv, qkv, qw, kw, cos, sin, rstd, hq, hkv, 128)), 0.0, 1.5 * byts
+    if op in ('conv_heads', 'conv_heads_step'):
+        # the step between projection and attention of a listed-layer stack: [q | k | v] in front of [gate | up] columns; prompts of
+        # --seq tokens written into a paged cache, or one token of --batch sequences
+        hq, hkv, d, taps, bs = a.heads, a.kv_heads, a.width, 4, 16
+        step = op.endswith('step')
+        T = a.batch if step else a.tokens
+        C = (hq + 2 * hkv) * d
+        proj = torch.randn(T, C + 6 * a.hidden, device=dev, dtype=bf)
+        w, lam, vf = torch.randn(C, taps, device=dev, dtype=bf), torch.rand(1, device=dev, dtype=bf), torch.randn(T, hkv, d, device=dev, dtype=bf)
+        pos = torch.full((T, ), a.seq - 1, device=dev) if step else torch.arange(T, device=dev) % a.seq
+        kp, vp = (torch.zeros(T * bs if step else T, hkv, d, device=dev, dtype=bf) for _ in range(2))
+        rows = torch.arange(T, device=dev) * (bs if step else 1)
+        hist = torch.zeros(T + 1, taps - 1, C, device=dev, dtype=bf)
+        slot = (torch.arange(T, device=dev, dtype=torch.int32) if step else (torch.arange(T, device=dev) // a.seq).int()) + 1
+        left = torch.zeros(T, device=dev, dtype=torch.int32) if step else (a.seq - 1 - pos).int()
+        # projection in; q, values (and keys of prompts) out, both pools; mixed-in values; history (all of it read and one row
+        # of it written by a step, negligible for prompts)
+        byts = 2.0 * T * d * (hq + 2 * hkv + hq + hkv + (0 if step else hkv) + 2 * hkv + hkv) + (2.0 * T * C * taps if step else 0.0)
+        return (lambda: E.conv_heads(proj, w, pos, hq, hkv, d, d, 1e-5, 0.1, 4096, vf, lam, step, hist, slot, left, rows, kp, vp, not step)), 0.0, byts
+    if op in ('stream_norm', 'add_rmsnorm'):
+        w, y = torch.ones(a.hidden, device=dev, dtype=bf), torch.randn(a.tokens, a.hidden, device=dev, dtype=bf)
+        if op == 'add_rmsnorm':
+            r = torch.randn_like(y)
+            return (lambda: E.rmsnorm_fwd(y, w, 1e-6, 0.0, r)), 0.0, 8.0 * a.tokens * a.hidden
+        x, y2 = torch.zeros(a.tokens, a.hidden, device=dev), torch.randn_like(y)
+        return (lambda: E.stream_rmsnorm(x, w, 1e-6, y, w, y2, w, 0.5)), 0.0, 14.0 * a.tokens * a.hidden
+    if op == 'glu_columns':
+        p = torch.randn(a.tokens, 6144 + 2 * a.hidden, device=dev, dtype=bf)
+        return (lambda: E.glu_columns(p, 6144, 6144 + a.hidden, a.hidden)), 0.0, 6.0 * a.tokens * a.hidden
+    if op in ('attn_packed', 'attn_packed32'):
+        # prefill attention at any head width (--width): the tensor-core kernel up to 128 in bf16, fp32 arithmetic beyond / in 32-bit
+        T, d, dt = a.tokens, a.width, bf if op == 'attn_packed' else torch.float32
+        n_seq = max(T // a.seq, 1)
+        cu = torch.arange(0, n_seq + 1, device=dev, dtype=torch.int32) * a.seq
+        q, k, v = (torch.randn(T, h, d, device=dev, dtype=dt) for h in (a.heads, a.kv_heads, a.kv_heads))
+        return ((lambda: ops.attention_packed(q, k, v, cu, a.seq, d**-0.5)), 4.0 * n_seq * a.seq * a.seq * a.heads * d / 2,
+                float(q.element_size()) * T * d * (2 * a.heads + 2 * a.kv_heads))
     if op == 'rmsnorm':
         x, w = torch.randn(a.tokens, a.hidden, device=dev, dtype=bf), torch.ones(a.hidden, device=dev, dtype=bf)
 
@@ -139,12 +176,12 @@ def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
     if op == 'paged_decode':
         B, bs, ctx = a.batch, 16, a.seq
         nb = B * ((ctx + bs - 1) // bs)
-        kc = torch.randn(nb, bs, a.kv_heads, 128, device=dev, dtype=bf)
+        kc = torch.randn(nb, bs, a.kv_heads, a.width, device=dev, dtype=bf)
         vc = torch.randn_like(kc)
         tables = torch.arange(nb, device=dev, dtype=torch.int32).view(B, -1)
         lens = torch.full((B, ), ctx, device=dev, dtype=torch.int32)
-        q = torch.randn(B, a.heads, 128, device=dev, dtype=bf)
-        return (lambda: ops.paged_attention_decode(q, kc, vc, tables, lens)), 0.0, 2.0 * 2 * B * ctx * a.kv_heads * 128
+        q = torch.randn(B, a.heads, a.width, device=dev, dtype=bf)
+        return (lambda: ops.paged_attention_decode(q, kc, vc, tables, lens)), 0.0, 2.0 * 2 * B * ctx * a.kv_heads * a.width
     if op == 'sample':
         lg = torch.randn(a.batch, a.vocab, device=dev)
         seeds = torch.arange(a.batch, device=dev, dtype=torch.int64)
@@ -219,6 +256,7 @@ def main() -> None:
     ap.add_argument('--seq', type=int, default=8192)
     ap.add_argument('--heads', type=int, default=32)
     ap.add_argument('--kv-heads', type=int, default=8)
+    ap.add_argument('--width', type=int, default=128, help='head width')
     ap.add_argument('--hidden', type=int, default=4096)
     ap.add_argument('--vocab', type=int, default=151936)
     ap.add_argument('--batch', type=int, default=256)

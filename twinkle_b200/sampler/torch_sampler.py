@@ -39,6 +39,8 @@ class TorchSampler(Sampler, CheckpointEngineMixin):
         self.device_mesh = device_mesh
         self.device = torch.device(device) if device is not None else Platform.current_device()
         if self.device.type == 'cuda':
+            if self.device.index is None:
+                self.device = torch.device('cuda', torch.cuda.current_device())
             torch.cuda.set_device(self.device)
         if isinstance(config, DecoderConfig):
             self.config = config
