@@ -96,8 +96,8 @@ template <> struct Raw8<float> {
 // as far as its position allows).  STEP: every row is a sequence of its own and takes its history from the pool.  What
 // depends on the row only (position, temperature, places in the cache) is worked out once per run, one row per lane.
 template <typename T, int TAPS, int NV, bool STEP>
-__global__ void __launch_bounds__(128) conv_heads_kernel(const ConvHeads<T> p, int run) {
-  constexpr int H = TAPS - 1, AHEAD = STEP ? 1 : (NV == 1 ? 4 : 2);
+__global__ void __launch_bounds__(128, (NV == 1 && sizeof(T) == 2) ? 4 : 1) conv_heads_kernel(const ConvHeads<T> p, int run) {
+  constexpr int H = TAPS - 1, AHEAD = STEP ? 1 : (NV == 1 ? 3 : 2);
   const int lane = threadIdx.x & 31, sub = lane & 15;
   const int heads = p.hq + 2 * p.hkv;
   int head = (blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5)) * 2 + (lane >> 4);
@@ -128,10 +128,18 @@ __global__ void __launch_bounds__(128) conv_heads_kernel(const ConvHeads<T> p, i
   for (int i = 0; i < NV; ++i) {
     const int el = (i * 16 + sub) * 8;
     own[i] = live && el < width;
+    // the taps of eight channels are 8 · TAPS consecutive elements
 #pragma unroll
-    for (int c = 0; c < 8; ++c)
+    for (int n = 0; n < TAPS; ++n) {
+      float v[8] = {1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f, 1.f};
+      if (own[i] && p.w != nullptr) {
+        Raw8<T> r;
+        r.load(p.w + static_cast<size_t>(c0 + el) * TAPS + n * 8);
+        r.get(v);
+      }
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) w[i][j][c] = own[i] && p.w != nullptr ? to_f(p.w[static_cast<size_t>(c0 + el + c) * TAPS + j]) : 1.f;
+      for (int c = 0; c < 8; ++c) w[i][(n * 8 + c) % TAPS][(n * 8 + c) / TAPS] = v[c];
+    }
   }
   const bool mixes = is_v && p.v_first != nullptr;
   const float lam = mixes ? to_f(p.lam[0]) : 0.f, inv_width = 1.f / width;
@@ -139,16 +147,14 @@ __global__ void __launch_bounds__(128) conv_heads_kernel(const ConvHeads<T> p, i
   T* dst = is_q ? p.q : (is_v ? p.v : p.k);          // + t · own_heads · width (keys of single steps have no copy of their own)
   const size_t off = static_cast<size_t>(gh) * width + sub * 8, pitch = static_cast<size_t>(own_heads) * width;
   T* pool = is_v ? p.v_pool : p.k_pool;
-  float h[H > 0 ? H : 1][NV][8];                     // h[j] = row t − 1 − j
+  Raw8<T> h[H > 0 ? H : 1][NV];                      // h[j] = row t − 1 − j, kept as it lies in memory (half the registers)
   if constexpr (!STEP) {
 #pragma unroll
     for (int j = 0; j < H; ++j)
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
-        Raw8<T> r;
-        r.zero();
-        if (own[i] && t0 - 1 - j >= 0) r.load(src + static_cast<size_t>(t0 - 1 - j) * p.ld + i * 128);
-        r.get(h[j][i]);
+        h[j][i].zero();
+        if (own[i] && t0 - 1 - j >= 0) h[j][i].load(src + static_cast<size_t>(t0 - 1 - j) * p.ld + i * 128);
       }
   }
   for (int tb = t0; tb < t1; tb += AHEAD) {
@@ -175,30 +181,27 @@ __global__ void __launch_bounds__(128) conv_heads_kernel(const ConvHeads<T> p, i
       const int kept = H > 0 ? __shfl_sync(0xffffffffu, m_hist, t - t0) : -1;
       if constexpr (STEP && H > 0) {
         const int slot = __shfl_sync(0xffffffffu, m_slot, t - t0);
-        Raw8<T> r[H][NV];
 #pragma unroll
         for (int j = 0; j < H; ++j)
 #pragma unroll
           for (int i = 0; i < NV; ++i) {
-            r[j][i].zero();
-            if (own[i] && j + 1 <= pos) r[j][i].load(p.hist + (static_cast<size_t>(slot) * H + (pos - 1 - j) % H) * C + c0 + sub * 8 + i * 128);
+            h[j][i].zero();
+            if (own[i] && j + 1 <= pos) h[j][i].load(p.hist + (static_cast<size_t>(slot) * H + (pos - 1 - j) % H) * C + c0 + sub * 8 + i * 128);
           }
-#pragma unroll
-        for (int j = 0; j < H; ++j)
-#pragma unroll
-          for (int i = 0; i < NV; ++i) r[j][i].get(h[j][i]);
       }
-      float x[NV][8], y[NV][8], ss = 0.f;
+      float y[NV][8], ss = 0.f;
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
-        cur[u][i].get(x[i]);
+        float x[8];
+        cur[u][i].get(x);
 #pragma unroll
-        for (int c = 0; c < 8; ++c) y[i][c] = w[i][H][c] * x[i][c];
+        for (int c = 0; c < 8; ++c) y[i][c] = w[i][H][c] * x[c];
 #pragma unroll
         for (int j = 0; j < H; ++j) {
           if (j + 1 <= pos) {
+            h[j][i].get(x);
 #pragma unroll
-            for (int c = 0; c < 8; ++c) y[i][c] += w[i][H - 1 - j][c] * h[j][i][c];
+            for (int c = 0; c < 8; ++c) y[i][c] += w[i][H - 1 - j][c] * x[c];
           }
         }
 #pragma unroll
@@ -229,13 +232,11 @@ __global__ void __launch_bounds__(128) conv_heads_kernel(const ConvHeads<T> p, i
       }
       if constexpr (!STEP && H > 0) {
 #pragma unroll
-        for (int i = 0; i < NV; ++i)
+        for (int i = 0; i < NV; ++i) {
 #pragma unroll
-          for (int c = 0; c < 8; ++c) {
-#pragma unroll
-            for (int j = H - 1; j > 0; --j) h[j][i][c] = h[j - 1][i][c];
-            h[0][i][c] = x[i][c];
-          }
+          for (int j = H - 1; j > 0; --j) h[j][i] = h[j - 1][i];
+          h[0][i] = cur[u][i];
+        }
       }
     }
   }
@@ -316,7 +317,7 @@ template <typename T>
 static void conv_heads_t(ConvHeads<T>& p, bool step) {
   auto stream = at::cuda::getCurrentCUDAStream();
   const int wmax = std::max(p.dp, p.ep);
-  const bool vec = p.d % 8 == 0 && p.e % 8 == 0 && p.ld % 8 == 0 && wmax <= 256 && p.taps <= 4 && aligned16(p.proj);
+  const bool vec = p.d % 8 == 0 && p.e % 8 == 0 && p.ld % 8 == 0 && wmax <= 256 && p.taps <= 4 && aligned16(p.proj) && aligned16(p.w);
   if (vec) {
     switch (p.taps) {
       case 4: launch_conv_heads<T, 4>(p, step, wmax > 128, stream); break;
