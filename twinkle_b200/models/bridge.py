@@ -158,36 +158,67 @@ def _nested(cfg: DecoderConfig) -> bool:
     return bool(cfg.vision) or cfg.model_type.startswith('qwen3_5')
 
 
-# Pomelix checkpoints: ``l<i>.mix.*`` / ``l<i>.mlp.*`` with one tensor per projection; here a layer's projections of the
-# same input are one matrix and its convolution filters one tensor
-_LISTED = {'input_layernorm.weight': ('norm1', ), 'conv_weight': ('mix.q.conv', 'mix.k.conv', 'mix.v.conv'), 'v_lambda': ('mix.vmix', ),
-           'o_proj.weight': ('mix.o', ), 'down_proj.weight': ('mlp.down', ), 'mixer_scale': ('ls1', ), 'mlp_scale': ('ls2', )}
+# Checkpoints with listed layers: ``l<i>.mix.*`` / ``l<i>.mlp.*`` with one tensor per projection; here a layer's projections of the
+# same input are one matrix, a layer's convolution filters one tensor and its experts one tensor per projection
+_LISTED = {'input_layernorm.weight': 'norm1', 'v_lambda': 'mix.vmix', 'o_proj.weight': 'mix.o', 'down_proj.weight': 'mlp.down', 'mixer_scale': 'ls1',
+           'mlp_scale': 'ls2', 'post_mixer_layernorm.weight': 'norm1b', 'pre_mlp_layernorm.weight': 'norm2', 'post_mlp_layernorm.weight': 'norm2b',
+           'mixer_gate_bias': 'rg1.b', 'mlp_gate_bias': 'rg2.b', 'mlp_gate.weight': 'rg2', 'mixer.q_norm.weight': 'mix.dq.norm',
+           'mixer.kv_norm.weight': 'mix.dkv.norm', 'mixer.q_up.weight': 'mix.uq', 'mixer.sinks': 'mix.sink', 'mixer.o_proj.weight': 'mix.o',
+           'mixer.f_bias': 'mix.f.b', 'mixer.lower': 'mix.lower', 'mixer.out_norm.weight': 'mix.norm', 'mlp.down_proj.weight': 'mlp.down',
+           'mlp.gate.weight': 'mlp.router', 'mlp.gate.bias': 'mlp.router.b'}
+_LISTED_PARTS = {'res_gate': 'rg1', 'q_proj': 'mix.q', 'k_proj': 'mix.k', 'v_proj': 'mix.v', 'f_proj': 'mix.f', 'dq_proj': 'mix.dq', 'dkv_proj': 'mix.dkv',
+                 'head_gate': 'mix.g', 'gate_proj': 'mlp.gate', 'up_proj': 'mlp.up'}
+
+
+def _listed_parts(rest: str, sp, width: int) -> List[Tuple[str, int]]:
+    """(checkpoint tensor, rows) of an internal tensor that joins several, in concatenation order; [] when it does not."""
+    if rest == 'conv_weight':
+        return [(f'mix.{p}.conv', n) for p, n in zip('qkv', sp.qkv_sizes)]
+    if rest == 'in_proj.weight':
+        parts = list(zip(('q_proj', 'k_proj', 'v_proj'), sp.qkv_sizes)) + ([('gate_proj', sp.ff), ('up_proj', sp.ff)] if sp.ff else [])
+    elif rest == 'mixer.in_proj.weight':
+        parts = [('res_gate', width)] + sp.mixer.in_parts()
+    elif rest == 'mlp.in_proj.weight':
+        return [('rg2', width), ('mlp.gate', sp.mlp.ff), ('mlp.up', sp.mlp.ff)]
+    elif rest == 'mixer.kv_up':
+        return [('mix.uk', sp.mixer.heads * sp.mixer.dim), ('mix.uv', sp.mixer.heads * sp.mixer.vdim)]
+    elif rest in ('mlp.experts.up_proj', 'mlp.experts.down_proj'):
+        which, rows = ('up', sp.mlp.ff) if rest.endswith('up_proj') else ('down', width)
+        return [(f'mlp.e{e}.{which}', rows) for e in range(sp.mlp.experts)]
+    else:
+        return []
+    return [(_LISTED_PARTS[n], rows) for n, rows in parts]
 
 
 def _listed_names(name: str, cfg: DecoderConfig) -> List[str]:
     """Checkpoint tensors that make up one internal tensor of a stack with listed layers, in concatenation order."""
-    if name == 'embed_tokens.weight':
-        return ['embed']
-    if name == 'norm.weight':
-        return ['final.norm']
+    top = {'embed_tokens.weight': 'embed', 'norm.weight': 'final.norm', 'lm_head.weight': 'head'}
+    if name in top:
+        return [top[name]]
     m = _LAYER.match(name)
     if not m:
         raise KeyError(f'no checkpoint mapping for {name}')
     i, rest = int(m.group(1)), m.group(2)
-    if rest == 'in_proj.weight':
-        return [f'l{i}.mix.{p}' for p in 'qkv'] + ([f'l{i}.mlp.gate', f'l{i}.mlp.up'] if cfg.layer_specs[i].ff else [])
-    return [f'l{i}.{p}' for p in _LISTED[rest]]
+    return [f'l{i}.{n}' for n, _ in _listed_parts(rest, cfg.layer_specs[i], cfg.hidden_size)] or [f'l{i}.{_LISTED[rest]}']
 
 
 def _listed_split(name: str, tensor: torch.Tensor, cfg: DecoderConfig) -> List[Tuple[str, torch.Tensor]]:
     names = _listed_names(name, cfg)
     if name.endswith('.v_lambda'):
         return [(names[0], tensor.reshape(()))]
-    if len(names) == 1:
+    if len(names) == 1 and '.experts.' not in name:
         return [(names[0], tensor)]
-    sp = cfg.layer_specs[int(_LAYER.match(name).group(1))]
-    sizes = list(sp.qkv_sizes) + ([sp.ff, sp.ff] if name.endswith('in_proj.weight') and sp.ff else [])
-    return list(zip(names, tensor.split(sizes, dim=0)))
+    m = _LAYER.match(name)
+    sizes = [n for _, n in _listed_parts(m.group(2), cfg.layer_specs[int(m.group(1))], cfg.hidden_size)]
+    return list(zip(names, tensor.reshape(-1, tensor.shape[-1]).split(sizes, dim=0)))
+
+
+def _listed_join(name: str, cfg: DecoderConfig, get: Callable[[str], torch.Tensor], expert_range: Optional[Tuple[int, int]] = None) -> torch.Tensor:
+    names = _listed_names(name, cfg)
+    if '.experts.' in name:
+        lo, hi = expert_range or (0, len(names))
+        return torch.stack([get(n) for n in names[lo:hi]])
+    return torch.cat([get(n).reshape(1) if n.endswith('.vmix') else get(n) for n in names], 0)
 
 
 def internal_to_hf(name: str, tensor: torch.Tensor, cfg: DecoderConfig) -> List[Tuple[str, torch.Tensor]]:
@@ -317,7 +348,7 @@ def hf_to_internal(name: str, cfg: DecoderConfig, get: Callable[[str], torch.Ten
     """Assemble one internal tensor from HF tensors fetched by ``get``.  An output head that the checkpoint does not carry
     (tied embeddings saved once) is read from the embedding."""
     if cfg.layer_specs is not None:
-        return torch.cat([get(n).reshape(1) if n.endswith('.vmix') else get(n) for n in _listed_names(name, cfg)], 0)
+        return _listed_join(name, cfg, get, expert_range)
     m = _LAYER.match(name)
     rest = m.group(2) if m else ''
     i = int(m.group(1)) if m else -1

@@ -72,8 +72,53 @@ def _pomelix_mapping(c: 'DecoderConfig') -> Dict[str, Any]:
     return d
 
 
+def _moronex_fields(cfg: Dict[str, Any]) -> Dict[str, Any]:
+    """``config.json`` of a Moronex checkpoint → keyword arguments of :class:`DecoderConfig`."""
+    specs = []
+    for i, layer in enumerate(cfg['layers']):
+        m, mlp = layer['mixer'], layer.get('mlp')
+        sizes = {k: int(m[k]) for k in ('heads', 'dim', 'vdim')}
+        if layer['type'] == 'latent_attention':
+            source = m.get('kv_from')
+            mixer = LatentSpec(**sizes, q_rank=int(m['q_rank']), kv_rank=int(m['kv_rank']), scale=float(m['scale']), kv_from=None if source is None else int(source))
+        elif layer['type'] == 'hgrn2':
+            mixer = HGRN2Spec(**sizes)
+        else:
+            raise NotImplementedError(f"layer {i}: mixer type {layer['type']!r} is not implemented (latent_attention and hgrn2 are)")
+        if mlp is None:
+            ff = None
+        elif mlp['kind'] == 'dense':
+            ff = FeedForwardSpec(ff=int(mlp['ff']))
+        elif mlp['kind'] == 'moe':
+            ff = FeedForwardSpec(ff=int(mlp['expert']['ff']), experts=int(mlp['router']['experts']), top=int(mlp['router']['top']))
+        else:
+            raise NotImplementedError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not implemented (dense and moe are)")
+        specs.append(SandwichSpec(mixer, ff))
+    return dict(model_type='moronex', vocab_size=int(cfg['vocab']), hidden_size=int(cfg['width']), rms_norm_eps=float(cfg['norm']['eps']), rms_norm_offset=1.0,
+                tie_word_embeddings=False, qk_norm=False, layer_specs=specs, eos_token_id=cfg.get('eos_token_id'), pad_token_id=cfg.get('pad_token_id'),
+                torch_dtype=str(cfg.get('torch_dtype', 'bfloat16')))
+
+
+def _moronex_mapping(c: 'DecoderConfig') -> Dict[str, Any]:
+    """The inverse of :func:`_moronex_fields`."""
+    layers = []
+    for sp in c.layer_specs:
+        m = {k: v for k, v in asdict(sp.mixer).items() if v is not None}
+        f = sp.mlp
+        mlp = None if f is None else ({'kind': 'moe', 'expert': {'ff': f.ff}, 'router': {'experts': f.experts, 'top': f.top}} if f.experts
+                                      else {'kind': 'dense', 'ff': f.ff})
+        layers.append({'type': sp.mixer.kind, 'mixer': m, 'mlp': mlp})
+    d = {'architecture': 'Moronex', 'vocab': c.vocab_size, 'width': c.hidden_size, 'norm': {'eps': c.rms_norm_eps}, 'layers': layers}
+    d.update({k: v for k, v in (('eos_token_id', c.eos_token_id), ('pad_token_id', c.pad_token_id)) if v is not None})
+    return d
+
+
 # checkpoints whose config.json names its ``architecture`` and lists every layer: (reader → DecoderConfig fields, writer)
-NATIVE_ARCHITECTURES = {'Pomelix': (_pomelix_fields, _pomelix_mapping)}
+NATIVE_ARCHITECTURES = {'Pomelix': (_pomelix_fields, _pomelix_mapping), 'Moronex': (_moronex_fields, _moronex_mapping)}
+
+
+def _up8(n: int) -> int:
+    return -(-n // 8) * 8
 
 
 @dataclass
@@ -95,9 +140,137 @@ class LayerSpec:
     v_mix: bool = False
     ff: int = 0
 
+    is_moe = False
+
     @property
     def qkv_sizes(self) -> Tuple[int, int, int]:
         return self.heads * self.dim, self.kv_heads * self.dim, self.kv_heads * self.vdim
+
+    # what a layer keeps per token, per sequence, and what it weighs (the same members exist on :class:`SandwichSpec`)
+    def kv_rows(self) -> Tuple[int, int, int]:
+        return self.kv_heads, _up8(self.dim), _up8(self.vdim)
+
+    def conv_rows(self) -> Optional[Tuple[int, int]]:
+        return (self.conv - 1, sum(self.qkv_sizes)) if self.conv > 1 else None
+
+    def state_shape(self) -> Optional[Tuple[int, int, int]]:
+        return None
+
+    def matmul_weights(self, width: int, active: bool = False) -> int:
+        return width * sum(self.qkv_sizes) + width * self.heads * self.vdim + 3 * width * self.ff
+
+    def small_weights(self, width: int) -> int:
+        return self.conv * sum(self.qkv_sizes) + width * (3 if self.ff else 2) + int(self.v_mix)
+
+    def attention_width(self) -> int:
+        """Multiply-adds per key and query of the score and value products."""
+        return (self.dim + self.vdim) * self.heads
+
+    @property
+    def ff_width(self) -> int:
+        return self.ff
+
+
+@dataclass
+class LatentSpec:
+    """Latent attention without positions: queries through a normed rank-``q_rank`` bottleneck, keys (``dim`` per head) and values
+    (``vdim``) expanded from one normed rank-``kv_rank`` latent per token, which is all the cache keeps; a sink logit per head in
+    the softmax, a sigmoid gate per head on the output.  ``kv_from``: index of the earlier layer whose latents this layer reads
+    instead of its own."""
+    heads: int
+    dim: int
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    kv_from: Optional[int] = None
+    kind = 'latent_attention'
+
+    def in_parts(self) -> List[Tuple[str, int]]:
+        """Projections of the layer input."""
+        return [('dq_proj', self.q_rank)] + ([('dkv_proj', self.kv_rank)] if self.kv_from is None else []) + [('head_gate', self.heads)]
+
+    def matmul_weights(self, width: int) -> int:
+        return width * sum(n for _, n in self.in_parts()) + self.heads * (self.dim * self.q_rank + (self.dim + self.vdim) * self.kv_rank + self.vdim * width)
+
+    def small_weights(self) -> int:
+        return self.q_rank + (self.kv_rank if self.kv_from is None else 0) + self.heads
+
+
+@dataclass
+class HGRN2Spec:
+    """Linear attention whose forget gate (per head and channel, bounded from below) also decides what is written; ``heads``
+    states of ``dim × vdim``."""
+    heads: int
+    dim: int
+    vdim: int
+    kind = 'hgrn2'
+
+    def in_parts(self) -> List[Tuple[str, int]]:
+        return [('q_proj', self.heads * self.dim), ('f_proj', self.heads * self.dim), ('v_proj', self.heads * self.vdim)]
+
+    def matmul_weights(self, width: int) -> int:
+        return width * self.heads * (2 * self.dim + 2 * self.vdim)
+
+    def small_weights(self) -> int:
+        return 2 * self.heads * self.dim + self.vdim
+
+
+@dataclass
+class FeedForwardSpec:
+    """Gated feed-forward block of width ``ff``, or, with ``experts``, that many two-matrix experts of which a token uses ``top``."""
+    ff: int
+    experts: int = 0
+    top: int = 0
+
+
+@dataclass
+class SandwichSpec:
+    """One layer with a norm in front of and behind each sub-layer and a sigmoid gate (read from the sub-layer's input) on its
+    result: a mixer and a feed-forward block (None: the layer has none)."""
+    mixer: Union[LatentSpec, HGRN2Spec]
+    mlp: Optional[FeedForwardSpec] = None
+
+    def __post_init__(self):
+        if isinstance(self.mixer, dict):
+            self.mixer = (LatentSpec if 'kv_rank' in self.mixer else HGRN2Spec)(**self.mixer)
+        if isinstance(self.mlp, dict):
+            self.mlp = FeedForwardSpec(**self.mlp)
+
+    heads = property(lambda self: self.mixer.heads)
+    kv_heads = property(lambda self: self.mixer.heads)
+    dim = property(lambda self: self.mixer.dim)
+    v_mix = False
+
+    @property
+    def is_moe(self) -> bool:
+        return self.mlp is not None and self.mlp.experts > 0
+
+    @property
+    def ff_width(self) -> int:
+        return self.mlp.ff if self.mlp is not None else 0
+
+    def kv_rows(self) -> Tuple[int, int, int]:
+        return (1, _up8(self.mixer.kv_rank), 0) if self.mixer.kind == 'latent_attention' and self.mixer.kv_from is None else (0, 0, 0)
+
+    def conv_rows(self) -> Optional[Tuple[int, int]]:
+        return None
+
+    def state_shape(self) -> Optional[Tuple[int, int, int]]:
+        return (self.mixer.heads, self.mixer.dim, self.mixer.vdim) if self.mixer.kind == 'hgrn2' else None
+
+    def matmul_weights(self, width: int, active: bool = False) -> int:
+        n = width * width + self.mixer.matmul_weights(width)
+        if self.mlp is not None:
+            per = (2 if self.mlp.experts else 3) * width * self.mlp.ff
+            n += width * width + (width * self.mlp.experts + (self.mlp.top if active else self.mlp.experts) * per if self.mlp.experts else per)
+        return n
+
+    def small_weights(self, width: int) -> int:
+        return 3 * width * (2 if self.mlp is not None else 1) + self.mixer.small_weights() + (self.mlp.experts if self.mlp is not None else 0)
+
+    def attention_width(self) -> int:
+        return (self.mixer.dim + self.mixer.vdim) * self.mixer.heads if self.mixer.kind == 'latent_attention' else 0
 
 
 @dataclass
@@ -206,24 +379,31 @@ class DecoderConfig:
     vision_end_token_id: Optional[int] = None
     mrope_section: Optional[List[int]] = None
     mrope_interleaved: bool = False  # Qwen3-VL lays the three position components out t h w t h w … instead of in blocks
-    # stacks whose layers are listed one by one and run mixer and feed-forward side by side on one norm (Pomelix): the
-    # residual stream is 32-bit, each sub-layer's result has a learned per-channel scale, positions enter through a short
-    # convolution and the query temperature only (no rotary embedding)
-    layer_specs: Optional[List[Union[LayerSpec, Dict[str, Any]]]] = None
+    # stacks whose layers are listed one by one, with a 32-bit residual stream and no rotary embedding: layers that run mixer and
+    # feed-forward side by side on one norm, each result with a learned per-channel scale (``LayerSpec``; Pomelix), or layers
+    # with norms around each sub-layer and a gate on its result (``SandwichSpec``; Moronex)
+    layer_specs: Optional[List[Union[LayerSpec, SandwichSpec, Dict[str, Any]]]] = None
 
     def __post_init__(self):
         if self.layer_specs is not None:
-            self.layer_specs = [LayerSpec(**sp) if isinstance(sp, dict) else sp for sp in self.layer_specs]
+            self.layer_specs = [(SandwichSpec if 'mixer' in sp else LayerSpec)(**sp) if isinstance(sp, dict) else sp for sp in self.layer_specs]
             first = self.layer_specs[0]
             self.num_hidden_layers = len(self.layer_specs)
             self.num_attention_heads, self.num_key_value_heads, self.head_dim = first.heads, first.kv_heads, first.dim
-            self.intermediate_size = max(sp.ff for sp in self.layer_specs)
+            self.intermediate_size = max(sp.ff_width for sp in self.layer_specs)
             for i, sp in enumerate(self.layer_specs):
                 if sp.heads % sp.kv_heads:
                     raise ValueError(f'layer {i}: {sp.heads} query heads do not divide over {sp.kv_heads} key / value heads')
             mixed = [sp for sp in self.layer_specs if sp.v_mix]
             if any((sp.kv_heads, sp.vdim) != (mixed[0].kv_heads, mixed[0].vdim) for sp in mixed):
                 raise ValueError('layers that mix values must agree on the number and width of the value heads')
+            for i, sp in enumerate(self.layer_specs):
+                j = getattr(getattr(sp, 'mixer', None), 'kv_from', None)
+                if j is None:
+                    continue
+                src = self.layer_specs[j].mixer if 0 <= j < i else None
+                if src is None or src.kind != 'latent_attention' or src.kv_from is not None or src.kv_rank != sp.mixer.kv_rank:
+                    raise ValueError(f'layer {i}: kv_from {j} is not an earlier latent-attention layer with latents of its own and rank {sp.mixer.kv_rank}')
         if self.vision is not None:
             from .vision import VisionConfig
             self.vision = VisionConfig.from_hf(self.vision).to_hf()  # only the fields the tower uses, in the family's spelling
@@ -243,14 +423,28 @@ class DecoderConfig:
 
     def kv_layout(self) -> List[Tuple[int, int, int]]:
         """Per layer ``(key / value heads, key row width, value row width)`` of the paged cache.  Layers with widths of their
-        own keep rows of whole 16-byte vectors (widths rounded up to a multiple of 8, the rest zero)."""
+        own keep rows of whole 16-byte vectors (widths rounded up to a multiple of 8, the rest zero); a latent is one key row
+        that also serves as the value; layers that keep nothing per token have 0 heads."""
         if self.layer_specs is None:
             return [(self.num_key_value_heads, self.head_dim, self.head_dim)] * self.num_hidden_layers
-        return [(sp.kv_heads, -(-sp.dim // 8) * 8, -(-sp.vdim // 8) * 8) for sp in self.layer_specs]
+        return [sp.kv_rows() for sp in self.layer_specs]
 
     def conv_layout(self) -> List[Optional[Tuple[int, int]]]:
         """Per layer ``(rows, channels)`` of the convolution history a sequence keeps between steps (None: no history)."""
-        return [(sp.conv - 1, sum(sp.qkv_sizes)) if sp.conv > 1 else None for sp in self.layer_specs or []]
+        return [sp.conv_rows() for sp in self.layer_specs or []]
+
+    def state_layout(self) -> List[Optional[Tuple[int, int, int]]]:
+        """Per layer shape of the (fp32) recurrent state a sequence carries from token to token (None: no state)."""
+        return [sp.state_shape() for sp in self.layer_specs or []]
+
+    def held_columns(self) -> List[Tuple[int, int]]:
+        """``(layer, columns)`` of what later layers take from earlier ones besides the stream: the values of the first mixing
+        layer, the latents of layers that others borrow."""
+        if self.first_mixing_layer is not None:
+            first = self.layer_specs[self.first_mixing_layer]
+            return [(self.first_mixing_layer, first.kv_heads * first.vdim)]
+        lent = sorted({sp.mixer.kv_from for sp in self.layer_specs or [] if getattr(getattr(sp, 'mixer', None), 'kv_from', None) is not None})
+        return [(j, self.layer_specs[j].mixer.kv_rank) for j in lent]
 
     def layer_is_moe(self, layer_idx: int) -> bool:
         return self.num_experts > 0 and layer_idx >= self.first_k_dense_replace
@@ -293,14 +487,13 @@ class DecoderConfig:
             return q + h * (self.kv_lora_rank + self.qk_rope_head_dim) + self.kv_lora_rank * nh * (self.qk_nope_head_dim + self.v_head_dim) + nh * self.v_head_dim * h
         return h * (self.q_size + 2 * self.kv_size) + self.q_size * h + (self.q_size * h if self.attn_output_gate else 0)
 
-    def _listed_matmul_weights(self) -> int:
-        h = self.hidden_size
-        return sum(h * sum(sp.qkv_sizes) + h * sp.heads * sp.vdim + 3 * h * sp.ff for sp in self.layer_specs)
+    def _listed_matmul_weights(self, active: bool = False) -> int:
+        return sum(sp.matmul_weights(self.hidden_size, active) for sp in self.layer_specs)
 
     def num_params(self) -> int:
         h, L = self.hidden_size, self.num_hidden_layers
         if self.layer_specs is not None:
-            small = sum(sp.conv * sum(sp.qkv_sizes) + h * (3 if sp.ff else 2) + int(sp.v_mix) for sp in self.layer_specs)
+            small = sum(sp.small_weights(h) for sp in self.layer_specs)
             return self._listed_matmul_weights() + small + self.vocab_size * h * (1 if self.tie_word_embeddings else 2) + h
         attn = self._attn_weights() + (2 * self.head_dim if self.qk_norm else 0)
         moe = self.num_experts * 3 * h * self.moe_intermediate_size + h * self.num_experts + 3 * h * self.shared_expert_intermediate_size
@@ -320,8 +513,9 @@ class DecoderConfig:
         """Forward+backward matmul FLOPs per token (6·N_active + attention)."""
         h, L = self.hidden_size, self.num_hidden_layers
         if self.layer_specs is not None:
-            attn = sum((sp.dim + sp.vdim) * sp.heads for sp in self.layer_specs) * avg_context
-            return 6.0 * (self._listed_matmul_weights() + self.vocab_size * h) + 6.0 * attn
+            attn = sum(sp.attention_width() for sp in self.layer_specs) * avg_context
+            state = 2 * sum(a * b * c for a, b, c in filter(None, self.state_layout()))       # a write and a read of every state element
+            return 6.0 * (self._listed_matmul_weights(active=True) + self.vocab_size * h + state) + 6.0 * attn
         attn_w = self._attn_weights()
         moe_w = self.num_experts_per_tok * 3 * h * self.moe_intermediate_size + h * self.num_experts + 3 * h * self.shared_expert_intermediate_size
         n_moe = sum(self.layer_is_moe(i) for i in range(L))
@@ -433,7 +627,7 @@ class DecoderConfig:
 
     def to_hf(self) -> Dict[str, Any]:
         if self.layer_specs is not None:
-            return NATIVE_ARCHITECTURES['Pomelix'][1](self)
+            return NATIVE_ARCHITECTURES[self.model_type.capitalize()][1](self)
         arch = 'Qwen3MoeForCausalLM' if self.is_moe else ('Qwen3ForCausalLM' if self.qk_norm else 'LlamaForCausalLM')
         arch = {'mixtral': 'MixtralForCausalLM', 'qwen2_moe': 'Qwen2MoeForCausalLM', 'qwen2': 'Qwen2ForCausalLM', 'mistral': 'MistralForCausalLM',
                 'seed_oss': 'SeedOssForCausalLM'}.get(self.model_type, arch)
@@ -646,6 +840,20 @@ PRESETS: Dict[str, Dict[str, Any]] = {
     'pomelix-8b': dict(vocab_size=151936, hidden_size=4096, tie_word_embeddings=True, qk_norm=False, model_type='pomelix', rms_norm_eps=1e-5,
                        residual_multiplier=0.5, layer_specs=[dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128**-0.5, conv=4, temp_coef=0.1,
                                                                   temp_every=4096, v_mix=True, ff=12288)] * 36),
+    # Moronex in small: recurrent and latent-attention layers of unequal sizes, a borrowed latent, dense / expert / no feed-forward
+    'tiny-moronex': dict(vocab_size=1024, hidden_size=192, tie_word_embeddings=False, qk_norm=False, torch_dtype='float32', model_type='moronex',
+                         rms_norm_eps=1e-5, rms_norm_offset=1.0,
+                         layer_specs=[dict(mixer=dict(heads=3, dim=24, vdim=48), mlp=dict(ff=320)),
+                                      dict(mixer=dict(heads=6, dim=40, vdim=24, q_rank=72, kv_rank=56, scale=0.2), mlp=dict(ff=64, experts=6, top=2)),
+                                      dict(mixer=dict(heads=2, dim=48, vdim=40)),
+                                      dict(mixer=dict(heads=4, dim=24, vdim=32, q_rank=48, kv_rank=56, scale=0.25, kv_from=1), mlp=dict(ff=80, experts=5, top=3))]),
+    # Moronex layers at the width, experts and depth of Qwen3-30B-A3B (benchmarks): three recurrent layers per latent-attention layer,
+    # every second of those borrowing the latents of the one before
+    'moronex-30b-a3b': dict(vocab_size=151936, hidden_size=2048, tie_word_embeddings=False, qk_norm=False, model_type='moronex', rms_norm_eps=1e-6,
+                            rms_norm_offset=1.0,
+                            layer_specs=[dict(mixer=dict(heads=16, dim=128, vdim=128) if i % 4 != 3 else
+                                              dict(heads=32, dim=128, vdim=128, q_rank=1024, kv_rank=512, scale=128**-0.5, kv_from=i - 4 if i % 8 == 7 else None),
+                                              mlp=dict(ff=6144) if i == 0 else dict(ff=1152, experts=128, top=8)) for i in range(48)]),
     'qwen3-0.6b': dict(hidden_size=1024, intermediate_size=3072, num_hidden_layers=28, num_attention_heads=16,
                        num_key_value_heads=8, head_dim=128, tie_word_embeddings=True),
     'qwen3-8b': dict(hidden_size=4096, intermediate_size=12288, num_hidden_layers=36, num_attention_heads=32,

@@ -22,7 +22,7 @@ import torch.nn as nn
 import torch.nn.functional as F
 
 from .. import ops
-from .config import DecoderConfig
+from .config import DecoderConfig, SandwichSpec
 from .layers import Embedding, Linear, RMSNorm
 from .parallel_layer import CacheView, ParallelLayer, Stream
 
@@ -249,21 +249,27 @@ class Experts(nn.Module):
         super().__init__()
         e = num_local if num_local is not None else cfg.num_experts
         self.num_local, self.first_expert = e, 0
-        self.gate_up_proj = nn.Parameter(torch.empty(e, 2 * cfg.moe_intermediate_size, cfg.hidden_size))
+        # 'relu2': two-matrix experts, the square of relu between them; otherwise a gated unit on [gate | up]
+        self.gated = cfg.expert_act != 'relu2'
+        if self.gated:
+            self.gate_up_proj = nn.Parameter(torch.empty(e, 2 * cfg.moe_intermediate_size, cfg.hidden_size))
+        else:
+            self.up_proj = nn.Parameter(torch.empty(e, cfg.moe_intermediate_size, cfg.hidden_size))
         self.down_proj = nn.Parameter(torch.empty(e, cfg.hidden_size, cfg.moe_intermediate_size))
         if cfg.expert_bias:
             self.gate_up_bias = nn.Parameter(torch.zeros(e, 2 * cfg.moe_intermediate_size))
             self.down_bias = nn.Parameter(torch.zeros(e, cfg.hidden_size))
         else:
             self.gate_up_bias = self.down_bias = None
-        self.act = ops.ref.clamped_glu if cfg.expert_act == 'clamped_glu' else ops.swiglu
+        self.act = {'clamped_glu': ops.ref.clamped_glu, 'relu2': ops.ref.relu2}.get(cfg.expert_act, ops.swiglu)
         self.lora = nn.ParameterDict()
         self.max_loras = 0
 
     def add_lora_pool(self, max_loras: int, max_r: int) -> None:
-        e, two_i, h = self.gate_up_proj.shape
-        i = two_i // 2
-        dev, dt = self.gate_up_proj.device, self.gate_up_proj.dtype
+        first, name = (self.gate_up_proj, 'gate_up') if self.gated else (self.up_proj, 'up')
+        e, out, h = first.shape
+        i = self.down_proj.shape[2]
+        dev, dt = first.device, first.dtype
         self.max_loras, self.max_r = max_loras, max_r
 
         def mk_a(inp):
@@ -271,8 +277,8 @@ class Experts(nn.Module):
             nn.init.kaiming_uniform_(a.view(-1, inp), a=math.sqrt(5))
             return nn.Parameter(a)
 
-        self.lora['gate_up_A'] = mk_a(h)
-        self.lora['gate_up_B'] = nn.Parameter(torch.zeros(max_loras, e, two_i, max_r, device=dev, dtype=dt))
+        self.lora[name + '_A'] = mk_a(h)
+        self.lora[name + '_B'] = nn.Parameter(torch.zeros(max_loras, e, out, max_r, device=dev, dtype=dt))
         self.lora['down_A'] = mk_a(i)
         self.lora['down_B'] = nn.Parameter(torch.zeros(max_loras, e, h, max_r, device=dev, dtype=dt))
 
@@ -298,6 +304,8 @@ class Experts(nn.Module):
 
     def forward(self, x_sorted: torch.Tensor, offsets: torch.Tensor) -> torch.Tensor:
         """``x_sorted`` rows grouped by local expert; ``offsets [E_local+1]``."""
+        if not self.gated:
+            return self._forward_plain(x_sorted, offsets)
         lo = self._expert_lora('gate_up')
         gu = ops.expert_linear(x_sorted, self.gate_up_proj, offsets, *(lo or ()))
         row_expert = None
@@ -310,6 +318,15 @@ class Experts(nn.Module):
         lo = self._expert_lora('down')
         y = ops.expert_linear(act, self.down_proj, offsets, *(lo or ()))
         return y if row_expert is None else y + self.down_bias[row_expert].to(y.dtype)
+
+    def _forward_plain(self, x_sorted: torch.Tensor, offsets: torch.Tensor) -> torch.Tensor:
+        """Two-matrix experts; without adapters and gradients the activation rides in the first product's epilogue."""
+        lo = self._expert_lora('up')
+        if lo is None and not ops._needs_grad(x_sorted, self.up_proj):
+            a = ops.grouped_gemm(x_sorted, self.up_proj, offsets, act='relu2')
+        else:
+            a = self.act(ops.expert_linear(x_sorted, self.up_proj, offsets, *(lo or ())))
+        return ops.expert_linear(a, self.down_proj, offsets, *(self._expert_lora('down') or ()))
 
 
 class MoEBlock(nn.Module):
@@ -388,6 +405,17 @@ class MoEBlock(nn.Module):
         if mp is not None:
             return self._with_shared(x, mp.forward(self, x, w, idx))
         return self._with_shared(x, self._routed_local(x, w, idx))
+
+    def rows(self, x: torch.Tensor, forced: Optional[torch.Tensor] = None):
+        """Inference form for blocks that choose by logit and weigh by a softmax over the chosen (``'topk_softmax'``): ``(expert rows
+        [T·k, H], their place [T, k], weights [T, k] fp32)``, left uncombined for a following kernel that reads them per token.
+        Router logits are fp32; rows of an expert are contiguous and nothing is padded."""
+        k = self.cfg.num_experts_per_tok
+        w, idx, hist = ops.moe_topk(ops.linear_f32(x, self.gate.weight), self.gate.bias, k, forced)
+        if self.record_routing:
+            self.last_routed = idx.detach()
+        xs, row_of, offsets = ops.moe_group_rows(x, idx, hist)
+        return self.experts(xs, offsets), row_of, w
 
     def _forward_expert_tp(self, x, w, idx):
         """Expert tensor parallelism (reference ``megatron/strategy/megatron.py:90-107``: ``expert_tensor_parallel_size``):
@@ -503,7 +531,7 @@ class DecoderModel(nn.Module):
         lo, hi = layer_range or (0, cfg.num_hidden_layers)
         self.layer_range = (lo, hi)
         self.embed_tokens = Embedding(cfg.vocab_size, cfg.hidden_size) if has_embed else None
-        self.layers = nn.ModuleList([(ParallelLayer if cfg.layer_specs is not None else DecoderLayer)(cfg, i) for i in range(lo, hi)])
+        self.layers = nn.ModuleList([self._layer_class(i)(cfg, i) for i in range(lo, hi)])
         self.norm = RMSNorm(cfg.hidden_size, cfg.rms_norm_eps, cfg.rms_norm_offset) if has_head else None
         if has_head and not cfg.tie_word_embeddings:
             self.lm_head = Linear(cfg.hidden_size, cfg.vocab_size, name='lm_head')
@@ -520,6 +548,14 @@ class DecoderModel(nn.Module):
                 m.full_name = name
         self.layer_runner = None  # engine hook: runs one layer (checkpoint / FSDP unshard)
         self.tp = None  # tensor-parallel context, set by parallel.tensor.apply_tensor_parallel
+
+    def _layer_class(self, i: int):
+        if self.cfg.layer_specs is None:
+            return DecoderLayer
+        if isinstance(self.cfg.layer_specs[i], SandwichSpec):
+            from .sandwich_layer import SandwichLayer
+            return SandwichLayer
+        return ParallelLayer
 
     # --------------------------------------------------------------- init
     @torch.no_grad()
@@ -538,10 +574,9 @@ class DecoderModel(nn.Module):
                 p.zero_()
                 continue
             if p.dim() == 1:
-                if name.endswith('bias'):
-                    p.zero_()
-                else:
-                    p.fill_(1.0 if self.cfg.rms_norm_offset == 0.0 else 0.0)
+                owner = self.get_submodule(name.rpartition('.')[0])
+                offset = owner.offset if isinstance(owner, RMSNorm) else self.cfg.rms_norm_offset
+                p.fill_(1.0 if offset == 0.0 else 0.0)
                 continue
             g = torch.Generator(device='cpu').manual_seed(stable_seed(seed, name))
             if p.numel() <= 2**24 or p.device.type == 'cpu':
@@ -586,18 +621,16 @@ class DecoderModel(nn.Module):
         """Stacks with listed layers: fp32 stream, final norm in the compute dtype (see ``models/parallel_layer.py``)."""
         cfg, run = self.cfg, self.layer_runner
         x = self.embed(batch)
-        mult = float(cfg.residual_multiplier)
         if run is None and not torch.is_grad_enabled():
             x = x.float().clone() if batch.inputs_embeds is not None else x.float()      # updated in place from here on
             st = Stream(x.contiguous())
             for layer in self.layers:
                 st = layer.advance(st, batch)
-            return ops.stream_rmsnorm(st.x, self.norm.weight, cfg.rms_norm_eps, st.adds, mult)[0]
-        first = cfg.layer_specs[cfg.first_mixing_layer] if cfg.first_mixing_layer is not None else None
-        x = F.pad(x.float(), (0, first.kv_heads * first.vdim if first is not None else 0))
+            return st.enter(self.norm)
+        x = F.pad(x.float(), (0, sum(n for _, n in cfg.held_columns())))
         for layer in self.layers:
             x = run(layer, x, None, None, batch) if run is not None else layer(x, None, None, batch)
-        return ops.stream_rmsnorm(x[:, :cfg.hidden_size].contiguous(), self.norm.weight, cfg.rms_norm_eps)[0]
+        return Stream(x[:, :cfg.hidden_size].contiguous()).enter(self.norm)
 
     def forward(self, batch: PackedBatch, hidden: Optional[torch.Tensor] = None, kv_sink=None) -> torch.Tensor:
         if self.cfg.layer_specs is not None:

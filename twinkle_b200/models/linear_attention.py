@@ -24,7 +24,7 @@ import torch
 import torch.nn as nn
 import torch.nn.functional as F
 
-from .layers import Linear
+from .layers import Linear, RMSNorm
 
 
 def gated_delta_rule_recurrent(q, k, v, g, beta, scale: Optional[float] = None, state=None):
@@ -246,3 +246,30 @@ class GatedDeltaNet(nn.Module):
         o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + self.eps) * self.norm_weight.float()
         o = o * F.silu(z.float().view(B, self.hv, self.dv))
         return self.out_proj(o.to(x.dtype).reshape(B, vd)), window[:, 1:].contiguous(), S
+
+
+class HGRN2(nn.Module):
+    """Linear attention whose forget gate also decides what is written: per head ``S ← f ⊙ S + (1 − f) vᵀ`` (f on the rows), ``o = Sᵀ q``,
+    with ``q = silu(W_q h)``, ``v = W_v h``, ``f = lower + (1 − lower) σ(W_f h + b)``; heads are RMS-normed over their width and
+    projected.  Everything between the two products is one kernel (``ops/csrc/hgrn2.cu``).  ``lead``: projections of the same input
+    that are not this block's, in the leading columns of its input product."""
+
+    def __init__(self, width: int, spec, eps: float, layer_idx: int, lead=()):
+        super().__init__()
+        self.spec, self.eps, self.layer_idx = spec, eps, layer_idx
+        parts = list(lead) + spec.in_parts()
+        self.in_proj = Linear(width, sum(n for _, n in parts), parts=parts)
+        self.first = sum(n for _, n in lead)
+        self.f_bias = nn.Parameter(torch.zeros(spec.heads * spec.dim))
+        self.lower = nn.Parameter(torch.zeros(spec.heads * spec.dim))
+        self.out_norm = RMSNorm(spec.vdim, eps)
+        self.o_proj = Linear(spec.heads * spec.vdim, width, name='o_proj')
+
+    def forward(self, h: torch.Tensor, batch, held=None):
+        """``(result [T, width], the input product)``."""
+        from .. import ops
+        sp, n = self.spec, self.spec.heads * self.spec.dim
+        p = self.in_proj(h)
+        o = ops.hgrn2(p, self.first, self.first + n, self.first + 2 * n, sp.heads, sp.dim, sp.vdim, self.f_bias, self.lower, self.out_norm.weight, self.eps,
+                      batch.cu_seqlens, batch.max_seqlen, batch.cache, self.layer_idx)
+        return self.o_proj(o), p

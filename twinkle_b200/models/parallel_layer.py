@@ -15,7 +15,7 @@ forward without gradients passes over the stream once per layer.  With gradients
 from __future__ import annotations
 
 from dataclasses import dataclass, field
-from typing import List, Optional, Tuple
+from typing import Dict, List, Optional, Tuple
 
 import torch
 import torch.nn as nn
@@ -32,7 +32,7 @@ class CacheView:
     packed, and their keys, values and convolution history are only written."""
     cache: object
     rows: torch.Tensor                          # [T] int64: row of each token in the flat key / value pools
-    slots: torch.Tensor                         # [T] int32: convolution-history slot of the token's sequence
+    slots: torch.Tensor                         # [T] int32: slot of the token's sequence in the history and state pools
     left: torch.Tensor                          # [T] int32: later tokens of the same sequence in this forward
     table: Optional[torch.Tensor] = None        # [B, blocks] int32
     seq_lens: Optional[torch.Tensor] = None     # [B] int32, the new token included
@@ -43,12 +43,36 @@ class CacheView:
 
 
 @dataclass
+class GatedResult:
+    """A sub-layer's result on its way into the stream: ``norm(σ(gate + bias) ⊙ result)``.  ``result [T, W]``, or expert rows
+    with the places ``row_of [T, k]`` and weights ``share [T, k]`` of every token's."""
+    result: torch.Tensor
+    gate: torch.Tensor                          # [T, ≥ W]: the gate's projection in the leading columns
+    bias: torch.Tensor
+    norm: RMSNorm
+    row_of: Optional[torch.Tensor] = None
+    share: Optional[torch.Tensor] = None
+
+
+@dataclass
 class Stream:
-    """The residual stream between layers: ``x`` (fp32) plus sub-layer results that have not joined it yet, and the values
-    of the first mixing layer."""
+    """The residual stream between layers: ``x`` (fp32) plus sub-layer results that have not joined it yet (``adds`` times
+    ``mult``, or one gated and normed result), and what later layers take from earlier ones (``held``: layer → tensor)."""
     x: torch.Tensor
     adds: List[Tuple[torch.Tensor, torch.Tensor]] = field(default_factory=list)
-    v_first: Optional[torch.Tensor] = None
+    held: Dict[int, torch.Tensor] = field(default_factory=dict)
+    mult: float = 1.0
+    gated: Optional[GatedResult] = None
+
+    def enter(self, norm: RMSNorm) -> torch.Tensor:
+        """What is pending joins the stream; returns its norm in the compute dtype — one kernel."""
+        if self.gated is not None:
+            g = self.gated
+            h, self.x = ops.stream_gated_rmsnorm(self.x, norm.weight, norm.eps, norm.offset, g.result, g.gate, g.bias, g.norm.weight, g.row_of, g.share)
+        else:
+            h, self.x = ops.stream_rmsnorm(self.x, norm.weight, norm.eps, self.adds, self.mult, norm.offset)
+        self.adds, self.gated = [], None
+        return h
 
 
 class ParallelLayer(nn.Module):
@@ -59,7 +83,8 @@ class ParallelLayer(nn.Module):
         sp = self.spec = cfg.layer_specs[layer_idx]
         self.layer_idx, self.eps, self.mult, self.width = layer_idx, cfg.rms_norm_eps, float(cfg.residual_multiplier), cfg.hidden_size
         q, k, v = sp.qkv_sizes
-        self.gives_values = layer_idx == cfg.first_mixing_layer
+        self.values_of = cfg.first_mixing_layer
+        self.gives_values = layer_idx == self.values_of
         self.takes_values = sp.v_mix and not self.gives_values
         self.input_layernorm = RMSNorm(cfg.hidden_size, cfg.rms_norm_eps)
         parts = [('q_proj', q), ('k_proj', k), ('v_proj', v)] + ([('gate_proj', sp.ff), ('up_proj', sp.ff)] if sp.ff else [])
@@ -91,9 +116,12 @@ class ParallelLayer(nn.Module):
 
     def advance(self, st: Stream, batch) -> Stream:
         """One layer without gradients: pending results of the layer below join the stream in this layer's norm kernel."""
-        h, x = ops.stream_rmsnorm(st.x, self.input_layernorm.weight, self.eps, st.adds, self.mult)
-        adds, v = self.sublayers(h, batch, st.v_first)
-        return Stream(x, adds, v if self.gives_values else st.v_first)
+        h = st.enter(self.input_layernorm)
+        st.adds, v = self.sublayers(h, batch, st.held.get(self.values_of))
+        st.mult = self.mult
+        if self.gives_values:
+            st.held[self.layer_idx] = v
+        return st
 
     def forward(self, x: torch.Tensor, cos, sin, batch, kv_sink=None) -> torch.Tensor:
         """``x [T, width + values]`` fp32 → the same after this layer (see the module's docstring)."""

@@ -285,13 +285,81 @@ def _needs_grad(*ts) -> bool:
     return torch.is_grad_enabled() and any(t is not None and t.requires_grad for t in ts)
 
 
-def stream_rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, adds=(), mult: float = 1.0):
+def stream_rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, adds=(), mult: float = 1.0, offset: float = 0.0):
     """fp32 residual stream ``x [T, W]``: ``x ← x + mult · Σ y_i ⊙ s_i`` for ``adds = [(y, s), …]`` (at most two) and its RMS
-    norm in ``weight``'s dtype, one kernel on CUDA.  Returns ``(norm, x)``; without gradients ``x`` is updated in place."""
+    norm (weight ``offset + w``) in ``weight``'s dtype, one kernel on CUDA.  Returns ``(norm, x)``; without gradients ``x`` is
+    updated in place."""
     if not _cuda(x) or _needs_grad(x, weight, *[t for a in adds for t in a]):
-        return ref.stream_rmsnorm(x, weight, eps, weight.dtype, adds, mult)
+        return ref.stream_rmsnorm(x, weight, eps, weight.dtype, adds, mult, offset)
     (y1, s1), (y2, s2) = (list(adds) + [(None, None)] * 2)[:2]
-    return ext().stream_rmsnorm(x, weight, eps, None if y1 is None else y1.contiguous(), s1, None if y2 is None else y2.contiguous(), s2, mult), x
+    return ext().stream_rmsnorm(x, weight, eps, None if y1 is None else y1.contiguous(), s1, None if y2 is None else y2.contiguous(), s2, mult, offset), x
+
+
+def stream_gated_rmsnorm(x, weight, eps: float, offset: float, result, gate, bias, post, row_of=None, share=None):
+    """fp32 residual stream ``x [T, W]``: ``x ← x + norm(σ(gate + bias) ⊙ result; post)`` and the norm of the sum in ``weight``'s
+    dtype (both norms with weights ``offset + w``), one kernel on CUDA.  ``gate``: leading ``W`` columns of a projection.
+    ``result``: ``[T, W]``, or expert rows combined on the way (``row_of [T, k]``, ``share [T, k]``).  Returns ``(norm, x)``; without
+    gradients ``x`` is updated in place."""
+    if not _cuda(x) or _needs_grad(x, weight, result, gate, bias, post, share):
+        return ref.stream_gated_rmsnorm(x, weight, eps, offset, result, gate, bias, post, row_of, share)
+    return ext().stream_gated_rmsnorm(x, weight, eps, offset, result.contiguous(), gate, bias, post, row_of, share), x
+
+
+# ------------------------------------------- latent attention, HGRN2
+def latent_norms(proj, q0: int, nq: int, wq, c0: int, nc: int, wc, eps: float, view=None, layer: int = -1):
+    """Column ranges of a projection → the normed query bottleneck ``[T, nq]`` and the normed latent ``[T, nc']`` (``nc'``: ``nc`` rounded
+    up to a multiple of 8, the rest zero; None for ``nc`` 0), which is also written to the cache that ``view`` names."""
+    pool = view.cache.k[layer] if view is not None and nc else None
+    if _cuda(proj) and not _needs_grad(proj, wq, wc):
+        q, c = ext().latent_norms(proj, q0, nq, wq, c0, nc, wc, eps, None if pool is None else pool, None if pool is None else view.rows)
+        return q, (c if nc else None)
+    q, c = ref.latent_norms(proj, q0, nq, wq, c0, nc, wc, eps)
+    if c is not None and not _needs_grad(proj, wq, wc):
+        c = torch.nn.functional.pad(c, (0, -nc % 8))
+        if pool is not None:
+            pool.view(-1, pool.shape[-1])[view.rows] = c
+    return q, c
+
+
+def head_linear(x, weight, transposed: bool = False):
+    """One small matrix per head: ``x [B, H, K]`` times ``weight[h]ᵀ`` for ``weight [H, N, K]``, or times ``weight[h]`` for ``[H, K, N]``
+    (``transposed``) → ``[B, H, N]``."""
+    n, k = (weight.shape[2], weight.shape[1]) if transposed else weight.shape[1:]
+    if _cuda(x) and x.dtype == torch.bfloat16 and n % 8 == 0 and k % 8 == 0 and not _needs_grad(x, weight):
+        return ext().head_gemm(x.contiguous(), weight, transposed)
+    w = weight if transposed else weight.transpose(1, 2)
+    return torch.bmm(x.transpose(0, 1), w).transpose(0, 1).contiguous()
+
+
+def latent_decode(q, pool, table, lens, scale: float, sinks, gate=None):
+    """One token per sequence, ``q [B, H, R]`` in latent space, against the cached latents ``pool [blocks, bs, 1, R']`` that are key and
+    value of every head; sink logits ``[H]`` in the denominator, result times ``σ(gate [B, H])``."""
+    if _cuda(q):
+        return ext().latent_decode(q.contiguous(), pool, table.to(torch.int32), lens.to(torch.int32), scale, sinks, gate)
+    return ref.latent_decode(q, pool, table, lens, scale, sinks, gate)
+
+
+def hgrn2(proj, q0: int, f0: int, v0: int, heads: int, dim: int, vdim: int, bias, lower, weight, eps: float, cu_seqlens=None, max_seqlen: int = 0,
+          view=None, layer: int = -1):
+    """The HGRN2 mixer between its projections: column ranges ``q``, ``f``, ``v`` of ``proj`` → the normed output ``[T, heads · vdim]``.  Prompts
+    start from an empty state; ``view`` (a ``CacheView``) says where the last states go, and single steps continue from there."""
+    step = view is not None and view.stepping
+    states = view.cache.state[layer] if view is not None else None
+    if _cuda(proj) and not _needs_grad(proj, bias, lower, weight):
+        args = (proj, q0, f0, v0, heads, dim, vdim, bias, lower, weight, eps)
+        if step:
+            return ext().hgrn2_step(*args, states, view.slots)
+        return ext().hgrn2_prefill(*args, cu_seqlens.to(torch.int32), int(max_seqlen), states, None if view is None else view.slots)
+    if step:
+        slots = view.slots.long()
+        o, last = ref.hgrn2(proj, q0, f0, v0, heads, dim, vdim, bias, lower, weight, eps, list(range(proj.shape[0] + 1)), list(states[slots]))
+        states[slots] = torch.stack(last)
+        return o
+    bounds = cu_seqlens.tolist()
+    o, last = ref.hgrn2(proj, q0, f0, v0, heads, dim, vdim, bias, lower, weight, eps, bounds)
+    if states is not None:
+        states[view.slots[cu_seqlens[:-1].long()].long()] = torch.stack(last)
+    return o
 
 
 def conv_heads(proj, weight, positions, hq: int, hkv: int, d: int, e: int, eps: float, coef: float = 0.0, every: int = 0, v_first=None, lam=None,
@@ -333,14 +401,18 @@ def glu_columns(proj: torch.Tensor, gate: int, up: int, width: int) -> torch.Ten
     return ref.swiglu(torch.cat([proj[:, gate:gate + width], proj[:, up:up + width]], -1))
 
 
-def attention_packed(q, k, v, cu_seqlens, max_seqlen: int, scale: float):
+def attention_packed(q, k, v, cu_seqlens, max_seqlen: int, scale: float, sinks=None, gate=None):
     """Causal packed attention for any key / value widths up to 256: tensor-core kernel for bf16 heads up to 128 wide, an
-    fp32-arithmetic kernel for wider heads and for 32-bit models."""
-    if not _cuda(q) or _needs_grad(q, k, v):
-        return flash_attn_varlen(q, k, v, cu_seqlens, max_seqlen, True, scale)
+    fp32-arithmetic kernel for wider heads and for 32-bit models.  ``sinks [Hq]``: a logit per head in the denominator;
+    ``gate [T, Hq]``: the output of a head is multiplied by its sigmoid.  ``k`` and ``v`` may be column ranges of one tensor."""
+    if not _cuda(q) or _needs_grad(q, k, v, sinks, gate):
+        o = flash_attn_varlen(q, k, v, cu_seqlens, max_seqlen, True, scale, sinks=sinks)
+        return o if gate is None else (o.float() * torch.sigmoid(gate.float())[..., None]).to(o.dtype)
+    cu = cu_seqlens.to(torch.int32)
     if _flash_widths(q, k, v):
-        return ext().flash_attn_fwd(q.contiguous(), k.contiguous(), v.contiguous(), cu_seqlens.to(torch.int32), int(max_seqlen), True, scale)[0]
-    return ext().attention_packed(q.contiguous(), k.contiguous(), v.contiguous(), cu_seqlens.to(torch.int32), int(max_seqlen), scale)
+        q, k, v = (t if t.stride(2) == 1 and t.stride(1) % 8 == 0 and t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 else t.contiguous() for t in (q, k, v))
+        return ext().flash_attn_fwd(q, k, v, cu, int(max_seqlen), True, scale, None, sinks, gate)[0]
+    return ext().attention_packed(q.contiguous(), k.contiguous(), v.contiguous(), cu, int(max_seqlen), scale, sinks, gate)
 
 
 # ------------------------------------------------------------------ swiglu
@@ -905,15 +977,52 @@ class _GroupedGemm(torch.autograd.Function):
         return gx, gw, None
 
 
-def grouped_gemm(x, weight, offsets):
-    """Per-expert GEMM over expert-sorted rows (``offsets [E+1]`` int32 on device)."""
+def grouped_gemm(x, weight, offsets, act: Optional[str] = None):
+    """Per-expert GEMM over expert-sorted rows (``offsets [E+1]`` int32 on device).  ``act='relu2'``: the square of relu in the
+    epilogue (no gradient)."""
     if _cuda(x) and x.dtype == torch.bfloat16:
+        n, k = weight.shape[1:]
+        if n % 8 or k % 8:      # TMA rows are whole 16-byte vectors: odd sizes are filled up with zero rows / columns
+            pad = torch.nn.functional.pad
+            return grouped_gemm(pad(x, (0, -k % 8)), pad(weight, (0, -k % 8, 0, -n % 8)), offsets, act)[:, :n]
+        if act is not None:
+            return ext().grouped_gemm(x, weight, offsets.to(torch.int32), 'nt', None, None, False, None, None, act)
         return _GroupedGemm.apply(x, weight, offsets.to(torch.int32))
+    if _cuda(x) and x.dtype == torch.float32 and not _needs_grad(x, weight):
+        return ext().grouped_gemm_f32(x.contiguous(), weight, offsets.to(torch.int32), act == 'relu2')
+    if act is not None:
+        return ref.relu2(grouped_gemm(x, weight, offsets))
     outs = []
     off = offsets.tolist()
     for e in range(weight.shape[0]):
         outs.append(x[off[e]:off[e + 1]] @ weight[e].t().to(x.dtype))
     return torch.cat(outs, 0)
+
+
+def moe_topk(logits, bias, k: int, forced=None):
+    """fp32 ``logits [T, E]`` (+ ``bias``) → weights ``[T, k]`` fp32 (softmax over the k largest), their experts ``[T, k]`` int64, and tokens
+    per expert ``[E]`` int32.  ``forced``: experts to take instead (rows of −1: none)."""
+    if _cuda(logits) and logits.shape[1] <= 256 and k <= 32:
+        return tuple(ext().moe_topk(logits, bias, k, None if forced is None else forced.to(logits.device).long().contiguous()))
+    z = logits.float() + (bias.float() if bias is not None else 0.0)
+    top, idx = z.topk(k, -1)
+    if forced is not None:
+        idx = torch.where(forced[:, :1] < 0, idx, forced.long())
+        top = z.gather(1, idx)
+    hist = torch.zeros(z.shape[1], dtype=torch.int32, device=z.device).scatter_add_(0, idx.reshape(-1), torch.ones(idx.numel(), dtype=torch.int32, device=z.device))
+    return torch.softmax(top, -1), idx, hist
+
+
+def moe_group_rows(x, idx, hist):
+    """Rows of ``x [T, H]`` once per chosen expert, those of an expert together and nothing between them: ``(rows [T·k, H], row_of [T, k]
+    int32, offsets [E+1] int32)``."""
+    if _cuda(x) and hist.numel() <= 256:
+        return tuple(ext().moe_group_rows(x.contiguous(), idx, hist))
+    order = torch.argsort(idx.reshape(-1), stable=True)
+    row_of = torch.empty(idx.numel(), dtype=torch.int32, device=x.device)
+    row_of[order] = torch.arange(idx.numel(), dtype=torch.int32, device=x.device)
+    offsets = torch.nn.functional.pad(hist.cumsum(0), (1, 0)).to(torch.int32)
+    return x[order // idx.shape[1]], row_of.view(idx.shape), offsets
 
 
 # ------------------------------------------------------- moe token permutation

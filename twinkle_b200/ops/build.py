@@ -27,7 +27,8 @@ _SO = os.path.join(_HERE, '_C.so')
 _STAMP = os.path.join(_HERE, '_C.stamp')
 _SERVING_SO = os.path.join(_HERE, '_C_serving.so')
 _SERVING_STAMP = os.path.join(_HERE, '_C_serving.stamp')
-_SERVING_SOURCES = ('bindings.cpp', 'host.cu', 'gemm.cu', 'gemm2.cu', 'attention_fwd.cu', 'attention_packed.cu', 'decode.cu', 'stream_ops.cu')
+_SERVING_SOURCES = ('bindings.cpp', 'host.cu', 'gemm.cu', 'gemm2.cu', 'attention_fwd.cu', 'attention_packed.cu', 'decode.cu', 'stream_ops.cu',
+                    'hgrn2.cu', 'latent.cu', 'latent_decode.cu', 'moe_serve.cu')
 _MOD = None
 _SERVING_ONLY = False
 

@@ -40,6 +40,9 @@ struct FwdParams {
   int T, hq, hkv;
   float scale_log2;   // softmax scale · log2(e)
   int causal;
+  const bf16* sinks;  // [Hq] logit of a key without a value that every row sees (nullptr: none)
+  const bf16* gate;   // [T, Hq] with row stride ldg: the output is multiplied by its sigmoid (nullptr: not)
+  long ldg;
   int* err;
 };
 
@@ -257,8 +260,10 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     l_sum += xsum[(wg ^ 1) * 128 + row];
     if (!dead && n_blocks > 0 && mbar_wait(o_done, (n_blocks - 1) & 1, p.err, ERR_ATTN_WAIT)) {
       tc_fence_after();
-      const float inv_l = (l_sum > 0.f) ? 1.f / l_sum : 0.f;
+      if (p.sinks != nullptr) l_sum += exp2f(__bfloat162float(p.sinks[head]) * 1.4426950408889634f - m_used);
+      float inv_l = (l_sum > 0.f) ? 1.f / l_sum : 0.f;
       const bool valid = q_pos < seq_len;
+      if (p.gate != nullptr && valid) inv_l /= 1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(seq_start + q_pos) * p.ldg + head]));
       bf16* orow = p.out + (static_cast<size_t>(seq_start + q_pos) * p.hq + head) * p.e;
 #pragma unroll 1
       for (int c = 2 * wg; c < 2 * wg + 2 && c * 32 < p.e; ++c) {
@@ -294,10 +299,13 @@ CUtensorMap make_head_tmap(const torch::Tensor& t, int rows) {
 }
 
 std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor& q, const torch::Tensor& k, const torch::Tensor& v, const torch::Tensor& cu,
-                                          int64_t max_seqlen, bool causal, double scale, const c10::optional<torch::Tensor>& cu_k) {
-  TORCH_CHECK(q.is_cuda() && q.scalar_type() == torch::kBFloat16 && q.dim() == 3 && q.is_contiguous(), "q [T,Hq,D] bf16 contiguous");
-  TORCH_CHECK(k.is_contiguous() && v.is_contiguous() && k.dim() == 3 && v.dim() == 3 && k.size(0) == v.size(0) && k.size(1) == v.size(1) &&
-                  k.scalar_type() == torch::kBFloat16 && v.scalar_type() == torch::kBFloat16, "k [T,Hkv,D], v [T,Hkv,E] bf16 contiguous");
+                                          int64_t max_seqlen, bool causal, double scale, const c10::optional<torch::Tensor>& cu_k,
+                                          const c10::optional<torch::Tensor>& sinks, const c10::optional<torch::Tensor>& gate) {
+  TORCH_CHECK(q.is_cuda() && q.scalar_type() == torch::kBFloat16 && q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && k.size(0) == v.size(0) && k.size(1) == v.size(1) &&
+                  k.scalar_type() == torch::kBFloat16 && v.scalar_type() == torch::kBFloat16, "q [T,Hq,D], k [T,Hkv,D], v [T,Hkv,E] bf16");
+  for (const auto* t : {&q, &k, &v})
+    TORCH_CHECK(t->stride(2) == 1 && t->stride(1) % 8 == 0 && t->stride(0) % 8 == 0 && reinterpret_cast<uintptr_t>(t->data_ptr()) % 16 == 0,
+                "q, k, v: unit stride inside a head, rows and heads on 16-byte boundaries");
   TORCH_CHECK(q.size(2) == k.size(2) && k.size(2) % 8 == 0 && v.size(2) % 8 == 0 && k.size(2) > 0 && v.size(2) > 0 && k.size(2) <= 128 && v.size(2) <= 128,
               "head widths: multiples of 8 up to 128");
   TORCH_CHECK(cu.is_cuda() && cu.scalar_type() == torch::kInt32 && cu.is_contiguous(), "cu_seqlens int32 on device");
@@ -314,6 +322,14 @@ std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor& q, const torch::T
   if (cu_k.has_value() && cu_k->defined()) {
     TORCH_CHECK(cu_k->is_cuda() && cu_k->scalar_type() == torch::kInt32 && cu_k->is_contiguous() && cu_k->numel() == cu.numel(), "cu_k like cu");
     p.cu_k = cu_k->data_ptr<int>();
+  }
+  if (sinks.has_value() && sinks->defined()) {
+    TORCH_CHECK(sinks->is_cuda() && sinks->scalar_type() == torch::kBFloat16 && sinks->is_contiguous() && sinks->numel() == hq, "sinks [Hq] bf16");
+    p.sinks = reinterpret_cast<const bf16*>(sinks->data_ptr());
+  }
+  if (gate.has_value() && gate->defined()) {
+    TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == torch::kBFloat16 && gate->dim() == 2 && gate->size(0) == T && gate->size(1) == hq && gate->stride(1) == 1, "gate [T, Hq] bf16");
+    p.gate = reinterpret_cast<const bf16*>(gate->data_ptr()); p.ldg = gate->stride(0);
   }
   p.T = T; p.hq = hq; p.hkv = hkv; p.scale_log2 = static_cast<float>(scale * 1.4426950408889634); p.causal = causal; p.err = error_word();
   const dim3 grid(hq, (static_cast<int>(max_seqlen) + fa::BQ - 1) / fa::BQ, nseq);

@@ -24,7 +24,8 @@ __device__ __forceinline__ void st(bf16* p, float v) { *p = __float2bfloat16(v);
 
 template <typename T, int EI>
 __global__ void __launch_bounds__(256) attention_packed_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, T* __restrict__ out,
-                                                               const int* __restrict__ cu, int hq, int hkv, int D, int E, float scale_log2) {
+                                                               const int* __restrict__ cu, int hq, int hkv, int D, int E, float scale_log2,
+                                                               const T* __restrict__ sinks, const T* __restrict__ gate, long ldg) {
   using namespace pa;
   extern __shared__ float sm[];
   const int head = blockIdx.x, seq = blockIdx.z, kvh = head / (hq / hkv);
@@ -97,19 +98,26 @@ __global__ void __launch_bounds__(256) attention_packed_kernel(const T* __restri
   }
   if (q0 + row < len) {
     T* o = out + (static_cast<size_t>(start + q0 + row) * hq + head) * E;
+    if (sinks != nullptr) l += exp2f(ld(sinks + head) * 1.4426950408889634f - m);      // a key without a value that every row sees
+    float f = 1.f / l;
+    if (gate != nullptr) f /= 1.f + __expf(-ld(gate + static_cast<size_t>(start + q0 + row) * ldg + head));
 #pragma unroll
     for (int i = 0; i < EI; ++i)
-      if (sub + 8 * i < E) st(o + sub + 8 * i, acc[i] / l);
+      if (sub + 8 * i < E) st(o + sub + 8 * i, acc[i] * f);
   }
 }
 
-torch::Tensor attention_packed(const torch::Tensor& q, const torch::Tensor& k, const torch::Tensor& v, const torch::Tensor& cu, int64_t max_seqlen, double scale) {
+torch::Tensor attention_packed(const torch::Tensor& q, const torch::Tensor& k, const torch::Tensor& v, const torch::Tensor& cu, int64_t max_seqlen, double scale,
+                               const c10::optional<torch::Tensor>& sinks, const c10::optional<torch::Tensor>& gate) {
   const auto st = q.scalar_type();
   TORCH_CHECK(q.is_cuda() && (st == torch::kBFloat16 || st == torch::kFloat32) && k.scalar_type() == st && v.scalar_type() == st, "q, k, v bf16 or fp32");
   TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && q.is_contiguous() && k.is_contiguous() && v.is_contiguous(), "[T, H, D] contiguous");
   TORCH_CHECK(q.size(2) == k.size(2) && k.size(0) == q.size(0) && v.size(0) == q.size(0) && k.size(1) == v.size(1) && q.size(1) % k.size(1) == 0, "shapes of q, k, v");
   TORCH_CHECK(q.size(2) <= 256 && v.size(2) <= 256, "head widths up to 256");
   TORCH_CHECK(cu.is_cuda() && cu.scalar_type() == torch::kInt32 && cu.is_contiguous(), "cu_seqlens int32 on device");
+  const bool has_sinks = sinks.has_value() && sinks->defined(), has_gate = gate.has_value() && gate->defined();
+  if (has_sinks) TORCH_CHECK(sinks->is_cuda() && sinks->scalar_type() == st && sinks->is_contiguous() && sinks->numel() == q.size(1), "sinks [Hq]");
+  if (has_gate) TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == st && gate->dim() == 2 && gate->size(0) == q.size(0) && gate->size(1) == q.size(1) && gate->stride(1) == 1, "gate [T, Hq]");
   c10::cuda::CUDAGuard guard(q.device());
   const int hq = q.size(1), hkv = k.size(1), D = q.size(2), E = v.size(2), nseq = cu.numel() - 1;
   auto out = torch::empty({q.size(0), hq, E}, q.options());
@@ -121,7 +129,9 @@ torch::Tensor attention_packed(const torch::Tensor& q, const torch::Tensor& k, c
     using T = decltype(tag);
     TK_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     kern<<<grid, 256, smem, stream>>>(reinterpret_cast<const T*>(q.data_ptr()), reinterpret_cast<const T*>(k.data_ptr()), reinterpret_cast<const T*>(v.data_ptr()),
-                                      reinterpret_cast<T*>(out.data_ptr()), cu.data_ptr<int>(), hq, hkv, D, E, static_cast<float>(scale * 1.4426950408889634));
+                                      reinterpret_cast<T*>(out.data_ptr()), cu.data_ptr<int>(), hq, hkv, D, E, static_cast<float>(scale * 1.4426950408889634),
+                                      has_sinks ? reinterpret_cast<const T*>(sinks->data_ptr()) : nullptr, has_gate ? reinterpret_cast<const T*>(gate->data_ptr()) : nullptr,
+                                      has_gate ? gate->stride(0) : 0L);
   };
   if (st == torch::kBFloat16) {
     if (E <= 64) go(attention_packed_kernel<bf16, 8>, bf16{});

@@ -8,8 +8,10 @@ namespace tk {
 torch::Tensor gemm(const torch::Tensor&, const torch::Tensor&, const std::string&, const c10::optional<torch::Tensor>&, bool,
                    c10::optional<torch::ScalarType>);
 std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t,
-                                          bool, double, const c10::optional<torch::Tensor>&);
-torch::Tensor attention_packed(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t, double);
+                                          bool, double, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&,
+                                          const c10::optional<torch::Tensor>&);
+torch::Tensor attention_packed(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t, double,
+                               const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
 torch::Tensor paged_attn_decode(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, double);
 std::vector<torch::Tensor> sample_tokens(const torch::Tensor&, double, int64_t, double, const torch::Tensor&);
 std::vector<torch::Tensor> conv_heads(const torch::Tensor&, const c10::optional<torch::Tensor>&, const torch::Tensor&, int64_t, int64_t, int64_t, int64_t,
@@ -17,13 +19,28 @@ std::vector<torch::Tensor> conv_heads(const torch::Tensor&, const c10::optional<
                                       const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&,
                                       const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, bool);
 torch::Tensor stream_rmsnorm(torch::Tensor, const torch::Tensor&, double, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&,
-                             const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, double);
+                             const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, double, double);
+torch::Tensor stream_gated_rmsnorm(torch::Tensor, const torch::Tensor&, double, double, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&,
+                                   const torch::Tensor&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
+std::vector<torch::Tensor> latent_norms(const torch::Tensor&, int64_t, int64_t, const torch::Tensor&, int64_t, int64_t, const c10::optional<torch::Tensor>&, double,
+                                        const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
+torch::Tensor latent_decode(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, double, const torch::Tensor&,
+                            const c10::optional<torch::Tensor>&);
+torch::Tensor hgrn2_prefill(const torch::Tensor&, int64_t, int64_t, int64_t, int64_t, int64_t, int64_t, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&,
+                            double, const torch::Tensor&, int64_t, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
+torch::Tensor hgrn2_step(const torch::Tensor&, int64_t, int64_t, int64_t, int64_t, int64_t, int64_t, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&,
+                         double, const torch::Tensor&, const torch::Tensor&);
+std::vector<torch::Tensor> moe_topk(const torch::Tensor&, const c10::optional<torch::Tensor>&, int64_t, const c10::optional<torch::Tensor>&);
+std::vector<torch::Tensor> moe_group_rows(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&);
+torch::Tensor grouped_gemm_f32(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, bool);
+torch::Tensor head_gemm(const torch::Tensor&, const torch::Tensor&, bool);
+torch::Tensor grouped_gemm(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const std::string&, const c10::optional<torch::Tensor>&,
+                           const c10::optional<torch::Tensor>&, bool, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&,
+                           const c10::optional<std::string>&);
 torch::Tensor glu_columns(const torch::Tensor&, int64_t, int64_t, int64_t);
 void set_gemm_pair(int64_t);
 void set_gemm_staged(int64_t);
 #ifndef TK_SERVING_ONLY
-torch::Tensor grouped_gemm(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const std::string&, const c10::optional<torch::Tensor>&,
-                           const c10::optional<torch::Tensor>&, bool, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
 torch::Tensor grouped_gemm_wgrad(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t);
 std::vector<torch::Tensor> rmsnorm_fwd(const torch::Tensor&, const torch::Tensor&, double, double, const c10::optional<torch::Tensor>&);
 std::vector<torch::Tensor> rmsnorm_bwd(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, double,
@@ -78,7 +95,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm", &tk::gemm, py::arg("a"), py::arg("b"), py::arg("layout") = "nt", py::arg("out") = py::none(),
         py::arg("accumulate") = false, py::arg("out_dtype") = py::none());
   m.def("flash_attn_fwd", &tk::flash_attn_fwd, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("cu"), py::arg("max_seqlen"), py::arg("causal"),
-        py::arg("scale"), py::arg("cu_k") = py::none());
+        py::arg("scale"), py::arg("cu_k") = py::none(), py::arg("sinks") = py::none(), py::arg("gate") = py::none());
   m.def("paged_attn_decode", &tk::paged_attn_decode);
   m.def("sample_tokens", &tk::sample_tokens);
   m.def("set_gemm_pair", &tk::set_gemm_pair);
@@ -86,17 +103,27 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("read_and_clear_error", &tk::read_and_clear_error, "Value of the device error word (0 = healthy); clears it.");
   m.def("num_sms", &tk::num_sms);
   m.def("launch_count", &tk::launch_count, "Number of kernels launched by this extension so far.");
-  m.def("attention_packed", &tk::attention_packed);
+  m.def("attention_packed", &tk::attention_packed, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("cu"), py::arg("max_seqlen"), py::arg("scale"),
+        py::arg("sinks") = py::none(), py::arg("gate") = py::none());
   m.def("conv_heads", &tk::conv_heads, py::arg("proj"), py::arg("weight"), py::arg("pos"), py::arg("hq"), py::arg("hkv"), py::arg("d"), py::arg("e"), py::arg("eps"),
         py::arg("coef") = 0.0, py::arg("every") = 0, py::arg("v_first") = py::none(), py::arg("lam") = py::none(), py::arg("step") = false,
         py::arg("hist") = py::none(), py::arg("slot") = py::none(), py::arg("left") = py::none(), py::arg("pool_row") = py::none(),
         py::arg("k_pool") = py::none(), py::arg("v_pool") = py::none(), py::arg("want_k") = true);
   m.def("stream_rmsnorm", &tk::stream_rmsnorm, py::arg("x"), py::arg("w"), py::arg("eps"), py::arg("y1") = py::none(), py::arg("s1") = py::none(),
-        py::arg("y2") = py::none(), py::arg("s2") = py::none(), py::arg("mult") = 1.0);
+        py::arg("y2") = py::none(), py::arg("s2") = py::none(), py::arg("mult") = 1.0, py::arg("offset") = 0.0);
+  m.def("stream_gated_rmsnorm", &tk::stream_gated_rmsnorm);
+  m.def("latent_norms", &tk::latent_norms);
+  m.def("latent_decode", &tk::latent_decode);
+  m.def("hgrn2_prefill", &tk::hgrn2_prefill);
+  m.def("hgrn2_step", &tk::hgrn2_step);
+  m.def("moe_topk", &tk::moe_topk);
+  m.def("moe_group_rows", &tk::moe_group_rows);
+  m.def("grouped_gemm_f32", &tk::grouped_gemm_f32);
+  m.def("head_gemm", &tk::head_gemm);
+  m.def("grouped_gemm", &tk::grouped_gemm, py::arg("x"), py::arg("w"), py::arg("offsets"), py::arg("layout") = "nt", py::arg("group_map") = py::none(),
+        py::arg("out") = py::none(), py::arg("accumulate") = false, py::arg("x2") = py::none(), py::arg("w2") = py::none(), py::arg("act") = py::none());
   m.def("glu_columns", &tk::glu_columns);
 #ifndef TK_SERVING_ONLY
-  m.def("grouped_gemm", &tk::grouped_gemm, py::arg("x"), py::arg("w"), py::arg("offsets"), py::arg("layout") = "nt", py::arg("group_map") = py::none(),
-        py::arg("out") = py::none(), py::arg("accumulate") = false, py::arg("x2") = py::none(), py::arg("w2") = py::none());
   m.def("grouped_gemm_wgrad", &tk::grouped_gemm_wgrad);
   m.def("rmsnorm_fwd", &tk::rmsnorm_fwd, py::arg("x"), py::arg("w"), py::arg("eps"), py::arg("offset"), py::arg("residual") = py::none());
   m.def("rmsnorm_bwd", &tk::rmsnorm_bwd, py::arg("g"), py::arg("x"), py::arg("w"), py::arg("rstd"), py::arg("offset"),

@@ -42,7 +42,8 @@ struct GemmParams {
   const int* offsets;  // [E+1] row offsets (aligned to BM) or nullptr
   int num_groups;
   int group_rows_b;    // rows of B per group (N for NT, K for NN)
-  int mode;            // 0 dense, 1 grouped over M (A rows by expert), 2 grouped wgrad (K range by expert)
+  int mode;            // 0 dense, 1 grouped over M (A rows by expert), 2 grouped wgrad (K range by expert), 3 one product per head
+  int act;             // 1: the square of relu on the result
   const int* group_map;  // optional: group g uses weight block group_map[g] (< 0: group skipped); nullptr = identity
   // second operand pair of the M-grouped mode (0 = none): out = A·B + A2·B2 accumulated in tensor memory before the
   // epilogue — how a low-rank (LoRA) term rides in the base GEMM instead of re-reading and re-writing the output
@@ -113,9 +114,25 @@ __device__ __forceinline__ bool grouped_k_tile(const GemmParams& p, int tile, Ti
   return true;
 }
 
+// One product per head: all heads have the same M rows, K columns of A (a 3-D tensor map) and N columns of the output.
+__device__ __forceinline__ bool head_tile(const GemmParams& p, int tile, TileCoord& t) {
+  int num_m = (p.M + BM - 1) / BM, num_n = (p.N + BN - 1) / BN;
+  int per = num_m * num_n;
+  if (tile >= per * p.num_groups) return false;
+  int g = tile / per, r = tile - g * per;
+  t.m0 = (r % num_m) * BM;
+  t.n0 = (r / num_m) * BN;
+  t.group = g;
+  t.k_begin = 0;
+  t.k_end = p.K;
+  t.m_limit = p.M;
+  return true;
+}
+
 template <int MODE>
 __device__ __forceinline__ bool next_tile(const GemmParams& p, int tile, GroupedCursor& c, TileCoord& t) {
   if constexpr (MODE == 0) return dense_tile(p, tile, t);
+  else if constexpr (MODE == 3) return head_tile(p, tile, t);
   else if constexpr (MODE == 1) return grouped_m_tile(p, tile, c, t);
   else return grouped_k_tile(p, tile, t);
 }
@@ -165,14 +182,16 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       TileCoord t;
       bool ok = true;
       for (int tile = blockIdx.x; ok && next_tile<MODE>(p, tile, cur, t); tile += gridDim.x) {
-        const int b_group = (MODE == 1) ? (p.group_map ? p.group_map[t.group] : t.group) : 0;
+        const int b_group = (MODE == 1) ? (p.group_map ? p.group_map[t.group] : t.group) : (MODE == 3 ? t.group : 0);
         const int b_row0 = b_group * p.group_rows_b;
         auto load_stage = [&](const CUtensorMap* mA, const CUtensorMap* mB, int k0, int brow) -> bool {
           if (!mbar_wait(&empty_bar[stage], phase ^ 1, p.err, ERR_PRODUCER_WAIT)) return false;
           uint8_t* sa = smem + stage * STAGE_BYTES;
           uint8_t* sb = sa + A_BYTES;
           mbar_expect_tx(&full_bar[stage], STAGE_BYTES);
-          if constexpr (!A_MN) {
+          if constexpr (MODE == 3) {
+            tma_load_3d(sa, mA, &full_bar[stage], k0, t.group, t.m0);   // columns past the head's K read as zero
+          } else if constexpr (!A_MN) {
             tma_load_2d(sa, mA, &full_bar[stage], k0, t.m0);            // box {64 (K), 128 rows}
           } else {
 #pragma unroll
@@ -257,6 +276,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       const bool row_ok = row < t.m_limit;
       size_t out_row = static_cast<size_t>(row);
       if constexpr (MODE == 2) out_row += static_cast<size_t>(t.group) * p.M;
+      const size_t head0 = MODE == 3 ? static_cast<size_t>(t.group) * p.N : 0;   // first output column of the head
 #pragma unroll 1
       for (int c = 0; c < BN / 32; ++c) {
         uint32_t r[32];
@@ -268,8 +288,15 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
 #pragma unroll
           for (int j = 0; j < 32; ++j) r[j] = 0u;
         }
+        if (MODE == 1 && p.act == 1) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            const float v = fmaxf(__uint_as_float(r[j]), 0.f);
+            r[j] = __float_as_uint(v * v);
+          }
+        }
         if (p.out_fp32) {
-          float* o = reinterpret_cast<float*>(p.out) + out_row * p.ldo + col0;
+          float* o = reinterpret_cast<float*>(p.out) + out_row * p.ldo + head0 + col0;
 #pragma unroll
           for (int j = 0; j < 32; j += 4) {
             if (col0 + j + 4 <= p.N) {
@@ -286,7 +313,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
             }
           }
         } else {
-          __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + out_row * p.ldo + col0;
+          __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + out_row * p.ldo + head0 + col0;
 #pragma unroll
           for (int j = 0; j < 32; j += 8) {
             if (col0 + j + 8 <= p.N) {
@@ -351,6 +378,9 @@ static void launch(bool a_mn, bool b_mn, int mode, const CUtensorMap& ta, const 
     if (!a_mn && !b_mn) TK_LAUNCH(false, false, 1);
     else if (!a_mn && b_mn) TK_LAUNCH(false, true, 1);
     else TORCH_CHECK(false, "unsupported grouped GEMM layout");
+  } else if (mode == 3) {
+    TORCH_CHECK(!a_mn, "unsupported per-head GEMM layout");
+    if (b_mn) TK_LAUNCH(false, true, 3); else TK_LAUNCH(false, false, 3);
   } else {
     TORCH_CHECK(a_mn && b_mn, "grouped wgrad is TN");
     TK_LAUNCH(true, true, 2);
@@ -425,14 +455,35 @@ torch::Tensor gemm(const torch::Tensor& a, const torch::Tensor& b, const std::st
   return out;
 }
 
-// Expert-grouped GEMM.  x [R, K] with expert e owning rows [offsets[e], offsets[e+1]) (offsets multiples of 128;
-// padding rows are zero); weight [E, N, K] (nt) or [E, K, N] (nn).  Returns [R, N].
+// One product per head: x [B, H, K] times w [H, N, K] transposed, or w [H, K, N] as it is (`nn`) → [B, H, N].
+torch::Tensor head_gemm(const torch::Tensor& x, const torch::Tensor& w, bool nn) {
+  TORCH_CHECK(x.is_cuda() && x.scalar_type() == torch::kBFloat16 && x.dim() == 3 && x.is_contiguous(), "x [B, H, K] bf16 contiguous");
+  TORCH_CHECK(w.is_cuda() && w.scalar_type() == torch::kBFloat16 && w.dim() == 3 && w.is_contiguous() && w.size(0) == x.size(1), "weight [H, *, *] bf16 contiguous");
+  c10::cuda::CUDAGuard guard(x.device());
+  const int B = x.size(0), H = x.size(1), K = x.size(2), N = nn ? w.size(2) : w.size(1);
+  TORCH_CHECK((nn ? w.size(1) : w.size(2)) == K && K % 8 == 0 && N % 8 == 0, "per-head product: widths that agree and are multiples of 8");
+  auto out = torch::empty({B, H, N}, x.options());
+  if (B == 0) return out;
+  auto w2 = w.view({w.size(0) * w.size(1), w.size(2)});
+  check_operand(w2, "weight");
+  CUtensorMap ta = make_tmap_3d(x.data_ptr(), K, H, B, K, static_cast<uint64_t>(H) * K, BK, 1, BM);
+  CUtensorMap tb = nn ? make_tmap_2d(w2.data_ptr(), w2.size(1), w2.size(0), w2.stride(0), 64, BK)
+                      : make_tmap_2d(w2.data_ptr(), w2.size(1), w2.size(0), w2.stride(0), BK, BN);
+  GemmParams p{};
+  p.out = out.data_ptr(); p.M = B; p.N = N; p.K = K; p.ldo = H * N; p.err = error_word();
+  p.num_groups = H; p.group_rows_b = w.size(1); p.mode = 3;
+  launch(false, nn, 3, ta, tb, p, ((B + BM - 1) / BM) * ((N + BN - 1) / BN) * H, at::cuda::getCurrentCUDAStream());
+  return out;
+}
+
+// Expert-grouped GEMM.  x [R, K] with expert e owning rows [offsets[e], offsets[e+1]); weight [E, N, K] (nt) or [E, K, N] (nn).  Returns [R, N].
 // Optional second pair (x2 [R, K2], w2 [E, N, K2] (nt) or [E, K2, N] (nn)): returns x·W + x2·W2 from one pass — the sum
 // is formed in tensor memory, the output is written once.
 torch::Tensor grouped_gemm(const torch::Tensor& x, const torch::Tensor& w, const torch::Tensor& offsets, const std::string& layout,
                            const c10::optional<torch::Tensor>& group_map, const c10::optional<torch::Tensor>& out_opt, bool accumulate,
-                           const c10::optional<torch::Tensor>& x2_opt, const c10::optional<torch::Tensor>& w2_opt) {
+                           const c10::optional<torch::Tensor>& x2_opt, const c10::optional<torch::Tensor>& w2_opt, const c10::optional<std::string>& act) {
   check_operand(x, "x");
+  TORCH_CHECK(!act.has_value() || (*act == "relu2" && !accumulate), "activation: relu2, without accumulation");
   TORCH_CHECK(w.is_cuda() && w.scalar_type() == torch::kBFloat16 && w.dim() == 3 && w.is_contiguous(), "weight [E, *, *] bf16 contiguous");
   TORCH_CHECK(offsets.is_cuda() && offsets.scalar_type() == torch::kInt32 && offsets.is_contiguous(), "offsets int32 on device");
   c10::cuda::CUDAGuard guard(x.device());
@@ -464,7 +515,7 @@ torch::Tensor grouped_gemm(const torch::Tensor& x, const torch::Tensor& w, const
                         : make_tmap_2d(w2.data_ptr(), w2.size(1), w2.size(0), w2.stride(0), BK, BN);
   GemmParams p{};
   p.out = out.data_ptr(); p.M = R; p.N = N; p.K = K; p.ldo = N; p.out_fp32 = 0; p.accumulate = accumulate ? 1 : 0; p.err = error_word();
-  p.offsets = offsets.data_ptr<int>(); p.num_groups = E; p.group_rows_b = w.size(1); p.mode = 1;
+  p.offsets = offsets.data_ptr<int>(); p.num_groups = E; p.group_rows_b = w.size(1); p.mode = 1; p.act = act.has_value() ? 1 : 0;
   p.group_map = mapped ? group_map->data_ptr<int>() : nullptr;
   // upper bound of tiles: every expert wastes at most one partial M-tile
   int tiles = ((R + BM - 1) / BM + E) * ((N + BN - 1) / BN);

@@ -3,6 +3,8 @@
 //   conv_heads      short causal convolution on q, k and v, q / k over their root mean square per head, query temperature,
 //                   value mixing, and the writes into the paged K/V pools and the convolution history — one pass
 //   stream_rmsnorm  x += mult · (y1 ⊙ s1 + y2 ⊙ s2) in fp32 and the RMS norm of the sum in the compute dtype — one pass
+//   stream_gated_rmsnorm  x += norm(σ(gate + bias) ⊙ y) in fp32 and the RMS norm of the sum — one pass; y is a row of its own or
+//                   the weighted sum of a token's expert rows
 //   glu_columns     silu(gate) · up on two column ranges of the projection
 // All are templated on the compute dtype (bf16 or fp32) and work for any width: vector kernels where rows are made of
 // whole vectors, plain ones otherwise.
@@ -396,7 +398,7 @@ std::vector<torch::Tensor> conv_heads(const torch::Tensor& proj, const OptT& wei
 // rows of any width, element-wise, the second pass re-reads what the thread wrote.
 template <typename T, int VPT>
 __global__ void stream_rmsnorm_kernel(float* __restrict__ x, const T* __restrict__ y1, const T* __restrict__ s1, const T* __restrict__ y2,
-                                      const T* __restrict__ s2, float mult, const T* __restrict__ w, T* __restrict__ h, int W, float eps) {
+                                      const T* __restrict__ s2, float mult, const T* __restrict__ w, T* __restrict__ h, int W, float eps, float offset) {
   __shared__ float sh[32];
   const size_t base = static_cast<size_t>(blockIdx.x) * W;
   float ss = 0.f;
@@ -427,7 +429,7 @@ __global__ void stream_rmsnorm_kernel(float* __restrict__ x, const T* __restrict
       const int c = (i * blockDim.x + threadIdx.x) * 4;
       if (c < W) {
         const float4 g = load4(w + c);
-        store4(h + base + c, make_float4(v[i].x * r * g.x, v[i].y * r * g.y, v[i].z * r * g.z, v[i].w * r * g.w));
+        store4(h + base + c, make_float4(v[i].x * r * (offset + g.x), v[i].y * r * (offset + g.y), v[i].z * r * (offset + g.z), v[i].w * r * (offset + g.w)));
       }
     }
   } else {
@@ -442,12 +444,13 @@ __global__ void stream_rmsnorm_kernel(float* __restrict__ x, const T* __restrict
       ss += v * v;
     }
     const float r = rsqrtf(block_sum(ss, sh) / W + eps);
-    for (int c = threadIdx.x; c < W; c += blockDim.x) h[base + c] = from_f<T>(x[base + c] * r * to_f(w[c]));
+    for (int c = threadIdx.x; c < W; c += blockDim.x) h[base + c] = from_f<T>(x[base + c] * r * (offset + to_f(w[c])));
   }
 }
 
-// x [rows, W] fp32 is updated in place when y1 is given; returns the norm in w's dtype.
-torch::Tensor stream_rmsnorm(torch::Tensor x, const torch::Tensor& w, double eps, const OptT& y1, const OptT& s1, const OptT& y2, const OptT& s2, double mult) {
+// x [rows, W] fp32 is updated in place when y1 is given; returns the norm (weights offset + w) in w's dtype.
+torch::Tensor stream_rmsnorm(torch::Tensor x, const torch::Tensor& w, double eps, const OptT& y1, const OptT& s1, const OptT& y2, const OptT& s2, double mult,
+                             double offset) {
   const auto st = w.scalar_type();
   TORCH_CHECK(x.is_cuda() && x.scalar_type() == torch::kFloat32 && x.is_contiguous() && x.dim() == 2, "stream [rows, W] fp32 contiguous");
   TORCH_CHECK((st == torch::kBFloat16 || st == torch::kFloat32) && w.is_contiguous() && w.numel() == x.size(1), "norm weight [W] bf16 or fp32");
@@ -471,7 +474,8 @@ torch::Tensor stream_rmsnorm(torch::Tensor x, const torch::Tensor& w, double eps
     auto ptr = [](const OptT& t) { return has(t) ? reinterpret_cast<const T*>(t->data_ptr()) : static_cast<const T*>(nullptr); };
     auto go = [&](auto kern, int threads) {
       kern<<<rows, threads, 0, stream>>>(x.data_ptr<float>(), ptr(y1), ptr(s1), ptr(y2), ptr(s2), static_cast<float>(mult),
-                                         reinterpret_cast<const T*>(w.data_ptr()), reinterpret_cast<T*>(h.data_ptr()), W, static_cast<float>(eps));
+                                         reinterpret_cast<const T*>(w.data_ptr()), reinterpret_cast<T*>(h.data_ptr()), W, static_cast<float>(eps),
+                                         static_cast<float>(offset));
     };
     const int nvec = (W + 3) / 4;
     const int vpt = nvec <= 512 ? 1 : (nvec <= 1024 ? 2 : 4);
@@ -480,6 +484,146 @@ torch::Tensor stream_rmsnorm(torch::Tensor x, const torch::Tensor& w, double eps
     else if (vpt == 1) go(stream_rmsnorm_kernel<T, 1>, threads);
     else if (vpt == 2) go(stream_rmsnorm_kernel<T, 2>, threads);
     else go(stream_rmsnorm_kernel<T, 4>, threads);
+  };
+  if (st == torch::kBFloat16) run(bf16{}); else run(float{});
+  count_launch();
+  TK_CUDA_CHECK(cudaGetLastError());
+  return h;
+}
+
+// -------------------------------------------------------- stream_gated_rmsnorm
+// One block per row, as above: gated result in registers, its mean square, the sum, the sum's mean square.  With k > 0 the result is
+// the weighted sum of the token's k ≤ 32 expert rows; their places and weights are read once per block.
+struct GatedNorm {
+  float* x;
+  const void *y, *gate, *bias, *post, *next;
+  void* h;
+  const int* row_of; const float* share;     // [rows, k] (k = 0: y has one row per token)
+  long ldg;                                  // row stride of the gate
+  int k, W;
+  float eps, offset;
+};
+
+template <typename T, int VPT>
+__global__ void stream_gated_rmsnorm_kernel(const GatedNorm p) {
+  __shared__ float sh[32];
+  __shared__ int s_row[32];
+  __shared__ float s_share[32];
+  const int W = p.W, t = blockIdx.x;
+  const T *y = reinterpret_cast<const T*>(p.y), *gate = reinterpret_cast<const T*>(p.gate) + t * p.ldg, *bias = reinterpret_cast<const T*>(p.bias);
+  const T *post = reinterpret_cast<const T*>(p.post), *next = reinterpret_cast<const T*>(p.next);
+  float* x = p.x + static_cast<size_t>(t) * W;
+  T* h = reinterpret_cast<T*>(p.h) + static_cast<size_t>(t) * W;
+  const int k = p.k;
+  if (k > 0) {
+    if (threadIdx.x < k) {
+      s_row[threadIdx.x] = p.row_of[static_cast<size_t>(t) * k + threadIdx.x];
+      s_share[threadIdx.x] = p.share[static_cast<size_t>(t) * k + threadIdx.x];
+    }
+    __syncthreads();
+  }
+  if constexpr (VPT > 0) {
+    float4 z[VPT], v[VPT];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * 4;
+      z[i] = v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < W) {
+        v[i] = load4(x + c);
+        const float4 g = load4(gate + c), b = load4(bias + c);
+        float4 a;
+        if (k == 0) {
+          a = load4(y + static_cast<size_t>(t) * W + c);
+        } else {
+          a = make_float4(0.f, 0.f, 0.f, 0.f);
+          for (int j = 0; j < k; ++j) {
+            const float4 e = load4(y + static_cast<size_t>(s_row[j]) * W + c);
+            const float w = s_share[j];
+            a.x += w * e.x; a.y += w * e.y; a.z += w * e.z; a.w += w * e.w;
+          }
+        }
+        z[i].x = a.x / (1.f + __expf(-(g.x + b.x))); z[i].y = a.y / (1.f + __expf(-(g.y + b.y)));
+        z[i].z = a.z / (1.f + __expf(-(g.z + b.z))); z[i].w = a.w / (1.f + __expf(-(g.w + b.w)));
+      }
+      ss += z[i].x * z[i].x + z[i].y * z[i].y + z[i].z * z[i].z + z[i].w * z[i].w;
+    }
+    const float r1 = rsqrtf(block_sum(ss, sh) / W + p.eps);
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * 4;
+      if (c < W) {
+        const float4 w = load4(post + c);
+        v[i].x += z[i].x * r1 * (p.offset + w.x); v[i].y += z[i].y * r1 * (p.offset + w.y);
+        v[i].z += z[i].z * r1 * (p.offset + w.z); v[i].w += z[i].w * r1 * (p.offset + w.w);
+        store4(x + c, v[i]);
+      }
+      ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    }
+    const float r2 = rsqrtf(block_sum(ss, sh) / W + p.eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * 4;
+      if (c < W) {
+        const float4 w = load4(next + c);
+        store4(h + c, make_float4(v[i].x * r2 * (p.offset + w.x), v[i].y * r2 * (p.offset + w.y), v[i].z * r2 * (p.offset + w.z), v[i].w * r2 * (p.offset + w.w)));
+      }
+    }
+  } else {                                   // any width: the gated result is formed twice
+    auto gated = [&](int c) {
+      float a = 0.f;
+      if (k == 0) a = to_f(y[static_cast<size_t>(t) * W + c]);
+      for (int j = 0; j < k; ++j) a += s_share[j] * to_f(y[static_cast<size_t>(s_row[j]) * W + c]);
+      return a / (1.f + __expf(-(to_f(gate[c]) + to_f(bias[c]))));
+    };
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < W; c += blockDim.x) { const float z = gated(c); ss += z * z; }
+    const float r1 = rsqrtf(block_sum(ss, sh) / W + p.eps);
+    ss = 0.f;
+    for (int c = threadIdx.x; c < W; c += blockDim.x) {
+      const float v = x[c] + gated(c) * r1 * (p.offset + to_f(post[c]));
+      x[c] = v;
+      ss += v * v;
+    }
+    const float r2 = rsqrtf(block_sum(ss, sh) / W + p.eps);
+    for (int c = threadIdx.x; c < W; c += blockDim.x) h[c] = from_f<T>(x[c] * r2 * (p.offset + to_f(next[c])));
+  }
+}
+
+// x [rows, W] fp32 is updated in place; returns the norm in w's dtype.  gate: [rows, ≥ W] with any row stride.
+torch::Tensor stream_gated_rmsnorm(torch::Tensor x, const torch::Tensor& w, double eps, double offset, const torch::Tensor& y, const torch::Tensor& gate,
+                                   const torch::Tensor& bias, const torch::Tensor& post, const OptT& row_of, const OptT& share) {
+  const auto st = w.scalar_type();
+  TORCH_CHECK(x.is_cuda() && x.scalar_type() == torch::kFloat32 && x.is_contiguous() && x.dim() == 2, "stream [rows, W] fp32 contiguous");
+  const int rows = x.size(0), W = x.size(1);
+  TORCH_CHECK(st == torch::kBFloat16 || st == torch::kFloat32, "bf16 or fp32");
+  for (const auto* t : {&w, &bias, &post}) TORCH_CHECK(t->scalar_type() == st && t->is_contiguous() && t->numel() == W, "norm weights and gate bias [W] in one dtype");
+  TORCH_CHECK(gate.scalar_type() == st && gate.dim() == 2 && gate.stride(1) == 1 && gate.size(0) == rows && gate.size(1) >= W, "gate [rows, >= W]");
+  TORCH_CHECK(y.scalar_type() == st && y.dim() == 2 && y.is_contiguous() && y.size(1) == W, "result [., W]");
+  GatedNorm p{};
+  if (has(row_of)) {
+    TORCH_CHECK(has(share) && row_of->scalar_type() == torch::kInt32 && share->scalar_type() == torch::kFloat32 && row_of->is_contiguous() && share->is_contiguous() &&
+                    row_of->dim() == 2 && row_of->size(0) == rows && share->sizes() == row_of->sizes() && row_of->size(1) >= 1 && row_of->size(1) <= 32, "row_of / share [rows, k], k <= 32");
+    p.k = row_of->size(1); p.row_of = row_of->data_ptr<int>(); p.share = share->data_ptr<float>();
+  } else {
+    TORCH_CHECK(y.size(0) == rows, "one result row per token");
+  }
+  c10::cuda::CUDAGuard guard(x.device());
+  auto h = torch::empty(x.sizes(), w.options());
+  if (rows == 0) return h;
+  p.x = x.data_ptr<float>(); p.y = y.data_ptr(); p.gate = gate.data_ptr(); p.bias = bias.data_ptr(); p.post = post.data_ptr(); p.next = w.data_ptr(); p.h = h.data_ptr();
+  p.ldg = gate.stride(0); p.W = W; p.eps = eps; p.offset = offset;
+  const bool vec = W % 4 == 0 && W <= 8192 && gate.stride(0) % 4 == 0 && aligned16(p.y) && aligned16(p.gate) && aligned16(p.bias) && aligned16(p.post) && aligned16(p.next);
+  const int nvec = (W + 3) / 4, vpt = nvec <= 512 ? 1 : (nvec <= 1024 ? 2 : 4);
+  auto stream = at::cuda::getCurrentCUDAStream();
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    const int threads = std::min(512, ((nvec + vpt - 1) / vpt + 31) / 32 * 32);
+    if (!vec) stream_gated_rmsnorm_kernel<T, 0><<<rows, std::min(512, (W + 31) / 32 * 32), 0, stream>>>(p);
+    else if (vpt == 1) stream_gated_rmsnorm_kernel<T, 1><<<rows, threads, 0, stream>>>(p);
+    else if (vpt == 2) stream_gated_rmsnorm_kernel<T, 2><<<rows, threads, 0, stream>>>(p);
+    else stream_gated_rmsnorm_kernel<T, 4><<<rows, threads, 0, stream>>>(p);
   };
   if (st == torch::kBFloat16) run(bf16{}); else run(float{});
   count_launch();

@@ -185,13 +185,71 @@ def conv_heads(proj: torch.Tensor, weight: Optional[torch.Tensor], positions: to
     return q.to(proj.dtype), k.to(proj.dtype), v.to(proj.dtype)
 
 
-def stream_rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype, adds=(), mult: float = 1.0):
-    """fp32 residual stream: ``x ← x + mult · Σ y_i ⊙ s_i`` over ``adds = [(y, s), …]``, then its RMS norm in ``out_dtype``.
-    Returns ``(norm, x)``."""
+def stream_rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype, adds=(), mult: float = 1.0, offset: float = 0.0):
+    """fp32 residual stream: ``x ← x + mult · Σ y_i ⊙ s_i`` over ``adds = [(y, s), …]``, then its RMS norm (weight ``offset + w``)
+    in ``out_dtype``.  Returns ``(norm, x)``."""
     x = x.float()
     if adds:
         x = x + mult * sum(y.float() * sc.float() for y, sc in adds)
-    return (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * weight.float()).to(out_dtype), x
+    return (x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * (weight.float() + offset)).to(out_dtype), x
+
+
+def stream_gated_rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, offset: float, result: torch.Tensor, gate: torch.Tensor, bias: torch.Tensor,
+                         post: torch.Tensor, row_of: Optional[torch.Tensor] = None, share: Optional[torch.Tensor] = None):
+    """fp32 residual stream: ``x ← x + norm(σ(gate + bias) ⊙ result; post)``, then the norm of the sum in ``weight``'s dtype; both
+    norms have weights ``offset + w``.  ``result [T, W]``, or expert rows of which token t has ``Σ_j share[t, j] · result[row_of[t, j]]``."""
+    y = result.float() if row_of is None else (result[row_of.long()].float() * share[..., None]).sum(1)
+    y = torch.sigmoid(gate[:, :x.shape[1]].float() + bias.float()) * y
+    x = x + y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * (post.float() + offset)
+    return stream_rmsnorm(x, weight, eps, weight.dtype, offset=offset)
+
+
+# ------------------------------------------- latent attention, HGRN2
+def latent_norms(proj: torch.Tensor, q0: int, nq: int, wq: torch.Tensor, c0: int, nc: int, wc: Optional[torch.Tensor], eps: float):
+    """RMS norms of the query-bottleneck and latent column ranges of a projection (``nc`` 0: no latent)."""
+    return rmsnorm(proj[:, q0:q0 + nq], wq, eps), rmsnorm(proj[:, c0:c0 + nc], wc, eps) if nc else None
+
+
+def latent_decode(q: torch.Tensor, pool: torch.Tensor, table: torch.Tensor, lens: torch.Tensor, scale: float, sinks: torch.Tensor, gate: Optional[torch.Tensor] = None):
+    """``q [B, H, R]`` against the cached latents of every sequence, which are key and value of all heads → ``[B, H, R]``."""
+    o = paged_attention_decode(q, pool[..., :q.shape[-1]], pool[..., :q.shape[-1]], table, lens, scale, sinks=sinks)
+    return o if gate is None else (o.float() * torch.sigmoid(gate.float())[..., None]).to(o.dtype)
+
+
+def hgrn2_gates(f: torch.Tensor, bias: torch.Tensor, lower: torch.Tensor) -> torch.Tensor:
+    """What a channel lets in, ``1 − forget gate = (1 − lower) · σ(−(f + bias))``, in fp32 (small values keep their digits)."""
+    return (1 - lower.float()) * torch.sigmoid(-(f.float() + bias.float()))
+
+
+def hgrn2_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, chunk: int = 16):
+    """``S ← (1 − k_t) ⊙ S + k_t v_tᵀ``, ``o_t = Sᵀ q_t`` over one sequence, fp32: ``q, k [T, H, d]``, ``v [T, H, e]``, ``state [H, d, e]`` →
+    ``(o [T, H, e], state)``.  Inside a chunk by the decay between every two tokens, one step per chunk."""
+    out = []
+    for a in range(0, q.shape[0], chunk):
+        qc, kc, vc = (t[a:a + chunk].transpose(0, 1) for t in (q, k, v))
+        G = torch.log1p(-kc).clamp_min(-60.0).cumsum(1)                                   # log decay since the chunk's start
+        n = G.shape[1]
+        past = torch.ones(n, n, dtype=torch.bool, device=q.device).tril()
+        D = (G[:, :, None] - G[:, None]).masked_fill(~past[None, :, :, None], float('-inf')).exp()       # [H, to, from, d]
+        A = torch.einsum('hid,hijd,hjd->hij', qc, D, kc)
+        out.append((A @ vc + (qc * G.exp()) @ state).transpose(0, 1))
+        state = state * G[:, -1].exp()[..., None] + (kc * D[:, -1]).transpose(1, 2) @ vc
+    return torch.cat(out), state
+
+
+def hgrn2(proj: torch.Tensor, q0: int, f0: int, v0: int, heads: int, dim: int, vdim: int, bias: torch.Tensor, lower: torch.Tensor, weight: torch.Tensor,
+          eps: float, bounds: List[int], states: Optional[List[torch.Tensor]] = None):
+    """The mixer between its projections, for packed rows of sequences at ``bounds``: ``(norm(o) [T, heads·vdim], last states)``."""
+    T, n, e = proj.shape[0], heads * dim, heads * vdim
+    q = F.silu(proj[:, q0:q0 + n].float()).view(T, heads, dim)
+    k = hgrn2_gates(proj[:, f0:f0 + n], bias, lower).view(T, heads, dim)
+    v = proj[:, v0:v0 + e].float().view(T, heads, vdim)
+    out, last = [], []
+    for i, (a, b) in enumerate(zip(bounds[:-1], bounds[1:])):
+        o, S = hgrn2_scan(q[a:b], k[a:b], v[a:b], states[i] if states is not None else q.new_zeros(heads, dim, vdim))
+        out.append(o)
+        last.append(S)
+    return rmsnorm(torch.cat(out), weight, eps).reshape(T, e).to(proj.dtype), last
 
 
 # -------------------------------------------------------------------- swiglu
@@ -212,6 +270,10 @@ def clamped_glu(gate_up: torch.Tensor, limit: float = 7.0, alpha: float = 1.702)
     g, u = gate_up.float().chunk(2, dim=-1)
     g, u = g.clamp(max=limit), u.clamp(-limit, limit)
     return ((u + 1.0) * g * torch.sigmoid(alpha * g)).to(gate_up.dtype)
+
+
+def relu2(x: torch.Tensor) -> torch.Tensor:
+    return F.relu(x.float()).square().to(x.dtype)
 
 
 # ----------------------------------------------------------------- attention

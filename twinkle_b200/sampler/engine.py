@@ -27,40 +27,46 @@ from ..models.parallel_layer import CacheView
 
 
 class PagedKVCache:
-    """Per layer K and V pools ``[num_blocks, block_size, Hkv, width]`` (key and value rows have the layer's own widths) + a
-    free list.  Layers with a short convolution in front of attention also have a history pool ``[num_slots, taps − 1,
-    channels]``; a sequence owns one slot of all of them.  Block 0 and slot 0 are never handed out so that the all-zero
-    rows that fill up a captured batch are harmless."""
+    """Per layer K and V pools ``[num_blocks, block_size, Hkv, width]`` (key and value rows have the layer's own widths; latent
+    attention keeps one row that serves as both, layers that keep nothing per token have no pool) + a free list.  Layers with a
+    short convolution in front of attention also have a history pool ``[num_slots, taps − 1, channels]``, recurrent layers an
+    fp32 state pool ``[num_slots, heads, dim, vdim]``; a sequence owns one slot of all of them.  Block 0 and slot 0 are never
+    handed out so that the all-zero rows that fill up a captured batch are harmless."""
 
     def __init__(self, cfg: DecoderConfig, num_blocks: int, block_size: int, device, dtype, num_slots: int = 0):
         self.cfg, self.block_size, self.num_blocks, self.device, self.dtype = cfg, block_size, num_blocks, device, dtype
-        self.num_slots = num_slots if any(cfg.conv_layout()) else 0
+        self.num_slots = num_slots if any(cfg.conv_layout()) or any(cfg.state_layout()) else 0
         self.build()
 
     def build(self) -> None:
         """(Re)create empty pools and free lists."""
         mk = lambda *shape: torch.zeros(shape, device=self.device, dtype=self.dtype)  # noqa: E731
         layout = self.cfg.kv_layout()
-        self.k = [mk(self.num_blocks, self.block_size, h, d) for h, d, _ in layout]
-        self.v = [mk(self.num_blocks, self.block_size, h, e) for h, _, e in layout]
-        conv = self.cfg.conv_layout() or [None] * len(layout)
-        self.conv = [mk(self.num_slots, *c) if c else None for c in conv]
+        self.k = [mk(self.num_blocks, self.block_size, h, d) if h * d else None for h, d, _ in layout]
+        self.v = [mk(self.num_blocks, self.block_size, h, e) if h * e else None for h, _, e in layout]
+        none = [None] * len(layout)
+        self.conv = [mk(self.num_slots, *c) if c else None for c in self.cfg.conv_layout() or none]
+        self.state = [torch.zeros(self.num_slots, *c, device=self.device) if c else None for c in self.cfg.state_layout() or none]
         self.free: List[int] = list(range(self.num_blocks - 1, 0, -1))
         self.free_slots: List[int] = list(range(self.num_slots - 1, 0, -1))
 
     def drop(self) -> None:
         """Give the pools' memory back (``build`` makes new ones)."""
-        self.k = self.v = self.conv = None
+        self.k = self.v = self.conv = self.state = None
 
     @staticmethod
     def block_bytes(cfg: DecoderConfig, block_size: int, elem: int) -> int:
         return elem * block_size * sum(h * (d + e) for h, d, e in cfg.kv_layout())
 
+    @staticmethod
+    def slot_bytes(cfg: DecoderConfig, elem: int) -> int:
+        return elem * sum(math.prod(c) for c in cfg.conv_layout() if c) + 4 * sum(math.prod(c) for c in cfg.state_layout() if c)
+
     def allocate_slot(self) -> int:
         if not self.num_slots:
             return 0
         if not self.free_slots:
-            raise RuntimeError(f'convolution history exhausted: {self.num_slots - 1} sequences are live')
+            raise RuntimeError(f'per-sequence state exhausted: {self.num_slots - 1} sequences are live')
         return self.free_slots.pop()
 
     def release_slot(self, slot: int) -> None:
@@ -98,7 +104,7 @@ class _Seq:
     lora_scale: float = 0.0
     lora_target: Any = None
     blocks: List[int] = field(default_factory=list)
-    state_slot: int = 0     # row of the convolution-history pools
+    state_slot: int = 0     # row of the convolution-history and state pools
     tokens: List[int] = field(default_factory=list)
     logprobs: List[float] = field(default_factory=list)
     topk: List[List[Tuple[int, float]]] = field(default_factory=list)
@@ -124,10 +130,12 @@ class NativeEngine:
         self.device = device or next(model.parameters()).device
         self.dtype = next(model.parameters()).dtype
         if num_blocks is None:
-            per_block = PagedKVCache.block_bytes(cfg, block_size, 2 if self.dtype != torch.float32 else 4)
-            if self.device.type == 'cuda':
+            elem = 2 if self.dtype != torch.float32 else 4
+            per_block = PagedKVCache.block_bytes(cfg, block_size, elem)
+            if self.device.type == 'cuda' and per_block:
                 free, _ = torch.cuda.mem_get_info(self.device)
-                num_blocks = max(int(free * gpu_memory_utilization * 0.9 // per_block), 64)
+                free = free * gpu_memory_utilization * 0.9 - (max_batch + 1) * PagedKVCache.slot_bytes(cfg, elem)
+                num_blocks = max(int(free // per_block), 64)
             else:
                 num_blocks = 1024
         self.cache = PagedKVCache(cfg, num_blocks, block_size, self.device, self.dtype, num_slots=max_batch + 1)
@@ -149,7 +157,7 @@ class NativeEngine:
 
     # -------------------------------------------------- what a sequence holds
     def admit(self, seqs: Sequence[_Seq]) -> None:
-        """Blocks for the prompt, the tokens it may generate and one more, and a convolution-history slot."""
+        """Blocks for the prompt, the tokens it may generate and one more, and a slot for convolution history and state."""
         for s in seqs:
             s.blocks = self.cache.allocate(self.cache.blocks_for(len(s.prompt) + (s.params.max_tokens or 0) + 1))
             s.state_slot = self.cache.allocate_slot()

@@ -82,7 +82,7 @@ class TorchSampler(Sampler, CheckpointEngineMixin):
             for n, p in self.model.named_parameters():
                 if 'lora' in n:
                     continue
-                if n == 'lm_head.weight' and 'lm_head.weight' not in loader:
+                if n == 'lm_head.weight' and self.config.layer_specs is None and 'lm_head.weight' not in loader:
                     p.copy_(loader.get('model.embed_tokens.weight'))
                 else:
                     p.copy_(hf_to_internal(n, self.config, loader.get).to(p.dtype))
