@@ -58,11 +58,12 @@ def parse():
     ap.add_argument('--sp', type=int, default=None, help='Ulysses degree (default min(4, gpus))')
     ap.add_argument('--ref-micro', type=int, default=1, help='reference arm: sequences per forward_backward call')
     ap.add_argument('--cpu-debug', action='store_true', help='reference arm: run on CPU/gloo (debug only, result invalid)')
-    ap.add_argument('--config', default='both', choices=['both', 'dense', 'moe', 'serve'],
+    ap.add_argument('--config', default='both', choices=['both', 'dense', 'moe', 'serve', 'serve-moe'],
                     help="dense: Qwen3-8B full-parameter SFT; moe: Qwen3-30B-A3B LoRA r=16 SFT with expert parallel = gpus; "
                          "both (default): the two halves of the headline metric one after the other, each in a process of its own, "
                          "printed as one line (the dense fields at top level, the mixture-of-experts result under 'moe'); "
-                         "serve: prefill and decode throughput of Pomelix stacks beside Qwen3 at equal sizes (one GPU, random weights)")
+                         "serve: prefill and decode throughput of Pomelix stacks beside Qwen3 at equal sizes (one GPU, random weights); "
+                         "serve-moe: likewise of a Moronex stack beside Qwen3-30B-A3B and a Qwen3-Next style hybrid (24 layers of each)")
     ap.add_argument('--moe-steps', type=int, default=10, help="cap on timed steps of the 'moe' half when --config both")
     return ap.parse_args()
 
@@ -198,32 +199,42 @@ def run_both(args):
 
 
 def run_serve(args):
-    """Prefill and decode throughput of the sampler's engine: Pomelix presets and the Qwen3 presets of the same sizes."""
+    """Prefill and decode throughput of the sampler's engine: Pomelix presets and the Qwen3 presets of the same sizes, or
+    (``serve-moe``) a Moronex preset beside the mixture-of-experts models of the same size."""
     import torch
     from twinkle_b200 import ops
     from twinkle_b200.models.config import preset
     from twinkle_b200.sampler.bench import measure
     torch.cuda.set_device(0)
-    over = {} if args.layers is None else {'num_hidden_layers': args.layers}
+    moe = args.config == 'serve-moe'
+    layers = args.layers or (24 if moe else None)
+    over = {} if layers is None else {'num_hidden_layers': layers}
+    if moe:
+        headline = 'moronex-30b-a3b'
+        # three Gated DeltaNet layers per attention layer, 16 heads of 128 x 128 state like the recurrent layers of the preset beside it
+        kinds = [('full_attention' if i % 4 == 3 else 'linear_attention') for i in range(layers)]
+        configs = {headline: preset(headline, **over), 'qwen3-30b-a3b': preset('qwen3-30b-a3b', **over),
+                   'qwen3-next style': preset('qwen3-30b-a3b', model_type='qwen3_next', layer_types=kinds, linear_num_key_heads=16, linear_num_value_heads=16, **over)}
+    else:
+        headline = 'pomelix-8b'
+        configs = {f'{f}-{n}': preset(f'{f}-{n}', tie_word_embeddings=True, **over) for n in ('0.6b', '8b') for f in ('qwen3', 'pomelix')}
     clock = ClockSampler(0)
     clock.start()
     launches, res = ops.ext().launch_count(), {}
-    for size in ('0.6b', '8b'):
-        for family in ('qwen3', 'pomelix'):
-            cfg = preset(f'{family}-{size}', tie_word_embeddings=True, **over)
-            res[f'{family}-{size}'] = dict(measure(cfg, [(8, 1024), (1, 8192)], [(1, 1024), (16, 1024), (64, 1024), (256, 1024)], args.steps, max(args.warmup, 3)),
-                                           parameters=cfg.num_params())
+    for name, cfg in configs.items():
+        res[name] = dict(measure(cfg, [(8, 1024), (1, 8192)], [(1, 1024), (16, 1024), (64, 1024), (256, 1024)], args.steps, max(args.warmup, 3)),
+                         parameters=cfg.num_params())
     clocks = clock.stop()
-    value = res['pomelix-8b']['decode'][2]['tokens_per_s']
-    print(json.dumps({'metric': 'decode tokens/s, pomelix-8b, 64 sequences of 1024 tokens', 'value': value, 'unit': 'tokens/s', 'n_gpus': 1, 'steps': args.steps,
+    value = res[headline]['decode'][2]['tokens_per_s']
+    print(json.dumps({'metric': f'decode tokens/s, {headline}, 64 sequences of 1024 tokens', 'value': value, 'unit': 'tokens/s', 'n_gpus': 1, 'steps': args.steps,
                       'warmup': max(args.warmup, 3), 'higher_is_better': True, 'vs_baseline': None, 'dtype': 'bf16', 'data': 'synthetic (random-init weights)', 'impl': 'ours',
-                      'config': {'l2': 'weights read per step exceed the 126 MB L2', 'layers': args.layers}, 'models': res, 'clocks': clocks,
+                      'config': {'l2': 'weights read per step exceed the 126 MB L2', 'layers': layers}, 'models': res, 'clocks': clocks,
                       'gpu_launches': int(ops.ext().launch_count() - launches), 'kernel_error_word': ops.ext().read_and_clear_error()}), flush=True)
 
 
 def main():
     args = parse()
-    if args.config == 'serve' and args.impl == 'ours':
+    if args.config.startswith('serve') and args.impl == 'ours':
         run_serve(args)
         return
     if args.config == 'both':

@@ -131,3 +131,88 @@ def forward(cfg, weights, tokens, dtype=torch.float64):
             x = join(x, y, h, W[p + 'rg2'], W[p + 'rg2.b'], W[p + 'norm2b'], eps)
         trail.append(x)
     return norm_about_one(x, W['final.norm'], eps) @ W['head'].t(), trail
+
+
+# ---------------------------------------------------------------- models for the tests
+def recurrent(heads, dim, vdim, mlp=None):
+    return {'type': 'hgrn2', 'mixer': {'heads': heads, 'dim': dim, 'vdim': vdim}, 'mlp': mlp}
+
+
+def latents(heads, dim, vdim, q_rank, kv_rank, scale, mlp=None, kv_from=None):
+    m = {'heads': heads, 'dim': dim, 'vdim': vdim, 'q_rank': q_rank, 'kv_rank': kv_rank, 'scale': scale}
+    if kv_from is not None:
+        m['kv_from'] = kv_from
+    return {'type': 'latent_attention', 'mixer': m, 'mlp': mlp}
+
+
+def dense(ff):
+    return {'kind': 'dense', 'ff': ff}
+
+
+def moe(experts, top, ff):
+    return {'kind': 'moe', 'expert': {'ff': ff}, 'router': {'experts': experts, 'top': top}}
+
+
+CONFIGS = {
+    # layers of unequal sizes and every kind of feed-forward; two layers borrow latents, one of them over a distance
+    'mixed': dict(vocab=120, width=96, norm={'eps': 1e-5},
+                  layers=[recurrent(3, 24, 40, dense(64)), latents(5, 24, 40, 56, 48, 0.3, moe(6, 2, 32)), recurrent(4, 32, 16),
+                          latents(2, 40, 24, 24, 48, 0.25, moe(5, 3, 40), kv_from=1), latents(4, 16, 32, 32, 64, 0.4), recurrent(2, 16, 64, moe(4, 4, 16)),
+                          latents(3, 32, 16, 40, 48, 0.2, dense(56), kv_from=1)]),
+    # sizes that are no whole vectors, attention first, one head, one expert, ranks below the head width
+    'odd': dict(vocab=97, width=52, norm={'eps': 1e-3},
+                layers=[latents(3, 7, 11, 9, 13, 0.5, moe(3, 1, 20)), recurrent(5, 6, 9, moe(1, 1, 36)), latents(1, 12, 5, 4, 13, 0.4, dense(18), kv_from=0),
+                        recurrent(1, 4, 6), recurrent(2, 33, 20, dense(12))]),
+    # head widths on both sides of 64, 128 and at 256, ranks up to 512
+    'wide': dict(vocab=64, width=72, norm={'eps': 1e-6},
+                 layers=[recurrent(1, 160, 256, dense(40)), latents(2, 160, 136, 40, 264, 0.08, moe(8, 3, 24)), recurrent(2, 128, 128), recurrent(2, 64, 136, dense(24)),
+                         latents(20, 64, 128, 96, 512, 0.1), latents(3, 128, 72, 96, 512, 0.09, kv_from=4)]),
+}
+for _c in CONFIGS.values():
+    _c['architecture'] = 'Moronex'
+
+
+def random_weights(cfg, seed=0):
+    """Weights under their checkpoint names, every value representable in bfloat16.  Forget gates reach from nearly open to nearly
+    closed, sinks weigh as much as a few keys."""
+    g = torch.Generator().manual_seed(seed)
+    rnd = lambda *s: torch.randn(*s, generator=g)  # noqa: E731
+    mat = lambda o, i: rnd(o, i) / i**0.5  # noqa: E731
+    width = cfg['width']
+    W = {'embed': rnd(cfg['vocab'], width), 'final.norm': 0.2 * rnd(width), 'head': mat(cfg['vocab'], width)}
+    for i, layer in enumerate(cfg['layers']):
+        p, m, f = f'l{i}.', layer['mixer'], layer['mlp']
+        H, d, e = m['heads'], m['dim'], m['vdim']
+        for n in ('1', '2') if f else ('1', ):
+            W[p + f'norm{n}'], W[p + f'norm{n}b'] = 0.2 * rnd(width), 0.2 * rnd(width)
+            W[p + f'rg{n}'], W[p + f'rg{n}.b'] = mat(width, width), rnd(width)
+        if layer['type'] == 'hgrn2':
+            W[p + 'mix.q'], W[p + 'mix.f'], W[p + 'mix.v'] = mat(H * d, width), mat(H * d, width), mat(H * e, width)
+            W[p + 'mix.f.b'], W[p + 'mix.lower'] = 2 + 3 * rnd(H * d), torch.rand(H * d, generator=g) * 0.9
+            W[p + 'mix.norm'] = 1 + 0.2 * rnd(e)
+        else:
+            r = m['kv_rank']
+            W[p + 'mix.dq'], W[p + 'mix.dq.norm'], W[p + 'mix.uq'] = mat(m['q_rank'], width), 1 + 0.2 * rnd(m['q_rank']), mat(H * d, m['q_rank'])
+            if m.get('kv_from') is None:
+                W[p + 'mix.dkv'], W[p + 'mix.dkv.norm'] = mat(r, width), 1 + 0.2 * rnd(r)
+            W[p + 'mix.uk'], W[p + 'mix.uv'], W[p + 'mix.sink'], W[p + 'mix.g'] = mat(H * d, r), mat(H * e, r), 2 + rnd(H), mat(H, width)
+        W[p + 'mix.o'] = mat(width, H * e)
+        if f and f['kind'] == 'dense':
+            W[p + 'mlp.gate'], W[p + 'mlp.up'], W[p + 'mlp.down'] = mat(f['ff'], width), mat(f['ff'], width), mat(width, f['ff'])
+        elif f:
+            n, ff = f['router']['experts'], f['expert']['ff']
+            W[p + 'mlp.router'], W[p + 'mlp.router.b'] = 2 * mat(n, width), 0.5 * rnd(n)
+            for x in range(n):
+                W[p + f'mlp.e{x}.up'], W[p + f'mlp.e{x}.down'] = mat(ff, width), mat(width, ff)
+    return {n: t.to(torch.bfloat16) for n, t in W.items()}
+
+
+def write_checkpoint(path, cfg, weights):
+    import json
+    import os
+    from safetensors.torch import save_file
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, 'config.json'), 'w') as f:
+        json.dump(cfg, f)
+    save_file({n: t.contiguous() for n, t in weights.items()}, os.path.join(path, 'model.safetensors'))
+    return str(path)

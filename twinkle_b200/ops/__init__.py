@@ -996,6 +996,8 @@ def grouped_gemm(x, weight, offsets, act: Optional[str] = None):
     off = offsets.tolist()
     for e in range(weight.shape[0]):
         outs.append(x[off[e]:off[e + 1]] @ weight[e].t().to(x.dtype))
+    if off[-1] < x.shape[0]:        # rows behind the last expert belong to nobody
+        outs.append(x.new_zeros(x.shape[0] - off[-1], weight.shape[1]))
     return torch.cat(outs, 0)
 
 

@@ -145,10 +145,13 @@ torch::Tensor moe_rows_gather(const torch::Tensor& x, const torch::Tensor& src, 
   switch (K) {                                                 \
     case 1: { constexpr int KK = 1; BODY; break; }             \
     case 2: { constexpr int KK = 2; BODY; break; }             \
+    case 3: { constexpr int KK = 3; BODY; break; }             \
     case 4: { constexpr int KK = 4; BODY; break; }             \
+    case 5: { constexpr int KK = 5; BODY; break; }             \
     case 6: { constexpr int KK = 6; BODY; break; }             \
+    case 7: { constexpr int KK = 7; BODY; break; }             \
     case 8: { constexpr int KK = 8; BODY; break; }             \
-    default: TORCH_CHECK(false, "top-k must be 1, 2, 4, 6 or 8"); \
+    default: TORCH_CHECK(false, "top-k must be 1 to 8");        \
   }
 
 torch::Tensor moe_rows_combine(const torch::Tensor& y, const torch::Tensor& row_of, const c10::optional<torch::Tensor>& w) {

@@ -106,6 +106,89 @@ def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
         # of it written by a step, negligible for prompts)
         byts = 2.0 * T * d * (hq + 2 * hkv + hq + hkv + (0 if step else hkv) + 2 * hkv + hkv) + (2.0 * T * C * taps if step else 0.0)
         return (lambda: E.conv_heads(proj, w, pos, hq, hkv, d, d, 1e-5, 0.1, 4096, vf, lam, step, hist, slot, left, rows, kp, vp, not step)), 0.0, byts
+    if op in ('hgrn2', 'hgrn2_step', 'gdn_step'):
+        # the recurrent mixer between its projections: --heads states of 128 x 128 (prompts of --seq tokens, or a token of --batch
+        # sequences); gdn_step: the Gated DeltaNet recurrence on one token of every sequence
+        H, d, step = a.heads, a.width, op != 'hgrn2'
+        T = a.batch if step else a.tokens
+        if op == 'gdn_step':
+            q, k, v = (torch.randn(T, H, d, device=dev, dtype=bf) for _ in range(3))
+            g, beta, S = -torch.rand(T, H, device=dev) * 0.1, torch.rand(T, H, device=dev), torch.zeros(T, H, d, d, device=dev)
+            cu = torch.arange(T + 1, device=dev, dtype=torch.int32)
+            return (lambda: ops.gated_delta_rule_varlen(q, k, v, g, beta, cu, init_state=S, return_states=True)), 0.0, 8.0 * T * H * d * d
+        proj = torch.randn(T, a.hidden + 3 * H * d, device=dev, dtype=bf)
+        bias, low, w = torch.zeros(H * d, device=dev, dtype=bf), torch.zeros(H * d, device=dev, dtype=bf), torch.ones(d, device=dev, dtype=bf)
+        n_seq = T if step else max(T // a.seq, 1)
+        pool = torch.zeros(n_seq + 1, H, d, d, device=dev)
+        args = (proj, a.hidden, a.hidden + H * d, a.hidden + 2 * H * d, H, d, d, bias, low, w, 1e-6)
+        if step:
+            slot = torch.arange(T, device=dev, dtype=torch.int32) + 1
+            return (lambda: E.hgrn2_step(*args, pool, slot)), 0.0, 8.0 * T * H * d * d + 8.0 * T * H * d
+        cu = torch.arange(0, n_seq + 1, device=dev, dtype=torch.int32) * a.seq
+        slot = (torch.arange(T, device=dev) // a.seq).int() + 1
+        # flops as for 'gdn' per state element and token: a write (multiply, add) and a read (multiply, add)
+        return (lambda: E.hgrn2_prefill(*args, cu, a.seq, pool, slot)), 2.0 * T * H * d * d * 2, 8.0 * T * H * d
+    if op == 'latent_decode':
+        # --heads heads against latents of --rank (the like kernel: paged_decode)
+        B, bs, ctx, R = a.batch, 16, a.seq, a.rank
+        nb = B * ((ctx + bs - 1) // bs) + 1
+        pool = torch.randn(nb, bs, 1, R, device=dev, dtype=bf)
+        tables = torch.arange(1, nb, device=dev, dtype=torch.int32).view(B, -1)
+        lens = torch.full((B, ), ctx, device=dev, dtype=torch.int32)
+        q, sinks, gate = torch.randn(B, a.heads, R, device=dev, dtype=bf), torch.zeros(a.heads, device=dev, dtype=bf), torch.zeros(B, a.heads, device=dev, dtype=bf)
+        return (lambda: E.latent_decode(q, pool, tables, lens, R**-0.5, sinks, gate)), 4.0 * B * ctx * a.heads * R, 2.0 * B * ctx * R + 4.0 * B * a.heads * R
+    if op == 'latent_norms':
+        p = torch.randn(a.tokens, a.hidden + 1536 + 32, device=dev, dtype=bf)
+        wq, wc = torch.ones(1024, device=dev, dtype=bf), torch.ones(512, device=dev, dtype=bf)
+        pool, rows = torch.zeros(a.tokens, 1, 1, 512, device=dev, dtype=bf), torch.arange(a.tokens, device=dev)
+        return (lambda: E.latent_norms(p, a.hidden, 1024, wq, a.hidden + 1024, 512, wc, 1e-6, pool, rows)), 0.0, 2.0 * a.tokens * (2 * 1536 + 512)
+    if op == 'head_gemm':
+        # the query into latent space: --batch tokens, --heads products of --width x --rank
+        x, w = torch.randn(a.batch, a.heads, a.width, device=dev, dtype=bf), torch.randn(a.heads, a.width, a.rank, device=dev, dtype=bf)
+        return (lambda: E.head_gemm(x, w, True)), 2.0 * a.batch * a.heads * a.width * a.rank, 2.0 * (x.numel() + w.numel() + a.batch * a.heads * a.rank)
+    if op in ('gated_norm', 'gated_norm_experts'):
+        W, k = a.hidden, 8
+        x, g, w = torch.zeros(a.tokens, W, device=dev), torch.randn(a.tokens, W + 4096, device=dev, dtype=bf), torch.zeros(W, device=dev, dtype=bf)
+        y = torch.randn(a.tokens * (k if op.endswith('experts') else 1), W, device=dev, dtype=bf)
+        row_of = torch.randperm(a.tokens * k, device=dev, dtype=torch.int32).view(-1, k) if op.endswith('experts') else None
+        share = torch.full((a.tokens, k), 1 / k, device=dev) if op.endswith('experts') else None
+        return (lambda: E.stream_gated_rmsnorm(x, w, 1e-6, 1.0, y, g, w, w, row_of, share)), 0.0, a.tokens * W * (12.0 + 2.0 * (k if op.endswith('experts') else 1))
+    if op in ('moe_topk', 'moe_group', 'moe_layout', 'moe_combine'):
+        # choice and grouping of --tokens rows of --hidden over 128 experts, top 8; moe_layout: sort, index maps and gather of the
+        # training block, moe_combine: its weighted sum
+        T, k, Ex = a.tokens, 8, 128
+        lg, x = torch.randn(T, Ex, device=dev), torch.randn(T, a.hidden, device=dev, dtype=bf)
+        if op == 'moe_topk':
+            return (lambda: E.moe_topk(lg, None, k, None)), 0.0, 4.0 * T * Ex + 12.0 * T * k
+        w, idx, hist = E.moe_topk(lg, None, k, None)
+        byts = 2.0 * T * a.hidden * (1 + k)
+        if op == 'moe_group':
+            return (lambda: E.moe_group_rows(x, idx, hist)), 0.0, byts
+        from twinkle_b200.parallel.expert import expert_layout
+
+        def layout():
+            order, rows, offsets, bound = expert_layout(idx.reshape(-1), Ex, 128, hist)
+            maps = ops.moe_index_maps(order, rows, bound, k)
+            return maps, ops.moe_dispatch(x, maps[1], maps[0])
+        if op == 'moe_layout':
+            return layout, 0.0, byts
+        (row_of, src, slot_of), xs = layout()
+        return (lambda: ops.moe_combine(xs, w, row_of, src, slot_of)), 0.0, byts
+    if op in ('experts_relu2', 'experts_swiglu'):
+        # both products of the experts of one layer: two matrices with the activation in the epilogue, or [gate | up] and down
+        T, k, Ex, W = a.tokens, 8, 128, a.hidden
+        ff = 1152 if op == 'experts_relu2' else 768
+        up = torch.randn(Ex, ff if op == 'experts_relu2' else 2 * ff, W, device=dev, dtype=bf) * 0.02
+        down = torch.randn(Ex, W, ff, device=dev, dtype=bf) * 0.02
+        _, idx, hist = E.moe_topk(torch.randn(T, Ex, device=dev), None, k, None)
+        xs, _, off = E.moe_group_rows(torch.randn(T, W, device=dev, dtype=bf), idx, hist)
+
+        def f():
+            with torch.no_grad():
+                h = ops.grouped_gemm(xs, up, off, act='relu2') if op == 'experts_relu2' else ops.swiglu(ops.grouped_gemm(xs, up, off))
+                ops.grouped_gemm(h, down, off)
+        used = min(Ex, T * k)
+        return f, 2.0 * T * k * (up.shape[1] * W + W * ff), 2.0 * used * (up.shape[1] * W + W * ff)
     if op in ('stream_norm', 'add_rmsnorm'):
         w, y = torch.ones(a.hidden, device=dev, dtype=bf), torch.randn(a.tokens, a.hidden, device=dev, dtype=bf)
         if op == 'add_rmsnorm':
@@ -122,7 +205,9 @@ def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
         n_seq = max(T // a.seq, 1)
         cu = torch.arange(0, n_seq + 1, device=dev, dtype=torch.int32) * a.seq
         q, k, v = (torch.randn(T, h, d, device=dev, dtype=dt) for h in (a.heads, a.kv_heads, a.kv_heads))
-        return ((lambda: ops.attention_packed(q, k, v, cu, a.seq, d**-0.5)), 4.0 * n_seq * a.seq * a.seq * a.heads * d / 2,
+        sinks = torch.zeros(a.heads, device=dev, dtype=dt) if a.sinks else None
+        gate = torch.zeros(T, a.heads, device=dev, dtype=dt) if a.sinks else None
+        return ((lambda: ops.attention_packed(q, k, v, cu, a.seq, d**-0.5, sinks, gate)), 4.0 * n_seq * a.seq * a.seq * a.heads * d / 2,
                 float(q.element_size()) * T * d * (2 * a.heads + 2 * a.kv_heads))
     if op == 'rmsnorm':
         x, w = torch.randn(a.tokens, a.hidden, device=dev, dtype=bf), torch.ones(a.hidden, device=dev, dtype=bf)
@@ -257,6 +342,7 @@ def main() -> None:
     ap.add_argument('--heads', type=int, default=32)
     ap.add_argument('--kv-heads', type=int, default=8)
     ap.add_argument('--width', type=int, default=128, help='head width')
+    ap.add_argument('--sinks', action='store_true', help='attn_packed: with sink logits and output gates')
     ap.add_argument('--hidden', type=int, default=4096)
     ap.add_argument('--vocab', type=int, default=151936)
     ap.add_argument('--batch', type=int, default=256)
