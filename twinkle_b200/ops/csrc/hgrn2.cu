@@ -5,12 +5,19 @@
 //
 // Forming k instead of the forget gate keeps the digits of gates close to one, and the update above needs no decay beside it.
 //
-//   hgrn2_prefill  packed prompts.  A block owns one head of one sequence (or of one time segment of it) and keeps the state in
-//                  registers: RS neighbouring lanes share two columns, each with RPT of the rows, so a token costs three
-//                  operations per state element, two 16-byte shared-memory broadcasts per twelve of them and a shuffle per column.
-//                  Sixteen tokens at a time are brought in by asynchronous copies while the sixteen before are worked on.
-//                  When sequences × heads do not fill the device, sequences are cut into time segments: a first pass forms each
-//                  segment's own contribution and decay, a scan over segments gives every segment its starting state.
+//   hgrn2_prefill  packed prompts; a block owns one head of one sequence (or of one time segment of it), the state is in registers.
+//     bf16: sixteen tokens per step on the tensor cores (``hgrn2_chunk_kernel``).  With P_t the product of the forget gates from
+//           the step's start through t, R_j the product behind j, and D the whole step's:
+//               o_t = Σ_{j ≤ t} A_tj v_j + Sᵀ (q_t P_t),   A_tj = Σ_d q_td k_jd Π_{j < s ≤ t} f_sd,   S ← D S + Σ_j (k_j R_j) v_jᵀ
+//           Only products of gates occur, never a quotient or a logarithm, so nothing overflows however fast a channel forgets.
+//           Operands that are not bf16 already (state, q P, k R, A) go in as a bf16 value plus the bf16 of what it left over:
+//           products keep 16 bits and more, sums are fp32, and the state itself is never rounded.
+//     else: token by token in fp32 (``hgrn2_prefill_kernel``): RS neighbouring lanes share two columns, each with RPT of the rows, so a
+//           token costs three operations per state element, two 16-byte shared-memory broadcasts per twelve of them and a shuffle
+//           per column.
+//     Tokens are brought in by asynchronous copies while those before are worked on.  When sequences × heads do not fill the
+//     device, sequences are cut into time segments: a first pass forms each segment's own contribution and decay, a scan over
+//     segments gives every segment its starting state.
 //   hgrn2_step     one token of every sequence: the state passes once through the block, 16 bytes per access.
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
@@ -227,6 +234,316 @@ __global__ void __launch_bounds__(256) hgrn2_prefill_kernel(const Hgrn2<T> p) {
   }
 }
 
+// ------------------------------------------------------------------ sixteen tokens per step on the tensor cores
+namespace hg {
+constexpr int TOK = 32;         // tokens per round: two steps
+
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const bf16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const bf16* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// two values as bf16 pairs: the rounded ones and what the rounding left over
+__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16(x, y);
+  const float2 h = unpack_bf16(hi);
+  lo = pack_bf16(x - h.x, y - h.y);
+}
+__device__ __forceinline__ void split(float x, bf16* hi, bf16* lo) {
+  const bf16 h = __float2bfloat16(x);
+  *hi = h;
+  *lo = __float2bfloat16(x - __bfloat162float(h));
+}
+// shared memory of a block, in bytes from its start
+struct Layout {
+  int q, k, qh, ql, kh, kl, a, v, rq, rf, d, low, ss, total, po;
+  __host__ __device__ Layout(int DP, int VP) {
+    const int pitch = DP + 8;
+    po = VP + 4;                                         // row pitch of the outputs, which take the place of q and k
+    q = 0;
+    k = q + TOK * DP * 4;
+    int at = k + TOK * DP * 4;
+    if (at < TOK * po * 4) at = TOK * po * 4;
+    qh = at; ql = qh + TOK * pitch * 2; kh = ql + TOK * pitch * 2; kl = kh + TOK * pitch * 2;
+    a = kl + TOK * pitch * 2;                            // [2 steps][hi, lo][16][24]
+    v = a + 2 * 2 * 16 * 24 * 2;                         // [2][TOK][VP + 8]
+    rq = v + 2 * TOK * (VP + 8) * 2; rf = rq + TOK * DP * 2;
+    d = rf + TOK * DP * 2;                               // [2 steps][DP]
+    low = d + 2 * DP * 4;                                // [DP] lower bound, [DP] bias
+    ss = low + 2 * DP * 4;                               // [8 warps][TOK]
+    total = ss + 8 * TOK * 4;
+  }
+};
+}  // namespace hg
+
+// A warp owns 16 columns of the head's values: Sᵀ [16, DP] lies in its registers as accumulators of Vᵀ (k R) and, packed, as the
+// left operand of Sᵀ (q P)ᵀ.  PART: only the state a segment builds up from nothing and its decay.
+template <int DP, bool PART>
+__global__ void __launch_bounds__(256, 2) hgrn2_chunk_kernel(const Hgrn2<bf16> p) {
+  using namespace hg;
+  extern __shared__ __align__(16) uint8_t sm_chunk[];
+  constexpr int PITCH = DP + 8, NT = DP / 8, DS = DP / 8;     // DS: lanes that share the sum over a head's width
+  const int head = blockIdx.x / p.slices, slice = blockIdx.x - head * p.slices, seg = blockIdx.y, seq = blockIdx.z;
+  const int s0 = p.cu[seq], len = p.cu[seq + 1] - s0;
+  const int a = seg * p.seg_len, b = min(len, a + p.seg_len);
+  if (a >= len || (PART && b >= len)) return;
+  const int col0 = slice * p.cols, ncol = min(p.cols, p.vdim - col0);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, warps = blockDim.x >> 5, VP = warps * 16, VPITCH = VP + 8;
+  const Layout L(DP, VP);
+  float *s_q = reinterpret_cast<float*>(sm_chunk + L.q), *s_k = reinterpret_cast<float*>(sm_chunk + L.k), *s_o = s_q;
+  bf16 *s_qh = reinterpret_cast<bf16*>(sm_chunk + L.qh), *s_ql = reinterpret_cast<bf16*>(sm_chunk + L.ql), *s_kh = reinterpret_cast<bf16*>(sm_chunk + L.kh),
+       *s_kl = reinterpret_cast<bf16*>(sm_chunk + L.kl), *s_a = reinterpret_cast<bf16*>(sm_chunk + L.a), *s_v = reinterpret_cast<bf16*>(sm_chunk + L.v),
+       *r_q = reinterpret_cast<bf16*>(sm_chunk + L.rq), *r_f = reinterpret_cast<bf16*>(sm_chunk + L.rf);
+  float *s_d = reinterpret_cast<float*>(sm_chunk + L.d), *s_low = reinterpret_cast<float*>(sm_chunk + L.low), *s_bias = s_low + DP,
+        *s_ss = reinterpret_cast<float*>(sm_chunk + L.ss);
+  for (int i = tid; i < DP; i += blockDim.x) {
+    s_low[i] = i < p.dim ? ld(p.lower + static_cast<size_t>(head) * p.dim + i) : 1.f;
+    s_bias[i] = i < p.dim ? ld(p.bias + static_cast<size_t>(head) * p.dim + i) : 0.f;
+  }
+  for (int i = tid; i < TOK * DP; i += blockDim.x) r_q[i] = r_f[i] = __float2bfloat16(0.f);      // columns past the head's width
+  for (int i = tid; i < 2 * TOK * VPITCH; i += blockDim.x) s_v[i] = __float2bfloat16(0.f);
+  __syncthreads();
+  const bf16* gq = p.q + static_cast<size_t>(s0) * p.ld + static_cast<size_t>(head) * p.dim;
+  const bf16* gf = p.f + static_cast<size_t>(s0) * p.ld + static_cast<size_t>(head) * p.dim;
+  const bf16* gv = p.v + static_cast<size_t>(s0) * p.ld + static_cast<size_t>(head) * p.vdim + col0;
+  auto fetch = [&](int t0, int buf) {
+    const int n = min(TOK, b - t0), dv = p.dim >> 3, vv = ncol >> 3;
+    for (int i = tid; i < n * dv; i += blockDim.x) {
+      const int t = i / dv, c = (i - t * dv) * 8;
+      const size_t g = static_cast<size_t>(t0 + t) * p.ld + c;
+      if constexpr (!PART) copy16(r_q + t * DP + c, gq + g);
+      copy16(r_f + t * DP + c, gf + g);
+    }
+    for (int i = tid; i < n * vv; i += blockDim.x) {
+      const int t = i / vv, c = (i - t * vv) * 8;
+      copy16(s_v + (buf * TOK + t) * VPITCH + c, gv + static_cast<size_t>(t0 + t) * p.ld + c);
+    }
+    copies_commit();
+  };
+  const int g = lane >> 2, tq = lane & 3;                // row and column pair of a lane in an accumulator
+  const size_t head_state = static_cast<size_t>(p.dim) * p.vdim;
+  const int v_lo = warp * 16 + g, v_hi = v_lo + 8;       // this lane's columns of the head (rows of Sᵀ), relative to col0
+  float S[NT][4];
+  {
+    const float* init = (!PART && seg > 0) ? p.part + ((static_cast<size_t>(seq) * (p.segments - 1) + seg - 1) * p.H + head) * head_state + col0 : nullptr;
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int r = n * 8 + tq * 2 + (e & 1), c = e < 2 ? v_lo : v_hi;
+        S[n][e] = init != nullptr && r < p.dim && c < ncol ? init[static_cast<size_t>(r) * p.vdim + c] : 0.f;
+      }
+  }
+  float keep[(DP + 31) / 32];
+  if constexpr (PART) {
+#pragma unroll
+    for (int i = 0; i < (DP + 31) / 32; ++i) keep[i] = 1.f;
+  }
+  fetch(a, 0);
+  int buf = 0;
+  for (int t0 = a; t0 < b; t0 += TOK, buf ^= 1) {
+    const int n = min(TOK, b - t0);
+    copies_wait();
+    __syncthreads();
+    // what enters the recurrence, in fp32; tokens past the end write nothing and decay nothing
+    for (int i = tid; i < TOK * DP / 2; i += blockDim.x) {
+      const int t = i / (DP / 2), c = (i - t * (DP / 2)) * 2;
+      float2 q = make_float2(0.f, 0.f), k = q;
+      if (t < n) {
+        if constexpr (!PART) {
+          q = unpack_bf16(reinterpret_cast<const uint32_t*>(r_q)[i]);
+          q.x = silu(q.x); q.y = silu(q.y);
+        }
+        const float2 f = unpack_bf16(reinterpret_cast<const uint32_t*>(r_f)[i]);
+        k.x = let_in(f.x + s_bias[c], s_low[c]); k.y = let_in(f.y + s_bias[c + 1], s_low[c + 1]);
+      }
+      if constexpr (!PART) reinterpret_cast<float2*>(s_q)[i] = q;
+      reinterpret_cast<float2*>(s_k)[i] = k;
+    }
+    if (n < TOK)
+      for (int i = tid; i < (TOK - n) * VP; i += blockDim.x) s_v[(buf * TOK + n + i / VP) * VPITCH + i % VP] = __float2bfloat16(0.f);
+    __syncthreads();
+    if (t0 + TOK < b) fetch(t0 + TOK, buf ^ 1);
+    // q P, k R and D: a thread follows one channel through one step
+    for (int i = tid; i < 2 * DP; i += blockDim.x) {
+      const int step = i / DP, c = i - step * DP, at = step * 16;
+      float w = 1.f;
+#pragma unroll
+      for (int t = 15; t >= 0; --t) {
+        const float k = s_k[(at + t) * DP + c];
+        split(k * w, s_kh + (at + t) * PITCH + c, s_kl + (at + t) * PITCH + c);
+        w *= 1.f - k;
+      }
+      s_d[i] = w;
+      if constexpr (!PART) {
+        w = 1.f;
+#pragma unroll
+        for (int t = 0; t < 16; ++t) {
+          w *= 1.f - s_k[(at + t) * DP + c];
+          split(s_q[(at + t) * DP + c] * w, s_qh + (at + t) * PITCH + c, s_ql + (at + t) * PITCH + c);
+        }
+      }
+    }
+    // A: DS lanes share token j's row of products and follow what j wrote through the tokens behind it
+    if constexpr (!PART) {
+      constexpr int JW = 32 / DS;                        // tokens j a warp follows at once
+      const int sub = lane % DS;
+      for (int i = warp; i < TOK / JW; i += warps) {
+        const int jj = i * JW + lane / DS, step = jj >> 4, j = jj & 15, first = (i * JW) & 15;
+        float w[8], acc[16];
+#pragma unroll
+        for (int t = 0; t < 16; ++t) acc[t] = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) w[e] = 0.f;
+#pragma unroll
+        for (int t = 0; t < 16; ++t) {
+          if (t >= first) {                              // nothing was written before the warp's first token
+            const float* qr = s_q + (step * 16 + t) * DP + sub * 4;
+            const float* kr = s_k + (step * 16 + t) * DP + sub * 4;
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+              const float4 q4 = *reinterpret_cast<const float4*>(qr + u * (DP / 2)), k4 = *reinterpret_cast<const float4*>(kr + u * (DP / 2));
+              w[4 * u] = t == j ? k4.x : w[4 * u] - w[4 * u] * k4.x; acc[t] = fmaf(q4.x, w[4 * u], acc[t]);
+              w[4 * u + 1] = t == j ? k4.y : w[4 * u + 1] - w[4 * u + 1] * k4.y; acc[t] = fmaf(q4.y, w[4 * u + 1], acc[t]);
+              w[4 * u + 2] = t == j ? k4.z : w[4 * u + 2] - w[4 * u + 2] * k4.z; acc[t] = fmaf(q4.z, w[4 * u + 2], acc[t]);
+              w[4 * u + 3] = t == j ? k4.w : w[4 * u + 3] - w[4 * u + 3] * k4.w; acc[t] = fmaf(q4.w, w[4 * u + 3], acc[t]);
+            }
+          }
+        }
+        // sum over the DS lanes; lane `sub` is left with 16 / DS of the sixteen
+        int left = 16, base = 0;
+#pragma unroll
+        for (int o = DS / 2; o > 0; o >>= 1) {
+          const bool upper = sub & o;
+          left >>= 1;
+#pragma unroll
+          for (int x = 0; x < 8; ++x) {
+            if (x < left) {
+              const float send = upper ? acc[x] : acc[x + left], kept = upper ? acc[x + left] : acc[x];
+              acc[x] = kept + __shfl_xor_sync(0xffffffffu, send, o);
+            }
+          }
+          base += upper ? left : 0;
+        }
+        bf16* ah = s_a + step * 2 * 16 * 24;
+#pragma unroll
+        for (int x = 0; x < 16 / DS; ++x) split(acc[x], ah + (base + x) * 24 + j, ah + 16 * 24 + (base + x) * 24 + j);
+      }
+    }
+    __syncthreads();
+#pragma unroll 1
+    for (int step = 0; step < 2; ++step) {
+      if (step * 16 >= n) break;
+      const int at = step * 16;
+      uint32_t va[4];                                    // Vᵀ of the step: [16 columns, 16 tokens]
+      ldsm4t(va, s_v + (buf * TOK + at + (lane >> 4) * 8 + (lane & 7)) * VPITCH + warp * 16 + (lane >> 3 & 1) * 8);
+      if constexpr (!PART) {
+        float o[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+        const int tok = at + (lane >> 4) * 8 + (lane & 7), kc = (lane >> 3 & 1) * 8;
+#pragma unroll
+        for (int s = 0; s < DP / 16; ++s) {
+          uint32_t sh[4], sl[4], qh[4], ql[4];
+          ldsm4(qh, s_qh + tok * PITCH + s * 16 + kc);
+          ldsm4(ql, s_ql + tok * PITCH + s * 16 + kc);
+          split2(S[2 * s][0], S[2 * s][1], sh[0], sl[0]);
+          split2(S[2 * s][2], S[2 * s][3], sh[1], sl[1]);
+          split2(S[2 * s + 1][0], S[2 * s + 1][1], sh[2], sl[2]);
+          split2(S[2 * s + 1][2], S[2 * s + 1][3], sh[3], sl[3]);
+          mma(o[0], sh, qh[0], qh[1]); mma(o[1], sh, qh[2], qh[3]);
+          mma(o[0], sl, qh[0], qh[1]); mma(o[1], sl, qh[2], qh[3]);
+          mma(o[0], sh, ql[0], ql[1]); mma(o[1], sh, ql[2], ql[3]);
+        }
+        uint32_t ah[4], al[4];
+        const bf16* ar = s_a + step * 2 * 16 * 24 + (tok - at) * 24 + kc;
+        ldsm4(ah, ar);
+        ldsm4(al, ar + 16 * 24);
+        mma(o[0], va, ah[0], ah[1]); mma(o[1], va, ah[2], ah[3]);
+        mma(o[0], va, al[0], al[1]); mma(o[1], va, al[2], al[3]);
+#pragma unroll
+        for (int h = 0; h < 2; ++h)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {                  // token 8 h + 2 tq + e: columns v_lo and v_hi
+            const int t = at + h * 8 + tq * 2 + e;
+            s_o[t * L.po + v_lo] = o[h][e];
+            s_o[t * L.po + v_hi] = o[h][e + 2];
+            float ss = o[h][e] * o[h][e] + o[h][e + 2] * o[h][e + 2];       // columns past the head's are zero
+            ss += __shfl_xor_sync(0xffffffffu, ss, 4);
+            ss += __shfl_xor_sync(0xffffffffu, ss, 8);
+            ss += __shfl_xor_sync(0xffffffffu, ss, 16);
+            if (g == 0) s_ss[warp * TOK + t] = ss;
+          }
+      }
+      const int ktok = at + (lane >> 3 & 1) * 8 + (lane & 7), kd = (lane >> 4) * 8;
+#pragma unroll
+      for (int s = 0; s < DP / 16; ++s) {
+        uint32_t kh[4], kl[4];
+        ldsm4t(kh, s_kh + ktok * PITCH + s * 16 + kd);
+        ldsm4t(kl, s_kl + ktok * PITCH + s * 16 + kd);
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const float2 d = *reinterpret_cast<const float2*>(s_d + step * DP + s * 16 + h * 8 + tq * 2);
+          float (&x)[4] = S[2 * s + h];
+          x[0] *= d.x; x[1] *= d.y; x[2] *= d.x; x[3] *= d.y;
+          mma(x, va, kh[2 * h], kh[2 * h + 1]);
+          mma(x, va, kl[2 * h], kl[2 * h + 1]);
+        }
+      }
+    }
+    if constexpr (PART) {
+#pragma unroll
+      for (int i = 0; i < (DP + 31) / 32; ++i) {
+        const int r = i * blockDim.x + tid;
+        if (r < DP) keep[i] *= s_d[r] * s_d[DP + r];
+      }
+    } else {
+      __syncthreads();
+      for (int t = warp; t < n; t += warps) {
+        const size_t out = static_cast<size_t>(s0 + t0 + t) * p.H * p.vdim + static_cast<size_t>(head) * p.vdim + col0;
+        if (p.raw != nullptr) {
+          for (int c = lane; c < ncol; c += 32) p.raw[out + c] = s_o[t * L.po + c];
+          continue;
+        }
+        float ss = 0.f;
+        for (int w = 0; w < warps; ++w) ss += s_ss[w * TOK + t];
+        const float r = rsqrtf(ss / p.vdim + p.eps);
+        for (int c = lane * 2; c < ncol; c += 64) {
+          const float2 x = *reinterpret_cast<const float2*>(s_o + t * L.po + c), w = unpack_bf16(*reinterpret_cast<const uint32_t*>(p.weight + c));
+          *reinterpret_cast<uint32_t*>(p.o + out + c) = pack_bf16(x.x * r * w.x, x.y * r * w.y);
+        }
+      }
+    }
+  }
+  float* out = nullptr;
+  if constexpr (PART) {
+    out = p.part + ((static_cast<size_t>(seq) * (p.segments - 1) + seg) * p.H + head) * head_state + col0;
+    if (slice == 0) {
+      float* d = p.decay + ((static_cast<size_t>(seq) * (p.segments - 1) + seg) * p.H + head) * p.dim;
+#pragma unroll
+      for (int i = 0; i < (DP + 31) / 32; ++i) {
+        const int r = i * blockDim.x + tid;
+        if (r < p.dim) d[r] = keep[i];
+      }
+    }
+  } else if (p.pool != nullptr && b == len) {
+    const int sl = p.slot[s0];
+    if (sl > 0) out = p.pool + (static_cast<size_t>(sl) * p.H + head) * head_state + col0;
+  }
+  if (out != nullptr) {
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int r = n * 8 + tq * 2 + (e & 1), c = e < 2 ? v_lo : v_hi;
+        if (r < p.dim && c < ncol) out[static_cast<size_t>(r) * p.vdim + c] = S[n][e];
+      }
+  }
+}
+
 // part[s] becomes the state behind segment s: a scan over the segments of every sequence, one thread per state element.
 __global__ void __launch_bounds__(256) hgrn2_scan_kernel(float* part, const float* __restrict__ decay, const int* __restrict__ cu, int H, int dim, int vdim,
                                                          int seg_len, int segments) {
@@ -375,8 +692,11 @@ torch::Tensor hgrn2_prefill(const torch::Tensor& proj, int64_t q0, int64_t f0, i
     using T = decltype(tag);
     auto p = hgrn2_args<T>(proj, q0, f0, v0, H, dim, vdim, bias, lower, weight, eps, o, pool, slot);
     p.cu = cu.data_ptr<int>();
+    constexpr int E = 16 / sizeof(T);
+    const bool whole = dim % E == 0 && vdim % E == 0 && p.ld % E == 0 && on16(p.q) && on16(p.f) && on16(p.v);      // 16-byte vectors everywhere
+    const bool chunks = sizeof(T) == 2 && whole && dim <= 128 && reinterpret_cast<uintptr_t>(p.weight) % 4 == 0;
     const int rpt = dim <= 64 ? 32 : 64, rs = dim <= 32 ? 1 : (dim <= 128 ? 2 : 4);
-    const int most = 256 / rs * 2;                               // columns a block can hold
+    const int most = chunks ? 128 : 256 / rs * 2;                // columns a block can hold
     p.slices = (vdim + most - 1) / most;
     p.cols = p.slices == 1 ? (vdim + 1) / 2 * 2 : most;
     torch::Tensor raw, part, decay;
@@ -393,10 +713,11 @@ torch::Tensor hgrn2_prefill(const torch::Tensor& proj, int64_t q0, int64_t f0, i
       p.part = part.data_ptr<float>(); p.decay = decay.data_ptr<float>();
     }
     TORCH_CHECK(n <= 65535, "too many sequences in one call");
-    constexpr int E = 16 / sizeof(T);
-    const bool vec = dim % E == 0 && vdim % E == 0 && p.cols % E == 0 && p.ld % E == 0 && on16(p.q) && on16(p.f) && on16(p.v);
-    const int threads = (((std::min<int>(p.cols, vdim) + 1) / 2) * rs + 31) / 32 * 32, dp = rpt * rs;
-    const size_t smem = sizeof(float) * (2 * hg::CH * dp + hg::CH * p.cols + 2 * dp) + (vec ? sizeof(T) * hg::CH * (2 * dim + p.cols) : 0);
+    const bool vec = whole && p.cols % E == 0;
+    const int warps = (p.cols + 15) / 16, dp = chunks ? (dim <= 32 ? 32 : (dim <= 64 ? 64 : 128)) : rpt * rs;
+    const int threads = chunks ? 32 * warps : (((std::min<int>(p.cols, vdim) + 1) / 2) * rs + 31) / 32 * 32;
+    const size_t smem = chunks ? hg::Layout(dp, warps * 16).total
+                               : sizeof(float) * (2 * hg::CH * dp + hg::CH * p.cols + 2 * dp) + (vec ? sizeof(T) * hg::CH * (2 * dim + p.cols) : 0);
     auto go = [&](auto kern, int segments) {
       TK_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
       kern<<<dim3(H * p.slices, segments, n), threads, smem, stream>>>(p);
@@ -405,6 +726,14 @@ torch::Tensor hgrn2_prefill(const torch::Tensor& proj, int64_t q0, int64_t f0, i
     };
 #define TK_HGRN2(PART, SEGS)                                                                                             \
   do {                                                                                                                   \
+    if constexpr (sizeof(T) == 2) {                                                                                      \
+      if (chunks) {                                                                                                      \
+        if (dp == 32) go(hgrn2_chunk_kernel<32, PART>, SEGS);                                                            \
+        else if (dp == 64) go(hgrn2_chunk_kernel<64, PART>, SEGS);                                                       \
+        else go(hgrn2_chunk_kernel<128, PART>, SEGS);                                                                    \
+        break;                                                                                                           \
+      }                                                                                                                  \
+    }                                                                                                                    \
     if (vec) {                                                                                                           \
       if (rpt == 32 && rs == 1) go(hgrn2_prefill_kernel<T, 32, 1, true, PART>, SEGS);                                    \
       else if (rpt == 32) go(hgrn2_prefill_kernel<T, 32, 2, true, PART>, SEGS);                                          \
