@@ -391,27 +391,31 @@ __global__ void __launch_bounds__(256, 2) hgrn2_chunk_kernel(const Hgrn2<bf16> p
     }
     // A: DS lanes share token j's row of products and follow what j wrote through the tokens behind it
     if constexpr (!PART) {
-      constexpr int JW = 32 / DS;                        // tokens j a warp follows at once
+      constexpr int JW = 32 / DS, ITEMS = 16 / JW;       // tokens j a warp follows at once, such groups in a step
       const int sub = lane % DS;
-      for (int i = warp; i < TOK / JW; i += warps) {
-        const int jj = i * JW + lane / DS, step = jj >> 4, j = jj & 15, first = (i * JW) & 15;
-        float w[8], acc[16];
+      for (int i = warp; i < 2 * ITEMS; i += warps) {
+        // the second step's groups in reverse: a warp that followed the longest rows follows the shortest next
+        const int step = i / ITEMS, first = (step ? 2 * ITEMS - 1 - i : i) * JW, j = first + lane / DS;
+        const float *qr = s_q + (step * 16 + first) * DP + sub * 4, *kr = s_k + (step * 16 + first) * DP + sub * 4;
+        float w[8], acc[16];                             // acc[r]: token first + r
 #pragma unroll
         for (int t = 0; t < 16; ++t) acc[t] = 0.f;
 #pragma unroll
         for (int e = 0; e < 8; ++e) w[e] = 0.f;
 #pragma unroll
-        for (int t = 0; t < 16; ++t) {
-          if (t >= first) {                              // nothing was written before the warp's first token
-            const float* qr = s_q + (step * 16 + t) * DP + sub * 4;
-            const float* kr = s_k + (step * 16 + t) * DP + sub * 4;
+        for (int r = 0; r < 16; ++r) {
+          if (first + r < 16) {
 #pragma unroll
             for (int u = 0; u < 2; ++u) {
-              const float4 q4 = *reinterpret_cast<const float4*>(qr + u * (DP / 2)), k4 = *reinterpret_cast<const float4*>(kr + u * (DP / 2));
-              w[4 * u] = t == j ? k4.x : w[4 * u] - w[4 * u] * k4.x; acc[t] = fmaf(q4.x, w[4 * u], acc[t]);
-              w[4 * u + 1] = t == j ? k4.y : w[4 * u + 1] - w[4 * u + 1] * k4.y; acc[t] = fmaf(q4.y, w[4 * u + 1], acc[t]);
-              w[4 * u + 2] = t == j ? k4.z : w[4 * u + 2] - w[4 * u + 2] * k4.z; acc[t] = fmaf(q4.z, w[4 * u + 2], acc[t]);
-              w[4 * u + 3] = t == j ? k4.w : w[4 * u + 3] - w[4 * u + 3] * k4.w; acc[t] = fmaf(q4.w, w[4 * u + 3], acc[t]);
+              const float4 q4 = *reinterpret_cast<const float4*>(qr + r * DP + u * (DP / 2)), k4 = *reinterpret_cast<const float4*>(kr + r * DP + u * (DP / 2));
+              const float q[4] = {q4.x, q4.y, q4.z, q4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                float& x = w[4 * u + e];
+                x = fmaf(-x, k[e], x);
+                if (r < JW && first + r == j) x = k[e];
+                acc[r] = fmaf(q[e], x, acc[r]);
+              }
             }
           }
         }
@@ -432,7 +436,11 @@ __global__ void __launch_bounds__(256, 2) hgrn2_chunk_kernel(const Hgrn2<bf16> p
         }
         bf16* ah = s_a + step * 2 * 16 * 24;
 #pragma unroll
-        for (int x = 0; x < 16 / DS; ++x) split(acc[x], ah + (base + x) * 24 + j, ah + 16 * 24 + (base + x) * 24 + j);
+        for (int x = 0; x < 16 / DS; ++x) {
+          const int t = first + base + x;                // tokens in front of the group's first see nothing of it
+          if (t < 16) split(acc[x], ah + t * 24 + j, ah + 16 * 24 + t * 24 + j);
+          else ah[(t - 16) * 24 + j] = ah[16 * 24 + (t - 16) * 24 + j] = __float2bfloat16(0.f);
+        }
       }
     }
     __syncthreads();
@@ -701,9 +709,9 @@ torch::Tensor hgrn2_prefill(const torch::Tensor& proj, int64_t q0, int64_t f0, i
     p.cols = p.slices == 1 ? (vdim + 1) / 2 * 2 : most;
     torch::Tensor raw, part, decay;
     if (p.slices > 1) { raw = torch::empty({rows, H * vdim}, f32); p.raw = raw.data_ptr<float>(); }
-    // time segments: enough blocks for two per SM, none shorter than 128 tokens (a segment costs a second pass over its state)
+    // time segments: at most two blocks per SM (one wave), none shorter than 128 tokens (a segment costs a second pass over its state)
     const long blocks = static_cast<long>(H) * p.slices * n;
-    long segs = blocks >= num_sms() ? 1 : std::min<long>((2L * num_sms() + blocks - 1) / blocks, max_seqlen / 128);
+    long segs = blocks >= num_sms() ? 1 : std::min<long>(2L * num_sms() / blocks, max_seqlen / 128);
     segs = std::max<long>(segs, 1);
     p.seg_len = static_cast<int>(((max_seqlen + segs - 1) / segs + hg::CH - 1) / hg::CH * hg::CH);
     p.segments = static_cast<int>((max_seqlen + p.seg_len - 1) / p.seg_len);
