@@ -10,7 +10,7 @@ from __future__ import annotations
 import json
 import math
 import os
-from dataclasses import asdict, dataclass, field
+from dataclasses import dataclass, field
 from typing import List, Any, Dict, Optional, Tuple, Union
 
 
@@ -103,7 +103,7 @@ def _moronex_mapping(c: 'DecoderConfig') -> Dict[str, Any]:
     """The inverse of :func:`_moronex_fields`."""
     layers = []
     for sp in c.layer_specs:
-        m = {k: v for k, v in asdict(sp.mixer).items() if v is not None}
+        m = {k: getattr(sp.mixer, k) for k in ('heads', 'dim', 'vdim', 'q_rank', 'kv_rank', 'scale', 'kv_from') if getattr(sp.mixer, k, None) is not None}
         f = sp.mlp
         mlp = None if f is None else ({'kind': 'moe', 'expert': {'ff': f.ff}, 'router': {'experts': f.experts, 'top': f.top}} if f.experts
                                       else {'kind': 'dense', 'ff': f.ff})
@@ -113,8 +113,76 @@ def _moronex_mapping(c: 'DecoderConfig') -> Dict[str, Any]:
     return d
 
 
+def _nilepel_rotary(rot: Dict[str, Any], interleaved: bool) -> 'RotarySpec':
+    return RotarySpec(dims=int(rot['dims']), base=float(rot['base']), interleaved=interleaved, scaling=dict(rot['scaling']) if rot.get('scaling') else None)
+
+
+def _nilepel_fields(cfg: Dict[str, Any]) -> Dict[str, Any]:
+    """``config.json`` of a Nilepel checkpoint → keyword arguments of :class:`DecoderConfig`."""
+    specs = []
+    for i, layer in enumerate(cfg['layers']):
+        kind, m, mlp = layer['type'], layer['mixer'], layer.get('mlp')
+        sizes = {k: int(m[k]) for k in ('heads', 'dim', 'vdim')}
+        size, scale, source = int(m['mask']['size']), float(m['scale']), None if m.get('kv_from') is None else int(m['kv_from'])
+        if kind == 'attention':
+            mixer = AttentionSpec(**sizes, kv_heads=int(m['kv_heads']), scale=scale, rotary=_nilepel_rotary(m['rot'], True), chunk=size, sinks=True, kv_from=source)
+        elif kind == 'attention_2':
+            mixer = AttentionSpec(**sizes, kv_heads=int(m['kv_heads']), scale=scale, rotary=_nilepel_rotary(m['rot'], False), window=size, bias=True, qk_norm=True,
+                                  sinks=True, head_gate=True, kv_from=source)
+        elif kind == 'latent_attention':
+            mixer = LatentSpec(**sizes, q_rank=0, kv_rank=int(m['kv_rank']), scale=scale, kv_from=source, rot_dim=int(m['rot_dim']),
+                               rotary=_nilepel_rotary(m['rot'], True), window=size, sinks=False, head_gate=False)
+        else:
+            raise NotImplementedError(f"layer {i}: mixer type {kind!r} is not implemented (attention, attention_2 and latent_attention are)")
+        if mlp is None:
+            ff = None
+        elif mlp['kind'] == 'dense':
+            ff = FeedForwardSpec(ff=int(mlp['ff']), limit=float(mlp['limit']))
+        elif mlp['kind'] == 'moe':
+            r, groups = mlp['router'], mlp['router'].get('groups') or {}
+            ff = FeedForwardSpec(ff=int(mlp['expert']['ff']), experts=int(r['experts']), top=int(r['top']), gated=True, scoring='softmax_grouped',
+                                 groups=int(groups.get('count', 1)), keep=int(groups.get('keep', 1)), scale=float(r.get('scale', 1.0)),
+                                 shared=int(mlp['shared']['ff']) if mlp.get('shared') else 0)
+        else:
+            raise NotImplementedError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not implemented (dense and moe are)")
+        specs.append(PreNormSpec(mixer, ff))
+    return dict(model_type='nilepel', vocab_size=int(cfg['vocab']), hidden_size=int(cfg['width']), rms_norm_eps=float(cfg['norm']['eps']),
+                embed_scale=float(cfg['embedding']['scale']), tie_word_embeddings=False, qk_norm=False, layer_specs=specs, eos_token_id=cfg.get('eos_token_id'),
+                pad_token_id=cfg.get('pad_token_id'), torch_dtype=str(cfg.get('torch_dtype', 'bfloat16')))
+
+
+def _nilepel_mapping(c: 'DecoderConfig') -> Dict[str, Any]:
+    """The inverse of :func:`_nilepel_fields`."""
+    layers = []
+    for sp in c.layer_specs:
+        m, f = sp.mixer, sp.mlp
+        rot = {'base': m.rotary.base, 'dims': m.rotary.dims}
+        if m.rotary.scaling:
+            rot['scaling'] = dict(m.rotary.scaling)
+        mixer = {'heads': m.heads, 'dim': m.dim, 'vdim': m.vdim, 'scale': m.scale, 'rot': rot, 'mask': {'size': m.window or m.chunk}}
+        if m.kind == 'latent_attention':
+            kind = m.kind
+            mixer.update(kv_rank=m.kv_rank, rot_dim=m.rot_dim)
+        else:
+            kind = 'attention' if m.chunk else 'attention_2'
+            mixer['kv_heads'] = m.kv_heads
+        if m.kv_from is not None:
+            mixer['kv_from'] = m.kv_from
+        mlp = None
+        if f is not None and f.experts:
+            mlp = {'kind': 'moe', 'expert': {'ff': f.ff}, 'router': {'experts': f.experts, 'top': f.top, 'scale': f.scale, 'groups': {'count': f.groups, 'keep': f.keep}}}
+            if f.shared:
+                mlp['shared'] = {'ff': f.shared}
+        elif f is not None:
+            mlp = {'kind': 'dense', 'ff': f.ff, 'limit': f.limit}
+        layers.append({'type': kind, 'mixer': mixer, 'mlp': mlp})
+    d = {'architecture': 'Nilepel', 'vocab': c.vocab_size, 'width': c.hidden_size, 'norm': {'eps': c.rms_norm_eps}, 'embedding': {'scale': c.embed_scale}, 'layers': layers}
+    d.update({k: v for k, v in (('eos_token_id', c.eos_token_id), ('pad_token_id', c.pad_token_id)) if v is not None})
+    return d
+
+
 # checkpoints whose config.json names its ``architecture`` and lists every layer: (reader → DecoderConfig fields, writer)
-NATIVE_ARCHITECTURES = {'Pomelix': (_pomelix_fields, _pomelix_mapping), 'Moronex': (_moronex_fields, _moronex_mapping)}
+NATIVE_ARCHITECTURES = {'Pomelix': (_pomelix_fields, _pomelix_mapping), 'Moronex': (_moronex_fields, _moronex_mapping), 'Nilepel': (_nilepel_fields, _nilepel_mapping)}
 
 
 def _up8(n: int) -> int:
@@ -172,11 +240,108 @@ class LayerSpec:
 
 
 @dataclass
+class RotarySpec:
+    """Rotation of the leading ``dims`` dimensions of a head by position: pair ``i`` turns by ``base^(−2i/dims)`` per position.  A pair is
+    ``(2i, 2i + 1)`` (``interleaved``) or ``(i, i + dims/2)``.  ``scaling`` (``factor``, ``low``, ``high``, ``original``): wavelengths above
+    ``original / low`` are slowed down by ``factor``, those below ``original / high`` kept, the ones between blended."""
+    dims: int
+    base: float
+    interleaved: bool = False
+    scaling: Optional[Dict[str, float]] = None
+
+    def __post_init__(self):
+        if self.dims < 2 or self.dims % 2:
+            raise ValueError(f'rotation over {self.dims} dimensions: a positive even number is needed')
+
+    @property
+    def pairs(self) -> int:
+        return self.dims // 2
+
+    def frequencies(self) -> List[float]:
+        """Angle per position of every pair."""
+        out = []
+        for i in range(self.pairs):
+            f = self.base**(-2.0 * i / self.dims)
+            if self.scaling:
+                factor, low, high, original = (float(self.scaling[k]) for k in ('factor', 'low', 'high', 'original'))
+                turns = original * f / (2 * math.pi)               # over the original context
+                if turns < low:
+                    f = f / factor
+                elif turns <= high:
+                    s = (turns - low) / (high - low)
+                    f = (1 - s) * f / factor + s * f
+            out.append(f)
+        return out
+
+
+@dataclass
+class AttentionSpec:
+    """Grouped-query attention over rotated queries and keys.  What a position sees: everything before it, its last ``window``
+    positions, or its own block of ``chunk`` positions counted from the first token.  ``bias`` on q, k and v, ``qk_norm`` per head before the
+    rotation, ``sinks`` (a logit per head in the denominator), ``head_gate`` (a sigmoid per head on the output).  ``kv_from``: index of the
+    earlier layer whose keys and values this layer reads instead of its own."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rotary: RotarySpec
+    window: int = 0
+    chunk: int = 0
+    bias: bool = False
+    qk_norm: bool = False
+    sinks: bool = False
+    head_gate: bool = False
+    kv_from: Optional[int] = None
+    kind = 'attention'
+
+    def __post_init__(self):
+        if isinstance(self.rotary, dict):
+            self.rotary = RotarySpec(**self.rotary)
+        if self.heads % self.kv_heads:
+            raise ValueError(f'{self.heads} query heads do not divide over {self.kv_heads} key / value heads')
+        if self.rotary.dims > self.dim:
+            raise ValueError(f'rotation over {self.rotary.dims} of {self.dim} dimensions')
+
+    @property
+    def qkv_sizes(self) -> Tuple[int, int, int]:
+        """Rows of the q, k and v projections (a layer that borrows keys and values has none of its own)."""
+        own = 0 if self.kv_from is not None else self.kv_heads
+        return self.heads * self.dim, own * self.dim, own * self.vdim
+
+    def in_parts(self) -> List[Tuple[str, int]]:
+        """Projections of the layer input."""
+        parts = [(n, w) for n, w in zip(('q_proj', 'k_proj', 'v_proj'), self.qkv_sizes) if w]
+        return parts + ([('head_gate', self.heads)] if self.head_gate else [])
+
+    def kept(self) -> Tuple[Any, ...]:
+        """What a borrowing layer must agree on with the layer it borrows from."""
+        return self.kind, self.kv_heads, self.dim, self.vdim, self.rotary
+
+    def lent_columns(self) -> int:
+        return self.kv_heads * (self.dim + self.vdim)
+
+    def kv_rows(self) -> Tuple[int, int, int]:
+        return (self.kv_heads, _up8(self.dim), _up8(self.vdim)) if self.kv_from is None else (0, 0, 0)
+
+    def matmul_weights(self, width: int) -> int:
+        return width * sum(n for _, n in self.in_parts()) + self.heads * self.vdim * width
+
+    def small_weights(self) -> int:
+        own = self.kv_from is None
+        return (sum(self.qkv_sizes) if self.bias else 0) + (self.dim * (2 if own else 1) if self.qk_norm else 0) + (self.heads if self.sinks else 0)
+
+    def attention_width(self) -> int:
+        return (self.dim + self.vdim) * self.heads
+
+
+@dataclass
 class LatentSpec:
-    """Latent attention without positions: queries through a normed rank-``q_rank`` bottleneck, keys (``dim`` per head) and values
-    (``vdim``) expanded from one normed rank-``kv_rank`` latent per token, which is all the cache keeps; a sink logit per head in
-    the softmax, a sigmoid gate per head on the output.  ``kv_from``: index of the earlier layer whose latents this layer reads
-    instead of its own."""
+    """Latent attention: keys (``dim`` per head) and values (``vdim``) expanded from one normed rank-``kv_rank`` latent per token, which
+    is all the cache keeps, together with ``rot_dim`` rotated key dimensions that all heads share (0: no positions).  Queries through a
+    normed rank-``q_rank`` bottleneck (0: a plain projection; a head's query is ``[dim | rot_dim]``).  ``window``: the last positions that a
+    position sees (0: all).  ``sinks`` (a logit per head in the softmax), ``head_gate`` (a sigmoid per head on the output).  ``kv_from``:
+    index of the earlier layer whose latents this layer reads instead of its own."""
     heads: int
     dim: int
     vdim: int
@@ -184,17 +349,49 @@ class LatentSpec:
     kv_rank: int
     scale: float
     kv_from: Optional[int] = None
+    rot_dim: int = 0
+    rotary: Optional[RotarySpec] = None
+    window: int = 0
+    sinks: bool = True
+    head_gate: bool = True
     kind = 'latent_attention'
+    chunk = 0
+
+    def __post_init__(self):
+        if isinstance(self.rotary, dict):
+            self.rotary = RotarySpec(**self.rotary)
+        if (self.rotary.dims if self.rotary else 0) != self.rot_dim:
+            raise ValueError(f'the rotation covers {self.rotary.dims if self.rotary else 0} dimensions of a rotated part of {self.rot_dim}')
+        if self.rot_dim and self.q_rank:
+            raise ValueError('rotated queries come from a plain projection (q_rank 0)')
+
+    @property
+    def qk_width(self) -> int:
+        return self.dim + self.rot_dim
 
     def in_parts(self) -> List[Tuple[str, int]]:
         """Projections of the layer input."""
-        return [('dq_proj', self.q_rank)] + ([('dkv_proj', self.kv_rank)] if self.kv_from is None else []) + [('head_gate', self.heads)]
+        q = [('dq_proj', self.q_rank)] if self.q_rank else [('q_proj', self.heads * self.qk_width)]
+        return q + ([('dkv_proj', self.kv_rank + self.rot_dim)] if self.kv_from is None else []) + ([('head_gate', self.heads)] if self.head_gate else [])
+
+    def kept(self) -> Tuple[Any, ...]:
+        """What a borrowing layer must agree on with the layer it borrows from."""
+        return self.kind, self.kv_rank, self.rot_dim, self.rotary
+
+    def lent_columns(self) -> int:
+        return self.kv_rank + self.rot_dim
+
+    def kv_rows(self) -> Tuple[int, int, int]:
+        return (1, _up8(self.kv_rank + self.rot_dim), 0) if self.kv_from is None else (0, 0, 0)
 
     def matmul_weights(self, width: int) -> int:
         return width * sum(n for _, n in self.in_parts()) + self.heads * (self.dim * self.q_rank + (self.dim + self.vdim) * self.kv_rank + self.vdim * width)
 
     def small_weights(self) -> int:
-        return self.q_rank + (self.kv_rank if self.kv_from is None else 0) + self.heads
+        return self.q_rank + (self.kv_rank if self.kv_from is None else 0) + (self.heads if self.sinks else 0)
+
+    def attention_width(self) -> int:
+        return (self.qk_width + self.vdim) * self.heads
 
 
 @dataclass
@@ -205,6 +402,13 @@ class HGRN2Spec:
     dim: int
     vdim: int
     kind = 'hgrn2'
+    kv_from = rotary = None
+
+    def kv_rows(self) -> Tuple[int, int, int]:
+        return 0, 0, 0
+
+    def attention_width(self) -> int:
+        return 0
 
     def in_parts(self) -> List[Tuple[str, int]]:
         return [('q_proj', self.heads * self.dim), ('f_proj', self.heads * self.dim), ('v_proj', self.heads * self.vdim)]
@@ -218,27 +422,60 @@ class HGRN2Spec:
 
 @dataclass
 class FeedForwardSpec:
-    """Gated feed-forward block of width ``ff``, or, with ``experts``, that many two-matrix experts of which a token uses ``top``."""
+    """Gated feed-forward block of width ``ff``, or, with ``experts``, that many experts of which a token uses ``top``.
+
+    Dense: ``silu(gate) · up``, or with a ``limit`` ``g σ(1.702 g) (u + 1)`` on ``g ≤ limit``, ``|u| ≤ limit``.
+    Experts: two matrices around the square of relu, or ``gated`` ones (three matrices, ``silu(gate) · up``).  ``scoring`` as in
+    ``DecoderConfig.router_scoring``: ``'topk_softmax'`` (biased logits, a softmax over the chosen) or ``'softmax_grouped'`` (softmax over all;
+    only experts of the ``keep`` best of ``groups`` groups of neighbours, each as good as its best expert; weights times ``scale``).
+    ``shared``: width of an expert beside them that runs for every token, scaled by a sigmoid per token (0: none)."""
     ff: int
     experts: int = 0
     top: int = 0
+    limit: float = 0.0
+    gated: bool = False
+    scoring: str = 'topk_softmax'
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
+    shared: int = 0
+
+    def __post_init__(self):
+        if not self.experts:
+            return
+        if self.experts % self.groups or not 1 <= self.keep <= self.groups:
+            raise ValueError(f'{self.experts} experts in {self.groups} groups of which {self.keep} are kept')
+        if not 1 <= self.top <= self.experts // self.groups * self.keep:
+            raise ValueError(f'top {self.top} of {self.experts // self.groups * self.keep} experts that can be chosen')
+
+    def matmul_weights(self, width: int, active: bool = False) -> int:
+        if not self.experts:
+            return 3 * width * self.ff
+        per = (3 if self.gated else 2) * width * self.ff
+        return width * self.experts + (self.top if active else self.experts) * per + (3 * width * self.shared + width if self.shared else 0)
+
+    def small_weights(self) -> int:
+        return self.experts if self.scoring == 'topk_softmax' else 0
+
+
+_MIXER_SPECS = ((LatentSpec, 'kv_rank'), (AttentionSpec, 'kv_heads'), (HGRN2Spec, 'heads'))
 
 
 @dataclass
 class SandwichSpec:
     """One layer with a norm in front of and behind each sub-layer and a sigmoid gate (read from the sub-layer's input) on its
     result: a mixer and a feed-forward block (None: the layer has none)."""
-    mixer: Union[LatentSpec, HGRN2Spec]
+    mixer: Union[LatentSpec, AttentionSpec, HGRN2Spec]
     mlp: Optional[FeedForwardSpec] = None
 
     def __post_init__(self):
         if isinstance(self.mixer, dict):
-            self.mixer = (LatentSpec if 'kv_rank' in self.mixer else HGRN2Spec)(**self.mixer)
+            self.mixer = next(c for c, key in _MIXER_SPECS if key in self.mixer)(**self.mixer)
         if isinstance(self.mlp, dict):
             self.mlp = FeedForwardSpec(**self.mlp)
 
     heads = property(lambda self: self.mixer.heads)
-    kv_heads = property(lambda self: self.mixer.heads)
+    kv_heads = property(lambda self: getattr(self.mixer, 'kv_heads', self.mixer.heads))
     dim = property(lambda self: self.mixer.dim)
     v_mix = False
 
@@ -251,7 +488,7 @@ class SandwichSpec:
         return self.mlp.ff if self.mlp is not None else 0
 
     def kv_rows(self) -> Tuple[int, int, int]:
-        return (1, _up8(self.mixer.kv_rank), 0) if self.mixer.kind == 'latent_attention' and self.mixer.kv_from is None else (0, 0, 0)
+        return self.mixer.kv_rows()
 
     def conv_rows(self) -> Optional[Tuple[int, int]]:
         return None
@@ -259,18 +496,35 @@ class SandwichSpec:
     def state_shape(self) -> Optional[Tuple[int, int, int]]:
         return (self.mixer.heads, self.mixer.dim, self.mixer.vdim) if self.mixer.kind == 'hgrn2' else None
 
+    def around(self, width: int) -> Tuple[int, int]:
+        """Weights of what stands around one sub-layer: in products, and others."""
+        return width * width, 3 * width
+
     def matmul_weights(self, width: int, active: bool = False) -> int:
-        n = width * width + self.mixer.matmul_weights(width)
-        if self.mlp is not None:
-            per = (2 if self.mlp.experts else 3) * width * self.mlp.ff
-            n += width * width + (width * self.mlp.experts + (self.mlp.top if active else self.mlp.experts) * per if self.mlp.experts else per)
-        return n
+        n = self.around(width)[0] + self.mixer.matmul_weights(width)
+        return n + (self.around(width)[0] + self.mlp.matmul_weights(width, active) if self.mlp is not None else 0)
 
     def small_weights(self, width: int) -> int:
-        return 3 * width * (2 if self.mlp is not None else 1) + self.mixer.small_weights() + (self.mlp.experts if self.mlp is not None else 0)
+        n = self.around(width)[1] + self.mixer.small_weights()
+        return n + (self.around(width)[1] + self.mlp.small_weights() if self.mlp is not None else 0)
 
     def attention_width(self) -> int:
-        return (self.mixer.dim + self.mixer.vdim) * self.mixer.heads if self.mixer.kind == 'latent_attention' else 0
+        return self.mixer.attention_width()
+
+
+@dataclass
+class PreNormSpec(SandwichSpec):
+    """One layer with a norm in front of each sub-layer, whose result joins the stream as it is."""
+    post: bool = False           # no norm behind the sub-layers (tells the two kinds apart when read from a mapping)
+
+    def around(self, width: int) -> Tuple[int, int]:
+        return 0, width
+
+
+def _layer_spec(sp: Any) -> Any:
+    if not isinstance(sp, dict):
+        return sp
+    return (LayerSpec if 'mixer' not in sp else (PreNormSpec if 'post' in sp else SandwichSpec))(**sp)
 
 
 @dataclass
@@ -379,14 +633,14 @@ class DecoderConfig:
     vision_end_token_id: Optional[int] = None
     mrope_section: Optional[List[int]] = None
     mrope_interleaved: bool = False  # Qwen3-VL lays the three position components out t h w t h w … instead of in blocks
-    # stacks whose layers are listed one by one, with a 32-bit residual stream and no rotary embedding: layers that run mixer and
-    # feed-forward side by side on one norm, each result with a learned per-channel scale (``LayerSpec``; Pomelix), or layers
-    # with norms around each sub-layer and a gate on its result (``SandwichSpec``; Moronex)
-    layer_specs: Optional[List[Union[LayerSpec, SandwichSpec, Dict[str, Any]]]] = None
+    # stacks whose layers are listed one by one, with a 32-bit residual stream: layers that run mixer and feed-forward side by side
+    # on one norm, each result with a learned per-channel scale (``LayerSpec``; Pomelix), layers with norms around each sub-layer and a
+    # gate on its result (``SandwichSpec``; Moronex), or layers with a norm in front of each sub-layer (``PreNormSpec``; Nilepel)
+    layer_specs: Optional[List[Union[LayerSpec, SandwichSpec, PreNormSpec, Dict[str, Any]]]] = None
 
     def __post_init__(self):
         if self.layer_specs is not None:
-            self.layer_specs = [(SandwichSpec if 'mixer' in sp else LayerSpec)(**sp) if isinstance(sp, dict) else sp for sp in self.layer_specs]
+            self.layer_specs = [_layer_spec(sp) for sp in self.layer_specs]
             first = self.layer_specs[0]
             self.num_hidden_layers = len(self.layer_specs)
             self.num_attention_heads, self.num_key_value_heads, self.head_dim = first.heads, first.kv_heads, first.dim
@@ -402,8 +656,8 @@ class DecoderConfig:
                 if j is None:
                     continue
                 src = self.layer_specs[j].mixer if 0 <= j < i else None
-                if src is None or src.kind != 'latent_attention' or src.kv_from is not None or src.kv_rank != sp.mixer.kv_rank:
-                    raise ValueError(f'layer {i}: kv_from {j} is not an earlier latent-attention layer with latents of its own and rank {sp.mixer.kv_rank}')
+                if src is None or src.kind == 'hgrn2' or src.kv_from is not None or src.kept() != sp.mixer.kept():
+                    raise ValueError(f'layer {i}: kv_from {j} is not an earlier layer with keys and values of its own and the same sizes and rotation {sp.mixer.kept()}')
         if self.vision is not None:
             from .vision import VisionConfig
             self.vision = VisionConfig.from_hf(self.vision).to_hf()  # only the fields the tower uses, in the family's spelling
@@ -444,7 +698,37 @@ class DecoderConfig:
             first = self.layer_specs[self.first_mixing_layer]
             return [(self.first_mixing_layer, first.kv_heads * first.vdim)]
         lent = sorted({sp.mixer.kv_from for sp in self.layer_specs or [] if getattr(getattr(sp, 'mixer', None), 'kv_from', None) is not None})
-        return [(j, self.layer_specs[j].mixer.kv_rank) for j in lent]
+        return [(j, self.layer_specs[j].mixer.lent_columns()) for j in lent]
+
+    def kernel_parts(self) -> List[str]:
+        """Mechanisms of a stack with listed layers whose kernels not every such stack needs (``ops/build.py``)."""
+        parts = set()
+        for sp in self.layer_specs or []:
+            m = getattr(sp, 'mixer', None)
+            if m is None:
+                parts.add('convolution')
+            else:
+                parts.update({'latent_attention': ['latent'], 'hgrn2': ['recurrent']}.get(m.kind, []) + (['rotary'] if m.rotary is not None or getattr(m, 'q_rank', 1) == 0 else []))
+                parts.update(['experts'] if sp.is_moe else [])
+        return sorted(parts)
+
+    def rotations(self) -> List[RotarySpec]:
+        """The distinct rotations of a stack with listed layers, in the order in which layers first use them."""
+        out: List[RotarySpec] = []
+        for sp in self.layer_specs or []:
+            rot = getattr(getattr(sp, 'mixer', None), 'rotary', None)
+            if rot is not None and rot not in out:
+                out.append(rot)
+        return out
+
+    def rotary_columns(self, layer_idx: int) -> Optional[Tuple[int, int]]:
+        """``(first, number)`` of a layer's pairs in the table of all :meth:`rotations` (None: the layer does not rotate)."""
+        at, mine = 0, getattr(self.layer_specs[layer_idx].mixer, 'rotary', None)
+        for rot in self.rotations():
+            if rot == mine:
+                return at, rot.pairs
+            at += rot.pairs
+        return None
 
     def layer_is_moe(self, layer_idx: int) -> bool:
         return self.num_experts > 0 and layer_idx >= self.first_k_dense_replace
