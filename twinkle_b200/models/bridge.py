@@ -165,7 +165,8 @@ _LISTED = {'input_layernorm.weight': 'norm1', 'v_lambda': 'mix.vmix', 'o_proj.we
            'mixer_gate_bias': 'rg1.b', 'mlp_gate_bias': 'rg2.b', 'mlp_gate.weight': 'rg2', 'mixer.q_norm.weight': 'mix.dq.norm',
            'mixer.kv_norm.weight': 'mix.dkv.norm', 'mixer.q_up.weight': 'mix.uq', 'mixer.sinks': 'mix.sink', 'mixer.o_proj.weight': 'mix.o',
            'mixer.f_bias': 'mix.f.b', 'mixer.lower': 'mix.lower', 'mixer.out_norm.weight': 'mix.norm', 'mlp.down_proj.weight': 'mlp.down',
-           'mlp.gate.weight': 'mlp.router', 'mlp.gate.bias': 'mlp.router.b'}
+           'mlp.gate.weight': 'mlp.router', 'mlp.gate.bias': 'mlp.router.b', 'mixer.head_q_norm.weight': 'mix.q.norm', 'mixer.head_k_norm.weight': 'mix.k.norm',
+           'mlp.shared_expert.down_proj.weight': 'mlp.shared.down', 'mlp.shared_expert_gate.weight': 'mlp.shared.sg'}
 _LISTED_PARTS = {'res_gate': 'rg1', 'q_proj': 'mix.q', 'k_proj': 'mix.k', 'v_proj': 'mix.v', 'f_proj': 'mix.f', 'dq_proj': 'mix.dq', 'dkv_proj': 'mix.dkv',
                  'head_gate': 'mix.g', 'gate_proj': 'mlp.gate', 'up_proj': 'mlp.up'}
 
@@ -177,9 +178,15 @@ def _listed_parts(rest: str, sp, width: int) -> List[Tuple[str, int]]:
     if rest == 'in_proj.weight':
         parts = list(zip(('q_proj', 'k_proj', 'v_proj'), sp.qkv_sizes)) + ([('gate_proj', sp.ff), ('up_proj', sp.ff)] if sp.ff else [])
     elif rest == 'mixer.in_proj.weight':
-        parts = [('res_gate', width)] + sp.mixer.in_parts()
+        parts = ([('res_gate', width)] if sp.around(width)[0] else []) + sp.mixer.in_parts()
+    elif rest == 'mixer.qkv_bias':
+        return [(f'mix.{p}.b', n) for p, n in zip('qkv', sp.mixer.qkv_sizes) if n]
     elif rest == 'mlp.in_proj.weight':
-        return [('rg2', width), ('mlp.gate', sp.mlp.ff), ('mlp.up', sp.mlp.ff)]
+        return ([('rg2', width)] if sp.around(width)[0] else []) + [('mlp.gate', sp.mlp.ff), ('mlp.up', sp.mlp.ff)]
+    elif rest == 'mlp.shared_expert.gate_up_proj.weight':
+        return [('mlp.shared.gate', sp.mlp.shared), ('mlp.shared.up', sp.mlp.shared)]
+    elif rest == 'mlp.experts.gate_up_proj':
+        return [(f'mlp.e{e}.{which}', sp.mlp.ff) for e in range(sp.mlp.experts) for which in ('gate', 'up')]
     elif rest == 'mixer.kv_up':
         return [('mix.uk', sp.mixer.heads * sp.mixer.dim), ('mix.uv', sp.mixer.heads * sp.mixer.vdim)]
     elif rest in ('mlp.experts.up_proj', 'mlp.experts.down_proj'):
@@ -210,14 +217,15 @@ def _listed_split(name: str, tensor: torch.Tensor, cfg: DecoderConfig) -> List[T
         return [(names[0], tensor)]
     m = _LAYER.match(name)
     sizes = [n for _, n in _listed_parts(m.group(2), cfg.layer_specs[int(m.group(1))], cfg.hidden_size)]
-    return list(zip(names, tensor.reshape(-1, tensor.shape[-1]).split(sizes, dim=0)))
+    return list(zip(names, (tensor if tensor.dim() == 1 else tensor.reshape(-1, tensor.shape[-1])).split(sizes, dim=0)))
 
 
 def _listed_join(name: str, cfg: DecoderConfig, get: Callable[[str], torch.Tensor], expert_range: Optional[Tuple[int, int]] = None) -> torch.Tensor:
     names = _listed_names(name, cfg)
     if '.experts.' in name:
-        lo, hi = expert_range or (0, len(names))
-        return torch.stack([get(n) for n in names[lo:hi]])
+        per = 2 if name.endswith('gate_up_proj') else 1
+        lo, hi = expert_range or (0, len(names) // per)
+        return torch.stack([torch.cat([get(n) for n in names[per * e:per * (e + 1)]], 0) for e in range(lo, hi)])
     return torch.cat([get(n).reshape(1) if n.endswith('.vmix') else get(n) for n in names], 0)
 
 

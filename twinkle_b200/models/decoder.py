@@ -22,7 +22,7 @@ import torch.nn as nn
 import torch.nn.functional as F
 
 from .. import ops
-from .config import DecoderConfig, SandwichSpec
+from .config import DecoderConfig, PreNormSpec, SandwichSpec
 from .layers import Embedding, Linear, RMSNorm
 from .parallel_layer import CacheView, ParallelLayer, Stream
 
@@ -52,6 +52,8 @@ class PackedBatch:
     deepstack: Optional[tuple] = None
     # stacks with listed layers: where the rows live in the sampler's cache (None: no cache is read or written)
     cache: Optional[CacheView] = None
+    # (cos, sin) of every row for all rotations of such a stack, [T, pairs, 2] fp32; set by the model forward
+    rotary: Optional[torch.Tensor] = None
     # under sequence / context parallelism: rows of the tower's output that belong to this rank's placeholder tokens
     vision_rows: Optional[torch.Tensor] = None
 
@@ -238,6 +240,11 @@ class MLP(nn.Module):
         callers that multiply or otherwise read the output pass ``False``."""
         return self.down_proj(self.act(self.gate_up_proj(x)), value_unused=value_unused)
 
+    def serve(self, x: torch.Tensor) -> torch.Tensor:
+        """:meth:`forward` without gradients, on the kernels of generation (any dtype)."""
+        gu = self.gate_up_proj(x)
+        return self.down_proj(ops.glu_columns(gu, 0, gu.shape[1] // 2, gu.shape[1] // 2) if self.act is ops.swiglu else self.act(gu))
+
 
 class Experts(nn.Module):
     """Fused expert weights ``gate_up_proj [E, 2I, H]`` and ``down_proj [E, H, I]``
@@ -302,8 +309,8 @@ class Experts(nn.Module):
             return None
         return self.lora[which + '_A'][slot, :, :r], self.lora[which + '_B'][slot, :, :, :r], scale
 
-    def forward(self, x_sorted: torch.Tensor, offsets: torch.Tensor) -> torch.Tensor:
-        """``x_sorted`` rows grouped by local expert; ``offsets [E_local+1]``."""
+    def forward(self, x_sorted: torch.Tensor, offsets: torch.Tensor, serving: bool = False) -> torch.Tensor:
+        """``x_sorted`` rows grouped by local expert; ``offsets [E_local+1]``.  ``serving``: no gradients, the kernels of generation."""
         if not self.gated:
             return self._forward_plain(x_sorted, offsets)
         lo = self._expert_lora('gate_up')
@@ -314,7 +321,7 @@ class Experts(nn.Module):
             row_expert = torch.bucketize(torch.arange(x_sorted.shape[0], device=x_sorted.device), offsets[1:].to(torch.long), right=True)
             row_expert = row_expert.clamp_(max=self.gate_up_proj.shape[0] - 1)
             gu = gu + self.gate_up_bias[row_expert].to(gu.dtype)
-        act = self.act(gu)
+        act = ops.glu_columns(gu, 0, gu.shape[1] // 2, gu.shape[1] // 2) if serving and self.act is ops.swiglu else self.act(gu)
         lo = self._expert_lora('down')
         y = ops.expert_linear(act, self.down_proj, offsets, *(lo or ()))
         return y if row_expert is None else y + self.down_bias[row_expert].to(y.dtype)
@@ -406,16 +413,23 @@ class MoEBlock(nn.Module):
             return self._with_shared(x, mp.forward(self, x, w, idx))
         return self._with_shared(x, self._routed_local(x, w, idx))
 
+    def rows_apply(self) -> bool:
+        """Whether :meth:`rows` serves this block now (no gradients, all experts here, a routing it has)."""
+        return self.moe_parallel is None and self.etp is None and not torch.is_grad_enabled() and self.cfg.router_scoring in ('topk_softmax', 'softmax_grouped')
+
     def rows(self, x: torch.Tensor, forced: Optional[torch.Tensor] = None):
-        """Inference form for blocks that choose by logit and weigh by a softmax over the chosen (``'topk_softmax'``): ``(expert rows
-        [T·k, H], their place [T, k], weights [T, k] fp32)``, left uncombined for a following kernel that reads them per token.
-        Router logits are fp32; rows of an expert are contiguous and nothing is padded."""
-        k = self.cfg.num_experts_per_tok
-        w, idx, hist = ops.moe_topk(ops.linear_f32(x, self.gate.weight), self.gate.bias, k, forced)
+        """Inference form: ``(expert rows [T·k, H], their place [T, k], weights [T, k] fp32, weight [T] fp32 of the shared expert or None)``,
+        left uncombined for a following kernel that reads them per token.  Router logits are fp32; rows of an expert are contiguous
+        and nothing is padded.  ``'topk_softmax'``: choice by biased logit, a softmax over the chosen; ``'softmax_grouped'``: a softmax over all
+        experts, a choice among the best groups."""
+        cfg, gate = self.cfg, self.shared_expert_gate if self.shared_expert is not None else None
+        grouped = dict(groups=cfg.n_group, keep=cfg.topk_group, factor=cfg.routed_scaling_factor) if cfg.router_scoring == 'softmax_grouped' else {}
+        w, idx, hist, *opened = ops.moe_topk(ops.linear_f32(x, self.gate.weight), self.gate.bias, cfg.num_experts_per_tok, forced, x=x,
+                                             shared=None if gate is None else gate.weight, **grouped)
         if self.record_routing:
             self.last_routed = idx.detach()
         xs, row_of, offsets = ops.moe_group_rows(x, idx, hist)
-        return self.experts(xs, offsets), row_of, w
+        return self.experts(xs, offsets, serving=True), row_of, w, opened[0] if opened else None
 
     def _forward_expert_tp(self, x, w, idx):
         """Expert tensor parallelism (reference ``megatron/strategy/megatron.py:90-107``: ``expert_tensor_parallel_size``):
@@ -548,10 +562,14 @@ class DecoderModel(nn.Module):
                 m.full_name = name
         self.layer_runner = None  # engine hook: runs one layer (checkpoint / FSDP unshard)
         self.tp = None  # tensor-parallel context, set by parallel.tensor.apply_tensor_parallel
+        self._frequencies: Dict[torch.device, torch.Tensor] = {}
 
     def _layer_class(self, i: int):
         if self.cfg.layer_specs is None:
             return DecoderLayer
+        if isinstance(self.cfg.layer_specs[i], PreNormSpec):
+            from .prenorm_layer import PreNormLayer
+            return PreNormLayer
         if isinstance(self.cfg.layer_specs[i], SandwichSpec):
             from .sandwich_layer import SandwichLayer
             return SandwichLayer
@@ -596,7 +614,9 @@ class DecoderModel(nn.Module):
             x = vocab_parallel_embedding(ids, self.embed_tokens.weight, self.tp)
         else:
             x = self.embed_tokens(ids)
-        if self.cfg.embed_scale != 1.0:
+        if self.cfg.embed_scale != 1.0 and self.cfg.layer_specs is not None:      # the start of a 32-bit stream
+            x = x.float() * self.cfg.embed_scale
+        elif self.cfg.embed_scale != 1.0:
             x = x * torch.tensor(self.cfg.embed_scale, dtype=x.dtype, device=x.device)
         return x
 
@@ -617,10 +637,21 @@ class DecoderModel(nn.Module):
             batch.deepstack = (where.nonzero(as_tuple=True)[0], deep) if deep else None
         return x
 
+    def rotary_table(self, positions: torch.Tensor) -> Optional[torch.Tensor]:
+        """Cosines and sines of all rotations of a stack with listed layers at these positions (None: it has none)."""
+        rots = self.cfg.rotations()
+        if not rots:
+            return None
+        f = self._frequencies.get(positions.device)
+        if f is None:       # kept per device; not a buffer, which would follow the model's dtype
+            f = self._frequencies[positions.device] = torch.tensor([v for r in rots for v in r.frequencies()], dtype=torch.float64, device=positions.device)
+        return ops.rotary_table(positions, f)
+
     def _forward_listed(self, batch: PackedBatch) -> torch.Tensor:
         """Stacks with listed layers: fp32 stream, final norm in the compute dtype (see ``models/parallel_layer.py``)."""
         cfg, run = self.cfg, self.layer_runner
         x = self.embed(batch)
+        batch.rotary = self.rotary_table(batch.position_ids)
         if run is None and not torch.is_grad_enabled():
             x = x.float().clone() if batch.inputs_embeds is not None else x.float()      # updated in place from here on
             st = Stream(x.contiguous())

@@ -254,7 +254,7 @@ class HGRN2(nn.Module):
     projected.  Everything between the two products is one kernel (``ops/csrc/hgrn2.cu``).  ``lead``: projections of the same input
     that are not this block's, in the leading columns of its input product."""
 
-    def __init__(self, width: int, spec, eps: float, layer_idx: int, lead=()):
+    def __init__(self, width: int, spec, eps: float, layer_idx: int, lead=(), table=None):
         super().__init__()
         self.spec, self.eps, self.layer_idx = spec, eps, layer_idx
         parts = list(lead) + spec.in_parts()

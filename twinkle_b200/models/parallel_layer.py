@@ -55,23 +55,38 @@ class GatedResult:
 
 
 @dataclass
+class PlainResult:
+    """A sub-layer's result on its way into the stream as it is: ``result [T, W]``, or expert rows with the places ``row_of [T, k]`` and
+    weights ``share [T, k]`` of every token's, plus ``beside [T, W]`` times ``open [T]`` (the shared expert)."""
+    result: torch.Tensor
+    row_of: Optional[torch.Tensor] = None
+    share: Optional[torch.Tensor] = None
+    beside: Optional[torch.Tensor] = None
+    open: Optional[torch.Tensor] = None
+
+
+@dataclass
 class Stream:
     """The residual stream between layers: ``x`` (fp32) plus sub-layer results that have not joined it yet (``adds`` times
-    ``mult``, or one gated and normed result), and what later layers take from earlier ones (``held``: layer → tensor)."""
+    ``mult``, one gated and normed result, or one plain result), and what later layers take from earlier ones (``held``: layer → tensor)."""
     x: torch.Tensor
     adds: List[Tuple[torch.Tensor, torch.Tensor]] = field(default_factory=list)
     held: Dict[int, torch.Tensor] = field(default_factory=dict)
     mult: float = 1.0
     gated: Optional[GatedResult] = None
+    plain: Optional[PlainResult] = None
 
     def enter(self, norm: RMSNorm) -> torch.Tensor:
         """What is pending joins the stream; returns its norm in the compute dtype — one kernel."""
         if self.gated is not None:
             g = self.gated
             h, self.x = ops.stream_gated_rmsnorm(self.x, norm.weight, norm.eps, norm.offset, g.result, g.gate, g.bias, g.norm.weight, g.row_of, g.share)
+        elif self.plain is not None:
+            y = self.plain
+            h, self.x = ops.stream_joined_rmsnorm(self.x, norm.weight, norm.eps, norm.offset, y.result, y.row_of, y.share, y.beside, y.open)
         else:
             h, self.x = ops.stream_rmsnorm(self.x, norm.weight, norm.eps, self.adds, self.mult, norm.offset)
-        self.adds, self.gated = [], None
+        self.adds, self.gated, self.plain = [], None, None
         return h
 
 

@@ -305,6 +305,67 @@ def stream_gated_rmsnorm(x, weight, eps: float, offset: float, result, gate, bia
     return ext().stream_gated_rmsnorm(x, weight, eps, offset, result.contiguous(), gate, bias, post, row_of, share), x
 
 
+def stream_joined_rmsnorm(x, weight, eps: float, offset: float, result, row_of=None, share=None, beside=None, open=None):
+    """fp32 residual stream ``x [T, W]``: ``x ← x + result + open · beside`` and the norm of the sum (weight ``offset + w``) in ``weight``'s dtype,
+    one kernel on CUDA.  ``result``: ``[T, W]``, or expert rows combined on the way (``row_of [T, k]``, ``share [T, k]``); ``beside [T, W]`` with a
+    weight ``open [T]`` per token, or None.  Returns ``(norm, x)``; without gradients ``x`` is updated in place."""
+    if not _cuda(x) or _needs_grad(x, weight, result, share, beside, open):
+        return ref.stream_joined_rmsnorm(x, weight, eps, offset, result, row_of, share, beside, open)
+    return ext().stream_joined_rmsnorm(x, weight, eps, offset, result.contiguous(), row_of, share, None if beside is None else beside.contiguous(), open), x
+
+
+# ------------------------------------------- rotated heads
+def rotary_table(positions, frequencies):
+    """``(cos, sin)`` of position times frequency (fp64 ``[n]``) as one fp32 tensor ``[T, n, 2]``."""
+    if _cuda(positions):
+        return ext().rotary_table(positions.contiguous(), frequencies)
+    return ref.rotary_table(positions, frequencies)
+
+
+def rotary_heads(proj, first: int, bias, q_weight, k_weight, table, at: int, pairs: int, interleaved: bool, hq: int, hkv: int, d: int, e: int, eps: float,
+                 view=None, layer: int = -1):
+    """Columns ``[q | k | v]`` of a fused projection from ``first`` on → ``(q [T,hq,d'], k [T,hkv,d'] | None, v [T,hkv,e'] | None)``: bias, RMS norm
+    of q and k per head (weights ``[d]``, None: none), rotation of the leading ``2 · pairs`` dimensions by columns ``at …`` of ``table``
+    (``rotary_table``).  ``hkv`` 0: queries only.  ``view`` (a ``CacheView``): keys and values are written to the cache; single steps return
+    queries only.  Widths ``d'``, ``e'`` are ``d``, ``e`` rounded up to multiples of 8, the rest zero; with gradients they are ``d`` and ``e``."""
+    step = view is not None and view.stepping
+    pools = (view.cache.k[layer], view.cache.v[layer], view.rows) if view is not None and hkv else (None, None, None)
+    if _cuda(proj) and not _needs_grad(proj, bias, q_weight, k_weight):
+        out = ext().rotary_heads(proj, first, bias, q_weight, k_weight, table, at, pairs, interleaved, hq, hkv, d, e, eps, *pools, not step)
+        return tuple(out) if len(out) == 3 else (out[0], None, None)
+    q, k, v = ref.rotary_heads(proj, first, bias, q_weight, k_weight, table[:, at:at + pairs], interleaved, hq, hkv, d, e, eps)
+    if _needs_grad(proj, bias, q_weight, k_weight):
+        return q, k, v
+    q, k, v = (None if t is None else torch.nn.functional.pad(t, (0, -t.shape[-1] % 8)) for t in (q, k, v))
+    if pools[0] is not None:
+        pools[0].view(-1, *k.shape[1:])[view.rows] = k
+        pools[1].view(-1, *v.shape[1:])[view.rows] = v
+    return (q, None, None) if step else (q, k, v)
+
+
+def latent_rotary(proj, q0: int, heads: int, d: int, r: int, c0: int, nc: int, wc, eps: float, table, at: int, pairs: int, interleaved: bool, rank: int, view=None,
+                  layer: int = -1):
+    """Queries ``[d | r]`` per head in columns ``q0 …`` and a latent with its key part ``[nc | r]`` in columns ``c0 …`` of a projection (``nc`` 0: the
+    layer borrows) → ``(q [T, heads, d + r], kept, ql)``.  The rotated dimensions ``r`` are turned by columns ``at …`` of ``table``, the latent is
+    RMS-normed; ``kept [T, n']`` is ``[latent | key part]`` (``n'``: rounded up to a multiple of 8, the rest zero), also written to the cache that
+    ``view`` names.  Prompts get the rotated query (without gradients ``proj`` is changed in place); single steps get ``ql [T, heads, rank + r]``
+    with the rotated part in its last ``r`` columns, ready for the rest of the query in latent space."""
+    T, step = proj.shape[0], view is not None and view.stepping
+    pool = view.cache.k[layer] if view is not None and nc else None
+    if _cuda(proj) and not _needs_grad(proj, wc):
+        ql = torch.empty(T, heads, rank + r, dtype=proj.dtype, device=proj.device) if step else None
+        kept = ext().latent_rotary(proj, q0, heads, d, r, c0, nc, wc, eps, table, at, pairs, interleaved, ql, pool, None if pool is None else view.rows, not step)
+        return proj[:, q0:q0 + heads * (d + r)].view(T, heads, d + r), (kept if nc and not step else None), ql
+    q, kept = ref.latent_rotary(proj, q0, heads, d, r, c0, nc, wc, eps, None if table is None else table[:, at:at + pairs], interleaved)
+    if _needs_grad(proj, wc):
+        return q, kept, None
+    if kept is not None:
+        kept = torch.nn.functional.pad(kept, (0, -kept.shape[-1] % 8))
+        if pool is not None:
+            pool.view(-1, pool.shape[-1])[view.rows] = kept
+    return q, kept, (torch.nn.functional.pad(q[..., d:], (rank, 0)) if step else None)
+
+
 # ------------------------------------------- latent attention, HGRN2
 def latent_norms(proj, q0: int, nq: int, wq, c0: int, nc: int, wc, eps: float, view=None, layer: int = -1):
     """Column ranges of a projection → the normed query bottleneck ``[T, nq]`` and the normed latent ``[T, nc']`` (``nc'``: ``nc`` rounded
@@ -321,22 +382,29 @@ def latent_norms(proj, q0: int, nq: int, wq, c0: int, nc: int, wc, eps: float, v
     return q, c
 
 
-def head_linear(x, weight, transposed: bool = False):
+def head_linear(x, weight, transposed: bool = False, out=None):
     """One small matrix per head: ``x [B, H, K]`` times ``weight[h]ᵀ`` for ``weight [H, N, K]``, or times ``weight[h]`` for ``[H, K, N]``
-    (``transposed``) → ``[B, H, N]``."""
+    (``transposed``) → ``[B, H, N]``.  ``out [B, H, ≥ N]``: the result goes into its leading columns, and it is returned."""
     n, k = (weight.shape[2], weight.shape[1]) if transposed else weight.shape[1:]
-    if _cuda(x) and x.dtype == torch.bfloat16 and n % 8 == 0 and k % 8 == 0 and not _needs_grad(x, weight):
-        return ext().head_gemm(x.contiguous(), weight, transposed)
+    if _cuda(x) and x.dtype == torch.bfloat16 and n % 8 == 0 and k % 8 == 0 and not _needs_grad(x, weight) and (out is None or out.shape[2] % 8 == 0):
+        y = ext().head_gemm(x if _tma_rows(x) else x.contiguous(), weight, transposed, None if out is None else out[..., :n])
+        return y if out is None else out
     w = weight if transposed else weight.transpose(1, 2)
-    return torch.bmm(x.transpose(0, 1), w).transpose(0, 1).contiguous()
+    y = torch.bmm(x.transpose(0, 1), w).transpose(0, 1)
+    if out is None:
+        return y.contiguous()
+    out[..., :n] = y
+    return out
 
 
-def latent_decode(q, pool, table, lens, scale: float, sinks, gate=None):
-    """One token per sequence, ``q [B, H, R]`` in latent space, against the cached latents ``pool [blocks, bs, 1, R']`` that are key and
-    value of every head; sink logits ``[H]`` in the denominator, result times ``σ(gate [B, H])``."""
+def latent_decode(q, pool, table, lens, scale: float, sinks=None, gate=None, rank: int = 0, window: int = 0):
+    """One token per sequence, ``q [B, H, K]`` in latent space, against the cached rows ``pool [blocks, bs, 1, K']``, keys of every head whose
+    first ``rank`` columns (0: all ``K``) are the values → ``[B, H, rank]``.  ``window``: only the last positions (0: all); sink logits
+    ``[H]`` in the denominator, result times ``σ(gate [B, H])``."""
+    rank = rank or q.shape[-1]
     if _cuda(q):
-        return ext().latent_decode(q.contiguous(), pool, table.to(torch.int32), lens.to(torch.int32), scale, sinks, gate)
-    return ref.latent_decode(q, pool, table, lens, scale, sinks, gate)
+        return ext().latent_decode(q.contiguous(), pool, table.to(torch.int32), lens.to(torch.int32), scale, sinks, gate, rank, window)
+    return ref.latent_decode(q, pool, table, lens, scale, sinks, gate, rank, window)
 
 
 def hgrn2(proj, q0: int, f0: int, v0: int, heads: int, dim: int, vdim: int, bias, lower, weight, eps: float, cu_seqlens=None, max_seqlen: int = 0,
@@ -394,25 +462,43 @@ def conv_heads(proj, weight, positions, hq: int, hkv: int, d: int, e: int, eps: 
     return q, (None if step else k), v
 
 
-def glu_columns(proj: torch.Tensor, gate: int, up: int, width: int) -> torch.Tensor:
-    """``silu(proj[:, gate : gate+width]) · proj[:, up : up+width]`` without copying the column ranges."""
+def glu_columns(proj: torch.Tensor, gate: int, up: int, width: int, limit: float = 0.0) -> torch.Tensor:
+    """``act(proj[:, gate : gate+width], proj[:, up : up+width])`` without copying the column ranges: ``silu(g) · u``, or with a ``limit``
+    ``g σ(1.702 g) (u + 1)`` on ``g ≤ limit`` and ``|u| ≤ limit``."""
     if _cuda(proj) and not _needs_grad(proj):
-        return ext().glu_columns(proj, gate, up, width)
-    return ref.swiglu(torch.cat([proj[:, gate:gate + width], proj[:, up:up + width]], -1))
+        return ext().glu_columns(proj, gate, up, width, limit)
+    gu = torch.cat([proj[:, gate:gate + width], proj[:, up:up + width]], -1)
+    return ref.clamped_glu(gu, limit) if limit else ref.swiglu(gu)
 
 
-def attention_packed(q, k, v, cu_seqlens, max_seqlen: int, scale: float, sinks=None, gate=None):
-    """Causal packed attention for any key / value widths up to 256: tensor-core kernel for bf16 heads up to 128 wide, an
-    fp32-arithmetic kernel for wider heads and for 32-bit models.  ``sinks [Hq]``: a logit per head in the denominator;
-    ``gate [T, Hq]``: the output of a head is multiplied by its sigmoid.  ``k`` and ``v`` may be column ranges of one tensor."""
-    if not _cuda(q) or _needs_grad(q, k, v, sinks, gate):
-        o = flash_attn_varlen(q, k, v, cu_seqlens, max_seqlen, True, scale, sinks=sinks)
+def _tma_rows(t) -> bool:
+    """Whether rows and heads of ``[T, H, D]`` start on 16-byte boundaries with unit stride inside a head (16-bit elements)."""
+    return t.stride(2) == 1 and t.stride(1) % 8 == 0 and t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0
+
+
+def attention_packed(q, k, v, cu_seqlens, max_seqlen: int, scale: float, sinks=None, gate=None, window: int = 0, chunk: int = 0, key_tail=None):
+    """Causal packed attention for any key / value widths up to 256: tensor-core kernel for bf16 heads (keys up to 192, values up to
+    128 wide), an fp32-arithmetic kernel for wider heads and for 32-bit models.  ``sinks [Hq]``: a logit per head in the denominator;
+    ``gate [T, Hq]``: the output of a head is multiplied by its sigmoid.  A position sees its last ``window`` keys, or its own block of
+    ``chunk`` positions (0: no bound).  ``k`` and ``v`` may be column ranges of one tensor; ``key_tail [T, r]``: further key dimensions that all
+    heads share (queries are ``[… | r]`` wide)."""
+    if not _cuda(q) or _needs_grad(q, k, v, sinks, gate, key_tail):
+        if key_tail is not None:
+            k = torch.cat([k, key_tail[:, None].expand(-1, k.shape[1], -1)], -1)
+        if window or chunk:
+            o = ref.attention_varlen(q, k, v, cu_seqlens, True, scale, window=window or None, sinks=sinks, chunk=chunk)
+        else:
+            o = flash_attn_varlen(q, k, v, cu_seqlens, max_seqlen, True, scale, sinks=sinks)
         return o if gate is None else (o.float() * torch.sigmoid(gate.float())[..., None]).to(o.dtype)
     cu = cu_seqlens.to(torch.int32)
-    if _flash_widths(q, k, v):
-        q, k, v = (t if t.stride(2) == 1 and t.stride(1) % 8 == 0 and t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0 else t.contiguous() for t in (q, k, v))
-        return ext().flash_attn_fwd(q, k, v, cu, int(max_seqlen), True, scale, None, sinks, gate)[0]
-    return ext().attention_packed(q.contiguous(), k.contiguous(), v.contiguous(), cu, int(max_seqlen), scale, sinks, gate)
+    if key_tail is not None:
+        d, r = k.shape[2], key_tail.shape[1]
+        if not (_flash_widths(q, k, v, 192) and d % 8 == 0 and r % 8 == 0 and d <= 128 and r <= 64 and key_tail.stride(0) % 8 == 0 and key_tail.data_ptr() % 16 == 0):
+            k, key_tail = torch.cat([k, key_tail[:, None].expand(-1, k.shape[1], -1)], -1), None
+    if _flash_widths(q, k, v, 192):
+        q, k, v = (t if _tma_rows(t) else t.contiguous() for t in (q, k, v))
+        return ext().flash_attn_fwd(q, k, v, cu, int(max_seqlen), True, scale, None, sinks, gate, window, chunk, key_tail)[0]
+    return ext().attention_packed(q.contiguous(), k.contiguous(), v.contiguous(), cu, int(max_seqlen), scale, sinks, gate, window, chunk)
 
 
 # ------------------------------------------------------------------ swiglu
@@ -514,10 +600,10 @@ class AttentionStash:
         AttentionStash.current = self._prev
 
 
-def _flash_widths(q, k, v) -> bool:
+def _flash_widths(q, k, v, widest: int = 128) -> bool:
     """Whether the forward kernel takes these heads (training also needs the backward kernel, which is for 128-wide heads)."""
     d, e = q.shape[-1], v.shape[-1]
-    return q.dtype == torch.bfloat16 and v.dtype == torch.bfloat16 and d <= 128 and e <= 128 and d % 8 == 0 and e % 8 == 0
+    return q.dtype == torch.bfloat16 and v.dtype == torch.bfloat16 and d <= widest and e <= 128 and d % 8 == 0 and e % 8 == 0
 
 
 def flash_attn_varlen(q, k, v, cu_seqlens, max_seqlen: int, causal: bool = True, scale: Optional[float] = None,
@@ -557,15 +643,16 @@ def flash_attn_varlen(q, k, v, cu_seqlens, max_seqlen: int, causal: bool = True,
 
 
 def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, scale: Optional[float] = None, window: Optional[int] = None,
-                           softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None):
+                           softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0, gate: Optional[torch.Tensor] = None):
+    """One query token per sequence against the paged cache.  It sees its last ``window`` keys, or its own block of ``chunk`` positions;
+    ``sinks [Hq]``: a logit per head in the denominator; ``gate [B, Hq]``: the output of a head is multiplied by its sigmoid."""
     scale = 1.0 / math.sqrt(q.shape[-1]) if scale is None else scale
-    if window is not None or softcap or sinks is not None:
-        return ref.paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, scale, window, softcap, sinks)
     vec = 16 // q.element_size()
-    if (_cuda(q) and q.dtype in (torch.bfloat16, torch.float32) and all(t.shape[-1] % vec == 0 and t.shape[-1] <= 256 for t in (q, v_cache))):
-        return ext().paged_attn_decode(q.contiguous(), k_cache, v_cache, block_tables.to(torch.int32),
-                                       seq_lens.to(torch.int32), scale)
-    return ref.paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, scale)
+    if (_cuda(q) and not softcap and q.dtype in (torch.bfloat16, torch.float32) and all(t.shape[-1] % vec == 0 and t.shape[-1] <= 256 for t in (q, v_cache))
+            and (sinks is None or sinks.dtype == q.dtype)):
+        return ext().paged_attn_decode(q.contiguous(), k_cache, v_cache, block_tables.to(torch.int32), seq_lens.to(torch.int32), scale, window or 0, chunk, sinks, gate)
+    o = ref.paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, scale, window, softcap, sinks, chunk)
+    return o if gate is None else (o.float() * torch.sigmoid(gate.float())[..., None]).to(o.dtype)
 
 
 # ------------------------------------------------------ gated delta net (linear attention)
@@ -1001,18 +1088,18 @@ def grouped_gemm(x, weight, offsets, act: Optional[str] = None):
     return torch.cat(outs, 0)
 
 
-def moe_topk(logits, bias, k: int, forced=None):
-    """fp32 ``logits [T, E]`` (+ ``bias``) → weights ``[T, k]`` fp32 (softmax over the k largest), their experts ``[T, k]`` int64, and tokens
-    per expert ``[E]`` int32.  ``forced``: experts to take instead (rows of −1: none)."""
+def moe_topk(logits, bias, k: int, forced=None, groups: int = 0, keep: int = 0, factor: float = 1.0, x=None, shared=None):
+    """fp32 ``logits [T, E]`` (+ ``bias``) → weights ``[T, k]`` fp32, their experts ``[T, k]`` int64, and tokens per expert ``[E]`` int32.
+    ``groups`` 0: the k largest, weighed by a softmax over just those.  Otherwise a softmax over all experts, the k largest inside the
+    ``keep`` best of ``groups`` groups of neighbours (a group is as good as its best expert), weighed by that softmax times ``factor``.
+    ``forced``: experts to take instead (rows of −1: none).  With ``shared [1, H]`` a fourth result is ``σ(x · shared)`` ``[T]`` fp32."""
     if _cuda(logits) and logits.shape[1] <= 256 and k <= 32:
-        return tuple(ext().moe_topk(logits, bias, k, None if forced is None else forced.to(logits.device).long().contiguous()))
+        return tuple(ext().moe_topk(logits, bias, k, None if forced is None else forced.to(logits.device).long().contiguous(), groups, keep, factor,
+                                    None if shared is None else x, shared))
     z = logits.float() + (bias.float() if bias is not None else 0.0)
-    top, idx = z.topk(k, -1)
-    if forced is not None:
-        idx = torch.where(forced[:, :1] < 0, idx, forced.long())
-        top = z.gather(1, idx)
+    w, idx = ref.moe_choice(z, k, forced, groups, keep, factor)
     hist = torch.zeros(z.shape[1], dtype=torch.int32, device=z.device).scatter_add_(0, idx.reshape(-1), torch.ones(idx.numel(), dtype=torch.int32, device=z.device))
-    return torch.softmax(top, -1), idx, hist
+    return (w, idx, hist) if shared is None else (w, idx, hist, torch.sigmoid(x.float() @ shared.float().t())[:, 0])
 
 
 def moe_group_rows(x, idx, hist):

@@ -204,15 +204,76 @@ def stream_gated_rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, offs
     return stream_rmsnorm(x, weight, eps, weight.dtype, offset=offset)
 
 
+def stream_joined_rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, offset: float, result: torch.Tensor, row_of: Optional[torch.Tensor] = None,
+                          share: Optional[torch.Tensor] = None, beside: Optional[torch.Tensor] = None, open: Optional[torch.Tensor] = None):
+    """fp32 residual stream: ``x ← x + result + open · beside``, then the norm of the sum (weight ``offset + w``) in ``weight``'s dtype.  ``result
+    [T, W]``, or expert rows of which token t has ``Σ_j share[t, j] · result[row_of[t, j]]``; ``open [T]``."""
+    y = result.float() if row_of is None else (result[row_of.long()].float() * share[..., None]).sum(1)
+    if beside is not None:
+        y = y + open.float()[:, None] * beside.float()
+    return stream_rmsnorm(x.float() + y, weight, eps, weight.dtype, offset=offset)
+
+
+# ------------------------------------------- rotated heads
+def rotary_table(positions: torch.Tensor, frequencies: torch.Tensor) -> torch.Tensor:
+    """``(cos, sin)`` of position times frequency ``[n]`` (fp64) as fp32 ``[T, n, 2]``."""
+    a = positions.double()[:, None] * frequencies
+    return torch.stack([a.cos(), a.sin()], -1).float()
+
+
+def rotate_pairs(x: torch.Tensor, table: torch.Tensor, interleaved: bool) -> torch.Tensor:
+    """``x [T, H, D]`` fp32, ``table [T, n, 2]``: the leading ``2n`` dimensions turned pair by pair, pairs ``(2i, 2i + 1)`` or ``(i, i + n)``."""
+    n = table.shape[1]
+    c, s = table[:, None, :, 0], table[:, None, :, 1]
+    a, b = (x[..., 0:2 * n:2], x[..., 1:2 * n:2]) if interleaved else (x[..., :n], x[..., n:2 * n])
+    ra, rb = a * c - b * s, b * c + a * s
+    return torch.cat([torch.stack([ra, rb], -1).flatten(-2) if interleaved else torch.cat([ra, rb], -1), x[..., 2 * n:]], -1)
+
+
+def rotary_heads(proj: torch.Tensor, first: int, bias: Optional[torch.Tensor], q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], table: torch.Tensor,
+                 interleaved: bool, hq: int, hkv: int, d: int, e: int, eps: float):
+    """Columns ``[q | k | v]`` from ``first`` on → ``(q [T,hq,d], k [T,hkv,d], v [T,hkv,e])`` (None without own keys): bias, RMS norm of q and k per
+    head, rotation.  fp32 inside; the results are rounded to the projection's dtype."""
+    T, n = proj.shape[0], hq * d + hkv * (d + e)
+    y = proj[:, first:first + n].float()
+    if bias is not None:
+        y = y + bias.float()
+    q, k, v = y[:, :hq * d].reshape(T, hq, d), y[:, hq * d:(hq + hkv) * d].reshape(T, hkv, d), y[:, (hq + hkv) * d:].reshape(T, hkv, e)
+    if q_weight is not None:
+        q = rmsnorm(q, q_weight, eps)
+    q = rotate_pairs(q, table, interleaved).to(proj.dtype)
+    if not hkv:
+        return q, None, None
+    if k_weight is not None:
+        k = rmsnorm(k, k_weight, eps)
+    return q, rotate_pairs(k, table, interleaved).to(proj.dtype), v.to(proj.dtype)
+
+
+def latent_rotary(proj: torch.Tensor, q0: int, heads: int, d: int, r: int, c0: int, nc: int, wc: Optional[torch.Tensor], eps: float, table: Optional[torch.Tensor],
+                  interleaved: bool):
+    """Queries ``[d | r]`` per head from column ``q0`` and ``[latent | key part]`` from column ``c0`` (``nc`` 0: none) → ``(q [T, heads, d + r], kept
+    [T, nc + r] | None)``: the ``r`` dimensions rotated, the latent RMS-normed."""
+    T = proj.shape[0]
+    q = proj[:, q0:q0 + heads * (d + r)].reshape(T, heads, d + r)
+    kept = rmsnorm(proj[:, c0:c0 + nc], wc, eps) if nc else None
+    if r:
+        q = torch.cat([q[..., :d], rotate_pairs(q[..., d:].float(), table, interleaved).to(proj.dtype)], -1)
+        if nc:
+            kept = torch.cat([kept, rotate_pairs(proj[:, None, c0 + nc:c0 + nc + r].float(), table, interleaved)[:, 0].to(proj.dtype)], -1)
+    return q, kept
+
+
 # ------------------------------------------- latent attention, HGRN2
 def latent_norms(proj: torch.Tensor, q0: int, nq: int, wq: torch.Tensor, c0: int, nc: int, wc: Optional[torch.Tensor], eps: float):
     """RMS norms of the query-bottleneck and latent column ranges of a projection (``nc`` 0: no latent)."""
     return rmsnorm(proj[:, q0:q0 + nq], wq, eps), rmsnorm(proj[:, c0:c0 + nc], wc, eps) if nc else None
 
 
-def latent_decode(q: torch.Tensor, pool: torch.Tensor, table: torch.Tensor, lens: torch.Tensor, scale: float, sinks: torch.Tensor, gate: Optional[torch.Tensor] = None):
-    """``q [B, H, R]`` against the cached latents of every sequence, which are key and value of all heads → ``[B, H, R]``."""
-    o = paged_attention_decode(q, pool[..., :q.shape[-1]], pool[..., :q.shape[-1]], table, lens, scale, sinks=sinks)
+def latent_decode(q: torch.Tensor, pool: torch.Tensor, table: torch.Tensor, lens: torch.Tensor, scale: float, sinks: Optional[torch.Tensor] = None,
+                  gate: Optional[torch.Tensor] = None, rank: int = 0, window: int = 0):
+    """``q [B, H, K]`` against the cached rows of every sequence, keys of all heads whose first ``rank`` columns (0: all) are the values →
+    ``[B, H, rank]``."""
+    o = paged_attention_decode(q, pool[..., :q.shape[-1]], pool[..., :rank or q.shape[-1]], table, lens, scale, window or None, sinks=sinks)
     return o if gate is None else (o.float() * torch.sigmoid(gate.float())[..., None]).to(o.dtype)
 
 
@@ -279,7 +340,7 @@ def relu2(x: torch.Tensor) -> torch.Tensor:
 # ----------------------------------------------------------------- attention
 def attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqlens: torch.Tensor, causal: bool = True,
                      scale: Optional[float] = None, return_lse: bool = False, cu_seqlens_k: Optional[torch.Tensor] = None,
-                     window: Optional[int] = None, softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None):
+                     window: Optional[int] = None, softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0):
     """Packed attention.  ``q [T,Hq,D]``, ``k,v [Tk,Hkv,D]``, ``cu_seqlens`` int
     ``[n+1]``; tokens of different segments never attend to each other; GQA by
     repeating each kv head ``Hq/Hkv`` times.  With ``cu_seqlens_k`` the keys of a segment may be longer than its
@@ -287,7 +348,7 @@ def attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqle
     ``window``: a query sees only the last ``window`` keys up to and including its own position (sliding-window
     checkpoints); ``softcap``: scores pass through ``cap · tanh(s / cap)`` before the softmax (Gemma-2); ``sinks [Hq]``: a
     learned logit per head that takes part in the softmax and carries no value (GPT-OSS), i.e. it only enlarges the
-    denominator."""
+    denominator; ``chunk``: a query sees only the keys of its own block of that many positions, counted from the sequence's start."""
     T, Hq, D = q.shape
     Hkv = k.shape[1]
     rep = Hq // Hkv
@@ -310,6 +371,9 @@ def attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqle
             s = s.masked_fill(torch.ones(L, Lk, dtype=torch.bool, device=q.device).triu(1 + Lk - L), float('-inf'))
             if window and Lk > window:
                 s = s.masked_fill(torch.ones(L, Lk, dtype=torch.bool, device=q.device).tril(Lk - L - window), float('-inf'))
+            if chunk and Lk > chunk:
+                block = torch.arange(Lk, device=q.device) // chunk
+                s = s.masked_fill(block[Lk - L:, None] != block, float('-inf'))
         l = torch.logsumexp(s, -1)
         if sinks is not None:
             l = torch.logaddexp(l, sinks.float()[:, None])
@@ -321,7 +385,7 @@ def attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqle
 
 def paged_attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_tables: torch.Tensor,
                            seq_lens: torch.Tensor, scale: Optional[float] = None, window: Optional[int] = None,
-                           softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                           softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0) -> torch.Tensor:
     """One query token per sequence against a paged KV cache.
     ``q [B,Hq,D]``; caches ``[num_blocks, block_size, Hkv, D]`` (values may have a width of their own); ``block_tables
     [B, max_blocks]`` int; ``seq_lens [B]`` (including the current token)."""
@@ -344,6 +408,8 @@ def paged_attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
             s = torch.tanh(s / softcap) * softcap
         if window and n > window:
             s[:, :n - window] = float('-inf')
+        if chunk:
+            s[:, :(n - 1) // chunk * chunk] = float('-inf')
         if sinks is not None:
             l = torch.logaddexp(torch.logsumexp(s, -1), sinks.float())
             out[b] = torch.einsum('hn,nhd->hd', torch.exp(s - l[:, None]), vv).to(q.dtype)
@@ -427,6 +493,21 @@ def moe_router(logits: torch.Tensor, top_k: int, renormalize: bool = True) -> Tu
     if renormalize:
         w = w / w.sum(-1, keepdim=True)
     return w, idx, probs
+
+
+def moe_choice(z: torch.Tensor, k: int, forced: Optional[torch.Tensor] = None, groups: int = 0, keep: int = 0, factor: float = 1.0):
+    """Weights ``[T, k]`` and experts ``[T, k]`` for router logits ``z [T, E]``.  ``groups`` 0: the k largest, a softmax over just those; otherwise a
+    softmax over all, choice among the ``keep`` groups with the best experts, weights times ``factor``.  ``forced``: see ``ops.moe_topk``."""
+    s = torch.softmax(z, -1)
+    c = z
+    if groups > 1:
+        best = z.view(z.shape[0], groups, -1).amax(-1).topk(keep, -1)[1]
+        allowed = torch.zeros(z.shape[0], groups, dtype=torch.bool, device=z.device).scatter_(1, best, True)
+        c = z.masked_fill(~allowed.repeat_interleave(z.shape[1] // groups, 1), float('-inf'))
+    idx = c.topk(k, -1)[1]
+    if forced is not None:
+        idx = torch.where(forced[:, :1] < 0, idx, forced.long())
+    return (s.gather(1, idx) * factor if groups else torch.softmax(z.gather(1, idx), -1)), idx
 
 
 def moe_aux_loss(probs: torch.Tensor, indices: torch.Tensor, num_experts: int) -> torch.Tensor:
