@@ -18,7 +18,7 @@ import os
 import sys
 from typing import Any, Dict, List
 
-MAX_LIVE = 1024     # sequences that may be live at a time (each needs a convolution-history slot)
+MAX_LIVE = 1024     # sequences that may be live at a time
 
 
 class TraceReplay:
@@ -85,7 +85,10 @@ def main(argv=None) -> int:
     torch.backends.cudnn.allow_tf32 = False
     from .. import ops
     from ..ops.build import prefer_serving
-    prefer_serving()
+    from ..models.config import DecoderConfig
+    cfg = DecoderConfig.from_pretrained(args.model)
+    if cfg.layer_specs is not None:
+        prefer_serving(cfg.kernel_parts())
     ops.ext()
     replay = TraceReplay(args.model, args.dtype, args.max_tokens)
     os.makedirs(args.out, exist_ok=True)

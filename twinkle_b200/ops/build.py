@@ -7,8 +7,8 @@ built module; when a GPU is present and the module is missing it is built on
 the spot, and any failure raises — there is no silent fallback on a GPU box.
 
 A process that only generates (``prefer_serving()``, e.g. the trace replayer) and finds no built ``_C.so`` compiles the
-serving subset into ``_C_serving.so`` instead: the kernels behind prefill, decode and sampling of listed-layer stacks.
-Objects are shared between the two builds.
+serving subset into ``_C_serving_….so`` instead: the kernels behind prefill, decode and sampling of listed-layer stacks, and of the
+mechanisms that not every such stack has (``_PARTS``) those of the model at hand.  Objects are shared between the builds.
 """
 from __future__ import annotations
 
@@ -19,33 +19,41 @@ import os
 import subprocess
 import sys
 import sysconfig
-from typing import List, Optional
+from typing import List, Optional, Sequence, Tuple
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 _CSRC = os.path.join(_HERE, 'csrc')
 _SO = os.path.join(_HERE, '_C.so')
 _STAMP = os.path.join(_HERE, '_C.stamp')
-_SERVING_SO = os.path.join(_HERE, '_C_serving.so')
-_SERVING_STAMP = os.path.join(_HERE, '_C_serving.stamp')
-_SERVING_SOURCES = ('bindings.cpp', 'host.cu', 'gemm.cu', 'gemm2.cu', 'attention_fwd.cu', 'attention_packed.cu', 'decode.cu', 'stream_ops.cu',
-                    'hgrn2.cu', 'latent.cu', 'latent_decode.cu', 'moe_serve.cu')
+_SERVING_SOURCES = ('bindings.cpp', 'host.cu', 'gemm.cu', 'gemm2.cu', 'attention_fwd.cu', 'attention_packed.cu', 'decode.cu', 'stream_ops.cu')
+# mechanism → its sources (``DecoderConfig.kernel_parts`` names those a model has)
+_PARTS = {'convolution': ('conv_heads.cu', ), 'experts': ('moe_serve.cu', ), 'latent': ('latent.cu', 'latent_decode.cu'), 'recurrent': ('hgrn2.cu', ), 'rotary': ('rotary.cu', )}
 _MOD = None
-_SERVING_ONLY = False
+_SERVING: Optional[Tuple[str, ...]] = None      # parts of the serving subset, when a process asked for it
 
 NVCC_FLAGS = ['-gencode', 'arch=compute_100a,code=sm_100a', '-lineinfo', '-O3', '-std=c++17', '--use_fast_math',
               '-Xcompiler', '-fPIC', '--expt-relaxed-constexpr', '--expt-extended-lambda', '-DNDEBUG',
               '-U__CUDA_NO_HALF_OPERATORS__', '-U__CUDA_NO_BFLOAT16_CONVERSIONS__', '-U__CUDA_NO_HALF_CONVERSIONS__']
 
 
-def prefer_serving() -> None:
-    """Let the serving subset stand in for the full extension when that is not built (call before the first kernel)."""
-    global _SERVING_ONLY
-    _SERVING_ONLY = True
+def prefer_serving(parts: Sequence[str] = tuple(_PARTS)) -> None:
+    """Let the serving subset with these mechanisms stand in for the full extension when that is not built (call before the first
+    kernel)."""
+    global _SERVING
+    _SERVING = tuple(sorted(set(parts)))
 
 
-def _sources(serving: bool = False) -> List[str]:
-    if serving:
-        return [os.path.join(_CSRC, f) for f in _SERVING_SOURCES]
+def _target(serving: Optional[Tuple[str, ...]] = None) -> Tuple[str, str]:
+    """Library and stamp of the full extension or of a serving subset."""
+    if serving is None:
+        return _SO, _STAMP
+    stem = os.path.join(_HERE, '_'.join(('_C_serving', ) + serving))
+    return stem + '.so', stem + '.stamp'
+
+
+def _sources(serving: Optional[Tuple[str, ...]] = None) -> List[str]:
+    if serving is not None:
+        return [os.path.join(_CSRC, f) for f in _SERVING_SOURCES + tuple(f for p in serving for f in _PARTS[p])]
     return sorted(glob.glob(os.path.join(_CSRC, '*.cu')) + glob.glob(os.path.join(_CSRC, '*.cpp')))
 
 
@@ -71,18 +79,18 @@ def _digest() -> str:
     return h.hexdigest()
 
 
-def is_built(serving: bool = False) -> bool:
-    so, stamp = (_SERVING_SO, _SERVING_STAMP) if serving else (_SO, _STAMP)
+def is_built(serving: Optional[Tuple[str, ...]] = None) -> bool:
+    so, stamp = _target(serving)
     if not os.path.isfile(so) or not os.path.isfile(stamp):
         return False
     with open(stamp) as f:
         return f.read().strip() == _digest()
 
 
-def build_extension(verbose: bool = False, jobs: Optional[int] = None, serving: bool = False) -> str:
+def build_extension(verbose: bool = False, jobs: Optional[int] = None, serving: Optional[Tuple[str, ...]] = None) -> str:
     """Compile each source to an object (in parallel) and link ``_C.so``.  Processes that arrive together (the ranks
     of one job) take a file lock in turn: the first builds, the others find the stamp current and return."""
-    so = _SERVING_SO if serving else _SO
+    so = _target(serving)[0]
     if is_built(serving):
         return so
     import fcntl
@@ -97,7 +105,7 @@ def build_extension(verbose: bool = False, jobs: Optional[int] = None, serving: 
         lock.close()
 
 
-def _build_locked(verbose: bool, jobs: Optional[int], serving: bool) -> str:
+def _build_locked(verbose: bool, jobs: Optional[int], serving: Optional[Tuple[str, ...]]) -> str:
     import torch
     from torch.utils import cpp_extension as ce
     from concurrent.futures import ThreadPoolExecutor
@@ -111,13 +119,16 @@ def _build_locked(verbose: bool, jobs: Optional[int], serving: bool) -> str:
     objs = []
 
     def compile_one(src: str) -> str:
-        own = ['-DTK_SERVING_ONLY'] if serving and src.endswith('bindings.cpp') else []
-        obj = os.path.join(build_dir, os.path.basename(src) + ('.serving' if own else '') + '.o')
+        own = []
+        if src.endswith('bindings.cpp'):
+            own = [f'-DTK_WITH_{p.upper()}' for p in (_PARTS if serving is None else serving)] + (['-DTK_SERVING_ONLY'] if serving is not None else [])
+        variant = '.' + '_'.join(('serving', ) + serving) if own and serving is not None else ''
+        obj = os.path.join(build_dir, os.path.basename(src) + variant + '.o')
         dep_stamp = obj + '.sha'
         h = hashlib.sha1(open(src, 'rb').read())
         for hdr in _local_includes(src):  # only the headers this source pulls in: touching one header rebuilds its users
             h.update(open(hdr, 'rb').read())
-        h.update(' '.join(NVCC_FLAGS).encode())
+        h.update(' '.join(NVCC_FLAGS + own).encode())
         if os.path.isfile(obj) and os.path.isfile(dep_stamp) and open(dep_stamp).read() == h.hexdigest():
             return obj
         cmd = [nvcc, '-c', src, '-o', obj] + NVCC_FLAGS + inc + defs + own
@@ -136,7 +147,7 @@ def _build_locked(verbose: bool, jobs: Optional[int], serving: bool) -> str:
     with ThreadPoolExecutor(max_workers=jobs or min(8, os.cpu_count() or 4)) as pool:
         objs = list(pool.map(compile_one, _sources(serving)))
     torch_lib = os.path.join(os.path.dirname(torch.__file__), 'lib')
-    so, stamp = (_SERVING_SO, _SERVING_STAMP) if serving else (_SO, _STAMP)
+    so, stamp = _target(serving)
     link = ['g++', '-shared', '-o', so] + objs + [
         '-L' + torch_lib, '-L' + os.path.join(cuda_home, 'lib64'), '-lc10', '-lc10_cuda', '-ltorch_cpu', '-ltorch_cuda',
         '-ltorch', '-ltorch_python', '-lcudart', '-Wl,-rpath,' + torch_lib, '-Wl,-rpath,' + os.path.join(cuda_home, 'lib64')]
@@ -154,8 +165,8 @@ def load_extension():
         return _MOD
     import torch  # noqa: F401  (libtorch must be loaded before the extension)
     so = _SO
-    if _SERVING_ONLY and not is_built():
-        so = build_extension(serving=True)
+    if _SERVING is not None and not is_built():
+        so = build_extension(serving=_SERVING)
     elif not is_built():
         if not torch.cuda.is_available() and os.environ.get('TWINKLE_B200_BUILD', '0') != '1' and not os.path.isfile(_SO):
             raise ImportError('twinkle_b200.ops._C is not built (run `python -c "import __graft_entry__ as g; g.build()"`)')

@@ -1,5 +1,8 @@
-// Flash-attention forward for sm_100a: causal, GQA, packed variable-length sequences, query / key and value widths up to 128.
-// A row narrower than its 64- or 128-wide tile is filled up with zeros by the TMA load (the tensor map ends at the row's width).
+// Flash-attention forward for sm_100a: causal, GQA, packed variable-length sequences, query / key widths up to 192, value widths up to
+// 128.  A row narrower than its tile of 64-wide chunks is filled up with zeros by the TMA load (the tensor map ends at the row's width).
+// Optional: only the last `window` keys or the query's block of `chunk` positions (key blocks before them are not loaded), sink logits, a
+// gate per head, and a last chunk of key dimensions that all heads share (rotated part of latent attention), loaded from a tensor of
+// its own so that nothing has to put the keys together.
 //
 // One CTA per (128-row query tile of one sequence, query head).  192 threads:
 //   warps 0-3  softmax: thread = one query row; reads S from tensor memory (tcgen05.ld), keeps the
@@ -24,9 +27,14 @@ namespace fa {
 constexpr int BQ = 128, BKV = 128, D = 128;
 constexpr int TILE_BYTES = 128 * 128 * 2;  // 32 KiB, two [128][64] swizzle atoms
 constexpr int ATOM_BYTES = 128 * 64 * 2;   // 16 KiB
-constexpr int SMEM_Q = 0, SMEM_K = TILE_BYTES, SMEM_V = 3 * TILE_BYTES, SMEM_P = 5 * TILE_BYTES, SMEM_BAR = 6 * TILE_BYTES;
-constexpr int SMEM_XCHG = SMEM_BAR + 256;           // row max (2 parities x 2 halves x 128) + row sums (2 x 128) floats
-constexpr int SMEM_TOTAL = SMEM_XCHG + 6 * 128 * 4 + 1024;
+// Q and two stages of K of KA atoms each, V in two stages (one when three-atom keys leave no room for more), P, barriers
+template <int KA>
+struct Smem {
+  static constexpr int K_TILE = KA > 2 ? 3 * ATOM_BYTES : TILE_BYTES, V_STAGES = KA > 2 ? 1 : 2;
+  static constexpr int Q = 0, K = K_TILE, V = 3 * K_TILE, P = V + V_STAGES * TILE_BYTES, BAR = P + TILE_BYTES;
+  static constexpr int XCHG = BAR + 256;            // row max (2 parities x 2 halves x 128) + row sums (2 x 128) floats
+  static constexpr int TOTAL = XCHG + 6 * 128 * 4 + 1024;
+};
 constexpr int THREADS = 320;  // warps 0-7 softmax (two groups of 4: each owns 64 of the 128 S columns), 8 producer, 9 MMA
 constexpr float RESCALE_THRESHOLD = 8.f;  // log2 units
 }  // namespace fa
@@ -43,15 +51,20 @@ struct FwdParams {
   const bf16* sinks;  // [Hq] logit of a key without a value that every row sees (nullptr: none)
   const bf16* gate;   // [T, Hq] with row stride ldg: the output is multiplied by its sigmoid (nullptr: not)
   long ldg;
+  int window, chunk;  // what a query sees of the keys before it (0: no bound)
+  int own_chunks;     // leading chunks of a key that are its head's own; the rest come from the shared tensor
+  int tail_col;       // first column of a query row that meets the shared part
   int* err;
 };
 
-// KA / VA: 64-wide chunks of a query / key row and of a value row (1 or 2).
+// KA / VA: 64-wide chunks of a query / key row (up to 3) and of a value row (1 or 2).
 template <int KA, int VA>
 __global__ void __launch_bounds__(fa::THREADS, 1)
 flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                 const __grid_constant__ CUtensorMap tmV, const FwdParams p) {
+                 const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmR, const FwdParams p) {
   using namespace fa;
+  using S = Smem<KA>;
+  constexpr int VS = S::V_STAGES;
   const int head = blockIdx.x, seq = blockIdx.z;
   const int seq_start = p.cu[seq], seq_len = p.cu[seq + 1] - seq_start;
   // longest-first: the heaviest (last) query tiles are scheduled first
@@ -65,11 +78,13 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   const int kv_start = p.cu_k[seq], kv_len = p.cu_k[seq + 1] - kv_start;
   const int q_off = kv_len - seq_len;
   const int kv_end = p.causal ? max(0, min(kv_len, q0 + BQ + q_off)) : kv_len;
-  const int n_blocks = (kv_end + BKV - 1) / BKV;
+  const bool bounded = p.window > 0 || p.chunk > 0;
+  const int jb0 = bounded ? first_visible(max(q0 + q_off, 0), p.window, p.chunk) / BKV : 0;    // first key block that any row sees
+  const int n_blocks = max(0, (kv_end + BKV - 1) / BKV - jb0);
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + SMEM_BAR);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + S::BAR);
   uint64_t* q_full = bars;            // 1
   uint64_t* k_full = bars + 1;        // 2
   uint64_t* v_full = bars + 3;        // 2
@@ -111,18 +126,26 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       tma_prefetch_desc(&tmK);
       tma_prefetch_desc(&tmV);
       mbar_expect_tx(q_full, KA * ATOM_BYTES);
-      tma_load_3d(smem + SMEM_Q, &tmQ, q_full, 0, head, seq_start + q0);
-      if constexpr (KA > 1) tma_load_3d(smem + SMEM_Q + ATOM_BYTES, &tmQ, q_full, 64, head, seq_start + q0);
+#pragma unroll
+      for (int c = 0; c < KA; ++c)
+        tma_load_3d(smem + S::Q + c * ATOM_BYTES, &tmQ, q_full, c < p.own_chunks ? c * 64 : p.tail_col, head, seq_start + q0);
       for (int j = 0; j < n_blocks; ++j) {
         const int st = j & 1;
         if (j >= 2 && !mbar_wait(&kv_empty[st], ((j >> 1) - 1) & 1, p.err, ERR_ATTN_WAIT)) break;
-        const int row = kv_start + j * BKV;
+        const int row = kv_start + (jb0 + j) * BKV;
         mbar_expect_tx(&k_full[st], KA * ATOM_BYTES);
-        tma_load_3d(smem + SMEM_K + st * TILE_BYTES, &tmK, &k_full[st], 0, kv_head, row);
-        if constexpr (KA > 1) tma_load_3d(smem + SMEM_K + st * TILE_BYTES + ATOM_BYTES, &tmK, &k_full[st], 64, kv_head, row);
-        mbar_expect_tx(&v_full[st], VA * ATOM_BYTES);
-        tma_load_3d(smem + SMEM_V + st * TILE_BYTES, &tmV, &v_full[st], 0, kv_head, row);
-        if constexpr (VA > 1) tma_load_3d(smem + SMEM_V + st * TILE_BYTES + ATOM_BYTES, &tmV, &v_full[st], 64, kv_head, row);
+#pragma unroll
+        for (int c = 0; c < KA; ++c) {
+          uint8_t* dst = smem + S::K + st * S::K_TILE + c * ATOM_BYTES;
+          if (c < p.own_chunks) tma_load_3d(dst, &tmK, &k_full[st], c * 64, kv_head, row);
+          else tma_load_3d(dst, &tmR, &k_full[st], 0, 0, row);
+        }
+        // a single stage of V is free once the product before has retired
+        if (VS == 1 && j >= 1 && !mbar_wait(&kv_empty[(j - 1) & 1], ((j - 1) >> 1) & 1, p.err, ERR_ATTN_WAIT)) break;
+        const int vs = j % VS;
+        mbar_expect_tx(&v_full[vs], VA * ATOM_BYTES);
+        tma_load_3d(smem + S::V + vs * TILE_BYTES, &tmV, &v_full[vs], 0, kv_head, row);
+        if constexpr (VA > 1) tma_load_3d(smem + S::V + vs * TILE_BYTES + ATOM_BYTES, &tmV, &v_full[vs], 64, kv_head, row);
       }
     }
   } else if (warp == 9) {
@@ -130,9 +153,9 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     if (lane == 0) {
       constexpr uint32_t idesc_s = umma_idesc_bf16(BQ, BKV, false, false);
       constexpr uint32_t idesc_o = umma_idesc_bf16(BQ, VA * 64, false, true);
-      const uint32_t sq = smem_u32(smem + SMEM_Q), sp = smem_u32(smem + SMEM_P);
+      const uint32_t sq = smem_u32(smem + S::Q), sp = smem_u32(smem + S::P);
       auto issue_s = [&](int j) {
-        const uint32_t sk = smem_u32(smem + SMEM_K + (j & 1) * TILE_BYTES);
+        const uint32_t sk = smem_u32(smem + S::K + (j & 1) * S::K_TILE);
 #pragma unroll
         for (int k = 0; k < KA * 4; ++k) {
           const uint32_t off = (k >> 2) * ATOM_BYTES + (k & 3) * 32;
@@ -154,10 +177,10 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           tc_fence_after();
           issue_s(n);
         }
-        ok = mbar_wait(p_ready, j & 1, p.err, ERR_ATTN_WAIT) && mbar_wait(&v_full[j & 1], (j >> 1) & 1, p.err, ERR_ATTN_WAIT);
+        ok = mbar_wait(p_ready, j & 1, p.err, ERR_ATTN_WAIT) && mbar_wait(&v_full[j % VS], (j / VS) & 1, p.err, ERR_ATTN_WAIT);
         if (!ok) break;
         tc_fence_after();
-        const uint32_t sv = smem_u32(smem + SMEM_V + (j & 1) * TILE_BYTES);
+        const uint32_t sv = smem_u32(smem + S::V + (j % VS) * TILE_BYTES);
 #pragma unroll
         for (int k = 0; k < BKV / 16; ++k) {
           // A = P (K-major over kv): atom k/4, 32-byte step inside; B = V (MN-major): 16 kv rows = 2048 B per step
@@ -179,13 +202,16 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const int row = (warp & 3) * 32 + lane;          // row inside the tile == TMEM lane
     const uint32_t lane_off = static_cast<uint32_t>((warp & 3) * 32) << 16;
     const int q_pos = q0 + row;                      // position inside the sequence
-    float* xmax = reinterpret_cast<float*>(smem + SMEM_XCHG);   // [parity][half][128]
+    float* xmax = reinterpret_cast<float*>(smem + S::XCHG);   // [parity][half][128]
     float* xsum = xmax + 4 * 128;                                 // [half][128]
+    // a row past the sequence's end keeps the bound of its place: what it computes is not stored
+    const int first = bounded ? first_visible(max(q_pos + q_off, 0), p.window, p.chunk) : 0;
+    const int first_last = bounded ? first_visible(max(q0 + BQ - 1 + q_off, 0), p.window, p.chunk) : 0;
     float m_used = -INFINITY, l_sum = 0.f;
     bool dead = false;
     for (int j = 0; j < n_blocks; ++j) {
       if (!dead && !mbar_wait(&s_full[j & 1], (j >> 1) & 1, p.err, ERR_ATTN_WAIT)) dead = true;
-      const int kv0 = j * BKV + wg * 64;
+      const int kv0 = (jb0 + j) * BKV + wg * 64;
       float sc[64];
       float mx = -INFINITY;
       if (!dead) {
@@ -197,13 +223,13 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         tmem_ld_wait();
         tc_fence_before();
         mbar_arrive(&s_empty[j & 1]);                 // scores are in registers: the TMEM buffer may be refilled
-        const bool need_mask = (kv0 + 64 > kv_end) || (p.causal && kv0 + 64 > q0 + q_off);
+        const bool need_mask = (kv0 + 64 > kv_end) || (p.causal && kv0 + 64 > q0 + q_off) || kv0 < first_last;
 #pragma unroll
         for (int i = 0; i < 64; ++i) {
           float sv = __uint_as_float(i < 32 ? r0[i] : r1[i - 32]) * p.scale_log2;
           if (need_mask) {
             const int col = kv0 + i;
-            if (col >= kv_end || (p.causal && col > q_pos + q_off)) sv = -INFINITY;
+            if (col >= kv_end || col < first || (p.causal && col > q_pos + q_off)) sv = -INFINITY;
           }
           sc[i] = sv;
           mx = fmaxf(mx, sv);
@@ -214,13 +240,14 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       mx = fmaxf(mx, xmax[((j & 1) * 2 + (wg ^ 1)) * 128 + row]);
       float alpha = 1.f;
       bool rescale = false;
-      if (mx > m_used + RESCALE_THRESHOLD || m_used == -INFINITY) {
-        const float m_new = (mx == -INFINITY) ? 0.f : mx;   // fully masked (garbage) rows stay finite
-        alpha = (m_used == -INFINITY) ? 0.f : exp2f(m_used - m_new);
+      // a row may see none of its first blocks: its maximum then stays at −∞ and its weights are zero
+      if (mx > m_used + RESCALE_THRESHOLD || (m_used == -INFINITY && mx != -INFINITY)) {
+        alpha = (m_used == -INFINITY) ? 0.f : exp2f(m_used - mx);
         rescale = (j > 0);
-        m_used = m_new;
+        m_used = mx;
         l_sum *= alpha;
       }
+      const float m_sub = m_used == -INFINITY ? 0.f : m_used;
       // P buffer and O accumulator are free once the previous P·V has retired
       if (!dead && j > 0 && !mbar_wait(o_done, (j - 1) & 1, p.err, ERR_ATTN_WAIT)) dead = true;
       if (dead) continue;
@@ -242,13 +269,13 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         uint32_t packed[16];
 #pragma unroll
         for (int i = 0; i < 32; i += 2) {
-          const float p0 = fast_exp2(sc[c * 32 + i] - m_used), p1 = fast_exp2(sc[c * 32 + i + 1] - m_used);
+          const float p0 = fast_exp2(sc[c * 32 + i] - m_sub), p1 = fast_exp2(sc[c * 32 + i + 1] - m_sub);
           // the sum uses the bf16-rounded values so that numerator and denominator match
           const __nv_bfloat162 pb = __floats2bfloat162_rn(p0, p1);
           l_sum += __low2float(pb) + __high2float(pb);
           packed[i >> 1] = *reinterpret_cast<const uint32_t*>(&pb);
         }
-        store_row_chunk_sw128(smem + SMEM_P, 128, row, wg * 64 + c * 32, packed);
+        store_row_chunk_sw128(smem + S::P, 128, row, wg * 64 + c * 32, packed);
       }
       tc_fence_before();
       fence_proxy_async();
@@ -300,14 +327,23 @@ CUtensorMap make_head_tmap(const torch::Tensor& t, int rows) {
 
 std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor& q, const torch::Tensor& k, const torch::Tensor& v, const torch::Tensor& cu,
                                           int64_t max_seqlen, bool causal, double scale, const c10::optional<torch::Tensor>& cu_k,
-                                          const c10::optional<torch::Tensor>& sinks, const c10::optional<torch::Tensor>& gate) {
+                                          const c10::optional<torch::Tensor>& sinks, const c10::optional<torch::Tensor>& gate, int64_t window, int64_t chunk,
+                                          const c10::optional<torch::Tensor>& key_tail) {
   TORCH_CHECK(q.is_cuda() && q.scalar_type() == torch::kBFloat16 && q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && k.size(0) == v.size(0) && k.size(1) == v.size(1) &&
                   k.scalar_type() == torch::kBFloat16 && v.scalar_type() == torch::kBFloat16, "q [T,Hq,D], k [T,Hkv,D], v [T,Hkv,E] bf16");
   for (const auto* t : {&q, &k, &v})
     TORCH_CHECK(t->stride(2) == 1 && t->stride(1) % 8 == 0 && t->stride(0) % 8 == 0 && reinterpret_cast<uintptr_t>(t->data_ptr()) % 16 == 0,
                 "q, k, v: unit stride inside a head, rows and heads on 16-byte boundaries");
-  TORCH_CHECK(q.size(2) == k.size(2) && k.size(2) % 8 == 0 && v.size(2) % 8 == 0 && k.size(2) > 0 && v.size(2) > 0 && k.size(2) <= 128 && v.size(2) <= 128,
-              "head widths: multiples of 8 up to 128");
+  const bool tail = key_tail.has_value() && key_tail->defined();
+  if (tail)
+    TORCH_CHECK(key_tail->is_cuda() && key_tail->scalar_type() == torch::kBFloat16 && key_tail->dim() == 2 && key_tail->size(0) == k.size(0) && key_tail->size(1) % 8 == 0 &&
+                    key_tail->size(1) > 0 && key_tail->size(1) <= 64 && key_tail->stride(1) == 1 && key_tail->stride(0) % 8 == 0 &&
+                    reinterpret_cast<uintptr_t>(key_tail->data_ptr()) % 16 == 0, "shared key part [T, up to 64] bf16 on 16-byte boundaries");
+  const int own_chunks = (static_cast<int>(k.size(2)) + 63) / 64, chunks = own_chunks + (tail ? 1 : 0);
+  TORCH_CHECK(q.size(2) == k.size(2) + (tail ? key_tail->size(1) : 0) && k.size(2) % 8 == 0 && v.size(2) % 8 == 0 && k.size(2) > 0 && v.size(2) > 0 && chunks <= 3 && v.size(2) <= 128,
+              "head widths: multiples of 8, keys up to 192 (three chunks of 64 with the shared part in one of its own), values up to 128");
+  TORCH_CHECK(window >= 0 && chunk >= 0 && window < (int64_t(1) << 30) && chunk < (int64_t(1) << 30), "window and chunk: 0 (none) or positive");
+  TORCH_CHECK(causal || (window == 0 && chunk == 0), "windows and chunks bound causal attention");
   TORCH_CHECK(cu.is_cuda() && cu.scalar_type() == torch::kInt32 && cu.is_contiguous(), "cu_seqlens int32 on device");
   TORCH_CHECK(q.size(1) % k.size(1) == 0, "Hq must be a multiple of Hkv");
   c10::cuda::CUDAGuard guard(q.device());
@@ -316,6 +352,7 @@ std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor& q, const torch::T
   auto lse = torch::empty({hq, T}, q.options().dtype(torch::kFloat32));
   if (T == 0 || nseq <= 0) return {out, lse};
   CUtensorMap tq = make_head_tmap(q, 128), tk_ = make_head_tmap(k, 128), tv = make_head_tmap(v, 128);
+  CUtensorMap tr = tail ? make_tmap_3d(key_tail->data_ptr(), key_tail->size(1), 1, key_tail->size(0), key_tail->stride(0), key_tail->stride(0), 64, 1, 128) : tk_;
   FwdParams p{};
   p.out = reinterpret_cast<bf16*>(out.data_ptr()); p.lse = lse.data_ptr<float>(); p.e = v.size(2); p.cu = cu.data_ptr<int>();
   p.cu_k = p.cu;
@@ -332,19 +369,22 @@ std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor& q, const torch::T
     p.gate = reinterpret_cast<const bf16*>(gate->data_ptr()); p.ldg = gate->stride(0);
   }
   p.T = T; p.hq = hq; p.hkv = hkv; p.scale_log2 = static_cast<float>(scale * 1.4426950408889634); p.causal = causal; p.err = error_word();
+  p.window = window; p.chunk = chunk; p.own_chunks = own_chunks; p.tail_col = k.size(2);
   const dim3 grid(hq, (static_cast<int>(max_seqlen) + fa::BQ - 1) / fa::BQ, nseq);
   auto stream = at::cuda::getCurrentCUDAStream();
 #define TK_FLASH(KA, VA)                                                                                                                \
   do {                                                                                                                                  \
     static bool configured = false;                                                                                                     \
     if (!configured) {                                                                                                                  \
-      TK_CUDA_CHECK(cudaFuncSetAttribute(flash_fwd_kernel<KA, VA>, cudaFuncAttributeMaxDynamicSharedMemorySize, fa::SMEM_TOTAL));       \
+      TK_CUDA_CHECK(cudaFuncSetAttribute(flash_fwd_kernel<KA, VA>, cudaFuncAttributeMaxDynamicSharedMemorySize, fa::Smem<KA>::TOTAL));  \
       configured = true;                                                                                                                \
     }                                                                                                                                   \
-    flash_fwd_kernel<KA, VA><<<grid, fa::THREADS, fa::SMEM_TOTAL, stream>>>(tq, tk_, tv, p);                                            \
+    flash_fwd_kernel<KA, VA><<<grid, fa::THREADS, fa::Smem<KA>::TOTAL, stream>>>(tq, tk_, tv, tr, p);                                   \
   } while (0)
-  const bool wide_k = q.size(2) > 64, wide_v = v.size(2) > 64;
-  if (wide_k && wide_v) TK_FLASH(2, 2);
+  const bool wide_k = chunks > 1, wide_v = v.size(2) > 64;
+  if (chunks == 3 && wide_v) TK_FLASH(3, 2);
+  else if (chunks == 3) TK_FLASH(3, 1);
+  else if (wide_k && wide_v) TK_FLASH(2, 2);
   else if (wide_k) TK_FLASH(2, 1);
   else if (wide_v) TK_FLASH(1, 2);
   else TK_FLASH(1, 1);

@@ -1,5 +1,5 @@
-// Causal attention over packed sequences in fp32 arithmetic, any key / value widths up to 256, grouped heads: the prefill
-// kernel for 32-bit models and for heads wider than the tensor-core kernel takes (attention_fwd.cu: bf16, up to 128).
+// Causal attention over packed sequences in fp32 arithmetic, any key / value widths up to 256, grouped heads, optionally within a
+// window or chunk: the prefill kernel for 32-bit models and for heads wider than the tensor-core kernel takes (attention_fwd.cu).
 //
 // One block per (32 query rows of one sequence, query head), 256 threads: eight threads per row.  Keys and values pass through
 // shared memory 32 rows at a time; a thread scores four keys of the tile and owns every eighth output column of its row.
@@ -25,7 +25,7 @@ __device__ __forceinline__ void st(bf16* p, float v) { *p = __float2bfloat16(v);
 template <typename T, int EI>
 __global__ void __launch_bounds__(256) attention_packed_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, T* __restrict__ out,
                                                                const int* __restrict__ cu, int hq, int hkv, int D, int E, float scale_log2,
-                                                               const T* __restrict__ sinks, const T* __restrict__ gate, long ldg) {
+                                                               const T* __restrict__ sinks, const T* __restrict__ gate, long ldg, int window, int chunk) {
   using namespace pa;
   extern __shared__ float sm[];
   const int head = blockIdx.x, seq = blockIdx.z, kvh = head / (hq / hkv);
@@ -47,8 +47,8 @@ __global__ void __launch_bounds__(256) attention_packed_kernel(const T* __restri
 #pragma unroll
   for (int i = 0; i < EI; ++i) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
-  const int end = min(len, q0 + BQ);
-  for (int k0 = 0; k0 < end; k0 += BK) {
+  const int end = min(len, q0 + BQ), first = first_visible(q0 + row, window, chunk);
+  for (int k0 = first_visible(q0, window, chunk) / BK * BK; k0 < end; k0 += BK) {
     __syncthreads();
     for (int i = threadIdx.x; i < BK * D; i += blockDim.x) {
       const int r = i / D, c = i - r * D;
@@ -68,17 +68,17 @@ __global__ void __launch_bounds__(256) attention_packed_kernel(const T* __restri
     float mx = m;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      if (k0 + sub + 8 * i > q0 + row || k0 + sub + 8 * i >= len) s[i] = -INFINITY;
+      if (k0 + sub + 8 * i > q0 + row || k0 + sub + 8 * i < first || k0 + sub + 8 * i >= len) s[i] = -INFINITY;
       mx = fmaxf(mx, s[i]);
     }
 #pragma unroll
     for (int o = 1; o < 8; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-    // key 0 is visible to every row, so mx is finite from the first tile on
-    const float corr = exp2f(m - mx);
+    // a row may not see any key of its tile's first keys
+    const float base = mx == -INFINITY ? 0.f : mx, corr = exp2f(m - base);
     float sum = 0.f;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      const float pr = exp2f(s[i] - mx);
+      const float pr = exp2f(s[i] - base);
       sp[row * (BK + 1) + sub + 8 * i] = pr;
       sum += pr;
     }
@@ -108,12 +108,13 @@ __global__ void __launch_bounds__(256) attention_packed_kernel(const T* __restri
 }
 
 torch::Tensor attention_packed(const torch::Tensor& q, const torch::Tensor& k, const torch::Tensor& v, const torch::Tensor& cu, int64_t max_seqlen, double scale,
-                               const c10::optional<torch::Tensor>& sinks, const c10::optional<torch::Tensor>& gate) {
+                               const c10::optional<torch::Tensor>& sinks, const c10::optional<torch::Tensor>& gate, int64_t window, int64_t chunk) {
   const auto st = q.scalar_type();
   TORCH_CHECK(q.is_cuda() && (st == torch::kBFloat16 || st == torch::kFloat32) && k.scalar_type() == st && v.scalar_type() == st, "q, k, v bf16 or fp32");
   TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && q.is_contiguous() && k.is_contiguous() && v.is_contiguous(), "[T, H, D] contiguous");
   TORCH_CHECK(q.size(2) == k.size(2) && k.size(0) == q.size(0) && v.size(0) == q.size(0) && k.size(1) == v.size(1) && q.size(1) % k.size(1) == 0, "shapes of q, k, v");
   TORCH_CHECK(q.size(2) <= 256 && v.size(2) <= 256, "head widths up to 256");
+  TORCH_CHECK(window >= 0 && chunk >= 0 && window < (int64_t(1) << 30) && chunk < (int64_t(1) << 30), "window and chunk: 0 (none) or positive");
   TORCH_CHECK(cu.is_cuda() && cu.scalar_type() == torch::kInt32 && cu.is_contiguous(), "cu_seqlens int32 on device");
   const bool has_sinks = sinks.has_value() && sinks->defined(), has_gate = gate.has_value() && gate->defined();
   if (has_sinks) TORCH_CHECK(sinks->is_cuda() && sinks->scalar_type() == st && sinks->is_contiguous() && sinks->numel() == q.size(1), "sinks [Hq]");
@@ -131,7 +132,7 @@ torch::Tensor attention_packed(const torch::Tensor& q, const torch::Tensor& k, c
     kern<<<grid, 256, smem, stream>>>(reinterpret_cast<const T*>(q.data_ptr()), reinterpret_cast<const T*>(k.data_ptr()), reinterpret_cast<const T*>(v.data_ptr()),
                                       reinterpret_cast<T*>(out.data_ptr()), cu.data_ptr<int>(), hq, hkv, D, E, static_cast<float>(scale * 1.4426950408889634),
                                       has_sinks ? reinterpret_cast<const T*>(sinks->data_ptr()) : nullptr, has_gate ? reinterpret_cast<const T*>(gate->data_ptr()) : nullptr,
-                                      has_gate ? gate->stride(0) : 0L);
+                                      has_gate ? gate->stride(0) : 0L, static_cast<int>(window), static_cast<int>(chunk));
   };
   if (st == torch::kBFloat16) {
     if (E <= 64) go(attention_packed_kernel<bf16, 8>, bf16{});

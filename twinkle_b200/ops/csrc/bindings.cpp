@@ -1,5 +1,6 @@
 // Python bindings of the sm_100a extension.  With TK_SERVING_ONLY the module holds just what generation with a
-// listed-layer stack launches (see ops/build.py): a box that only serves does not compile the training kernels.
+// listed-layer stack launches (see ops/build.py): a box that only serves does not compile the training kernels, nor those of
+// mechanisms that the model it serves does not have (TK_WITH_…).
 #include <torch/extension.h>
 
 #include "host.h"
@@ -9,10 +10,11 @@ torch::Tensor gemm(const torch::Tensor&, const torch::Tensor&, const std::string
                    c10::optional<torch::ScalarType>);
 std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t,
                                           bool, double, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&,
-                                          const c10::optional<torch::Tensor>&);
+                                          const c10::optional<torch::Tensor>&, int64_t, int64_t, const c10::optional<torch::Tensor>&);
 torch::Tensor attention_packed(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t, double,
-                               const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
-torch::Tensor paged_attn_decode(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, double);
+                               const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, int64_t, int64_t);
+torch::Tensor paged_attn_decode(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, double, int64_t, int64_t,
+                                const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
 std::vector<torch::Tensor> sample_tokens(const torch::Tensor&, double, int64_t, double, const torch::Tensor&);
 std::vector<torch::Tensor> conv_heads(const torch::Tensor&, const c10::optional<torch::Tensor>&, const torch::Tensor&, int64_t, int64_t, int64_t, int64_t,
                                       double, double, int64_t, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, bool,
@@ -20,24 +22,34 @@ std::vector<torch::Tensor> conv_heads(const torch::Tensor&, const c10::optional<
                                       const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, bool);
 torch::Tensor stream_rmsnorm(torch::Tensor, const torch::Tensor&, double, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&,
                              const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, double, double);
+torch::Tensor stream_joined_rmsnorm(torch::Tensor, const torch::Tensor&, double, double, const torch::Tensor&, const c10::optional<torch::Tensor>&,
+                                    const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
+torch::Tensor rotary_table(const torch::Tensor&, const torch::Tensor&);
+std::vector<torch::Tensor> rotary_heads(const torch::Tensor&, int64_t, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&,
+                                        const torch::Tensor&, int64_t, int64_t, bool, int64_t, int64_t, int64_t, int64_t, double, const c10::optional<torch::Tensor>&,
+                                        const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, bool);
+torch::Tensor latent_rotary(const torch::Tensor&, int64_t, int64_t, int64_t, int64_t, int64_t, int64_t, const c10::optional<torch::Tensor>&, double,
+                            const c10::optional<torch::Tensor>&, int64_t, int64_t, bool, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&,
+                            const c10::optional<torch::Tensor>&, bool);
 torch::Tensor stream_gated_rmsnorm(torch::Tensor, const torch::Tensor&, double, double, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&,
                                    const torch::Tensor&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
 std::vector<torch::Tensor> latent_norms(const torch::Tensor&, int64_t, int64_t, const torch::Tensor&, int64_t, int64_t, const c10::optional<torch::Tensor>&, double,
                                         const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
-torch::Tensor latent_decode(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, double, const torch::Tensor&,
-                            const c10::optional<torch::Tensor>&);
+torch::Tensor latent_decode(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, double, const c10::optional<torch::Tensor>&,
+                            const c10::optional<torch::Tensor>&, int64_t, int64_t);
 torch::Tensor hgrn2_prefill(const torch::Tensor&, int64_t, int64_t, int64_t, int64_t, int64_t, int64_t, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&,
                             double, const torch::Tensor&, int64_t, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
 torch::Tensor hgrn2_step(const torch::Tensor&, int64_t, int64_t, int64_t, int64_t, int64_t, int64_t, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&,
                          double, const torch::Tensor&, const torch::Tensor&);
-std::vector<torch::Tensor> moe_topk(const torch::Tensor&, const c10::optional<torch::Tensor>&, int64_t, const c10::optional<torch::Tensor>&);
+std::vector<torch::Tensor> moe_topk(const torch::Tensor&, const c10::optional<torch::Tensor>&, int64_t, const c10::optional<torch::Tensor>&, int64_t, int64_t, double,
+                                    const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
 std::vector<torch::Tensor> moe_group_rows(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&);
 torch::Tensor grouped_gemm_f32(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, bool);
-torch::Tensor head_gemm(const torch::Tensor&, const torch::Tensor&, bool);
+torch::Tensor head_gemm(const torch::Tensor&, const torch::Tensor&, bool, const c10::optional<torch::Tensor>&);
 torch::Tensor grouped_gemm(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const std::string&, const c10::optional<torch::Tensor>&,
                            const c10::optional<torch::Tensor>&, bool, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&,
                            const c10::optional<std::string>&);
-torch::Tensor glu_columns(const torch::Tensor&, int64_t, int64_t, int64_t);
+torch::Tensor glu_columns(const torch::Tensor&, int64_t, int64_t, int64_t, double);
 void set_gemm_pair(int64_t);
 void set_gemm_staged(int64_t);
 #ifndef TK_SERVING_ONLY
@@ -95,8 +107,10 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm", &tk::gemm, py::arg("a"), py::arg("b"), py::arg("layout") = "nt", py::arg("out") = py::none(),
         py::arg("accumulate") = false, py::arg("out_dtype") = py::none());
   m.def("flash_attn_fwd", &tk::flash_attn_fwd, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("cu"), py::arg("max_seqlen"), py::arg("causal"),
-        py::arg("scale"), py::arg("cu_k") = py::none(), py::arg("sinks") = py::none(), py::arg("gate") = py::none());
-  m.def("paged_attn_decode", &tk::paged_attn_decode);
+        py::arg("scale"), py::arg("cu_k") = py::none(), py::arg("sinks") = py::none(), py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("chunk") = 0,
+        py::arg("key_tail") = py::none());
+  m.def("paged_attn_decode", &tk::paged_attn_decode, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("tables"), py::arg("seq_lens"), py::arg("scale"),
+        py::arg("window") = 0, py::arg("chunk") = 0, py::arg("sinks") = py::none(), py::arg("gate") = py::none());
   m.def("sample_tokens", &tk::sample_tokens);
   m.def("set_gemm_pair", &tk::set_gemm_pair);
   m.def("set_gemm_staged", &tk::set_gemm_staged);
@@ -104,25 +118,42 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("num_sms", &tk::num_sms);
   m.def("launch_count", &tk::launch_count, "Number of kernels launched by this extension so far.");
   m.def("attention_packed", &tk::attention_packed, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("cu"), py::arg("max_seqlen"), py::arg("scale"),
-        py::arg("sinks") = py::none(), py::arg("gate") = py::none());
+        py::arg("sinks") = py::none(), py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("chunk") = 0);
+#ifdef TK_WITH_CONVOLUTION
   m.def("conv_heads", &tk::conv_heads, py::arg("proj"), py::arg("weight"), py::arg("pos"), py::arg("hq"), py::arg("hkv"), py::arg("d"), py::arg("e"), py::arg("eps"),
         py::arg("coef") = 0.0, py::arg("every") = 0, py::arg("v_first") = py::none(), py::arg("lam") = py::none(), py::arg("step") = false,
         py::arg("hist") = py::none(), py::arg("slot") = py::none(), py::arg("left") = py::none(), py::arg("pool_row") = py::none(),
         py::arg("k_pool") = py::none(), py::arg("v_pool") = py::none(), py::arg("want_k") = true);
+#endif
+#ifdef TK_WITH_ROTARY
+  m.def("rotary_table", &tk::rotary_table);
+  m.def("rotary_heads", &tk::rotary_heads);
+  m.def("latent_rotary", &tk::latent_rotary);
+#endif
   m.def("stream_rmsnorm", &tk::stream_rmsnorm, py::arg("x"), py::arg("w"), py::arg("eps"), py::arg("y1") = py::none(), py::arg("s1") = py::none(),
         py::arg("y2") = py::none(), py::arg("s2") = py::none(), py::arg("mult") = 1.0, py::arg("offset") = 0.0);
   m.def("stream_gated_rmsnorm", &tk::stream_gated_rmsnorm);
+  m.def("stream_joined_rmsnorm", &tk::stream_joined_rmsnorm, py::arg("x"), py::arg("w"), py::arg("eps"), py::arg("offset"), py::arg("y"), py::arg("row_of") = py::none(),
+        py::arg("share") = py::none(), py::arg("beside") = py::none(), py::arg("open") = py::none());
+#ifdef TK_WITH_LATENT
   m.def("latent_norms", &tk::latent_norms);
-  m.def("latent_decode", &tk::latent_decode);
+  m.def("latent_decode", &tk::latent_decode, py::arg("q"), py::arg("pool"), py::arg("tables"), py::arg("lens"), py::arg("scale"), py::arg("sinks"), py::arg("gate"),
+        py::arg("rank"), py::arg("window") = 0);
+#endif
+#ifdef TK_WITH_RECURRENT
   m.def("hgrn2_prefill", &tk::hgrn2_prefill);
   m.def("hgrn2_step", &tk::hgrn2_step);
-  m.def("moe_topk", &tk::moe_topk);
+#endif
+#ifdef TK_WITH_EXPERTS
+  m.def("moe_topk", &tk::moe_topk, py::arg("logits"), py::arg("bias"), py::arg("k"), py::arg("forced") = py::none(), py::arg("groups") = 0, py::arg("keep") = 0,
+        py::arg("factor") = 1.0, py::arg("x") = py::none(), py::arg("shared") = py::none());
   m.def("moe_group_rows", &tk::moe_group_rows);
   m.def("grouped_gemm_f32", &tk::grouped_gemm_f32);
-  m.def("head_gemm", &tk::head_gemm);
+#endif
+  m.def("head_gemm", &tk::head_gemm, py::arg("x"), py::arg("w"), py::arg("nn"), py::arg("out") = py::none());
   m.def("grouped_gemm", &tk::grouped_gemm, py::arg("x"), py::arg("w"), py::arg("offsets"), py::arg("layout") = "nt", py::arg("group_map") = py::none(),
         py::arg("out") = py::none(), py::arg("accumulate") = false, py::arg("x2") = py::none(), py::arg("w2") = py::none(), py::arg("act") = py::none());
-  m.def("glu_columns", &tk::glu_columns);
+  m.def("glu_columns", &tk::glu_columns, py::arg("p"), py::arg("gate"), py::arg("up"), py::arg("width"), py::arg("limit") = 0.0);
 #ifndef TK_SERVING_ONLY
   m.def("grouped_gemm_wgrad", &tk::grouped_gemm_wgrad);
   m.def("rmsnorm_fwd", &tk::rmsnorm_fwd, py::arg("x"), py::arg("w"), py::arg("eps"), py::arg("offset"), py::arg("residual") = py::none());

@@ -200,6 +200,13 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
+// First key that a query at `pos` sees: of its last `window` positions, or of its own block of `chunk` positions (0: no such bound).
+__device__ __forceinline__ int first_visible(int pos, int window, int chunk) {
+  int a = window > 0 ? max(0, pos - window + 1) : 0;
+  if (chunk > 0) a = max(a, pos / chunk * chunk);
+  return a;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

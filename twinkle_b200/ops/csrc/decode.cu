@@ -18,6 +18,13 @@ using bf16 = __nv_bfloat16;
 // per token, each lane NC 16-byte vectors of the K row and of the V row — and U steps are issued back to back (two for rows
 // of up to 256 bytes: 32 token rows per CTA in flight).  Every lane group keeps an online-softmax state per query head;
 // lane groups and warps are merged at the end.  Key and value rows are `d` and `e` elements wide, whole 16-byte vectors.
+// Optional: only the last `window` keys or the query's block of `chunk` positions, a sink logit per head in the denominator, a
+// sigmoid gate per head on the result.
+struct PagedExtras {
+  const void *sinks, *gate;   // [hq], [B, hq] with row stride ldg (nullptr: none)
+  long ldg;
+  int window, chunk;
+};
 __device__ __forceinline__ void unpack_vec(const uint4& u, float (&x)[8], const bf16*) {
   const uint32_t w[4] = {u.x, u.y, u.z, u.w};
 #pragma unroll
@@ -37,11 +44,11 @@ __device__ __forceinline__ void put(float* p, float v) { *p = v; }
 template <typename T, int GH, int NC, int U>
 __global__ void __launch_bounds__(128) paged_decode_kernel(const T* __restrict__ q, const T* __restrict__ kc, const T* __restrict__ vc,
                                                             const int* __restrict__ tables, const int* __restrict__ seq_lens, T* __restrict__ out,
-                                                            int hq, int hkv, int d, int e, int block_size, int max_blocks, float scale_log2, int G) {
+                                                            int hq, int hkv, int d, int e, int block_size, int max_blocks, float scale_log2, int G, const PagedExtras x) {
   constexpr int V = 16 / sizeof(T), D = NC * 8 * V;   // elements per vector, widest row of this instance
   const int b = blockIdx.x, kvh = blockIdx.y, g0 = blockIdx.z * GH, h0 = kvh * G + g0;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, grp = lane >> 3, sub = lane & 7;  // vector c of a lane: elements [(8c + sub)·V, …+V)
-  const int n = seq_lens[b];
+  const int n = seq_lens[b], first = n > 0 ? first_visible(n - 1, x.window, x.chunk) : 0;
   // the query (pre-scaled, fp32) lives in shared memory: registers are kept for two iterations' worth of K/V rows
   __shared__ __align__(16) float s_q[GH][D];
   for (int i = threadIdx.x; i < GH * D; i += blockDim.x) {
@@ -77,8 +84,8 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const T* __restrict__
       }
     }
   };
-  if (warp * 4 < n) fetch(warp * 4, kr, vr);
-  for (int base = warp * 4; base < n; base += 16 * U) {
+  if (first + warp * 4 < n) fetch(first + warp * 4, kr, vr);
+  for (int base = first + warp * 4; base < n; base += 16 * U) {
     if (base + 16 * U < n) fetch(base + 16 * U, kn, vn);
 #pragma unroll
     for (int u = 0; u < U; ++u) {
@@ -149,14 +156,20 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const T* __restrict__
 #pragma unroll
     for (int g = 0; g < GH; ++g) {
       if (g0 + g >= G) break;
-      const float mm = fmaxf(fmaxf(s_m[0][g], s_m[1][g]), fmaxf(s_m[2][g], s_m[3][g]));
+      float mm = fmaxf(fmaxf(s_m[0][g], s_m[1][g]), fmaxf(s_m[2][g], s_m[3][g]));
       float ll = 0.f, o = 0.f;
+      if (x.sinks != nullptr) {
+        const float sink = to_float(reinterpret_cast<const T*>(x.sinks)[h0 + g]) * 1.4426950408889634f;
+        mm = fmaxf(mm, sink);
+        ll = exp2f(sink - mm);
+      }
 #pragma unroll
       for (int w = 0; w < 4; ++w) {
         const float c = (s_m[w][g] == -INFINITY) ? 0.f : exp2f(s_m[w][g] - mm);
         ll += s_l[w][g] * c;
         o += s_acc[w][g][i] * c;
       }
+      if (x.gate != nullptr) ll *= 1.f + __expf(-to_float(reinterpret_cast<const T*>(x.gate)[b * x.ldg + h0 + g]));
       put(out + (static_cast<size_t>(b) * hq + h0 + g) * e + i, ll > 0.f ? o / ll : 0.f);
     }
   }
@@ -164,14 +177,14 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const T* __restrict__
 
 template <typename T>
 static void launch_paged_decode(const torch::Tensor& q, const torch::Tensor& kc, const torch::Tensor& vc, const torch::Tensor& tables,
-                                const torch::Tensor& seq_lens, torch::Tensor& out, float sl2, cudaStream_t stream) {
+                                const torch::Tensor& seq_lens, torch::Tensor& out, float sl2, const PagedExtras& extras, cudaStream_t stream) {
   constexpr int V = 16 / sizeof(T);
   const int B = q.size(0), hq = q.size(1), hkv = kc.size(2), G = hq / hkv, d = q.size(2), e = vc.size(3);
   auto go = [&](auto kern, int GH) {
     // query heads of a group are processed GH at a time (register budget): G = 8 → two CTAs per (sequence, kv head)
     kern<<<dim3(B, hkv, (G + GH - 1) / GH), 128, 0, stream>>>(reinterpret_cast<const T*>(q.data_ptr()), reinterpret_cast<const T*>(kc.data_ptr()),
         reinterpret_cast<const T*>(vc.data_ptr()), tables.data_ptr<int>(), seq_lens.data_ptr<int>(), reinterpret_cast<T*>(out.data_ptr()), hq, hkv, d, e,
-        static_cast<int>(kc.size(1)), static_cast<int>(tables.size(1)), sl2, G);
+        static_cast<int>(kc.size(1)), static_cast<int>(tables.size(1)), sl2, G, extras);
   };
   const int vectors = (std::max(d, e) + 8 * V - 1) / (8 * V);   // per lane
   if (vectors <= 1) {
@@ -186,7 +199,8 @@ static void launch_paged_decode(const torch::Tensor& q, const torch::Tensor& kc,
 }
 
 torch::Tensor paged_attn_decode(const torch::Tensor& q, const torch::Tensor& kc, const torch::Tensor& vc, const torch::Tensor& tables,
-                                const torch::Tensor& seq_lens, double scale) {
+                                const torch::Tensor& seq_lens, double scale, int64_t window, int64_t chunk, const c10::optional<torch::Tensor>& sinks,
+                                const c10::optional<torch::Tensor>& gate) {
   const auto st = q.scalar_type();
   TORCH_CHECK(q.is_cuda() && (st == torch::kBFloat16 || st == torch::kFloat32) && q.is_contiguous() && q.dim() == 3, "q [B,Hq,D] bf16 or fp32");
   TORCH_CHECK(kc.is_contiguous() && vc.is_contiguous() && kc.dim() == 4 && vc.dim() == 4 && kc.scalar_type() == st && vc.scalar_type() == st, "caches [blocks,bs,Hkv,·] in q's dtype");
@@ -194,13 +208,24 @@ torch::Tensor paged_attn_decode(const torch::Tensor& q, const torch::Tensor& kc,
   TORCH_CHECK(kc.size(3) == q.size(2) && kc.size(3) % V == 0 && vc.size(3) % V == 0 && kc.size(3) <= 256 && vc.size(3) <= 256, "rows of whole 16-byte vectors, up to 256 wide");
   TORCH_CHECK(kc.size(0) == vc.size(0) && kc.size(1) == vc.size(1) && kc.size(2) == vc.size(2) && q.size(1) % kc.size(2) == 0, "shapes of the caches");
   TORCH_CHECK(tables.scalar_type() == torch::kInt32 && tables.is_contiguous() && seq_lens.scalar_type() == torch::kInt32, "int32 tables / lens");
+  PagedExtras x{};
+  TORCH_CHECK(window >= 0 && chunk >= 0 && window < (int64_t(1) << 30) && chunk < (int64_t(1) << 30), "window and chunk: 0 (none) or positive");
+  x.window = window; x.chunk = chunk;
+  if (sinks.has_value() && sinks->defined()) {
+    TORCH_CHECK(sinks->is_cuda() && sinks->scalar_type() == st && sinks->is_contiguous() && sinks->numel() == q.size(1), "sinks [Hq] in q's dtype");
+    x.sinks = sinks->data_ptr();
+  }
+  if (gate.has_value() && gate->defined()) {
+    TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == st && gate->dim() == 2 && gate->size(0) == q.size(0) && gate->size(1) == q.size(1) && gate->stride(1) == 1, "gate [B, Hq]");
+    x.gate = gate->data_ptr(); x.ldg = gate->stride(0);
+  }
   c10::cuda::CUDAGuard guard(q.device());
   auto out = torch::empty({q.size(0), q.size(1), vc.size(3)}, q.options());
   if (q.size(0) == 0) return out;
   const float sl2 = static_cast<float>(scale * 1.4426950408889634);
   auto stream = at::cuda::getCurrentCUDAStream();
-  if (st == torch::kBFloat16) launch_paged_decode<bf16>(q, kc, vc, tables, seq_lens, out, sl2, stream);
-  else launch_paged_decode<float>(q, kc, vc, tables, seq_lens, out, sl2, stream);
+  if (st == torch::kBFloat16) launch_paged_decode<bf16>(q, kc, vc, tables, seq_lens, out, sl2, x, stream);
+  else launch_paged_decode<float>(q, kc, vc, tables, seq_lens, out, sl2, x, stream);
   count_launch();
   TK_CUDA_CHECK(cudaGetLastError());
   return out;

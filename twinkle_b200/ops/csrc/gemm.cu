@@ -44,6 +44,7 @@ struct GemmParams {
   int group_rows_b;    // rows of B per group (N for NT, K for NN)
   int mode;            // 0 dense, 1 grouped over M (A rows by expert), 2 grouped wgrad (K range by expert), 3 one product per head
   int act;             // 1: the square of relu on the result
+  int head_cols;       // one product per head: output columns from one head to the next
   const int* group_map;  // optional: group g uses weight block group_map[g] (< 0: group skipped); nullptr = identity
   // second operand pair of the M-grouped mode (0 = none): out = A·B + A2·B2 accumulated in tensor memory before the
   // epilogue — how a low-rank (LoRA) term rides in the base GEMM instead of re-reading and re-writing the output
@@ -276,7 +277,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_consta
       const bool row_ok = row < t.m_limit;
       size_t out_row = static_cast<size_t>(row);
       if constexpr (MODE == 2) out_row += static_cast<size_t>(t.group) * p.M;
-      const size_t head0 = MODE == 3 ? static_cast<size_t>(t.group) * p.N : 0;   // first output column of the head
+      const size_t head0 = MODE == 3 ? static_cast<size_t>(t.group) * p.head_cols : 0;   // first output column of the head
 #pragma unroll 1
       for (int c = 0; c < BN / 32; ++c) {
         uint32_t r[32];
@@ -455,22 +456,30 @@ torch::Tensor gemm(const torch::Tensor& a, const torch::Tensor& b, const std::st
   return out;
 }
 
-// One product per head: x [B, H, K] times w [H, N, K] transposed, or w [H, K, N] as it is (`nn`) → [B, H, N].
-torch::Tensor head_gemm(const torch::Tensor& x, const torch::Tensor& w, bool nn) {
-  TORCH_CHECK(x.is_cuda() && x.scalar_type() == torch::kBFloat16 && x.dim() == 3 && x.is_contiguous(), "x [B, H, K] bf16 contiguous");
+// One product per head: x [B, H, K] times w [H, N, K] transposed, or w [H, K, N] as it is (`nn`) → [B, H, N].  x and out may be ranges of
+// the last dimension of wider tensors.
+torch::Tensor head_gemm(const torch::Tensor& x, const torch::Tensor& w, bool nn, const c10::optional<torch::Tensor>& out_opt) {
+  auto rows16 = [](const torch::Tensor& t) { return t.stride(2) == 1 && t.stride(1) % 8 == 0 && t.stride(0) % 8 == 0 && reinterpret_cast<uintptr_t>(t.data_ptr()) % 16 == 0; };
+  TORCH_CHECK(x.is_cuda() && x.scalar_type() == torch::kBFloat16 && x.dim() == 3 && rows16(x), "x [B, H, K] bf16, rows and heads on 16-byte boundaries");
   TORCH_CHECK(w.is_cuda() && w.scalar_type() == torch::kBFloat16 && w.dim() == 3 && w.is_contiguous() && w.size(0) == x.size(1), "weight [H, *, *] bf16 contiguous");
   c10::cuda::CUDAGuard guard(x.device());
   const int B = x.size(0), H = x.size(1), K = x.size(2), N = nn ? w.size(2) : w.size(1);
   TORCH_CHECK((nn ? w.size(1) : w.size(2)) == K && K % 8 == 0 && N % 8 == 0, "per-head product: widths that agree and are multiples of 8");
-  auto out = torch::empty({B, H, N}, x.options());
+  torch::Tensor out;
+  if (out_opt.has_value() && out_opt->defined()) {
+    out = *out_opt;
+    TORCH_CHECK(out.is_cuda() && out.scalar_type() == torch::kBFloat16 && out.dim() == 3 && out.size(0) == B && out.size(1) == H && out.size(2) == N && rows16(out), "out [B, H, N]");
+  } else {
+    out = torch::empty({B, H, N}, x.options());
+  }
   if (B == 0) return out;
   auto w2 = w.view({w.size(0) * w.size(1), w.size(2)});
   check_operand(w2, "weight");
-  CUtensorMap ta = make_tmap_3d(x.data_ptr(), K, H, B, K, static_cast<uint64_t>(H) * K, BK, 1, BM);
+  CUtensorMap ta = make_tmap_3d(x.data_ptr(), K, H, B, x.stride(1), x.stride(0), BK, 1, BM);
   CUtensorMap tb = nn ? make_tmap_2d(w2.data_ptr(), w2.size(1), w2.size(0), w2.stride(0), 64, BK)
                       : make_tmap_2d(w2.data_ptr(), w2.size(1), w2.size(0), w2.stride(0), BK, BN);
   GemmParams p{};
-  p.out = out.data_ptr(); p.M = B; p.N = N; p.K = K; p.ldo = H * N; p.err = error_word();
+  p.out = out.data_ptr(); p.M = B; p.N = N; p.K = K; p.ldo = out.stride(0); p.head_cols = out.stride(1); p.err = error_word();
   p.num_groups = H; p.group_rows_b = w.size(1); p.mode = 3;
   launch(false, nn, 3, ta, tb, p, ((B + BM - 1) / BM) * ((N + BN - 1) / BN) * H, at::cuda::getCurrentCUDAStream());
   return out;

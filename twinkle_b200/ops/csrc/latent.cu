@@ -1,7 +1,8 @@
 // Latent attention (keys and values expanded from one cached vector per token, which serves as both in latent space):
 //   latent_norms   RMS norms of the query bottleneck and of the new latents, and the write into the paged cache — one pass
-//   latent_decode  one token per sequence, all heads against the same cached rows, sink logit in the denominator, sigmoid gate on
-//                  the result.  This file holds the fp32-arithmetic form for any rank up to 1024 (32-bit models, odd sizes, small
+//   latent_decode  one token per sequence, all heads against the same cached rows, optionally the last `window` of them, a sink logit in
+//                  the denominator and a sigmoid gate on the result.  A cached row may be wider than its value (rotated key
+//                  dimensions).  This file holds the fp32-arithmetic form for any rank up to 1024 (32-bit models, odd sizes, small
 //                  pages); latent_decode.cu the tensor-core form for bf16.
 #include <ATen/cuda/CUDAContext.h>
 #include <c10/cuda/CUDAGuard.h>
@@ -108,42 +109,43 @@ std::vector<torch::Tensor> latent_norms(const torch::Tensor& proj, int64_t q0, i
 }
 
 // ---------------------------------------------------------------- latent decode, fp32 arithmetic
-// Block = (GH heads, sequence), 256 threads.  Sixteen cached rows at a time in shared memory; four threads form a score, a thread
-// owns RI of the latent columns of every head.
+// Block = (GH heads, sequence), 256 threads.  Sixteen cached rows at a time in shared memory; four threads form a score over the K
+// columns of a row, a thread owns RI of the R ≤ K value columns of every head.
 template <typename T, int RI>
 __global__ void __launch_bounds__(256) latent_decode_plain_kernel(const T* __restrict__ q, const T* __restrict__ pool, const int* __restrict__ tables,
                                                                   const int* __restrict__ lens, const T* __restrict__ sinks, const T* __restrict__ gate, long ldg,
-                                                                  T* __restrict__ out, int H, int R, int RP, int block_size, int max_blocks, float scale) {
+                                                                  T* __restrict__ out, int H, int K, int R, int RP, int block_size, int max_blocks, int window, float scale) {
   constexpr int GH = 4, TK = 16;
   extern __shared__ float sm_latent[];
   __shared__ float s_s[GH][TK];
   const int h0 = blockIdx.x * GH, b = blockIdx.y, tid = threadIdx.x, n = lens[b];
-  const int pitch = R + 1;
+  const int pitch = K + 1;
   float *s_q = sm_latent, *s_c = s_q + GH * pitch;
-  for (int i = tid; i < GH * R; i += 256) {
-    const int g = i / R, c = i - g * R;
-    s_q[g * pitch + c] = h0 + g < H ? lt::ld(q + (static_cast<size_t>(b) * H + h0 + g) * R + c) * scale : 0.f;
+  for (int i = tid; i < GH * K; i += 256) {
+    const int g = i / K, c = i - g * K;
+    s_q[g * pitch + c] = h0 + g < H ? lt::ld(q + (static_cast<size_t>(b) * H + h0 + g) * K + c) * scale : 0.f;
   }
   float acc[GH][RI], m[GH], l[GH];
 #pragma unroll
   for (int g = 0; g < GH; ++g) {
-    m[g] = h0 + g < H ? lt::ld(sinks + h0 + g) : 0.f;      // the sink is a key without a value that every step already sees
-    l[g] = 1.f;
+    // the sink is a key without a value that every step already sees
+    m[g] = sinks == nullptr ? -1e30f : (h0 + g < H ? lt::ld(sinks + h0 + g) : 0.f);
+    l[g] = sinks == nullptr ? 0.f : 1.f;
 #pragma unroll
     for (int i = 0; i < RI; ++i) acc[g][i] = 0.f;
   }
   const int* table = tables + static_cast<size_t>(b) * max_blocks;
-  for (int t0 = 0; t0 < n; t0 += TK) {
+  for (int t0 = window > 0 ? max(0, n - window) : 0; t0 < n; t0 += TK) {
     __syncthreads();
-    for (int i = tid; i < TK * R; i += 256) {
-      const int t = i / R, c = i - t * R, p = t0 + t;
+    for (int i = tid; i < TK * K; i += 256) {
+      const int t = i / K, c = i - t * K, p = t0 + t;
       s_c[t * pitch + c] = p < n ? lt::ld(pool + (static_cast<size_t>(table[p / block_size]) * block_size + p % block_size) * RP + c) : 0.f;
     }
     __syncthreads();
     {
       const int pair = tid >> 2, sub = tid & 3, g = pair / TK, t = pair % TK;
       float s = 0.f;
-      for (int c = sub; c < R; c += 4) s += s_q[g * pitch + c] * s_c[t * pitch + c];
+      for (int c = sub; c < K; c += 4) s += s_q[g * pitch + c] * s_c[t * pitch + c];
       s += __shfl_xor_sync(0xffffffffu, s, 1);
       s += __shfl_xor_sync(0xffffffffu, s, 2);
       if (sub == 0) s_s[g][t] = t0 + t < n ? s : -INFINITY;
@@ -172,7 +174,7 @@ __global__ void __launch_bounds__(256) latent_decode_plain_kernel(const T* __res
 #pragma unroll
   for (int g = 0; g < GH; ++g) {
     if (h0 + g >= H) break;
-    float f = 1.f / l[g];
+    float f = l[g] > 0.f ? 1.f / l[g] : 0.f;
     if (gate != nullptr) f /= 1.f + __expf(-lt::ld(gate + b * ldg + h0 + g));
 #pragma unroll
     for (int i = 0; i < RI; ++i)
@@ -180,36 +182,37 @@ __global__ void __launch_bounds__(256) latent_decode_plain_kernel(const T* __res
   }
 }
 
-bool latent_decode_tc(const torch::Tensor& q, const torch::Tensor& pool, const torch::Tensor& tables, const torch::Tensor& lens, double scale, const torch::Tensor& sinks,
-                      const OptT& gate, torch::Tensor& out);
+bool latent_decode_tc(const torch::Tensor& q, const torch::Tensor& pool, const torch::Tensor& tables, const torch::Tensor& lens, double scale, const OptT& sinks,
+                      const OptT& gate, int window, torch::Tensor& out);
 
-// q [B, H, R], pool [blocks, bs, 1, R rounded up to 8], tables int32 [B, ·], lens int32 [B] → [B, H, R]
+// q [B, H, K], pool [blocks, bs, 1, K rounded up to 8], tables int32 [B, ·], lens int32 [B] → [B, H, R] (values: the first R ≤ K columns)
 torch::Tensor latent_decode(const torch::Tensor& q, const torch::Tensor& pool, const torch::Tensor& tables, const torch::Tensor& lens, double scale,
-                            const torch::Tensor& sinks, const OptT& gate) {
+                            const OptT& sinks, const OptT& gate, int64_t rank, int64_t window) {
   const auto st = q.scalar_type();
-  TORCH_CHECK(q.is_cuda() && q.dim() == 3 && q.is_contiguous() && (st == torch::kBFloat16 || st == torch::kFloat32), "q [B, H, R] bf16 or fp32");
-  const int B = q.size(0), H = q.size(1), R = q.size(2);
-  TORCH_CHECK(pool.scalar_type() == st && pool.is_contiguous() && pool.dim() == 4 && pool.size(2) == 1 && pool.size(3) >= R, "latent pool [blocks, bs, 1, >= R]");
+  TORCH_CHECK(q.is_cuda() && q.dim() == 3 && q.is_contiguous() && (st == torch::kBFloat16 || st == torch::kFloat32), "q [B, H, K] bf16 or fp32");
+  const int B = q.size(0), H = q.size(1), K = q.size(2), R = rank;
+  TORCH_CHECK(R >= 1 && R <= K && window >= 0 && window < (int64_t(1) << 30), "value columns within the key's, window 0 (none) or positive");
+  TORCH_CHECK(pool.scalar_type() == st && pool.is_contiguous() && pool.dim() == 4 && pool.size(2) == 1 && pool.size(3) >= K, "latent pool [blocks, bs, 1, >= K]");
   TORCH_CHECK(tables.scalar_type() == torch::kInt32 && tables.is_contiguous() && tables.dim() == 2 && tables.size(0) == B && lens.scalar_type() == torch::kInt32 &&
                   lens.is_contiguous() && lens.numel() == B, "int32 tables / lens");
-  TORCH_CHECK(sinks.scalar_type() == st && sinks.is_contiguous() && sinks.numel() == H, "sinks [H]");
+  if (lt::has(sinks)) TORCH_CHECK(sinks->scalar_type() == st && sinks->is_contiguous() && sinks->numel() == H, "sinks [H]");
   if (lt::has(gate)) TORCH_CHECK(gate->scalar_type() == st && gate->dim() == 2 && gate->size(0) == B && gate->size(1) == H && gate->stride(1) == 1, "gate [B, H]");
-  TORCH_CHECK(R <= 1024, "latent rank up to 1024");
+  TORCH_CHECK(R <= 1024 && K <= 2048, "latent rank up to 1024, rows up to 2048 wide");
   c10::cuda::CUDAGuard guard(q.device());
   auto out = torch::empty({B, H, R}, q.options());
   if (B == 0) return out;
-  if (latent_decode_tc(q, pool, tables, lens, scale, sinks, gate, out)) return out;
+  if (latent_decode_tc(q, pool, tables, lens, scale, sinks, gate, static_cast<int>(window), out)) return out;
   auto stream = at::cuda::getCurrentCUDAStream();
-  const size_t smem = sizeof(float) * 20 * (R + 1);
+  const size_t smem = sizeof(float) * 20 * (K + 1);
   auto run = [&](auto tag) {
     using T = decltype(tag);
     auto go = [&](auto kern) {
       TK_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
       kern<<<dim3((H + 3) / 4, B), 256, smem, stream>>>(
           reinterpret_cast<const T*>(q.data_ptr()), reinterpret_cast<const T*>(pool.data_ptr()), tables.data_ptr<int>(), lens.data_ptr<int>(),
-          reinterpret_cast<const T*>(sinks.data_ptr()), lt::has(gate) ? reinterpret_cast<const T*>(gate->data_ptr()) : nullptr, lt::has(gate) ? gate->stride(0) : 0L,
-          reinterpret_cast<T*>(out.data_ptr()), H, R, static_cast<int>(pool.size(3)), static_cast<int>(pool.size(1)), static_cast<int>(tables.size(1)),
-          static_cast<float>(scale));
+          lt::has(sinks) ? reinterpret_cast<const T*>(sinks->data_ptr()) : nullptr, lt::has(gate) ? reinterpret_cast<const T*>(gate->data_ptr()) : nullptr, lt::has(gate) ? gate->stride(0) : 0L,
+          reinterpret_cast<T*>(out.data_ptr()), H, K, R, static_cast<int>(pool.size(3)), static_cast<int>(pool.size(1)), static_cast<int>(tables.size(1)),
+          static_cast<int>(window), static_cast<float>(scale));
     };
     if (R <= 256) go(latent_decode_plain_kernel<T, 1>);
     else if (R <= 512) go(latent_decode_plain_kernel<T, 2>);

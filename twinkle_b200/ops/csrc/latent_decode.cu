@@ -4,7 +4,8 @@
 // once and used by two products with the tokens (or the rank) on the 128 rows of the tensor core and the heads as columns:
 //     Sᵀ [tokens, heads] = C · Qᵀ                 C as it lies: tokens are rows, the rank is reduced
 //     Oᵀ [rank, heads]  += Cᵀ · Pᵀ                the same shared memory read the other way round: tokens are reduced
-// Heads need not fill a 128-row tile, which a product with heads as rows would leave mostly empty.
+// Heads need not fill a 128-row tile, which a product with heads as rows would leave mostly empty.  A row's value is its first R columns;
+// rotated key dimensions behind them enter the first product only.  With a window the tiles start at the first token it reaches.
 //
 // One CTA per (part of the context, group of up to 64 heads, sequence), 192 threads:
 //   warps 0-3  softmax: thread = one token; maxima over tokens by a transposing butterfly in each warp, then over warps; weights go
@@ -30,7 +31,8 @@ namespace ld {
 constexpr int TT = 128;                       // tokens per tile
 constexpr int CHUNK = TT * 64 * 2;            // 64 columns of a tile
 constexpr int PIECE = 2 * CHUNK;              // 128 columns: the unit of the ring
-constexpr int MAX_RING = 6, MAX_PIECES = 4;
+constexpr int MAX_RING = 6, MAX_VALUE_PIECES = 4;
+constexpr float FAR = -1e30f;                 // running maximum before the first score
 constexpr int THREADS = 192;
 constexpr float RESCALE = 8.f;                // log2 units
 constexpr float LOG2E = 1.4426950408889634f;
@@ -42,9 +44,9 @@ struct LatentDecode {
   const int* lens;
   const bf16* sinks;
   const bf16* gate; long ldg;
-  bf16* out;                                  // [B, H, R]
+  bf16* out;                                  // [B, H, R]; scores run over K ≥ R columns
   float *part_o, *part_m, *part_l;            // [parts, B, H, R], [parts, B, H] twice (parts > 1)
-  int B, H, R, page, max_pages, parts, ring;
+  int B, H, K, R, page, max_pages, parts, ring, window;
   float scale_log2;
   int* err;
 };
@@ -76,10 +78,11 @@ __global__ void __launch_bounds__(ld::THREADS, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmC, const LatentDecode p) {
   using namespace ld;
   constexpr int W = N < 32 ? N : 32;          // heads per butterfly
-  const int part = blockIdx.x, h0 = blockIdx.y * 64, b = blockIdx.z;
-  const int n = p.lens[b], tiles_all = (n + TT - 1) / TT, per = (tiles_all + p.parts - 1) / p.parts;
-  const int first = part * per, tiles = max(0, min(tiles_all - first, per));
-  const int pieces = (p.R + 127) / 128, ring = p.ring;
+  const int part = blockIdx.x, h0 = blockIdx.y * N, b = blockIdx.z;
+  const int n = p.lens[b], lo = p.window > 0 ? max(0, n - p.window) : 0;
+  const int tiles_all = (n + TT - 1) / TT - lo / TT, per = (tiles_all + p.parts - 1) / p.parts;
+  const int first = lo / TT + part * per, tiles = max(0, min(tiles_all - part * per, per));
+  const int pieces = (p.K + 127) / 128, value_pieces = (p.R + 127) / 128, ring = p.ring;
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -103,7 +106,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     mbar_init(o_done, 1);
     fence_barrier_init();
   }
-  if (threadIdx.x < N) s_m[threadIdx.x] = h0 + static_cast<int>(threadIdx.x) < p.H ? __bfloat162float(p.sinks[h0 + threadIdx.x]) * LOG2E : 0.f;
+  if (threadIdx.x < N) s_m[threadIdx.x] = p.sinks == nullptr ? FAR : (h0 + static_cast<int>(threadIdx.x) < p.H ? __bfloat162float(p.sinks[h0 + threadIdx.x]) * LOG2E : 0.f);
   if (warp == 5) {
     tmem_alloc(tmem_slot, 512);
     tmem_relinquish();
@@ -177,10 +180,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         if (!ok) break;
         tc_fence_after();
         for (int c = 0; c < pieces; ++c) {
+          if (c < value_pieces) {
 #pragma unroll
-          for (int k = 0; k < TT / 16; ++k)
-            umma_bf16(tmem_o + c * N, umma_desc(a_c + o_slot * PIECE + k * 2048, CHUNK, 1024), umma_desc(a_p + (k >> 2) * N * 128 + (k & 3) * 32, 16, 1024), idesc_o,
-                      j > 0 || k > 0 ? 1u : 0u);
+            for (int k = 0; k < TT / 16; ++k)
+              umma_bf16(tmem_o + c * N, umma_desc(a_c + o_slot * PIECE + k * 2048, CHUNK, 1024), umma_desc(a_p + (k >> 2) * N * 128 + (k & 3) * 32, 16, 1024), idesc_o,
+                        j > 0 || k > 0 ? 1u : 0u);
+          }
           umma_commit(&c_empty[o_slot]);
           if (++o_slot == ring) o_slot = 0;
         }
@@ -206,7 +211,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
           uint32_t r[32];
           tmem_ld32(tmem + (j & 1) * 64 + c * 32 + lanes, r);      // N = 16: columns 16-31 are not used
           tmem_ld_wait();
-          const bool live = (first + j) * TT + t < n;
+          const int at = (first + j) * TT + t;
+          const bool live = at < n && at >= lo;
 #pragma unroll
           for (int i = 0; i < W; ++i) s[c * 32 + i] = live ? __uint_as_float(r[i]) * p.scale_log2 : -INFINITY;
         }
@@ -245,7 +251,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         for (int i = 0; i < N; ++i) l[i] *= s_alpha[i];
         if (!dead && j > 0) {
           tc_fence_after();
-          for (int c = 0; c < pieces * N / W; ++c) {
+          for (int c = 0; c < value_pieces * N / W; ++c) {
             uint32_t r[32];
             const uint32_t at = tmem_o + c * W + lanes;
             tmem_ld32(at, r);                             // N = 16: the second half is the next piece's and goes back unchanged
@@ -280,13 +286,13 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     asm volatile("bar.sync 1, 128;" ::: "memory");
     if (t < N && h0 + t < p.H) {
       float sum = s_w[t] + s_w[64 + t] + s_w[128 + t] + s_w[192 + t];
-      if (part == 0) sum += exp2f(__bfloat162float(p.sinks[h0 + t]) * LOG2E - s_m[t]);
+      if (part == 0 && p.sinks != nullptr) sum += exp2f(__bfloat162float(p.sinks[h0 + t]) * LOG2E - s_m[t]);
       const size_t at = (static_cast<size_t>(part) * p.B + b) * p.H + h0 + t;
       if (p.parts > 1) {
         p.part_m[at] = s_m[t];
         p.part_l[at] = sum;
       } else {
-        float f = 1.f / sum;
+        float f = sum > 0.f ? 1.f / sum : 0.f;
         if (p.gate != nullptr) f /= 1.f + __expf(-__bfloat162float(p.gate[b * p.ldg + h0 + t]));
         s_alpha[t] = f;
       }
@@ -295,7 +301,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     bool done = tiles == 0 || (!dead && mbar_wait(o_done, (tiles - 1) & 1, p.err, ERR_ATTN_WAIT));
     if (done) {
       tc_fence_after();
-      for (int c = 0; c < pieces; ++c) {
+      for (int c = 0; c < value_pieces; ++c) {
         const int rank = c * 128 + t;
 #pragma unroll
         for (int q = 0; q < N / W; ++q) {
@@ -336,7 +342,7 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentDecode 
   float m = -INFINITY, l = 0.f;
   for (int s = 0; s < p.parts; ++s) m = fmaxf(m, p.part_m[s * step + at]);
   for (int s = 0; s < p.parts; ++s) l += p.part_l[s * step + at] * exp2f(p.part_m[s * step + at] - m);
-  float f = 1.f / l;
+  float f = l > 0.f ? 1.f / l : 0.f;
   if (p.gate != nullptr) f /= 1.f + __expf(-__bfloat162float(p.gate[b * p.ldg + h]));
   for (int r = threadIdx.x; r < p.R; r += 128) {
     float o = 0.f;
@@ -346,21 +352,27 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentDecode 
 }
 
 // Whether the tensor-core form takes these operands; if so, runs it.
-bool latent_decode_tc(const torch::Tensor& q, const torch::Tensor& pool, const torch::Tensor& tables, const torch::Tensor& lens, double scale, const torch::Tensor& sinks,
-                      const OptT& gate, torch::Tensor& out) {
-  const int B = q.size(0), H = q.size(1), R = q.size(2), page = pool.size(1);
-  if (q.scalar_type() != torch::kBFloat16 || R % 8 != 0 || R > 128 * ld::MAX_PIECES || pool.size(3) != R || page < 8 || ld::TT % page != 0) return false;
+bool latent_decode_tc(const torch::Tensor& q, const torch::Tensor& pool, const torch::Tensor& tables, const torch::Tensor& lens, double scale, const OptT& sinks,
+                      const OptT& gate, int window, torch::Tensor& out) {
+  const int B = q.size(0), H = q.size(1), K = q.size(2), R = out.size(2), page = pool.size(1);
+  if (q.scalar_type() != torch::kBFloat16 || K % 8 != 0 || R % 8 != 0 || R > 128 * ld::MAX_VALUE_PIECES || pool.size(3) != K || page < 8 || ld::TT % page != 0) return false;
   if (reinterpret_cast<uintptr_t>(q.data_ptr()) % 16 != 0 || reinterpret_cast<uintptr_t>(pool.data_ptr()) % 16 != 0 || B > 65535) return false;
-  const int N = H <= 16 ? 16 : (H <= 32 ? 32 : 64), groups = (H + 63) / 64, pieces = (R + 127) / 128;
-  const int fixed = 2 * pieces * N * 128 + 2 * N * 128 + 1024 + 4096;
+  const int pieces = (K + 127) / 128;
   LatentDecode p{};
-  p.ring = std::min((227 * 1024 - fixed) / ld::PIECE, ld::MAX_RING);
+  int N = H <= 16 ? 16 : (H <= 32 ? 32 : 64), fixed = 0;
+  for (;; N /= 2) {                     // rows too wide for 64 heads at a time: fewer heads per block
+    fixed = 2 * pieces * N * 128 + 2 * N * 128 + 1024 + 4096;
+    p.ring = std::min((227 * 1024 - fixed) / ld::PIECE, ld::MAX_RING);
+    if (p.ring >= pieces || N == 16) break;
+  }
   if (p.ring < pieces) return false;
-  p.B = B; p.H = H; p.R = R; p.page = page; p.max_pages = tables.size(1);
-  const int most = (p.max_pages * page + ld::TT - 1) / ld::TT;
+  const int groups = (H + N - 1) / N;
+  p.B = B; p.H = H; p.K = K; p.R = R; p.page = page; p.max_pages = tables.size(1); p.window = window;
+  int most = (p.max_pages * page + ld::TT - 1) / ld::TT;
+  if (window > 0) most = std::min(most, (window + ld::TT - 2) / ld::TT + 1);
   p.parts = std::max(1, std::min({most, num_sms() / (B * groups), 32}));
   p.tables = tables.data_ptr<int>(); p.lens = lens.data_ptr<int>();
-  p.sinks = reinterpret_cast<const bf16*>(sinks.data_ptr());
+  if (sinks.has_value() && sinks->defined()) p.sinks = reinterpret_cast<const bf16*>(sinks->data_ptr());
   if (gate.has_value() && gate->defined()) { p.gate = reinterpret_cast<const bf16*>(gate->data_ptr()); p.ldg = gate->stride(0); }
   p.out = reinterpret_cast<bf16*>(out.data_ptr());
   p.scale_log2 = static_cast<float>(scale) * ld::LOG2E;
@@ -372,8 +384,8 @@ bool latent_decode_tc(const torch::Tensor& q, const torch::Tensor& pool, const t
     pml = torch::empty({2, p.parts, B, H}, f32);
     p.part_o = po.data_ptr<float>(); p.part_m = pml.data_ptr<float>(); p.part_l = p.part_m + static_cast<size_t>(p.parts) * B * H;
   }
-  CUtensorMap tq = make_tmap_2d(q.data_ptr(), R, static_cast<uint64_t>(B) * H, R, 64, N);
-  CUtensorMap tc = make_tmap_2d(pool.data_ptr(), R, static_cast<uint64_t>(pool.size(0)) * page, R, 64, page);
+  CUtensorMap tq = make_tmap_2d(q.data_ptr(), K, static_cast<uint64_t>(B) * H, K, 64, N);
+  CUtensorMap tc = make_tmap_2d(pool.data_ptr(), K, static_cast<uint64_t>(pool.size(0)) * page, K, 64, page);
   const int smem = p.ring * ld::PIECE + fixed;
   auto stream = at::cuda::getCurrentCUDAStream();
   auto go = [&](auto kern) {

@@ -1,5 +1,6 @@
 // Mixture-of-experts steps of inference, all without host reads (they are captured into decode graphs):
-//   moe_topk          fp32 router logits (+ bias) → the k largest, a softmax over just those, and tokens per expert
+//   moe_topk          fp32 router logits (+ bias) → the k largest, a softmax over just those, and tokens per expert; or a softmax over
+//                     all and a choice among the best groups; the shared expert's sigmoid weight on the way
 //   moe_group_rows    token rows copied next to the rows of the same expert, nothing between experts: every expert's range comes
 //                     from the histogram, a row's place inside it from an atomic counter (rows do not interact, so their order
 //                     inside an expert does not matter)
@@ -10,29 +11,69 @@
 
 #include "common.cuh"
 #include "host.h"
+#include "vec.cuh"
 
 namespace tk {
-
-using bf16 = __nv_bfloat16;
-using OptT = c10::optional<torch::Tensor>;
 
 namespace ms {
 __device__ __forceinline__ float ld(const float* p) { return *p; }
 __device__ __forceinline__ float ld(const bf16* p) { return __bfloat162float(*p); }
 }  // namespace ms
 
+struct Choice {
+  int rows, E, k;
+  int groups, keep;                      // groups 0: a softmax over the chosen; otherwise over all, and only the `keep` best groups count
+  float factor;                          // on the weights of the second form
+  const void *x, *shared; long ldx;      // [rows, width], [width]: open[t] = σ(x_t · shared) (nullptr: not wanted)
+  float* open; int width;
+};
+
 // One warp per token, up to 32·PER experts.
 template <typename T, int PER>
 __global__ void __launch_bounds__(256) moe_topk_kernel(const float* __restrict__ logits, long ld, const T* __restrict__ bias, const int64_t* __restrict__ forced,
-                                                       float* __restrict__ weights, int64_t* __restrict__ indices, int* __restrict__ hist, int rows, int E, int k) {
-  const int lane = threadIdx.x & 31;
+                                                       float* __restrict__ weights, int64_t* __restrict__ indices, int* __restrict__ hist, const Choice p) {
+  const int lane = threadIdx.x & 31, rows = p.rows, E = p.E, k = p.k, size = p.groups > 0 ? E / p.groups : E;
   for (int t = blockIdx.x * 8 + (threadIdx.x >> 5); t < rows; t += gridDim.x * 8) {
+    if (p.shared != nullptr) {
+      const T *x = reinterpret_cast<const T*>(p.x) + t * p.ldx, *w = reinterpret_cast<const T*>(p.shared);
+      float s = 0.f;
+      if (p.width % 8 == 0 && p.ldx % 8 == 0 && aligned16(p.x) && aligned16(p.shared)) {
+        for (int c = lane * 8; c < p.width; c += 256) {
+          Raw8<T> a, b;
+          a.load(x + c);
+          b.load(w + c);
+          float u[8], v[8];
+          a.get(u);
+          b.get(v);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) s += u[i] * v[i];
+        }
+      } else {
+        for (int c = lane; c < p.width; c += 32) s += ms::ld(x + c) * ms::ld(w + c);
+      }
+      s = warp_sum(s);
+      if (lane == 0) p.open[t] = 1.f / (1.f + __expf(-s));
+    }
     float z[PER];
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
       const int e = j * 32 + lane;
       z[j] = e < E ? logits[t * ld + e] + (bias != nullptr ? ms::ld(bias + e) : 0.f) : -INFINITY;
     }
+    // the largest logit among experts outside `taken`: same result in every lane
+    auto largest = [&](uint32_t taken, float& best, int& be) {
+      best = -INFINITY;
+      be = 1 << 30;
+#pragma unroll
+      for (int j = 0; j < PER; ++j)
+        if (!(taken >> j & 1) && j * 32 + lane < E && (z[j] > best || be == 1 << 30)) { best = z[j]; be = j * 32 + lane; }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oe = __shfl_xor_sync(0xffffffffu, be, o);
+        if (ob > best || (ob == best && oe < be)) { best = ob; be = oe; }
+      }
+    };
     float mine = -INFINITY;
     int my_e = 0;
     const bool given = forced != nullptr && forced[static_cast<size_t>(t) * k] >= 0;
@@ -43,59 +84,89 @@ __global__ void __launch_bounds__(256) moe_topk_kernel(const float* __restrict__
       }
     } else {
       uint32_t taken = 0;
-      for (int r = 0; r < k; ++r) {
-        float best = -INFINITY;
-        int be = 1 << 30;
+      if (p.groups > 1 && p.keep < p.groups) {         // a group is as good as its best expert: the next best outside the groups so far names one
+        uint32_t inside = 0;
+        for (int r = 0; r < p.keep; ++r) {
+          float best;
+          int be;
+          largest(inside, best, be);
 #pragma unroll
-        for (int j = 0; j < PER; ++j)
-          if (!(taken >> j & 1) && j * 32 + lane < E && (z[j] > best || be == 1 << 30)) { best = z[j]; be = j * 32 + lane; }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-          const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-          const int oe = __shfl_xor_sync(0xffffffffu, be, o);
-          if (ob > best || (ob == best && oe < be)) { best = ob; be = oe; }
+          for (int j = 0; j < PER; ++j)
+            if ((j * 32 + lane) / size == be / size) inside |= 1u << j;
         }
+        taken = ~inside;
+      }
+      for (int r = 0; r < k; ++r) {
+        float best;
+        int be;
+        largest(taken, best, be);
         if ((be & 31) == lane && be < (1 << 30)) taken |= 1u << (be >> 5);
         if (lane == r) { mine = best; my_e = min(be, E - 1); }   // logits that are not numbers still name an expert that exists
       }
     }
-    const float mx = warp_max(mine);
-    const float w = lane < k ? __expf(mine - mx) : 0.f, sum = warp_sum(w);
+    float over = mine;                                  // the softmax runs over the chosen, or over all
+    if (p.groups > 0) {
+#pragma unroll
+      for (int j = 0; j < PER; ++j) over = j == 0 ? z[0] : fmaxf(over, z[j]);
+    }
+    const float mx = warp_max(over), w = lane < k ? __expf(mine - mx) : 0.f;
+    float part = w;
+    if (p.groups > 0) {
+      part = 0.f;
+#pragma unroll
+      for (int j = 0; j < PER; ++j) part += j * 32 + lane < E ? __expf(z[j] - mx) : 0.f;
+    }
+    const float sum = warp_sum(part);
     if (lane < k) {
-      weights[static_cast<size_t>(t) * k + lane] = w / sum;
+      weights[static_cast<size_t>(t) * k + lane] = p.groups > 0 ? w / sum * p.factor : w / sum;
       indices[static_cast<size_t>(t) * k + lane] = my_e;
       atomicAdd(hist + my_e, 1);
     }
   }
 }
 
-std::vector<torch::Tensor> moe_topk(const torch::Tensor& logits, const OptT& bias, int64_t k, const OptT& forced) {
+// Returns {weights, experts, tokens per expert} and, with `shared`, its weight per token.
+std::vector<torch::Tensor> moe_topk(const torch::Tensor& logits, const OptT& bias, int64_t k, const OptT& forced, int64_t groups, int64_t keep, double factor,
+                                    const OptT& x, const OptT& shared) {
   TORCH_CHECK(logits.is_cuda() && logits.dim() == 2 && logits.scalar_type() == torch::kFloat32 && logits.stride(1) == 1, "router logits [T, E] fp32");
   const int rows = logits.size(0), E = logits.size(1);
   TORCH_CHECK(E >= 1 && E <= 256 && k >= 1 && k <= 32 && k <= E, "up to 256 experts and top-32");
-  const bool has_bias = bias.has_value() && bias->defined(), has_forced = forced.has_value() && forced->defined();
+  TORCH_CHECK(groups >= 0 && (groups == 0 || (E % groups == 0 && keep >= 1 && keep <= groups && k <= E / groups * keep)), "equal groups that hold enough experts");
+  const bool has_bias = has(bias), has_forced = has(forced), has_shared = has(shared);
+  auto dt = has_bias ? bias->scalar_type() : torch::kFloat32;
+  if (has_shared) {
+    TORCH_CHECK(has(x) && x->is_cuda() && x->dim() == 2 && x->size(0) == rows && x->stride(1) == 1 && shared->is_cuda() && shared->is_contiguous() && shared->numel() == x->size(1) &&
+                    shared->scalar_type() == x->scalar_type() && (x->scalar_type() == torch::kBFloat16 || x->scalar_type() == torch::kFloat32), "x [T, H] and shared [H] in one dtype");
+    TORCH_CHECK(!has_bias || dt == x->scalar_type(), "bias in x's dtype");
+    dt = x->scalar_type();
+  }
   if (has_bias) TORCH_CHECK(bias->is_cuda() && bias->is_contiguous() && bias->numel() == E && (bias->scalar_type() == torch::kBFloat16 || bias->scalar_type() == torch::kFloat32), "router bias [E]");
   if (has_forced) TORCH_CHECK(forced->is_cuda() && forced->scalar_type() == torch::kInt64 && forced->is_contiguous() && forced->numel() == rows * k, "forced experts int64 [T, k]");
   c10::cuda::CUDAGuard guard(logits.device());
   auto w = torch::empty({rows, k}, logits.options());
   auto idx = torch::empty({rows, k}, logits.options().dtype(torch::kInt64));
   auto hist = torch::zeros({E}, logits.options().dtype(torch::kInt32));
-  if (rows == 0) return {w, idx, hist};
+  auto open = torch::empty({has_shared ? rows : 0}, logits.options());
+  std::vector<torch::Tensor> out{w, idx, hist};
+  if (has_shared) out.push_back(open);
+  if (rows == 0) return out;
+  Choice p{};
+  p.rows = rows; p.E = E; p.k = k; p.groups = groups; p.keep = keep; p.factor = factor;
+  if (has_shared) { p.x = x->data_ptr(); p.ldx = x->stride(0); p.shared = shared->data_ptr(); p.open = open.data_ptr<float>(); p.width = x->size(1); }
   const int blocks = std::min((rows + 7) / 8, num_sms() * 8);
   auto stream = at::cuda::getCurrentCUDAStream();
   auto run = [&](auto tag) {
     using T = decltype(tag);
     auto go = [&](auto kern) {
       kern<<<blocks, 256, 0, stream>>>(logits.data_ptr<float>(), logits.stride(0), has_bias ? reinterpret_cast<const T*>(bias->data_ptr()) : nullptr,
-                                       has_forced ? forced->data_ptr<int64_t>() : nullptr, w.data_ptr<float>(), idx.data_ptr<int64_t>(), hist.data_ptr<int>(), rows, E,
-                                       static_cast<int>(k));
+                                       has_forced ? forced->data_ptr<int64_t>() : nullptr, w.data_ptr<float>(), idx.data_ptr<int64_t>(), hist.data_ptr<int>(), p);
     };
     if (E <= 32) go(moe_topk_kernel<T, 1>); else if (E <= 64) go(moe_topk_kernel<T, 2>); else if (E <= 128) go(moe_topk_kernel<T, 4>); else go(moe_topk_kernel<T, 8>);
   };
-  if (has_bias && bias->scalar_type() == torch::kBFloat16) run(bf16{}); else run(float{});
+  if (dt == torch::kBFloat16) run(bf16{}); else run(float{});
   count_launch();
   TK_CUDA_CHECK(cudaGetLastError());
-  return {w, idx, hist};
+  return out;
 }
 
 // One warp per (token, choice).  Every block forms the expert ranges from the histogram for itself (≤ 256 numbers).
