@@ -1138,6 +1138,17 @@ PRESETS: Dict[str, Dict[str, Any]] = {
                             layer_specs=[dict(mixer=dict(heads=16, dim=128, vdim=128) if i % 4 != 3 else
                                               dict(heads=32, dim=128, vdim=128, q_rank=1024, kv_rank=512, scale=128**-0.5, kv_from=i - 4 if i % 8 == 7 else None),
                                               mlp=dict(ff=6144) if i == 0 else dict(ff=1152, experts=128, top=8)) for i in range(48)]),
+    # Nilepel in small: a window with experts beside a shared one, a chunk, rotated latents, borrowed keys and values
+    'tiny-nilepel': dict(vocab_size=1024, hidden_size=192, tie_word_embeddings=False, qk_norm=False, torch_dtype='float32', model_type='nilepel', rms_norm_eps=1e-5, embed_scale=4.0,
+                         layer_specs=[dict(mixer=dict(heads=6, kv_heads=2, dim=24, vdim=40, scale=0.2, rotary=dict(dims=16, base=1e4), window=48, bias=True, qk_norm=True,
+                                                      sinks=True, head_gate=True),
+                                           mlp=dict(ff=64, experts=6, top=2, gated=True, scoring='softmax_grouped', groups=3, keep=2, scale=1.5, shared=48), post=False),
+                                      dict(mixer=dict(heads=4, kv_heads=4, dim=32, vdim=32, scale=0.2, rotary=dict(dims=32, base=1e3, interleaved=True), chunk=40, sinks=True),
+                                           mlp=dict(ff=256, limit=2.0), post=False),
+                                      dict(mixer=dict(heads=5, dim=24, vdim=24, q_rank=0, kv_rank=56, scale=0.2, rot_dim=16, rotary=dict(dims=16, base=1e4, interleaved=True), window=64,
+                                                      sinks=False, head_gate=False), mlp=None, post=False),
+                                      dict(mixer=dict(heads=4, kv_heads=2, dim=24, vdim=40, scale=0.2, rotary=dict(dims=16, base=1e4), window=32, bias=True, qk_norm=True,
+                                                      sinks=True, head_gate=True, kv_from=0), mlp=dict(ff=128, limit=1.0), post=False)]),
     'qwen3-0.6b': dict(hidden_size=1024, intermediate_size=3072, num_hidden_layers=28, num_attention_heads=16,
                        num_key_value_heads=8, head_dim=128, tie_word_embeddings=True),
     'qwen3-8b': dict(hidden_size=4096, intermediate_size=12288, num_hidden_layers=36, num_attention_heads=32,
