@@ -1,5 +1,5 @@
 """A plain, slow evaluation of the Nilepel decoder: one function per mechanism, one sequence at a time, whole sequence from its first
-token, loops over positions, heads and experts where that is the clearest statement.  It shares no code with the package.
+token, loops over heads, experts and pairs of dimensions where that is the clearest statement.  It shares no code with the package.
 
 Weights come as a mapping from checkpoint names to tensors; a configuration is the checkpoint's ``config.json`` mapping.
 """
@@ -65,16 +65,16 @@ def attend(q, k, v, scale, first, sink=None):
     """One sequence: ``q [T, H, d]``, ``k [T, G, d]``, ``v [T, G, e]``; position i sees ``first(i) … i``.  ``sink [H]``: a logit in the
     denominator that belongs to no key."""
     T, H = q.shape[:2]
+    j = torch.arange(T)
+    seen = (j[None] <= j[:, None]) & (j[None] >= torch.tensor([first(i) for i in range(T)])[:, None])
     out = q.new_zeros(T, H, v.shape[-1])
     for h in range(H):
         g = h // (H // k.shape[1])
-        for i in range(T):
-            a = first(i)
-            s = (k[a:i + 1, g] @ q[i, h]) * scale
-            top = s.max() if sink is None else torch.maximum(s.max(), sink[h])
-            p = torch.exp(s - top)
-            total = p.sum() if sink is None else p.sum() + torch.exp(sink[h] - top)
-            out[i, h] = p @ v[a:i + 1, g] / total
+        s = (q[:, h] @ k[:, g].t() * scale).masked_fill(~seen, -math.inf)
+        top = s.amax(-1) if sink is None else torch.maximum(s.amax(-1), sink[h])
+        p = torch.exp(s - top[:, None])
+        total = p.sum(-1) if sink is None else p.sum(-1) + torch.exp(sink[h] - top)
+        out[:, h] = p @ v[:, g] / total[:, None]
     return out
 
 
@@ -159,9 +159,9 @@ def route(z, r):
 def mixture(h, m, w):
     idx, share = route(h @ w['router'].t(), m['router'])
     out = torch.zeros_like(h)
-    for t in range(h.shape[0]):
-        for n, p in zip(idx[t].tolist(), share[t]):
-            out[t] += p * expert(h[t], w[f'e{n}.gate'], w[f'e{n}.up'], w[f'e{n}.down'])
+    for n in range(m['router']['experts']):
+        p = (share * (idx == n)).sum(-1, keepdim=True)          # 0 for tokens that did not choose it
+        out = out + p * expert(h, w[f'e{n}.gate'], w[f'e{n}.up'], w[f'e{n}.down'])
     if m.get('shared'):
         out = out + sigmoid(h @ w['shared.sg'].t()) * expert(h, w['shared.gate'], w['shared.up'], w['shared.down'])
     return out

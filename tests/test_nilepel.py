@@ -273,7 +273,7 @@ def _paged(G, lens, bs, *shapes):
     for i, n in enumerate(lens):
         for j in range(-(-n // bs)):
             table[i, j] = order.pop()
-    return pools, table, lambda pool, i: torch.stack([pool[table[i, p // bs], p % bs] for p in range(lens[i])])
+    return pools, table, lambda pool, i: pool[table[i].long()].flatten(0, 1)[:lens[i]]
 
 
 @BACKENDS
@@ -310,13 +310,12 @@ def test_decode_attention_inside_bounds(where, kind, size, hq, hkv, d, e, bs):
 
 def _one(q, k, v, scale, sink):
     """One query ``[H, d]`` over all of ``k [n, G, d]``."""
-    out = []
-    for h in range(q.shape[0]):
-        s = k[:, h // (q.shape[0] // k.shape[1])] @ q[h] * scale
-        top = s.max() if sink is None else torch.maximum(s.max(), sink[h])
-        p = torch.exp(s - top)
-        out.append(p @ v[:, h // (q.shape[0] // k.shape[1])] / (p.sum() + (0 if sink is None else torch.exp(sink[h] - top))))
-    return torch.stack(out)
+    share = q.shape[0] // k.shape[1]
+    s = torch.einsum('hd,nhd->hn', q, k.repeat_interleave(share, 1) if k.shape[1] > 1 else k.expand(-1, share, -1)) * scale
+    top = s.amax(-1) if sink is None else torch.maximum(s.amax(-1), sink)
+    p = torch.exp(s - top[:, None])
+    o = torch.einsum('hn,nhe->he', p, v.repeat_interleave(share, 1) if v.shape[1] > 1 else v.expand(-1, share, -1))
+    return o / (p.sum(-1) + (0 if sink is None else torch.exp(sink - top)))[:, None]
 
 
 @BACKENDS
