@@ -58,12 +58,13 @@ def parse():
     ap.add_argument('--sp', type=int, default=None, help='Ulysses degree (default min(4, gpus))')
     ap.add_argument('--ref-micro', type=int, default=1, help='reference arm: sequences per forward_backward call')
     ap.add_argument('--cpu-debug', action='store_true', help='reference arm: run on CPU/gloo (debug only, result invalid)')
-    ap.add_argument('--config', default='both', choices=['both', 'dense', 'moe', 'serve', 'serve-moe'],
+    ap.add_argument('--config', default='both', choices=['both', 'dense', 'moe', 'serve', 'serve-moe', 'serve-windows'],
                     help="dense: Qwen3-8B full-parameter SFT; moe: Qwen3-30B-A3B LoRA r=16 SFT with expert parallel = gpus; "
                          "both (default): the two halves of the headline metric one after the other, each in a process of its own, "
                          "printed as one line (the dense fields at top level, the mixture-of-experts result under 'moe'); "
                          "serve: prefill and decode throughput of Pomelix stacks beside Qwen3 at equal sizes (one GPU, random weights); "
-                         "serve-moe: likewise of a Moronex stack beside Qwen3-30B-A3B and a Qwen3-Next style hybrid (24 layers of each)")
+                         "serve-moe: likewise of a Moronex stack beside Qwen3-30B-A3B and a Qwen3-Next style hybrid (24 layers of each); "
+                         "serve-windows: likewise of a Nilepel stack beside a Moronex stack and Qwen3-30B-A3B, with longer contexts (24 layers of each)")
     ap.add_argument('--moe-steps', type=int, default=10, help="cap on timed steps of the 'moe' half when --config both")
     return ap.parse_args()
 
@@ -200,16 +201,23 @@ def run_both(args):
 
 def run_serve(args):
     """Prefill and decode throughput of the sampler's engine: Pomelix presets and the Qwen3 presets of the same sizes, or
-    (``serve-moe``) a Moronex preset beside the mixture-of-experts models of the same size."""
+    (``serve-moe``) a Moronex preset beside the mixture-of-experts models of the same size, or (``serve-windows``) a Nilepel preset
+    beside those."""
     import torch
     from twinkle_b200 import ops
     from twinkle_b200.models.config import preset
     from twinkle_b200.sampler.bench import measure
     torch.cuda.set_device(0)
-    moe = args.config == 'serve-moe'
+    windows = args.config == 'serve-windows'
+    moe = args.config == 'serve-moe' or windows
     layers = args.layers or (24 if moe else None)
     over = {} if layers is None else {'num_hidden_layers': layers}
-    if moe:
+    prompts, batches = [(8, 1024), (1, 8192)], [(1, 1024), (16, 1024), (64, 1024), (256, 1024)]
+    if windows:
+        headline = 'nilepel-30b-a3b'
+        configs = {n: preset(n, **over) for n in (headline, 'moronex-30b-a3b', 'qwen3-30b-a3b')}
+        batches += [(16, 8192), (64, 8192)]
+    elif moe:
         headline = 'moronex-30b-a3b'
         # three Gated DeltaNet layers per attention layer, 16 heads of 128 x 128 state like the recurrent layers of the preset beside it
         kinds = [('full_attention' if i % 4 == 3 else 'linear_attention') for i in range(layers)]
@@ -222,7 +230,7 @@ def run_serve(args):
     clock.start()
     launches, res = ops.ext().launch_count(), {}
     for name, cfg in configs.items():
-        res[name] = dict(measure(cfg, [(8, 1024), (1, 8192)], [(1, 1024), (16, 1024), (64, 1024), (256, 1024)], args.steps, max(args.warmup, 3)),
+        res[name] = dict(measure(cfg, prompts, batches, args.steps, max(args.warmup, 3)),
                          parameters=cfg.num_params())
     clocks = clock.stop()
     value = res[headline]['decode'][2]['tokens_per_s']

@@ -147,7 +147,7 @@ def _nilepel_fields(cfg: Dict[str, Any]) -> Dict[str, Any]:
             raise NotImplementedError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not implemented (dense and moe are)")
         specs.append(PreNormSpec(mixer, ff))
     return dict(model_type='nilepel', vocab_size=int(cfg['vocab']), hidden_size=int(cfg['width']), rms_norm_eps=float(cfg['norm']['eps']),
-                embed_scale=float(cfg['embedding']['scale']), tie_word_embeddings=False, qk_norm=False, layer_specs=specs, eos_token_id=cfg.get('eos_token_id'),
+                embed_scale=float((cfg.get('embedding') or {}).get('scale', 1.0)), tie_word_embeddings=False, qk_norm=False, layer_specs=specs, eos_token_id=cfg.get('eos_token_id'),
                 pad_token_id=cfg.get('pad_token_id'), torch_dtype=str(cfg.get('torch_dtype', 'bfloat16')))
 
 
@@ -1055,6 +1055,18 @@ class DecoderConfig:
             json.dump(self.to_hf(), f, indent=2)
 
 
+def _nilepel_bench_mixer(i: int) -> Dict[str, Any]:
+    """Mixer of layer ``i`` of the Nilepel benchmark preset."""
+    heads = dict(heads=32, dim=128, vdim=128)
+    if i % 4 == 1:
+        return dict(heads, q_rank=0, kv_rank=512, scale=192**-0.5, rot_dim=64, rotary=dict(dims=64, base=1e4, interleaved=True), window=4096, sinks=False, head_gate=False)
+    grouped = dict(heads, kv_heads=4, scale=128**-0.5, sinks=True)
+    if i % 4 == 2:
+        return dict(grouped, rotary=dict(dims=128, base=5e5, interleaved=True), chunk=4096)
+    return dict(grouped, rotary=dict(dims=128, base=1e6, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192)), window=1024, bias=True, qk_norm=True, head_gate=True,
+                kv_from=i - 3 if i % 4 == 3 else None)
+
+
 PRESETS: Dict[str, Dict[str, Any]] = {
     # the smallest end-to-end configuration (LoRA SFT on CPU)
     'tiny-dense': dict(vocab_size=1024, hidden_size=256, intermediate_size=688, num_hidden_layers=2, num_attention_heads=4,
@@ -1149,6 +1161,12 @@ PRESETS: Dict[str, Dict[str, Any]] = {
                                                       sinks=False, head_gate=False), mlp=None, post=False),
                                       dict(mixer=dict(heads=4, kv_heads=2, dim=24, vdim=40, scale=0.2, rotary=dict(dims=16, base=1e4), window=32, bias=True, qk_norm=True,
                                                       sinks=True, head_gate=True, kv_from=0), mlp=dict(ff=128, limit=1.0), post=False)]),
+    # Nilepel layers at the width, experts and depth of Qwen3-30B-A3B (benchmarks): of four layers a window of 1024, rotated latents in a
+    # window of 4096, a chunk of 4096, and a window on the first one's keys and values
+    'nilepel-30b-a3b': dict(vocab_size=151936, hidden_size=2048, tie_word_embeddings=False, qk_norm=False, model_type='nilepel', rms_norm_eps=1e-6, embed_scale=2048**0.5,
+                            layer_specs=[dict(mixer=_nilepel_bench_mixer(i), mlp=dict(ff=6144, limit=7.0) if i == 0 else
+                                              dict(ff=768, experts=128, top=8, gated=True, scoring='softmax_grouped', groups=8, keep=4, scale=1.0, shared=768), post=False)
+                                         for i in range(48)]),
     'qwen3-0.6b': dict(hidden_size=1024, intermediate_size=3072, num_hidden_layers=28, num_attention_heads=16,
                        num_key_value_heads=8, head_dim=128, tie_word_embeddings=True),
     'qwen3-8b': dict(hidden_size=4096, intermediate_size=12288, num_hidden_layers=36, num_attention_heads=32,

@@ -68,16 +68,18 @@ __global__ void __launch_bounds__(128) rotary_heads_kernel(const RotaryHeads<T> 
   const int n = p.pairs, dims = 2 * n;
   float cs[8], sn[8];
   {
-    const float2* a = p.table + static_cast<size_t>(t) * p.table_ld;
+    // rotate-half: el < 2n and n a multiple of 8, so the eight pairs lie side by side
+    const float2* a = p.table + static_cast<size_t>(t) * p.table_ld + (INTER ? el / 2 : (el < n ? el : el - n));
 #pragma unroll
     for (int c = 0; c < 8; ++c) {
       float2 v = make_float2(1.f, 0.f);
-      if (el + c < dims) v = a[INTER ? (el + c) / 2 : (el + c) % n];
+      if (el + c < dims) v = a[INTER ? c / 2 : c];
       cs[c] = v.x; sn[c] = v.y;
     }
   }
   // rotate-half: n is a multiple of 8, so the partners of these eight elements are another thread's eight
   const bool lower = el < n, turns = el < dims;
+  const float inv_d = 1.f / p.d;
   const int lane = threadIdx.x & 31, partner = INTER || !turns ? lane : (lower ? lane + n / 8 : lane - n / 8);
   auto column = [&](int h) { return h < p.hq + p.hkv ? h * p.d : (p.hq + p.hkv) * p.d + (h - p.hq - p.hkv) * p.e; };
   auto fetch = [&](int h, Raw8<T>& r) {
@@ -112,7 +114,7 @@ __global__ void __launch_bounds__(128) rotary_heads_kernel(const RotaryHeads<T> 
       Raw8<T> r;
       r.load(w + el);
       r.get(g);
-      const float f = rsqrtf(ss / p.d + p.eps);
+      const float f = rsqrtf(ss * inv_d + p.eps);
 #pragma unroll
       for (int c = 0; c < 8; ++c) y[c] *= f * g[c];
     }

@@ -106,6 +106,43 @@ def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
         # of it written by a step, negligible for prompts)
         byts = 2.0 * T * d * (hq + 2 * hkv + hq + hkv + (0 if step else hkv) + 2 * hkv + hkv) + (2.0 * T * C * taps if step else 0.0)
         return (lambda: E.conv_heads(proj, w, pos, hq, hkv, d, d, 1e-5, 0.1, 4096, vf, lam, step, hist, slot, left, rows, kp, vp, not step)), 0.0, byts
+    if op in ('rotary_heads', 'rotary_heads_step'):
+        # bias, per-head norm, rotation and cache writes between projection and attention (the like kernel: rope, which norms and rotates)
+        hq, hkv, d, bs, step = a.heads, a.kv_heads, a.width, 16, op.endswith('step')
+        T = a.batch if step else a.tokens
+        C = (hq + 2 * hkv) * d
+        proj, bias, w = torch.randn(T, C + hq, device=dev, dtype=bf), torch.zeros(C, device=dev, dtype=bf), torch.ones(d, device=dev, dtype=bf)
+        pos = torch.full((T, ), a.seq - 1, device=dev) if step else torch.arange(T, device=dev) % a.seq
+        table = E.rotary_table(pos, torch.rand(d // 2, device=dev, dtype=torch.float64))
+        kp, vp = (torch.zeros(T * bs if step else T, hkv, d, device=dev, dtype=bf) for _ in range(2))
+        rows = torch.arange(T, device=dev) * (bs if step else 1)
+        byts = 2.0 * T * d * (2 * hq + 2 * hkv + (2 if step else 4) * hkv)      # in; q; both pools; keys and values of prompts
+        return (lambda: E.rotary_heads(proj, 0, bias, w, w, table, 0, d // 2, False, hq, hkv, d, d, 1e-6, kp, vp, rows, not step)), 0.0, byts
+    if op == 'rotary_table':
+        pos, f = torch.arange(a.tokens, device=dev) % a.seq, torch.rand(160, device=dev, dtype=torch.float64)
+        return (lambda: E.rotary_table(pos, f)), 0.0, 8.0 * a.tokens * 160
+    if op in ('latent_rotary', 'latent_rotary_step'):
+        # norm of the latents (--rank), rotated parts (--tail) of keys and queries, cache write (the like kernel: latent_norms)
+        H, d, r, R, step = a.heads, a.width, a.tail or 64, a.rank, op.endswith('step')
+        T = a.batch if step else a.tokens
+        proj, w = torch.randn(T, H * (d + r) + R + r, device=dev, dtype=bf), torch.ones(R, device=dev, dtype=bf)
+        table = E.rotary_table(torch.arange(T, device=dev), torch.rand(r // 2, device=dev, dtype=torch.float64))
+        pool, rows = torch.zeros(T, 1, 1, R + r, device=dev, dtype=bf), torch.arange(T, device=dev)
+        ql = torch.empty(T, H, R + r, device=dev, dtype=bf) if step else None
+        return ((lambda: E.latent_rotary(proj, 0, H, d, r, H * (d + r), R, w, 1e-6, table, 0, r // 2, True, ql, pool, rows, not step)), 0.0,
+                2.0 * T * (2 * H * r + (2 if step else 3) * (R + r)))
+    if op in ('joined_norm', 'joined_norm_experts'):
+        W, k = a.hidden, 8
+        x, w, b = torch.zeros(a.tokens, W, device=dev), torch.ones(W, device=dev, dtype=bf), torch.randn(a.tokens, W, device=dev, dtype=bf)
+        if op == 'joined_norm':
+            return (lambda: E.stream_joined_rmsnorm(x, w, 1e-6, 0.0, b)), 0.0, 12.0 * a.tokens * W
+        y, o = torch.randn(a.tokens * k, W, device=dev, dtype=bf), torch.rand(a.tokens, device=dev)
+        row_of, share = torch.randperm(a.tokens * k, device=dev, dtype=torch.int32).view(-1, k), torch.full((a.tokens, k), 1 / k, device=dev)
+        return (lambda: E.stream_joined_rmsnorm(x, w, 1e-6, 0.0, y, row_of, share, b, o)), 0.0, a.tokens * W * (12.0 + 2.0 * k)
+    if op == 'moe_topk_grouped':
+        T, k, Ex = a.tokens, 8, 128
+        lg, x, w = torch.randn(T, Ex, device=dev), torch.randn(T, a.hidden, device=dev, dtype=bf), torch.randn(1, a.hidden, device=dev, dtype=bf)
+        return (lambda: E.moe_topk(lg, None, k, None, 8, 4, 1.0, x, w)), 0.0, 4.0 * T * Ex + 12.0 * T * k + 2.0 * T * a.hidden
     if op in ('hgrn2', 'hgrn2_step', 'gdn_step'):
         # the recurrent mixer between its projections: --heads states of 128 x 128 (prompts of --seq tokens, or a token of --batch
         # sequences); gdn_step: the Gated DeltaNet recurrence on one token of every sequence
@@ -129,14 +166,18 @@ def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
         # flops as for 'gdn' per state element and token: a write (multiply, add) and a read (multiply, add)
         return (lambda: E.hgrn2_prefill(*args, cu, a.seq, pool, slot)), 2.0 * T * H * d * d * 2, 8.0 * T * H * d
     if op == 'latent_decode':
-        # --heads heads against latents of --rank (the like kernel: paged_decode)
+        # --heads heads against latents of --rank with --tail rotated key dimensions inside --window (the like kernel: paged_decode)
         B, bs, ctx, R = a.batch, 16, a.seq, a.rank
+        K, seen = R + a.tail, min(ctx, a.window or ctx)
         nb = B * ((ctx + bs - 1) // bs) + 1
-        pool = torch.randn(nb, bs, 1, R, device=dev, dtype=bf)
+        pool = torch.randn(nb, bs, 1, K, device=dev, dtype=bf)
         tables = torch.arange(1, nb, device=dev, dtype=torch.int32).view(B, -1)
         lens = torch.full((B, ), ctx, device=dev, dtype=torch.int32)
-        q, sinks, gate = torch.randn(B, a.heads, R, device=dev, dtype=bf), torch.zeros(a.heads, device=dev, dtype=bf), torch.zeros(B, a.heads, device=dev, dtype=bf)
-        return (lambda: E.latent_decode(q, pool, tables, lens, R**-0.5, sinks, gate)), 4.0 * B * ctx * a.heads * R, 2.0 * B * ctx * R + 4.0 * B * a.heads * R
+        q, sinks, gate = torch.randn(B, a.heads, K, device=dev, dtype=bf), torch.zeros(a.heads, device=dev, dtype=bf), torch.zeros(B, a.heads, device=dev, dtype=bf)
+        if a.tail:
+            sinks = gate = None
+        return ((lambda: E.latent_decode(q, pool, tables, lens, K**-0.5, sinks, gate, R, a.window)), 2.0 * B * seen * a.heads * (K + R),
+                2.0 * B * seen * K + 2.0 * B * a.heads * (K + R))
     if op == 'latent_norms':
         p = torch.randn(a.tokens, a.hidden + 1536 + 32, device=dev, dtype=bf)
         wq, wc = torch.ones(1024, device=dev, dtype=bf), torch.ones(512, device=dev, dtype=bf)
@@ -174,7 +215,7 @@ def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
             return layout, 0.0, byts
         (row_of, src, slot_of), xs = layout()
         return (lambda: ops.moe_combine(xs, w, row_of, src, slot_of)), 0.0, byts
-    if op in ('experts_relu2', 'experts_swiglu'):
+    if op in ('experts_relu2', 'experts_swiglu', 'experts_columns'):
         # both products of the experts of one layer: two matrices with the activation in the epilogue, or [gate | up] and down
         T, k, Ex, W = a.tokens, 8, 128, a.hidden
         ff = 1152 if op == 'experts_relu2' else 768
@@ -185,7 +226,10 @@ def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
 
         def f():
             with torch.no_grad():
-                h = ops.grouped_gemm(xs, up, off, act='relu2') if op == 'experts_relu2' else ops.swiglu(ops.grouped_gemm(xs, up, off))
+                if op == 'experts_columns':          # the unit as generation runs it
+                    h = ops.glu_columns(ops.grouped_gemm(xs, up, off), 0, ff, ff)
+                else:
+                    h = ops.grouped_gemm(xs, up, off, act='relu2') if op == 'experts_relu2' else ops.swiglu(ops.grouped_gemm(xs, up, off))
                 ops.grouped_gemm(h, down, off)
         used = min(Ex, T * k)
         return f, 2.0 * T * k * (up.shape[1] * W + W * ff), 2.0 * used * (up.shape[1] * W + W * ff)
@@ -198,17 +242,21 @@ def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
         return (lambda: E.stream_rmsnorm(x, w, 1e-6, y, w, y2, w, 0.5)), 0.0, 14.0 * a.tokens * a.hidden
     if op == 'glu_columns':
         p = torch.randn(a.tokens, 6144 + 2 * a.hidden, device=dev, dtype=bf)
-        return (lambda: E.glu_columns(p, 6144, 6144 + a.hidden, a.hidden)), 0.0, 6.0 * a.tokens * a.hidden
+        return (lambda: E.glu_columns(p, 6144, 6144 + a.hidden, a.hidden, a.limit)), 0.0, 6.0 * a.tokens * a.hidden
     if op in ('attn_packed', 'attn_packed32'):
-        # prefill attention at any head width (--width): the tensor-core kernel up to 128 in bf16, fp32 arithmetic beyond / in 32-bit
+        # prefill attention at any head width (--width): the tensor-core kernel up to 192 in bf16, fp32 arithmetic beyond / in 32-bit;
+        # --window / --chunk bound what a position sees, --tail adds key dimensions that all heads share
         T, d, dt = a.tokens, a.width, bf if op == 'attn_packed' else torch.float32
         n_seq = max(T // a.seq, 1)
         cu = torch.arange(0, n_seq + 1, device=dev, dtype=torch.int32) * a.seq
-        q, k, v = (torch.randn(T, h, d, device=dev, dtype=dt) for h in (a.heads, a.kv_heads, a.kv_heads))
+        q, k, v = (torch.randn(T, h, w, device=dev, dtype=dt) for h, w in ((a.heads, d + a.tail), (a.kv_heads, d), (a.kv_heads, d)))
+        tail = torch.randn(T, a.tail, device=dev, dtype=dt) if a.tail else None
+        first = [max(0, i - a.window + 1) if a.window else (i // a.chunk * a.chunk if a.chunk else 0) for i in range(a.seq)]
+        pairs = n_seq * sum(i + 1 - f for i, f in enumerate(first))
         sinks = torch.zeros(a.heads, device=dev, dtype=dt) if a.sinks else None
         gate = torch.zeros(T, a.heads, device=dev, dtype=dt) if a.sinks else None
-        return ((lambda: ops.attention_packed(q, k, v, cu, a.seq, d**-0.5, sinks, gate)), 4.0 * n_seq * a.seq * a.seq * a.heads * d / 2,
-                float(q.element_size()) * T * d * (2 * a.heads + 2 * a.kv_heads))
+        return ((lambda: ops.attention_packed(q, k, v, cu, a.seq, d**-0.5, sinks, gate, a.window, a.chunk, tail)), 2.0 * pairs * a.heads * (2 * d + a.tail),
+                float(q.element_size()) * T * (d * (2 * a.heads + 2 * a.kv_heads) + a.tail * (a.heads + 1)))
     if op == 'rmsnorm':
         x, w = torch.randn(a.tokens, a.hidden, device=dev, dtype=bf), torch.ones(a.hidden, device=dev, dtype=bf)
 
@@ -266,7 +314,10 @@ def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
         tables = torch.arange(nb, device=dev, dtype=torch.int32).view(B, -1)
         lens = torch.full((B, ), ctx, device=dev, dtype=torch.int32)
         q = torch.randn(B, a.heads, a.width, device=dev, dtype=bf)
-        return (lambda: ops.paged_attention_decode(q, kc, vc, tables, lens)), 0.0, 2.0 * 2 * B * ctx * a.kv_heads * a.width
+        sinks, gate = (torch.zeros(a.heads, device=dev, dtype=bf), torch.zeros(B, a.heads, device=dev, dtype=bf)) if a.sinks else (None, None)
+        seen = min(ctx, a.window or ctx) if not a.chunk else (ctx - 1) % a.chunk + 1
+        return ((lambda: ops.paged_attention_decode(q, kc, vc, tables, lens, window=a.window or None, chunk=a.chunk, sinks=sinks, gate=gate)), 0.0,
+                2.0 * 2 * B * seen * a.kv_heads * a.width)
     if op == 'sample':
         lg = torch.randn(a.batch, a.vocab, device=dev)
         seeds = torch.arange(a.batch, device=dev, dtype=torch.int64)
@@ -342,7 +393,11 @@ def main() -> None:
     ap.add_argument('--heads', type=int, default=32)
     ap.add_argument('--kv-heads', type=int, default=8)
     ap.add_argument('--width', type=int, default=128, help='head width')
-    ap.add_argument('--sinks', action='store_true', help='attn_packed: with sink logits and output gates')
+    ap.add_argument('--sinks', action='store_true', help='attn_packed, paged_decode: with sink logits and output gates')
+    ap.add_argument('--window', type=int, default=0, help='attention: the last positions that a position sees (0: all)')
+    ap.add_argument('--chunk', type=int, default=0, help='attention: positions of a block that sees only itself (0: none)')
+    ap.add_argument('--tail', type=int, default=0, help='attention: key dimensions that all heads share')
+    ap.add_argument('--limit', type=float, default=0.0, help='glu_columns: bound of the clamped unit (0: silu)')
     ap.add_argument('--hidden', type=int, default=4096)
     ap.add_argument('--vocab', type=int, default=151936)
     ap.add_argument('--batch', type=int, default=256)
