@@ -24,7 +24,7 @@ from typing import Callable, Dict, Iterable, Iterator, List, Optional, Tuple
 
 import torch
 
-from .config import DecoderConfig
+from .config import DecoderConfig, PostNormSpec
 
 _LAYER = re.compile(r'^layers\.(\d+)\.(.+)$')
 
@@ -166,13 +166,29 @@ _LISTED = {'input_layernorm.weight': 'norm1', 'v_lambda': 'mix.vmix', 'o_proj.we
            'mixer.kv_norm.weight': 'mix.dkv.norm', 'mixer.q_up.weight': 'mix.uq', 'mixer.sinks': 'mix.sink', 'mixer.o_proj.weight': 'mix.o',
            'mixer.f_bias': 'mix.f.b', 'mixer.lower': 'mix.lower', 'mixer.out_norm.weight': 'mix.norm', 'mlp.down_proj.weight': 'mlp.down',
            'mlp.gate.weight': 'mlp.router', 'mlp.gate.bias': 'mlp.router.b', 'mixer.head_q_norm.weight': 'mix.q.norm', 'mixer.head_k_norm.weight': 'mix.k.norm',
-           'mlp.shared_expert.down_proj.weight': 'mlp.shared.down', 'mlp.shared_expert_gate.weight': 'mlp.shared.sg'}
+           'mlp.shared_expert.down_proj.weight': 'mlp.shared.down', 'mlp.shared_expert_gate.weight': 'mlp.shared.sg',
+           'mixer.temperature': 'mix.temp', 'mixer.log_slope': 'mix.r1', 'mixer.log_rate': 'mix.r2', 'mixer.distance_table': 'mix.rel', 'mixer.o_bias': 'mix.o.b',
+           'mixer.conv_weight': 'mix.conv', 'mixer.conv_bias': 'mix.conv.b', 'mixer.x_proj.weight': 'mix.x', 'mixer.dt_proj.weight': 'mix.dt',
+           'mixer.dt_bias': 'mix.dt.b', 'mixer.A_log': 'mix.A_log', 'mixer.D': 'mix.D', 'mixer.i_bias': 'mix.i.b',
+           'mixer.left_norm.weight': 'mix.left.out', 'mixer.right_norm.weight': 'mix.right.out'}
+# layers without norms in front of their sub-layers name those behind them
+_LISTED_POST = {'post_mixer_layernorm.weight': 'norm1', 'post_mlp_layernorm.weight': 'norm2'}
 _LISTED_PARTS = {'res_gate': 'rg1', 'q_proj': 'mix.q', 'k_proj': 'mix.k', 'v_proj': 'mix.v', 'f_proj': 'mix.f', 'dq_proj': 'mix.dq', 'dkv_proj': 'mix.dkv',
-                 'head_gate': 'mix.g', 'gate_proj': 'mlp.gate', 'up_proj': 'mlp.up'}
+                 'head_gate': 'mix.g', 'gate_proj': 'mlp.gate', 'up_proj': 'mlp.up', 'out_gate': 'mix.g', 'in_proj': 'mix.in', 'i_gate': 'mix.i', 'f_gate': 'mix.f'}
+
+
+def _listed_part(name: str) -> str:
+    """Checkpoint tensor of one projection of a joined matrix; those of two mixers side by side begin with their side."""
+    side, _, rest = name.partition('_')
+    return _LISTED_PARTS[rest].replace('mix.', f'mix.{side}.') if side in ('left', 'right') else _LISTED_PARTS[name]
 
 
 def _listed_parts(rest: str, sp, width: int) -> List[Tuple[str, int]]:
     """(checkpoint tensor, rows) of an internal tensor that joins several, in concatenation order; [] when it does not."""
+    side = re.match(r'mixer\.(left|right)\.(.*)', rest)
+    if side:
+        sub = type(sp)(getattr(sp.mixer, side.group(1)))
+        return [(n.replace('mix.', f'mix.{side.group(1)}.'), rows) for n, rows in _listed_parts(f'mixer.{side.group(2)}', sub, width)]
     if rest == 'conv_weight':
         return [(f'mix.{p}.conv', n) for p, n in zip('qkv', sp.qkv_sizes)]
     if rest == 'in_proj.weight':
@@ -194,7 +210,15 @@ def _listed_parts(rest: str, sp, width: int) -> List[Tuple[str, int]]:
         return [(f'mlp.e{e}.{which}', rows) for e in range(sp.mlp.experts)]
     else:
         return []
-    return [(_LISTED_PARTS[n], rows) for n, rows in parts]
+    return [(_listed_part(n), rows) for n, rows in parts]
+
+
+def _listed_single(rest: str, sp) -> str:
+    """Checkpoint tensor of an internal tensor that is just one."""
+    side = re.match(r'mixer\.(left|right)\.(.*)', rest)
+    if side:
+        return _LISTED[f'mixer.{side.group(2)}'].replace('mix.', f'mix.{side.group(1)}.')
+    return (_LISTED_POST if isinstance(sp, PostNormSpec) and rest in _LISTED_POST else _LISTED)[rest]
 
 
 def _listed_names(name: str, cfg: DecoderConfig) -> List[str]:
@@ -206,7 +230,7 @@ def _listed_names(name: str, cfg: DecoderConfig) -> List[str]:
     if not m:
         raise KeyError(f'no checkpoint mapping for {name}')
     i, rest = int(m.group(1)), m.group(2)
-    return [f'l{i}.{n}' for n, _ in _listed_parts(rest, cfg.layer_specs[i], cfg.hidden_size)] or [f'l{i}.{_LISTED[rest]}']
+    return [f'l{i}.{n}' for n, _ in _listed_parts(rest, cfg.layer_specs[i], cfg.hidden_size)] or [f'l{i}.{_listed_single(rest, cfg.layer_specs[i])}']
 
 
 def _listed_split(name: str, tensor: torch.Tensor, cfg: DecoderConfig) -> List[Tuple[str, torch.Tensor]]:

@@ -11,7 +11,7 @@ import json
 import math
 import os
 from dataclasses import dataclass, field
-from typing import List, Any, Dict, Optional, Tuple, Union
+from typing import Any, Callable, Dict, List, Optional, Sequence, Tuple, Union
 
 
 # config.json ``model_type`` values whose layer maths is what ``models/decoder.py`` computes (each checked against transformers)
@@ -181,8 +181,72 @@ def _nilepel_mapping(c: 'DecoderConfig') -> Dict[str, Any]:
     return d
 
 
+def _puzonex_attention(m: Dict[str, Any], **kinds) -> 'AttentionSpec':
+    return AttentionSpec(**{k: int(m[k]) for k in ('heads', 'kv_heads', 'dim', 'vdim')}, scale=float(m['scale']), window=int(m['mask']['size']), bias=True,
+                         softcap=float(m['softcap']), **kinds)
+
+
+def _puzonex_fields(cfg: Dict[str, Any]) -> Dict[str, Any]:
+    """``config.json`` of a Puzonex checkpoint → keyword arguments of :class:`DecoderConfig`.  The number of rows of a distance table
+    (``left.buckets``) is not in the original file: it is the shape of a tensor, and :func:`_puzonex_sizes` adds it."""
+    specs = []
+    for i, layer in enumerate(cfg['layers']):
+        kind, m, mlp = layer['type'], layer['mixer'], layer.get('mlp')
+        if kind == 'attention':
+            mixer = _puzonex_attention(m, qk_norm=True, value_norm=True, log_bias=True, sinks=True)
+        elif kind == 'mamba1':
+            mixer = Mamba1Spec(**{k: int(m[k]) for k in ('inner', 'state', 'dt_rank', 'conv')})
+        elif kind == 'parallel':
+            left, right = m['left'], m['right']
+            if 'buckets' not in left:
+                raise ValueError(f"layer {i}: the size of its distance table is known from the checkpoint's tensors only; read the configuration with from_pretrained, "
+                                 "or give left.buckets")
+            mixer = SideBySideSpec(_puzonex_attention(left, qk_norm='whole', values_are_keys=True, temperature=True, buckets=int(left['buckets']), bias_max=float(left['bias_max']),
+                                                      out_gate=True, out_bias=True),
+                                   MatrixMemorySpec(**{k: int(right[k]) for k in ('heads', 'dim', 'vdim')}, gate_cap=float(right['gate_cap'])))
+        else:
+            raise NotImplementedError(f"layer {i}: mixer type {kind!r} is not implemented (attention, mamba1 and parallel are)")
+        if mlp is not None and mlp['kind'] != 'dense':
+            raise NotImplementedError(f"layer {i}: feed-forward kind {mlp['kind']!r} is not implemented (dense is)")
+        specs.append(PostNormSpec(mixer, None if mlp is None else FeedForwardSpec(ff=int(mlp['ff']), act='gelu_tanh')))
+    return dict(model_type='puzonex', vocab_size=int(cfg['vocab']), hidden_size=int(cfg['width']), rms_norm_eps=float(cfg['norm']['eps']), sinusoidal_base=10000.0,
+                tie_word_embeddings=False, qk_norm=False, layer_specs=specs, eos_token_id=cfg.get('eos_token_id'), pad_token_id=cfg.get('pad_token_id'),
+                torch_dtype=str(cfg.get('torch_dtype', 'bfloat16')))
+
+
+def _puzonex_mapping(c: 'DecoderConfig') -> Dict[str, Any]:
+    """The inverse of :func:`_puzonex_fields`."""
+    def attention(a: 'AttentionSpec') -> Dict[str, Any]:
+        return {**{k: getattr(a, k) for k in ('heads', 'kv_heads', 'dim', 'vdim', 'scale', 'softcap')}, 'mask': {'size': a.window}}
+
+    layers = []
+    for sp in c.layer_specs:
+        m = sp.mixer
+        if m.kind == 'attention':
+            mixer = attention(m)
+        elif m.kind == 'mamba1':
+            mixer = {k: getattr(m, k) for k in ('inner', 'state', 'dt_rank', 'conv')}
+        else:
+            mixer = {'left': {**attention(m.left), 'bias_max': m.left.bias_max, 'buckets': m.left.buckets},
+                     'right': {k: getattr(m.right, k) for k in ('heads', 'dim', 'vdim', 'gate_cap')}}
+        layers.append({'type': m.kind, 'mixer': mixer, 'mlp': None if sp.mlp is None else {'kind': 'dense', 'ff': sp.mlp.ff}})
+    d = {'architecture': 'Puzonex', 'vocab': c.vocab_size, 'width': c.hidden_size, 'norm': {'eps': c.rms_norm_eps}, 'layers': layers}
+    d.update({k: v for k, v in (('eos_token_id', c.eos_token_id), ('pad_token_id', c.pad_token_id)) if v is not None})
+    return d
+
+
+def _puzonex_sizes(cfg: Dict[str, Any], shape: Callable[[str], Sequence[int]]) -> None:
+    """What the file leaves to the checkpoint's tensors: ``shape`` gives a tensor's by its name."""
+    for i, layer in enumerate(cfg['layers']):
+        if layer['type'] == 'parallel':
+            layer['mixer']['left']['buckets'] = int(shape(f'l{i}.mix.left.rel')[0])
+
+
 # checkpoints whose config.json names its ``architecture`` and lists every layer: (reader → DecoderConfig fields, writer)
-NATIVE_ARCHITECTURES = {'Pomelix': (_pomelix_fields, _pomelix_mapping), 'Moronex': (_moronex_fields, _moronex_mapping), 'Nilepel': (_nilepel_fields, _nilepel_mapping)}
+NATIVE_ARCHITECTURES = {'Pomelix': (_pomelix_fields, _pomelix_mapping), 'Moronex': (_moronex_fields, _moronex_mapping), 'Nilepel': (_nilepel_fields, _nilepel_mapping),
+                        'Puzonex': (_puzonex_fields, _puzonex_mapping)}
+# architectures whose files leave sizes to the tensors' shapes
+_SIZES_FROM_TENSORS = {'Puzonex': _puzonex_sizes}
 
 
 def _up8(n: int) -> int:
@@ -221,8 +285,11 @@ class LayerSpec:
     def conv_rows(self) -> Optional[Tuple[int, int]]:
         return (self.conv - 1, sum(self.qkv_sizes)) if self.conv > 1 else None
 
-    def state_shape(self) -> Optional[Tuple[int, int, int]]:
+    def state_shape(self) -> Optional[Tuple[int, ...]]:
         return None
+
+    def state_width(self) -> int:
+        return 0
 
     def matmul_weights(self, width: int, active: bool = False) -> int:
         return width * sum(self.qkv_sizes) + width * self.heads * self.vdim + 3 * width * self.ff
@@ -274,25 +341,65 @@ class RotarySpec:
         return out
 
 
+class MixerSpec:
+    """What every kind of mixer answers for: what it keeps per token (``kv_rows``) and per sequence (``conv_rows``, ``state_shape``), what it
+    borrows and how it rotates."""
+    kv_from = rotary = None
+
+    def kv_rows(self) -> Tuple[int, int, int]:
+        return 0, 0, 0
+
+    def conv_rows(self) -> Optional[Tuple[int, int]]:
+        return None
+
+    def state_shape(self) -> Optional[Tuple[int, ...]]:
+        return None
+
+    def state_width(self) -> int:
+        """Elements of the state that a token writes and reads."""
+        return math.prod(self.state_shape() or (0, ))
+
+    def attention_width(self) -> int:
+        """Multiply-adds per key and query of the score and value products."""
+        return 0
+
+    def kernel_parts(self) -> List[str]:
+        """Kernels that not every stack needs (``ops/build.py``)."""
+        return []
+
+
 @dataclass
-class AttentionSpec:
-    """Grouped-query attention over rotated queries and keys.  What a position sees: everything before it, its last ``window``
-    positions, or its own block of ``chunk`` positions counted from the first token.  ``bias`` on q, k and v, ``qk_norm`` per head before the
-    rotation, ``sinks`` (a logit per head in the denominator), ``head_gate`` (a sigmoid per head on the output).  ``kv_from``: index of the
-    earlier layer whose keys and values this layer reads instead of its own."""
+class AttentionSpec(MixerSpec):
+    """Grouped-query attention.  Positions enter through a rotation of queries and keys (``rotary``) or through a number per head that is
+    added to a score: ``log_bias`` (``−r1 ln(1 + r2 · distance)``) or a learned table of ``buckets`` rows over distances (exact up to half of them,
+    then logarithmic up to ``bias_max``).  What a position sees: everything before it, its last ``window`` positions, or its own block
+    of ``chunk`` positions counted from the first token.  Projections: ``bias`` on q, k and v; ``values_are_keys`` (the projected keys,
+    before their norm); ``out_bias``.  Norms: ``qk_norm`` per head (True) or over all heads together (``'whole'``); ``value_norm`` (values
+    over their root mean square).  Scores: times ``temperature`` (a number per head), through ``softcap · tanh(s / softcap)``, then the number for the
+    distance; ``sinks`` (a logit per head in the denominator).  Output: ``head_gate`` (a sigmoid per head) or ``out_gate`` (one per element).
+    ``kv_from``: index of the earlier layer whose keys and values this layer reads instead of its own."""
     heads: int
     kv_heads: int
     dim: int
     vdim: int
     scale: float
-    rotary: RotarySpec
+    rotary: Optional[RotarySpec] = None
     window: int = 0
     chunk: int = 0
     bias: bool = False
-    qk_norm: bool = False
+    qk_norm: Union[bool, str] = False
     sinks: bool = False
     head_gate: bool = False
     kv_from: Optional[int] = None
+    values_are_keys: bool = False
+    value_norm: bool = False
+    softcap: float = 0.0
+    temperature: bool = False
+    log_bias: bool = False
+    buckets: int = 0
+    bias_max: float = 0.0
+    out_gate: bool = False
+    out_bias: bool = False
     kind = 'attention'
 
     def __post_init__(self):
@@ -300,19 +407,38 @@ class AttentionSpec:
             self.rotary = RotarySpec(**self.rotary)
         if self.heads % self.kv_heads:
             raise ValueError(f'{self.heads} query heads do not divide over {self.kv_heads} key / value heads')
-        if self.rotary.dims > self.dim:
+        if self.rotary is not None and self.rotary.dims > self.dim:
             raise ValueError(f'rotation over {self.rotary.dims} of {self.dim} dimensions')
+        if self.values_are_keys and self.vdim != self.dim:
+            raise ValueError(f'values that are the keys: {self.vdim} wide, keys are {self.dim} wide')
+        if self.rotary is not None and (self.values_are_keys or self.value_norm or self.qk_norm == 'whole'):
+            raise ValueError('values_are_keys, value_norm and norms over all heads go with attention that does not rotate')
+        if self.rotary is None and self.kv_from is not None:
+            raise ValueError('attention that does not rotate has keys and values of its own')
+        if self.buckets and (self.log_bias or self.buckets < 2 or not self.bias_max > self.buckets // 2):
+            raise ValueError(f'a distance table of {self.buckets} rows up to {self.bias_max}: at least two rows, and a last distance beyond the exact half')
 
     @property
     def qkv_sizes(self) -> Tuple[int, int, int]:
         """Rows of the q, k and v projections (a layer that borrows keys and values has none of its own)."""
         own = 0 if self.kv_from is not None else self.kv_heads
-        return self.heads * self.dim, own * self.dim, own * self.vdim
+        return self.heads * self.dim, own * self.dim, 0 if self.values_are_keys else own * self.vdim
 
     def in_parts(self) -> List[Tuple[str, int]]:
         """Projections of the layer input."""
         parts = [(n, w) for n, w in zip(('q_proj', 'k_proj', 'v_proj'), self.qkv_sizes) if w]
-        return parts + ([('head_gate', self.heads)] if self.head_gate else [])
+        return parts + ([('head_gate', self.heads)] if self.head_gate else []) + ([('out_gate', self.heads * self.vdim)] if self.out_gate else [])
+
+    def distance_buckets(self) -> List[int]:
+        """Row of the distance table for the distances 0 … ``bias_max``; all farther ones share the last."""
+        half, far, out = self.buckets // 2, self.bias_max, []
+        for n in range(int(math.ceil(far)) + 1):
+            # the small term keeps a distance that lies on a boundary in the bucket that begins there
+            out.append(n if n < half else min(self.buckets - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (self.buckets - half) + 1e-9)))
+        return out
+
+    def kernel_parts(self) -> List[str]:
+        return ['rotary' if self.rotary is not None else 'heads']
 
     def kept(self) -> Tuple[Any, ...]:
         """What a borrowing layer must agree on with the layer it borrows from."""
@@ -329,14 +455,16 @@ class AttentionSpec:
 
     def small_weights(self) -> int:
         own = self.kv_from is None
-        return (sum(self.qkv_sizes) if self.bias else 0) + (self.dim * (2 if own else 1) if self.qk_norm else 0) + (self.heads if self.sinks else 0)
+        norms = self.dim * (self.heads + self.kv_heads) if self.qk_norm == 'whole' else self.dim * (2 if own else 1) if self.qk_norm else 0
+        per_head = (1 if self.sinks else 0) + (1 if self.temperature else 0) + (2 if self.log_bias else 0) + self.buckets
+        return (sum(self.qkv_sizes) if self.bias else 0) + norms + per_head * self.heads
 
     def attention_width(self) -> int:
         return (self.dim + self.vdim) * self.heads
 
 
 @dataclass
-class LatentSpec:
+class LatentSpec(MixerSpec):
     """Latent attention: keys (``dim`` per head) and values (``vdim``) expanded from one normed rank-``kv_rank`` latent per token, which
     is all the cache keeps, together with ``rot_dim`` rotated key dimensions that all heads share (0: no positions).  Queries through a
     normed rank-``q_rank`` bottleneck (0: a plain projection; a head's query is ``[dim | rot_dim]``).  ``window``: the last positions that a
@@ -390,25 +518,27 @@ class LatentSpec:
     def small_weights(self) -> int:
         return self.q_rank + (self.kv_rank if self.kv_from is None else 0) + (self.heads if self.sinks else 0)
 
+    def kernel_parts(self) -> List[str]:
+        return ['latent'] + (['rotary'] if self.rotary is not None or not self.q_rank else [])
+
     def attention_width(self) -> int:
         return (self.qk_width + self.vdim) * self.heads
 
 
 @dataclass
-class HGRN2Spec:
+class HGRN2Spec(MixerSpec):
     """Linear attention whose forget gate (per head and channel, bounded from below) also decides what is written; ``heads``
     states of ``dim × vdim``."""
     heads: int
     dim: int
     vdim: int
     kind = 'hgrn2'
-    kv_from = rotary = None
 
-    def kv_rows(self) -> Tuple[int, int, int]:
-        return 0, 0, 0
+    def state_shape(self) -> Tuple[int, ...]:
+        return self.heads, self.dim, self.vdim
 
-    def attention_width(self) -> int:
-        return 0
+    def kernel_parts(self) -> List[str]:
+        return ['recurrent']
 
     def in_parts(self) -> List[Tuple[str, int]]:
         return [('q_proj', self.heads * self.dim), ('f_proj', self.heads * self.dim), ('v_proj', self.heads * self.vdim)]
@@ -421,10 +551,124 @@ class HGRN2Spec:
 
 
 @dataclass
+class Mamba1Spec(MixerSpec):
+    """Selective scan: ``inner`` channels with ``state`` fp32 numbers each, whose decay and input depend on the token through a step size
+    (of rank ``dt_rank``) behind a causal convolution of ``conv`` taps."""
+    inner: int
+    state: int
+    dt_rank: int
+    conv: int
+    kind = 'mamba1'
+    heads = 1
+
+    def __post_init__(self):
+        if self.conv < 1:
+            raise ValueError(f'a convolution of {self.conv} taps')
+
+    @property
+    def dim(self) -> int:
+        return self.inner
+
+    def conv_rows(self) -> Optional[Tuple[int, int]]:
+        return (self.conv - 1, self.inner) if self.conv > 1 else None
+
+    def state_shape(self) -> Tuple[int, ...]:
+        return self.inner, self.state
+
+    def in_parts(self) -> List[Tuple[str, int]]:
+        return [('in_proj', 2 * self.inner)]
+
+    def matmul_weights(self, width: int) -> int:
+        return 3 * width * self.inner + self.inner * (2 * self.dt_rank + 2 * self.state)
+
+    def small_weights(self) -> int:
+        return self.inner * (self.conv + 1 + 1 + self.state + 1)
+
+    def kernel_parts(self) -> List[str]:
+        return ['selective']
+
+
+@dataclass
+class MatrixMemorySpec(MixerSpec):
+    """mLSTM: ``heads`` matrix memories of ``dim × vdim`` with a normaliser of ``dim`` and a running maximum, exponential input gates and
+    sigmoid forget gates in the logarithm, both capped at ``gate_cap``."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+    kind = 'mlstm'
+
+    def state_shape(self) -> Tuple[int, ...]:
+        """Per head the matrix by rows, the normaliser (filled up to whole vectors) and a vector that begins with the maximum."""
+        return self.heads, -(-self.dim * self.vdim // 4) * 4 + -(-self.dim // 4) * 4 + 4
+
+    def state_width(self) -> int:
+        return self.heads * self.dim * (self.vdim + 1)
+
+    def in_parts(self) -> List[Tuple[str, int]]:
+        d, e = self.heads * self.dim, self.heads * self.vdim
+        return [('q_proj', d), ('k_proj', d), ('v_proj', e), ('out_gate', e), ('i_gate', self.heads), ('f_gate', self.heads)]
+
+    def matmul_weights(self, width: int) -> int:
+        return width * (sum(n for _, n in self.in_parts()) + self.heads * self.vdim)
+
+    def small_weights(self) -> int:
+        return self.heads * (self.vdim + 2)
+
+    def kernel_parts(self) -> List[str]:
+        return ['memory']
+
+
+@dataclass
+class SideBySideSpec(MixerSpec):
+    """Attention and a matrix memory on the same input; the result is half the sum of both, each RMS-normed over the model's width."""
+    left: AttentionSpec
+    right: MatrixMemorySpec
+    kind = 'parallel'
+
+    def __post_init__(self):
+        if isinstance(self.left, dict):
+            self.left = AttentionSpec(**self.left)
+        if isinstance(self.right, dict):
+            self.right = MatrixMemorySpec(**self.right)
+        if self.left.kv_from is not None:
+            raise ValueError('attention beside another mixer has keys and values of its own')
+
+    heads = property(lambda self: self.left.heads)
+    kv_heads = property(lambda self: self.left.kv_heads)
+    dim = property(lambda self: self.left.dim)
+    rotary = property(lambda self: self.left.rotary)
+
+    def kv_rows(self) -> Tuple[int, int, int]:
+        return self.left.kv_rows()
+
+    def state_shape(self) -> Tuple[int, ...]:
+        return self.right.state_shape()
+
+    def state_width(self) -> int:
+        return self.right.state_width()
+
+    def in_parts(self) -> List[Tuple[str, int]]:
+        return [(f'{side}_{n}', w) for side in ('left', 'right') for n, w in getattr(self, side).in_parts()]
+
+    def matmul_weights(self, width: int) -> int:
+        return self.left.matmul_weights(width) + self.right.matmul_weights(width)
+
+    def small_weights(self) -> int:
+        return self.left.small_weights() + self.right.small_weights()
+
+    def attention_width(self) -> int:
+        return self.left.attention_width()
+
+    def kernel_parts(self) -> List[str]:
+        return self.left.kernel_parts() + self.right.kernel_parts()
+
+
+@dataclass
 class FeedForwardSpec:
     """Gated feed-forward block of width ``ff``, or, with ``experts``, that many experts of which a token uses ``top``.
 
-    Dense: ``silu(gate) · up``, or with a ``limit`` ``g σ(1.702 g) (u + 1)`` on ``g ≤ limit``, ``|u| ≤ limit``.
+    Dense: ``act(gate) · up`` with ``act`` ``'silu'`` or ``'gelu_tanh'``, or with a ``limit`` ``g σ(1.702 g) (u + 1)`` on ``g ≤ limit``, ``|u| ≤ limit``.
     Experts: two matrices around the square of relu, or ``gated`` ones (three matrices, ``silu(gate) · up``).  ``scoring`` as in
     ``DecoderConfig.router_scoring``: ``'topk_softmax'`` (biased logits, a softmax over the chosen) or ``'softmax_grouped'`` (softmax over all;
     only experts of the ``keep`` best of ``groups`` groups of neighbours, each as good as its best expert; weights times ``scale``).
@@ -439,8 +683,11 @@ class FeedForwardSpec:
     keep: int = 1
     scale: float = 1.0
     shared: int = 0
+    act: str = 'silu'
 
     def __post_init__(self):
+        if self.act not in ('silu', 'gelu_tanh') or (self.act != 'silu' and (self.limit or self.experts)):
+            raise ValueError(f'activation {self.act!r}: silu, or gelu_tanh in a dense block without a limit')
         if not self.experts:
             return
         if self.experts % self.groups or not 1 <= self.keep <= self.groups:
@@ -458,14 +705,14 @@ class FeedForwardSpec:
         return self.experts if self.scoring == 'topk_softmax' else 0
 
 
-_MIXER_SPECS = ((LatentSpec, 'kv_rank'), (AttentionSpec, 'kv_heads'), (HGRN2Spec, 'heads'))
+_MIXER_SPECS = ((SideBySideSpec, 'left'), (LatentSpec, 'kv_rank'), (AttentionSpec, 'kv_heads'), (Mamba1Spec, 'inner'), (MatrixMemorySpec, 'gate_cap'), (HGRN2Spec, 'heads'))
 
 
 @dataclass
 class SandwichSpec:
     """One layer with a norm in front of and behind each sub-layer and a sigmoid gate (read from the sub-layer's input) on its
     result: a mixer and a feed-forward block (None: the layer has none)."""
-    mixer: Union[LatentSpec, AttentionSpec, HGRN2Spec]
+    mixer: MixerSpec
     mlp: Optional[FeedForwardSpec] = None
 
     def __post_init__(self):
@@ -491,10 +738,13 @@ class SandwichSpec:
         return self.mixer.kv_rows()
 
     def conv_rows(self) -> Optional[Tuple[int, int]]:
-        return None
+        return self.mixer.conv_rows()
 
-    def state_shape(self) -> Optional[Tuple[int, int, int]]:
-        return (self.mixer.heads, self.mixer.dim, self.mixer.vdim) if self.mixer.kind == 'hgrn2' else None
+    def state_shape(self) -> Optional[Tuple[int, ...]]:
+        return self.mixer.state_shape()
+
+    def state_width(self) -> int:
+        return self.mixer.state_width()
 
     def around(self, width: int) -> Tuple[int, int]:
         """Weights of what stands around one sub-layer: in products, and others."""
@@ -505,17 +755,31 @@ class SandwichSpec:
         return n + (self.around(width)[0] + self.mlp.matmul_weights(width, active) if self.mlp is not None else 0)
 
     def small_weights(self, width: int) -> int:
-        n = self.around(width)[1] + self.mixer.small_weights()
+        n = self.around(width)[1] + self.inside(width) + self.mixer.small_weights()
         return n + (self.around(width)[1] + self.mlp.small_weights() if self.mlp is not None else 0)
 
     def attention_width(self) -> int:
         return self.mixer.attention_width()
 
+    def inside(self, width: int) -> int:
+        """Weights inside the mixer that are as wide as the model: norms of two results, the bias of an output projection."""
+        m = self.mixer
+        return (2 * width if m.kind == 'parallel' else 0) + (width if getattr(getattr(m, 'left', m), 'out_bias', False) else 0)
+
 
 @dataclass
 class PreNormSpec(SandwichSpec):
     """One layer with a norm in front of each sub-layer, whose result joins the stream as it is."""
-    post: bool = False           # no norm behind the sub-layers (tells the two kinds apart when read from a mapping)
+    post: bool = False           # no norm behind the sub-layers (tells the kinds apart when read from a mapping)
+
+    def around(self, width: int) -> Tuple[int, int]:
+        return 0, width
+
+
+@dataclass
+class PostNormSpec(SandwichSpec):
+    """One layer whose sub-layers read the stream as it is; a norm on each sub-layer's result before it joins."""
+    pre: bool = False            # no norm in front of the sub-layers (tells the kinds apart when read from a mapping)
 
     def around(self, width: int) -> Tuple[int, int]:
         return 0, width
@@ -524,7 +788,9 @@ class PreNormSpec(SandwichSpec):
 def _layer_spec(sp: Any) -> Any:
     if not isinstance(sp, dict):
         return sp
-    return (LayerSpec if 'mixer' not in sp else (PreNormSpec if 'post' in sp else SandwichSpec))(**sp)
+    if 'mixer' not in sp:
+        return LayerSpec(**sp)
+    return (PreNormSpec if 'post' in sp else PostNormSpec if 'pre' in sp else SandwichSpec)(**sp)
 
 
 @dataclass
@@ -635,8 +901,11 @@ class DecoderConfig:
     mrope_interleaved: bool = False  # Qwen3-VL lays the three position components out t h w t h w … instead of in blocks
     # stacks whose layers are listed one by one, with a 32-bit residual stream: layers that run mixer and feed-forward side by side
     # on one norm, each result with a learned per-channel scale (``LayerSpec``; Pomelix), layers with norms around each sub-layer and a
-    # gate on its result (``SandwichSpec``; Moronex), or layers with a norm in front of each sub-layer (``PreNormSpec``; Nilepel)
-    layer_specs: Optional[List[Union[LayerSpec, SandwichSpec, PreNormSpec, Dict[str, Any]]]] = None
+    # gate on its result (``SandwichSpec``; Moronex), layers with a norm in front of each sub-layer (``PreNormSpec``; Nilepel), or layers with a
+    # norm on each sub-layer's result only (``PostNormSpec``; Puzonex)
+    layer_specs: Optional[List[Union[LayerSpec, SandwichSpec, PreNormSpec, PostNormSpec, Dict[str, Any]]]] = None
+    # such stacks: sines and cosines of the position on top of the token embeddings, pair ``i`` at ``base^(−2i/hidden)`` per position (0: none)
+    sinusoidal_base: float = 0.0
 
     def __post_init__(self):
         if self.layer_specs is not None:
@@ -656,7 +925,7 @@ class DecoderConfig:
                 if j is None:
                     continue
                 src = self.layer_specs[j].mixer if 0 <= j < i else None
-                if src is None or src.kind == 'hgrn2' or src.kv_from is not None or src.kept() != sp.mixer.kept():
+                if src is None or src.kind not in ('attention', 'latent_attention') or src.kv_from is not None or src.kept() != sp.mixer.kept():
                     raise ValueError(f'layer {i}: kv_from {j} is not an earlier layer with keys and values of its own and the same sizes and rotation {sp.mixer.kept()}')
         if self.vision is not None:
             from .vision import VisionConfig
@@ -687,7 +956,7 @@ class DecoderConfig:
         """Per layer ``(rows, channels)`` of the convolution history a sequence keeps between steps (None: no history)."""
         return [sp.conv_rows() for sp in self.layer_specs or []]
 
-    def state_layout(self) -> List[Optional[Tuple[int, int, int]]]:
+    def state_layout(self) -> List[Optional[Tuple[int, ...]]]:
         """Per layer shape of the (fp32) recurrent state a sequence carries from token to token (None: no state)."""
         return [sp.state_shape() for sp in self.layer_specs or []]
 
@@ -708,7 +977,7 @@ class DecoderConfig:
             if m is None:
                 parts.add('convolution')
             else:
-                parts.update({'latent_attention': ['latent'], 'hgrn2': ['recurrent']}.get(m.kind, []) + (['rotary'] if m.rotary is not None or getattr(m, 'q_rank', 1) == 0 else []))
+                parts.update(m.kernel_parts())
                 parts.update(['experts'] if sp.is_moe else [])
         return sorted(parts)
 
@@ -798,7 +1067,7 @@ class DecoderConfig:
         h, L = self.hidden_size, self.num_hidden_layers
         if self.layer_specs is not None:
             attn = sum(sp.attention_width() for sp in self.layer_specs) * avg_context
-            state = 2 * sum(a * b * c for a, b, c in filter(None, self.state_layout()))       # a write and a read of every state element
+            state = 2 * sum(sp.state_width() for sp in self.layer_specs)       # a write and a read of every state element
             return 6.0 * (self._listed_matmul_weights(active=True) + self.vocab_size * h + state) + 6.0 * attn
         attn_w = self._attn_weights()
         moe_w = self.num_experts_per_tok * 3 * h * self.moe_intermediate_size + h * self.num_experts + 3 * h * self.shared_expert_intermediate_size
@@ -907,7 +1176,14 @@ class DecoderConfig:
     @classmethod
     def from_pretrained(cls, path: str) -> 'DecoderConfig':
         with open(os.path.join(path, 'config.json')) as f:
-            return cls.from_hf(json.load(f))
+            cfg = json.load(f)
+        sizes = _SIZES_FROM_TENSORS.get(cfg.get('architecture'))
+        if sizes is not None:
+            from ..utils.safetensors_io import SafetensorLazyLoader
+            loader = SafetensorLazyLoader(path)
+            sizes(cfg, lambda name: loader.get_slice(name).get_shape())
+            loader.close()
+        return cls.from_hf(cfg)
 
     def to_hf(self) -> Dict[str, Any]:
         if self.layer_specs is not None:

@@ -22,7 +22,7 @@ import torch.nn as nn
 import torch.nn.functional as F
 
 from .. import ops
-from .config import DecoderConfig, PreNormSpec, SandwichSpec
+from .config import DecoderConfig, PostNormSpec, PreNormSpec, SandwichSpec
 from .layers import Embedding, Linear, RMSNorm
 from .parallel_layer import CacheView, ParallelLayer, Stream
 
@@ -562,7 +562,7 @@ class DecoderModel(nn.Module):
                 m.full_name = name
         self.layer_runner = None  # engine hook: runs one layer (checkpoint / FSDP unshard)
         self.tp = None  # tensor-parallel context, set by parallel.tensor.apply_tensor_parallel
-        self._frequencies: Dict[torch.device, torch.Tensor] = {}
+        self._frequencies: Dict[Tuple[str, torch.device], torch.Tensor] = {}
 
     def _layer_class(self, i: int):
         if self.cfg.layer_specs is None:
@@ -570,6 +570,9 @@ class DecoderModel(nn.Module):
         if isinstance(self.cfg.layer_specs[i], PreNormSpec):
             from .prenorm_layer import PreNormLayer
             return PreNormLayer
+        if isinstance(self.cfg.layer_specs[i], PostNormSpec):
+            from .postnorm_layer import PostNormLayer
+            return PostNormLayer
         if isinstance(self.cfg.layer_specs[i], SandwichSpec):
             from .sandwich_layer import SandwichLayer
             return SandwichLayer
@@ -642,15 +645,26 @@ class DecoderModel(nn.Module):
         rots = self.cfg.rotations()
         if not rots:
             return None
-        f = self._frequencies.get(positions.device)
+        f = self._frequencies.get(('rotations', positions.device))
         if f is None:       # kept per device; not a buffer, which would follow the model's dtype
-            f = self._frequencies[positions.device] = torch.tensor([v for r in rots for v in r.frequencies()], dtype=torch.float64, device=positions.device)
+            f = self._frequencies['rotations', positions.device] = torch.tensor([v for r in rots for v in r.frequencies()], dtype=torch.float64, device=positions.device)
         return ops.rotary_table(positions, f)
+
+    def embed_positions(self, batch: PackedBatch) -> torch.Tensor:
+        """Token embeddings with sines and cosines of the position on top, the start of a 32-bit stream."""
+        cfg, dev = self.cfg, batch.position_ids.device
+        f = self._frequencies.get(('waves', dev))
+        if f is None:
+            W = cfg.hidden_size
+            f = self._frequencies['waves', dev] = torch.tensor([cfg.sinusoidal_base**(-2.0 * i / W) for i in range((W + 1) // 2)], dtype=torch.float64, device=dev)
+        if batch.inputs_embeds is None and self.layer_runner is None and not torch.is_grad_enabled():
+            return ops.embed_positions(batch.input_ids, self.embed_tokens.weight, batch.position_ids, f)
+        return self.embed(batch).float() + ops.position_waves(batch.position_ids, f, cfg.hidden_size)
 
     def _forward_listed(self, batch: PackedBatch) -> torch.Tensor:
         """Stacks with listed layers: fp32 stream, final norm in the compute dtype (see ``models/parallel_layer.py``)."""
         cfg, run = self.cfg, self.layer_runner
-        x = self.embed(batch)
+        x = self.embed_positions(batch) if cfg.sinusoidal_base else self.embed(batch)
         batch.rotary = self.rotary_table(batch.position_ids)
         if run is None and not torch.is_grad_enabled():
             x = x.float().clone() if batch.inputs_embeds is not None else x.float()      # updated in place from here on

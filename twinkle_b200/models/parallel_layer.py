@@ -66,19 +66,37 @@ class PlainResult:
 
 
 @dataclass
+class NormedResult:
+    """A sub-layer's result on its way into the stream: ``norm(result + bias)``, or with a second one ``norm(½ (inner(result + bias) +
+    beside_inner(beside)))``."""
+    result: torch.Tensor
+    norm: RMSNorm
+    bias: Optional[torch.Tensor] = None
+    inner: Optional[RMSNorm] = None
+    beside: Optional[torch.Tensor] = None
+    beside_inner: Optional[RMSNorm] = None
+
+
+@dataclass
 class Stream:
     """The residual stream between layers: ``x`` (fp32) plus sub-layer results that have not joined it yet (``adds`` times
-    ``mult``, one gated and normed result, or one plain result), and what later layers take from earlier ones (``held``: layer → tensor)."""
+    ``mult``, one gated and normed result, one plain or one normed result), and what later layers take from earlier ones (``held``: layer → tensor)."""
     x: torch.Tensor
     adds: List[Tuple[torch.Tensor, torch.Tensor]] = field(default_factory=list)
     held: Dict[int, torch.Tensor] = field(default_factory=dict)
     mult: float = 1.0
     gated: Optional[GatedResult] = None
     plain: Optional[PlainResult] = None
+    normed: Optional[NormedResult] = None
 
-    def enter(self, norm: RMSNorm) -> torch.Tensor:
-        """What is pending joins the stream; returns its norm in the compute dtype — one kernel."""
-        if self.gated is not None:
+    def enter(self, norm: Optional[RMSNorm], dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+        """What is pending joins the stream; returns its norm (None: the stream itself, in ``dtype``) in the compute dtype — one kernel."""
+        if self.normed is not None:
+            y, w = self.normed, lambda n: None if n is None else n.weight  # noqa: E731
+            h, self.x = ops.stream_normed(self.x, w(norm), y.norm.eps, y.result, y.bias, y.norm.weight, w(y.inner), y.beside, w(y.beside_inner))
+        elif norm is None and self.gated is self.plain is None and not self.adds:
+            h = self.x.to(dtype)
+        elif self.gated is not None:
             g = self.gated
             h, self.x = ops.stream_gated_rmsnorm(self.x, norm.weight, norm.eps, norm.offset, g.result, g.gate, g.bias, g.norm.weight, g.row_of, g.share)
         elif self.plain is not None:
@@ -86,7 +104,7 @@ class Stream:
             h, self.x = ops.stream_joined_rmsnorm(self.x, norm.weight, norm.eps, norm.offset, y.result, y.row_of, y.share, y.beside, y.open)
         else:
             h, self.x = ops.stream_rmsnorm(self.x, norm.weight, norm.eps, self.adds, self.mult, norm.offset)
-        self.adds, self.gated, self.plain = [], None, None
+        self.adds, self.gated, self.plain, self.normed = [], None, None, None
         return h
 
 

@@ -25,7 +25,7 @@ class PreNormLayer(MixerLayer):
         if f is None:
             return
         self.pre_mlp_layernorm = self.norm(cfg)
-        self.mlp = self.experts(cfg) if self.is_moe else GatedFeedForward(cfg.hidden_size, f.ff, limit=f.limit)
+        self.mlp = self.experts(cfg) if self.is_moe else GatedFeedForward(cfg.hidden_size, f.ff, limit=f.limit, act=f.act)
 
     def feed_forward(self, h: torch.Tensor, batch) -> PlainResult:
         if not self.is_moe:

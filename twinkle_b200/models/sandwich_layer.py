@@ -36,7 +36,7 @@ class SandwichLayer(MixerLayer):
             self.mlp_gate = Linear(cfg.hidden_size, cfg.hidden_size, name='res_gate')
             self.mlp = self.experts(cfg)
         else:
-            self.mlp = GatedFeedForward(cfg.hidden_size, sp.mlp.ff, lead, sp.mlp.limit)
+            self.mlp = GatedFeedForward(cfg.hidden_size, sp.mlp.ff, lead, sp.mlp.limit, sp.mlp.act)
 
     def feed_forward(self, h: torch.Tensor, batch) -> GatedResult:
         if not self.is_moe:

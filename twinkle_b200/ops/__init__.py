@@ -19,7 +19,7 @@ from __future__ import annotations
 
 import math
 import os
-from typing import Optional, Tuple
+from typing import NamedTuple, Optional, Tuple
 
 import torch
 
@@ -314,6 +314,163 @@ def stream_joined_rmsnorm(x, weight, eps: float, offset: float, result, row_of=N
     return ext().stream_joined_rmsnorm(x, weight, eps, offset, result.contiguous(), row_of, share, None if beside is None else beside.contiguous(), open), x
 
 
+def stream_normed(x, weight, eps: float, y, bias, post, inner=None, beside=None, beside_inner=None):
+    """fp32 residual stream ``x [T, W]``: ``x ← x + norm(y + bias; post)``, or with a second result ``x ← x + norm(½ (norm(y + bias; inner) +
+    norm(beside; beside_inner)); post)``, and the norm of the sum (``weight`` None: the sum itself) in ``y``'s dtype, one kernel on CUDA.  Returns
+    ``(norm, x)``; without gradients ``x`` is updated in place."""
+    if not _cuda(x) or _needs_grad(x, weight, y, bias, post, inner, beside, beside_inner):
+        return ref.stream_normed(x, weight, eps, y.dtype, y, bias, post, inner, beside, beside_inner)
+    return ext().stream_normed(x, weight, eps, y.contiguous(), bias, post, inner, None if beside is None else beside.contiguous(), beside_inner), x
+
+
+def position_waves(positions, frequencies, width: int):
+    """``[T, width]`` fp32: sine and cosine of position times frequency (fp64) side by side."""
+    return ref.position_waves(positions, frequencies, width)
+
+
+def embed_positions(ids, weight, positions, frequencies):
+    """Rows of an embedding plus :func:`position_waves`, fp32; one kernel on CUDA (no gradient)."""
+    if _cuda(weight):
+        return ext().embed_positions(ids.contiguous(), weight, positions.contiguous(), frequencies)
+    return torch.nn.functional.embedding(ids, weight).float() + ref.position_waves(positions, frequencies, weight.shape[1])
+
+
+# ------------------------------------------- heads without a rotation
+def plain_heads(proj, first: int, bias, q_weight, k_weight, value_norm: bool, values_are_keys: bool, hq: int, hkv: int, d: int, e: int, eps: float, view=None, layer: int = -1):
+    """Columns ``[q | k | v]`` (``[q | k]`` when the values are the projected keys) of a fused projection from ``first`` on → ``(q [T,hq,d'], k
+    [T,hkv,d'] | None, v [T,hkv,e'] | None)``: bias, RMS norm of q and k per head (weights ``[d]``) or over all heads together (``[hq · d]``, ``[hkv ·
+    d]``), values over their root mean square per head (``value_norm``).  ``view`` and the widths ``d'``, ``e'``: see :func:`rotary_heads`."""
+    step = view is not None and view.stepping
+    pools = (view.cache.k[layer], view.cache.v[layer], view.rows) if view is not None else (None, None, None)
+    if _cuda(proj) and not _needs_grad(proj, bias, q_weight, k_weight):
+        out = ext().plain_heads(proj, first, bias, q_weight, k_weight, value_norm, values_are_keys, hq, hkv, d, e, eps, *pools, not step)
+        return tuple(out) if len(out) == 3 else (out[0], None, None)
+    q, k, v = ref.plain_heads(proj, first, bias, q_weight, k_weight, value_norm, values_are_keys, hq, hkv, d, e, eps)
+    if _needs_grad(proj, bias, q_weight, k_weight):
+        return q, k, v
+    q, k, v = (torch.nn.functional.pad(t, (0, -t.shape[-1] % 8)) for t in (q, k, v))
+    if pools[0] is not None:
+        pools[0].view(-1, *k.shape[1:])[view.rows] = k
+        pools[1].view(-1, *v.shape[1:])[view.rows] = v
+    return (q, None, None) if step else (q, k, v)
+
+
+class ScoreTerms(NamedTuple):
+    """What happens to an attention score beyond its scale, in this order: times a number per head (``temp [H]``), ``softcap · tanh(s / softcap)``, and a number
+    for the distance ``n`` between query and key: ``−slope[h] ln(1 + rate[h] n)``, or ``table[bucket[min(n, last)], h]``."""
+    softcap: float = 0.0
+    temp: Optional[torch.Tensor] = None
+    slope: Optional[torch.Tensor] = None
+    rate: Optional[torch.Tensor] = None
+    table: Optional[torch.Tensor] = None        # [rows, H]
+    bucket: Optional[torch.Tensor] = None       # [distances] int32
+
+    def apply(self, s, distance):
+        """Scores ``[H, Lq, Lk]`` (scaled) at distances ``[Lq, Lk]``."""
+        n = distance.clamp(min=0)
+        if self.temp is not None:
+            s = s * self.temp.float()[:, None, None]
+        if self.softcap:
+            s = self.softcap * torch.tanh(s / self.softcap)
+        if self.slope is not None:
+            s = s - self.slope.float()[:, None, None] * torch.log1p(self.rate.float()[:, None, None] * n)
+        if self.table is not None:
+            s = s + self.table.float()[self.bucket[n.clamp(max=self.bucket.numel() - 1)].long()].permute(2, 0, 1)
+        return s
+
+    @property
+    def tensors(self):
+        return self.temp, self.slope, self.rate, self.table, self.bucket
+
+
+def _score_args(terms: Optional[ScoreTerms], softcap: float = 0.0):
+    """A kernel's arguments for ``terms`` (or just a cap)."""
+    if terms is None:
+        return float(softcap or 0.0), None, None, None, None, None
+    return (float(terms.softcap), *terms.tensors)
+
+
+def _open_gate(o, gate):
+    """The output of heads ``[T, H, e]`` times the sigmoid of a gate per head ``[T, H]`` or per element ``[T, H · e]``."""
+    if gate is None:
+        return o
+    g = torch.sigmoid(gate.float())
+    if g.shape[1] == o.shape[1]:
+        return (o.float() * g[..., None]).to(o.dtype)
+    g = g.view(*o.shape[:2], -1)
+    return (o.float() * torch.nn.functional.pad(g, (0, o.shape[-1] - g.shape[-1]))).to(o.dtype)      # rows may be filled up with zeros
+
+
+# ------------------------------------------- selective scan, matrix memory
+def conv_silu(proj, first: int, channels: int, weight, bias, positions, view=None, layer: int = -1):
+    """Causal depth-wise convolution (``weight [channels, taps]``, ``bias``) and silu on columns of a projection → ``[T, channels]``.  ``view`` (a
+    ``CacheView``): the last inputs are kept in the history pool, a ring over positions, and single steps take their past from it."""
+    step = view is not None and view.stepping
+    hist = view.cache.conv[layer] if view is not None else None
+    if _cuda(proj) and not _needs_grad(proj, weight, bias):
+        return ext().conv_silu(proj, first, weight, bias, positions, step, hist, *((view.slots, view.left) if view is not None else (None, None)))
+    x = proj[:, first:first + channels]
+    y = ref.conv_silu(x, weight, bias, positions, hist if step else None, view.slots if step else None)
+    if hist is not None:
+        n = hist.shape[1]
+        keep = (view.left < n).nonzero(as_tuple=True)[0]
+        hist[view.slots[keep].long(), positions[keep] % n] = x[keep]
+    return y
+
+
+def selective_scan(u, dt, dt_bias, A_log, proj, b0: int, c0: int, D, gate, z0: int, cu_seqlens=None, max_seqlen: int = 0, view=None, layer: int = -1):
+    """The selective scan behind its projections: inputs ``u [T, inner]``, step sizes ``softplus(dt + dt_bias)``, ``B`` and ``C`` in columns ``b0``, ``c0`` of
+    ``proj``, ``A = −e^A_log``, skip ``D``, output gate ``silu`` of columns ``z0 …`` of ``gate`` → ``[T, inner]``.  Prompts start from an empty
+    state; ``view`` (a ``CacheView``) says where the last states go, and single steps continue from there."""
+    inner, n = A_log.shape
+    step = view is not None and view.stepping
+    states = view.cache.state[layer] if view is not None else None
+    if _cuda(u) and not _needs_grad(u, dt, dt_bias, A_log, proj, D, gate):
+        args = (u, dt, dt_bias, A_log, proj, b0, c0, D, gate, z0)
+        if step:
+            return ext().selective_step(*args, states, view.slots)
+        return ext().selective_prefill(*args, cu_seqlens.to(torch.int32), int(max_seqlen), states, None if view is None else view.slots)
+    args = (u, dt, dt_bias, A_log, proj[:, b0:b0 + n], proj[:, c0:c0 + n], D, gate[:, z0:z0 + inner])
+    if step:
+        slots = view.slots.long()
+        y, last = ref.selective_scan(*args, list(range(u.shape[0] + 1)), list(states[slots]))
+        states[slots] = torch.stack(last)
+        return y
+    y, last = ref.selective_scan(*args, cu_seqlens.tolist())
+    if states is not None:
+        states[view.slots[cu_seqlens[:-1].long()].long()] = torch.stack(last)
+    return y
+
+
+def matrix_memory(proj, first: int, heads: int, dim: int, vdim: int, i_bias, f_bias, cap: float, weight, eps: float, cu_seqlens=None, max_seqlen: int = 0, view=None,
+                  layer: int = -1):
+    """The matrix memory between its projections: columns ``[q | k | v | gate | i | f]`` of ``proj`` from ``first`` on → the normed and gated output ``[T, heads · vdim]``.
+    Prompts start from an empty state; ``view`` (a ``CacheView``) says where the last states go, and single steps continue from there.  A
+    state is a row of ``[heads, ·]``: the matrix by rows, the normaliser, the running maximum, each from a 16-byte boundary on."""
+    step = view is not None and view.stepping
+    states = view.cache.state[layer] if view is not None else None
+    args = (proj, first, heads, dim, vdim, i_bias, f_bias, cap, weight, eps)
+    if _cuda(proj) and not _needs_grad(proj, i_bias, f_bias, weight):
+        if step:
+            return ext().mlstm_step(*args, states, view.slots)
+        return ext().mlstm_prefill(*args, cu_seqlens.to(torch.int32), int(max_seqlen), states, None if view is None else view.slots)
+    n0 = -(-dim * vdim // 4) * 4
+    m0 = n0 + -(-dim // 4) * 4
+
+    def keep(slots, last):
+        for s, (S, n, m) in zip(slots.tolist(), last):
+            states[s, :, :dim * vdim], states[s, :, n0:n0 + dim], states[s, :, m0] = S.flatten(1), n, m
+    if step:
+        old = [(s[:, :dim * vdim].view(heads, dim, vdim), s[:, n0:n0 + dim], s[:, m0]) for s in states[view.slots.long()]]
+        o, last = ref.matrix_memory(*args, list(range(proj.shape[0] + 1)), old)
+        keep(view.slots, last)
+        return o
+    o, last = ref.matrix_memory(*args, cu_seqlens.tolist())
+    if states is not None:
+        keep(view.slots[cu_seqlens[:-1].long()], last)
+    return o
+
+
 # ------------------------------------------- rotated heads
 def rotary_table(positions, frequencies):
     """``(cos, sin)`` of position times frequency (fp64 ``[n]``) as one fp32 tensor ``[T, n, 2]``."""
@@ -462,13 +619,13 @@ def conv_heads(proj, weight, positions, hq: int, hkv: int, d: int, e: int, eps: 
     return q, (None if step else k), v
 
 
-def glu_columns(proj: torch.Tensor, gate: int, up: int, width: int, limit: float = 0.0) -> torch.Tensor:
-    """``act(proj[:, gate : gate+width], proj[:, up : up+width])`` without copying the column ranges: ``silu(g) · u``, or with a ``limit``
-    ``g σ(1.702 g) (u + 1)`` on ``g ≤ limit`` and ``|u| ≤ limit``."""
+def glu_columns(proj: torch.Tensor, gate: int, up: int, width: int, limit: float = 0.0, act: str = 'silu') -> torch.Tensor:
+    """``act(proj[:, gate : gate+width], proj[:, up : up+width])`` without copying the column ranges: ``silu(g) · u``, ``gelu_tanh(g) · u``, or with a
+    ``limit`` ``g σ(1.702 g) (u + 1)`` on ``g ≤ limit`` and ``|u| ≤ limit``."""
     if _cuda(proj) and not _needs_grad(proj):
-        return ext().glu_columns(proj, gate, up, width, limit)
+        return ext().glu_columns(proj, gate, up, width, limit, act == 'gelu_tanh')
     gu = torch.cat([proj[:, gate:gate + width], proj[:, up:up + width]], -1)
-    return ref.clamped_glu(gu, limit) if limit else ref.swiglu(gu)
+    return ref.geglu(gu) if act == 'gelu_tanh' else ref.clamped_glu(gu, limit) if limit else ref.swiglu(gu)
 
 
 def _tma_rows(t) -> bool:
@@ -476,20 +633,22 @@ def _tma_rows(t) -> bool:
     return t.stride(2) == 1 and t.stride(1) % 8 == 0 and t.stride(0) % 8 == 0 and t.data_ptr() % 16 == 0
 
 
-def attention_packed(q, k, v, cu_seqlens, max_seqlen: int, scale: float, sinks=None, gate=None, window: int = 0, chunk: int = 0, key_tail=None):
+def attention_packed(q, k, v, cu_seqlens, max_seqlen: int, scale: float, sinks=None, gate=None, window: int = 0, chunk: int = 0, key_tail=None,
+                     terms: Optional[ScoreTerms] = None):
     """Causal packed attention for any key / value widths up to 256: tensor-core kernel for bf16 heads (keys up to 192, values up to
     128 wide), an fp32-arithmetic kernel for wider heads and for 32-bit models.  ``sinks [Hq]``: a logit per head in the denominator;
-    ``gate [T, Hq]``: the output of a head is multiplied by its sigmoid.  A position sees its last ``window`` keys, or its own block of
-    ``chunk`` positions (0: no bound).  ``k`` and ``v`` may be column ranges of one tensor; ``key_tail [T, r]``: further key dimensions that all
-    heads share (queries are ``[… | r]`` wide)."""
-    if not _cuda(q) or _needs_grad(q, k, v, sinks, gate, key_tail):
+    ``gate``: the output is multiplied by its sigmoid, per head ``[T, Hq]`` or per element ``[T, Hq · e]``.  A position sees its last ``window`` keys,
+    or its own block of ``chunk`` positions (0: no bound).  ``k`` and ``v`` may be column ranges of one tensor; ``key_tail [T, r]``: further key
+    dimensions that all heads share (queries are ``[… | r]`` wide).  ``terms``: what else happens to scores."""
+    extra = terms.tensors if terms is not None else ()
+    if not _cuda(q) or _needs_grad(q, k, v, sinks, gate, key_tail, *extra):
         if key_tail is not None:
             k = torch.cat([k, key_tail[:, None].expand(-1, k.shape[1], -1)], -1)
-        if window or chunk:
-            o = ref.attention_varlen(q, k, v, cu_seqlens, True, scale, window=window or None, sinks=sinks, chunk=chunk)
+        if window or chunk or terms is not None:
+            o = ref.attention_varlen(q, k, v, cu_seqlens, True, scale, window=window or None, sinks=sinks, chunk=chunk, terms=terms)
         else:
             o = flash_attn_varlen(q, k, v, cu_seqlens, max_seqlen, True, scale, sinks=sinks)
-        return o if gate is None else (o.float() * torch.sigmoid(gate.float())[..., None]).to(o.dtype)
+        return _open_gate(o, gate)
     cu = cu_seqlens.to(torch.int32)
     if key_tail is not None:
         d, r = k.shape[2], key_tail.shape[1]
@@ -497,8 +656,8 @@ def attention_packed(q, k, v, cu_seqlens, max_seqlen: int, scale: float, sinks=N
             k, key_tail = torch.cat([k, key_tail[:, None].expand(-1, k.shape[1], -1)], -1), None
     if _flash_widths(q, k, v, 192):
         q, k, v = (t if _tma_rows(t) else t.contiguous() for t in (q, k, v))
-        return ext().flash_attn_fwd(q, k, v, cu, int(max_seqlen), True, scale, None, sinks, gate, window, chunk, key_tail)[0]
-    return ext().attention_packed(q.contiguous(), k.contiguous(), v.contiguous(), cu, int(max_seqlen), scale, sinks, gate, window, chunk)
+        return ext().flash_attn_fwd(q, k, v, cu, int(max_seqlen), True, scale, None, sinks, gate, window, chunk, key_tail, *_score_args(terms))[0]
+    return ext().attention_packed(q.contiguous(), k.contiguous(), v.contiguous(), cu, int(max_seqlen), scale, sinks, gate, window, chunk, *_score_args(terms))
 
 
 # ------------------------------------------------------------------ swiglu
@@ -643,16 +802,18 @@ def flash_attn_varlen(q, k, v, cu_seqlens, max_seqlen: int, causal: bool = True,
 
 
 def paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, scale: Optional[float] = None, window: Optional[int] = None,
-                           softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0, gate: Optional[torch.Tensor] = None):
+                           softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0, gate: Optional[torch.Tensor] = None,
+                           terms: Optional[ScoreTerms] = None):
     """One query token per sequence against the paged cache.  It sees its last ``window`` keys, or its own block of ``chunk`` positions;
-    ``sinks [Hq]``: a logit per head in the denominator; ``gate [B, Hq]``: the output of a head is multiplied by its sigmoid."""
+    ``sinks [Hq]``: a logit per head in the denominator; ``gate``: the output is multiplied by its sigmoid, per head ``[B, Hq]`` or per element ``[B,
+    Hq · e]``; ``softcap`` alone or all of ``terms``: what else happens to scores."""
     scale = 1.0 / math.sqrt(q.shape[-1]) if scale is None else scale
     vec = 16 // q.element_size()
-    if (_cuda(q) and not softcap and q.dtype in (torch.bfloat16, torch.float32) and all(t.shape[-1] % vec == 0 and t.shape[-1] <= 256 for t in (q, v_cache))
+    if (_cuda(q) and q.dtype in (torch.bfloat16, torch.float32) and all(t.shape[-1] % vec == 0 and t.shape[-1] <= 256 for t in (q, v_cache))
             and (sinks is None or sinks.dtype == q.dtype)):
-        return ext().paged_attn_decode(q.contiguous(), k_cache, v_cache, block_tables.to(torch.int32), seq_lens.to(torch.int32), scale, window or 0, chunk, sinks, gate)
-    o = ref.paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, scale, window, softcap, sinks, chunk)
-    return o if gate is None else (o.float() * torch.sigmoid(gate.float())[..., None]).to(o.dtype)
+        return ext().paged_attn_decode(q.contiguous(), k_cache, v_cache, block_tables.to(torch.int32), seq_lens.to(torch.int32), scale, window or 0, chunk, sinks, gate,
+                                       *_score_args(terms, softcap))
+    return _open_gate(ref.paged_attention_decode(q, k_cache, v_cache, block_tables, seq_lens, scale, window, softcap, sinks, chunk, terms), gate)
 
 
 # ------------------------------------------------------ gated delta net (linear attention)

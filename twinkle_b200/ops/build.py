@@ -27,7 +27,8 @@ _SO = os.path.join(_HERE, '_C.so')
 _STAMP = os.path.join(_HERE, '_C.stamp')
 _SERVING_SOURCES = ('bindings.cpp', 'host.cu', 'gemm.cu', 'gemm2.cu', 'attention_fwd.cu', 'attention_packed.cu', 'decode.cu', 'stream_ops.cu')
 # mechanism → its sources (``DecoderConfig.kernel_parts`` names those a model has)
-_PARTS = {'convolution': ('conv_heads.cu', ), 'experts': ('moe_serve.cu', ), 'latent': ('latent.cu', 'latent_decode.cu'), 'recurrent': ('hgrn2.cu', ), 'rotary': ('rotary.cu', )}
+_PARTS = {'convolution': ('conv_heads.cu', ), 'experts': ('moe_serve.cu', ), 'heads': ('heads.cu', ), 'latent': ('latent.cu', 'latent_decode.cu'), 'memory': ('mlstm.cu', ),
+          'recurrent': ('hgrn2.cu', ), 'rotary': ('rotary.cu', ), 'selective': ('selective.cu', )}
 _MOD = None
 _SERVING: Optional[Tuple[str, ...]] = None      # parts of the serving subset, when a process asked for it
 

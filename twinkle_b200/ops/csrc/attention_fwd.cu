@@ -1,7 +1,8 @@
 // Flash-attention forward for sm_100a: causal, GQA, packed variable-length sequences, query / key widths up to 192, value widths up to
 // 128.  A row narrower than its tile of 64-wide chunks is filled up with zeros by the TMA load (the tensor map ends at the row's width).
 // Optional: only the last `window` keys or the query's block of `chunk` positions (key blocks before them are not loaded), sink logits, a
-// gate per head, and a last chunk of key dimensions that all heads share (rotated part of latent attention), loaded from a tensor of
+// gate per head or element, score terms (TERMS: cap, factor per head, a number for the distance; the 255 distances of a tile are looked up or
+// formed once per tile, one per softmax thread), and a last chunk of key dimensions that all heads share (rotated part of latent attention), loaded from a tensor of
 // its own so that nothing has to put the keys together.
 //
 // One CTA per (128-row query tile of one sequence, query head).  192 threads:
@@ -18,6 +19,7 @@
 
 #include "common.cuh"
 #include "host.h"
+#include "scores.cuh"
 
 namespace tk {
 
@@ -33,7 +35,8 @@ struct Smem {
   static constexpr int K_TILE = KA > 2 ? 3 * ATOM_BYTES : TILE_BYTES, V_STAGES = KA > 2 ? 1 : 2;
   static constexpr int Q = 0, K = K_TILE, V = 3 * K_TILE, P = V + V_STAGES * TILE_BYTES, BAR = P + TILE_BYTES;
   static constexpr int XCHG = BAR + 256;            // row max (2 parities x 2 halves x 128) + row sums (2 x 128) floats
-  static constexpr int TOTAL = XCHG + 6 * 128 * 4 + 1024;
+  static constexpr int BAND = XCHG + 6 * 128 * 4;   // numbers of the tile's distances, two tiles
+  static constexpr int TOTAL = BAND + 2 * 256 * 4 + 1024;
 };
 constexpr int THREADS = 320;  // warps 0-7 softmax (two groups of 4: each owns 64 of the 128 S columns), 8 producer, 9 MMA
 constexpr float RESCALE_THRESHOLD = 8.f;  // log2 units
@@ -49,8 +52,9 @@ struct FwdParams {
   float scale_log2;   // softmax scale · log2(e)
   int causal;
   const bf16* sinks;  // [Hq] logit of a key without a value that every row sees (nullptr: none)
-  const bf16* gate;   // [T, Hq] with row stride ldg: the output is multiplied by its sigmoid (nullptr: not)
-  long ldg;
+  OutGate gate;       // the output is multiplied by its sigmoid
+  bool gate_vec;      // gates per element on 16-byte boundaries
+  ScoreTerms terms;
   int window, chunk;  // what a query sees of the keys before it (0: no bound)
   int own_chunks;     // leading chunks of a key that are its head's own; the rest come from the shared tensor
   int tail_col;       // first column of a query row that meets the shared part
@@ -58,7 +62,7 @@ struct FwdParams {
 };
 
 // KA / VA: 64-wide chunks of a query / key row (up to 3) and of a value row (1 or 2).
-template <int KA, int VA>
+template <int KA, int VA, bool TERMS>
 __global__ void __launch_bounds__(fa::THREADS, 1)
 flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                  const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmR, const FwdParams p) {
@@ -209,6 +213,18 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const int first_last = bounded ? first_visible(max(q0 + BQ - 1 + q_off, 0), p.window, p.chunk) : 0;
     float m_used = -INFINITY, l_sum = 0.f;
     bool dead = false;
+    // TERMS: band[j & 1][i] is the number for distance i − 127 between the tile's first query and key, in log2 units
+    float* band = reinterpret_cast<float*>(smem + S::BAND);
+    const DistanceNumber<bf16> number(p.terms, TERMS ? head : 0);
+    const float score_scale = TERMS ? p.scale_log2 * 0.6931471805599453f * score_temp<bf16>(p.terms, head) : p.scale_log2;
+    auto fill_band = [&](int j) {
+      const int i = wg * 128 + row;
+      band[(j & 1) * 256 + i] = number.at(max(q0 + q_off - (jb0 + j) * BKV + i - 127, 0)) * 1.4426950408889634f;
+    };
+    if constexpr (TERMS) {
+      fill_band(0);
+      asm volatile("bar.sync 1, 256;" ::: "memory");
+    }
     for (int j = 0; j < n_blocks; ++j) {
       if (!dead && !mbar_wait(&s_full[j & 1], (j >> 1) & 1, p.err, ERR_ATTN_WAIT)) dead = true;
       const int kv0 = (jb0 + j) * BKV + wg * 64;
@@ -224,9 +240,33 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
         tc_fence_before();
         mbar_arrive(&s_empty[j & 1]);                 // scores are in registers: the TMEM buffer may be refilled
         const bool need_mask = (kv0 + 64 > kv_end) || (p.causal && kv0 + 64 > q0 + q_off) || kv0 < first_last;
+        if constexpr (TERMS) {
+          if (p.terms.cap > 0.f) {
+            const float to_u = score_scale * p.terms.inv_cap, cap_log2 = p.terms.cap * 1.4426950408889634f;
+            float top = 0.f;
+#pragma unroll
+            for (int i = 0; i < 64; ++i) {
+              sc[i] = __uint_as_float(i < 32 ? r0[i] : r1[i - 32]) * to_u;
+              top = fmaxf(top, fabsf(sc[i]));
+            }
+            if (__any_sync(0xffffffffu, !(top <= kTanhNear))) {
+#pragma unroll
+              for (int i = 0; i < 64; ++i) sc[i] = cap_log2 * tanh_any(sc[i]);
+            } else {           // the usual case: scores well inside the cap
+#pragma unroll
+              for (int i = 0; i < 64; ++i) sc[i] = cap_log2 * tanh_near(sc[i]);
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < 64; ++i) sc[i] = __uint_as_float(i < 32 ? r0[i] : r1[i - 32]) * (score_scale * 1.4426950408889634f);
+          }
+          const float* mine = band + (j & 1) * 256 + row + 127 - wg * 64;
+#pragma unroll
+          for (int i = 0; i < 64; ++i) sc[i] += mine[-i];
+        }
 #pragma unroll
         for (int i = 0; i < 64; ++i) {
-          float sv = __uint_as_float(i < 32 ? r0[i] : r1[i - 32]) * p.scale_log2;
+          float sv = TERMS ? sc[i] : __uint_as_float(i < 32 ? r0[i] : r1[i - 32]) * p.scale_log2;
           if (need_mask) {
             const int col = kv0 + i;
             if (col >= kv_end || col < first || (p.causal && col > q_pos + q_off)) sv = -INFINITY;
@@ -235,6 +275,7 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
           mx = fmaxf(mx, sv);
         }
       }
+      if constexpr (TERMS) fill_band(j + 1);
       xmax[((j & 1) * 2 + wg) * 128 + row] = mx;
       asm volatile("bar.sync 1, 256;" ::: "memory");
       mx = fmaxf(mx, xmax[((j & 1) * 2 + (wg ^ 1)) * 128 + row]);
@@ -290,7 +331,9 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       if (p.sinks != nullptr) l_sum += exp2f(__bfloat162float(p.sinks[head]) * 1.4426950408889634f - m_used);
       float inv_l = (l_sum > 0.f) ? 1.f / l_sum : 0.f;
       const bool valid = q_pos < seq_len;
-      if (p.gate != nullptr && valid) inv_l /= 1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(seq_start + q_pos) * p.ldg + head]));
+      const bf16* gate = p.gate.p != nullptr && valid ? reinterpret_cast<const bf16*>(p.gate.p) + static_cast<size_t>(seq_start + q_pos) * p.gate.ld + static_cast<size_t>(head) * max(p.gate.e, 1)
+                                                      : nullptr;
+      if (gate != nullptr && p.gate.e == 0) inv_l *= sigmoid_of(__bfloat162float(*gate));
       bf16* orow = p.out + (static_cast<size_t>(seq_start + q_pos) * p.hq + head) * p.e;
 #pragma unroll 1
       for (int c = 2 * wg; c < 2 * wg + 2 && c * 32 < p.e; ++c) {
@@ -301,6 +344,22 @@ flash_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
 #pragma unroll
           for (int i = 0; i < 32; i += 8) {
             if (VA == 1 || c >= 2) { if (c * 32 + i >= p.e) break; }
+            if (gate != nullptr && p.gate.e > 0) {
+              if (p.gate_vec) {
+                const uint4 g = *reinterpret_cast<const uint4*>(gate + c * 32 + i);
+                const uint32_t gw[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+                for (int x = 0; x < 4; ++x) {
+                  const float2 z = unpack_bf16(gw[x]);
+                  r[i + 2 * x] = __float_as_uint(__uint_as_float(r[i + 2 * x]) * sigmoid_of(z.x));
+                  r[i + 2 * x + 1] = __float_as_uint(__uint_as_float(r[i + 2 * x + 1]) * sigmoid_of(z.y));
+                }
+              } else {
+#pragma unroll
+                for (int x = 0; x < 8; ++x)
+                  if (c * 32 + i + x < p.gate.e) r[i + x] = __float_as_uint(__uint_as_float(r[i + x]) * sigmoid_of(__bfloat162float(gate[c * 32 + i + x])));
+              }
+            }
             uint4 v = make_uint4(pack_bf16(__uint_as_float(r[i]) * inv_l, __uint_as_float(r[i + 1]) * inv_l),
                                  pack_bf16(__uint_as_float(r[i + 2]) * inv_l, __uint_as_float(r[i + 3]) * inv_l),
                                  pack_bf16(__uint_as_float(r[i + 4]) * inv_l, __uint_as_float(r[i + 5]) * inv_l),
@@ -328,7 +387,7 @@ CUtensorMap make_head_tmap(const torch::Tensor& t, int rows) {
 std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor& q, const torch::Tensor& k, const torch::Tensor& v, const torch::Tensor& cu,
                                           int64_t max_seqlen, bool causal, double scale, const c10::optional<torch::Tensor>& cu_k,
                                           const c10::optional<torch::Tensor>& sinks, const c10::optional<torch::Tensor>& gate, int64_t window, int64_t chunk,
-                                          const c10::optional<torch::Tensor>& key_tail) {
+                                          const c10::optional<torch::Tensor>& key_tail, double cap, const c10::optional<torch::Tensor>& temp, const c10::optional<torch::Tensor>& slope, const c10::optional<torch::Tensor>& rate, const c10::optional<torch::Tensor>& table, const c10::optional<torch::Tensor>& bucket) {
   TORCH_CHECK(q.is_cuda() && q.scalar_type() == torch::kBFloat16 && q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && k.size(0) == v.size(0) && k.size(1) == v.size(1) &&
                   k.scalar_type() == torch::kBFloat16 && v.scalar_type() == torch::kBFloat16, "q [T,Hq,D], k [T,Hkv,D], v [T,Hkv,E] bf16");
   for (const auto* t : {&q, &k, &v})
@@ -364,22 +423,22 @@ std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor& q, const torch::T
     TORCH_CHECK(sinks->is_cuda() && sinks->scalar_type() == torch::kBFloat16 && sinks->is_contiguous() && sinks->numel() == hq, "sinks [Hq] bf16");
     p.sinks = reinterpret_cast<const bf16*>(sinks->data_ptr());
   }
-  if (gate.has_value() && gate->defined()) {
-    TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == torch::kBFloat16 && gate->dim() == 2 && gate->size(0) == T && gate->size(1) == hq && gate->stride(1) == 1, "gate [T, Hq] bf16");
-    p.gate = reinterpret_cast<const bf16*>(gate->data_ptr()); p.ldg = gate->stride(0);
-  }
+  p.gate = out_gate(gate, T, hq, v.size(2), torch::kBFloat16);
+  p.gate_vec = p.gate.e == v.size(2) && p.gate.ld % 8 == 0 && reinterpret_cast<uintptr_t>(p.gate.p) % 16 == 0;
+  p.terms = score_terms(cap, temp, slope, rate, table, bucket, hq, torch::kBFloat16);
   p.T = T; p.hq = hq; p.hkv = hkv; p.scale_log2 = static_cast<float>(scale * 1.4426950408889634); p.causal = causal; p.err = error_word();
   p.window = window; p.chunk = chunk; p.own_chunks = own_chunks; p.tail_col = k.size(2);
   const dim3 grid(hq, (static_cast<int>(max_seqlen) + fa::BQ - 1) / fa::BQ, nseq);
   auto stream = at::cuda::getCurrentCUDAStream();
-#define TK_FLASH(KA, VA)                                                                                                                \
+#define TK_FLASH(KA, VA) do { if (p.terms.used) TK_FLASH_RUN(KA, VA, true); else TK_FLASH_RUN(KA, VA, false); } while (0)
+#define TK_FLASH_RUN(KA, VA, TERMS)                                                                                                     \
   do {                                                                                                                                  \
     static bool configured = false;                                                                                                     \
     if (!configured) {                                                                                                                  \
-      TK_CUDA_CHECK(cudaFuncSetAttribute(flash_fwd_kernel<KA, VA>, cudaFuncAttributeMaxDynamicSharedMemorySize, fa::Smem<KA>::TOTAL));  \
+      TK_CUDA_CHECK(cudaFuncSetAttribute(flash_fwd_kernel<KA, VA, TERMS>, cudaFuncAttributeMaxDynamicSharedMemorySize, fa::Smem<KA>::TOTAL));  \
       configured = true;                                                                                                                \
     }                                                                                                                                   \
-    flash_fwd_kernel<KA, VA><<<grid, fa::THREADS, fa::Smem<KA>::TOTAL, stream>>>(tq, tk_, tv, tr, p);                                   \
+    flash_fwd_kernel<KA, VA, TERMS><<<grid, fa::THREADS, fa::Smem<KA>::TOTAL, stream>>>(tq, tk_, tv, tr, p);                                   \
   } while (0)
   const bool wide_k = chunks > 1, wide_v = v.size(2) > 64;
   if (chunks == 3 && wide_v) TK_FLASH(3, 2);
@@ -389,6 +448,7 @@ std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor& q, const torch::T
   else if (wide_v) TK_FLASH(1, 2);
   else TK_FLASH(1, 1);
 #undef TK_FLASH
+#undef TK_FLASH_RUN
   count_launch();
   TK_CUDA_CHECK(cudaGetLastError());
   return {out, lse};

@@ -9,6 +9,7 @@
 
 #include "common.cuh"
 #include "host.h"
+#include "scores.cuh"
 
 namespace tk {
 
@@ -25,7 +26,7 @@ __device__ __forceinline__ void st(bf16* p, float v) { *p = __float2bfloat16(v);
 template <typename T, int EI>
 __global__ void __launch_bounds__(256) attention_packed_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, T* __restrict__ out,
                                                                const int* __restrict__ cu, int hq, int hkv, int D, int E, float scale_log2,
-                                                               const T* __restrict__ sinks, const T* __restrict__ gate, long ldg, int window, int chunk) {
+                                                               const T* __restrict__ sinks, const OutGate gate, int window, int chunk, const ScoreTerms terms) {
   using namespace pa;
   extern __shared__ float sm[];
   const int head = blockIdx.x, seq = blockIdx.z, kvh = head / (hq / hkv);
@@ -39,9 +40,11 @@ __global__ void __launch_bounds__(256) attention_packed_kernel(const T* __restri
   float* sv = sk + BK * ds;
   float* sp = sv + BK * E;
   const int row = threadIdx.x >> 3, sub = threadIdx.x & 7;
+  const DistanceNumber<T> number(terms, head);
+  const float q_scale = terms.used ? scale_log2 * 0.6931471805599453f * score_temp<T>(terms, head) : scale_log2;
   for (int i = threadIdx.x; i < BQ * D; i += blockDim.x) {
     const int r = i / D, c = i - r * D;
-    sq[r * ds + c] = q0 + r < len ? ld(q + (static_cast<size_t>(start + q0 + r) * hq + head) * D + c) * scale_log2 : 0.f;
+    sq[r * ds + c] = q0 + r < len ? ld(q + (static_cast<size_t>(start + q0 + r) * hq + head) * D + c) * q_scale : 0.f;
   }
   float acc[EI];
 #pragma unroll
@@ -64,6 +67,13 @@ __global__ void __launch_bounds__(256) attention_packed_kernel(const T* __restri
       const float a = sq[row * ds + c];
 #pragma unroll
       for (int i = 0; i < 4; ++i) s[i] += a * sk[(sub + 8 * i) * ds + c];
+    }
+    if (terms.used) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        if (terms.cap > 0.f) s[i] = terms.cap * tanh_any(s[i] * terms.inv_cap);
+        s[i] = (s[i] + number.at(max(q0 + row - k0 - sub - 8 * i, 0))) * 1.4426950408889634f;
+      }
     }
     float mx = m;
 #pragma unroll
@@ -100,15 +110,19 @@ __global__ void __launch_bounds__(256) attention_packed_kernel(const T* __restri
     T* o = out + (static_cast<size_t>(start + q0 + row) * hq + head) * E;
     if (sinks != nullptr) l += exp2f(ld(sinks + head) * 1.4426950408889634f - m);      // a key without a value that every row sees
     float f = 1.f / l;
-    if (gate != nullptr) f /= 1.f + __expf(-ld(gate + static_cast<size_t>(start + q0 + row) * ldg + head));
+    const T* g = gate.p != nullptr ? reinterpret_cast<const T*>(gate.p) + static_cast<size_t>(start + q0 + row) * gate.ld + static_cast<size_t>(head) * max(gate.e, 1) : nullptr;
+    if (g != nullptr && gate.e == 0) f *= sigmoid_of(ld(g));
 #pragma unroll
-    for (int i = 0; i < EI; ++i)
-      if (sub + 8 * i < E) st(o + sub + 8 * i, acc[i] * f);
+    for (int i = 0; i < EI; ++i) {
+      const int c = sub + 8 * i;
+      if (c < E) st(o + c, acc[i] * f * (g != nullptr && c < gate.e ? sigmoid_of(ld(g + c)) : 1.f));
+    }
   }
 }
 
 torch::Tensor attention_packed(const torch::Tensor& q, const torch::Tensor& k, const torch::Tensor& v, const torch::Tensor& cu, int64_t max_seqlen, double scale,
-                               const c10::optional<torch::Tensor>& sinks, const c10::optional<torch::Tensor>& gate, int64_t window, int64_t chunk) {
+                               const c10::optional<torch::Tensor>& sinks, const c10::optional<torch::Tensor>& gate, int64_t window, int64_t chunk,
+                               double cap, const c10::optional<torch::Tensor>& temp, const c10::optional<torch::Tensor>& slope, const c10::optional<torch::Tensor>& rate, const c10::optional<torch::Tensor>& table, const c10::optional<torch::Tensor>& bucket) {
   const auto st = q.scalar_type();
   TORCH_CHECK(q.is_cuda() && (st == torch::kBFloat16 || st == torch::kFloat32) && k.scalar_type() == st && v.scalar_type() == st, "q, k, v bf16 or fp32");
   TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && q.is_contiguous() && k.is_contiguous() && v.is_contiguous(), "[T, H, D] contiguous");
@@ -116,9 +130,10 @@ torch::Tensor attention_packed(const torch::Tensor& q, const torch::Tensor& k, c
   TORCH_CHECK(q.size(2) <= 256 && v.size(2) <= 256, "head widths up to 256");
   TORCH_CHECK(window >= 0 && chunk >= 0 && window < (int64_t(1) << 30) && chunk < (int64_t(1) << 30), "window and chunk: 0 (none) or positive");
   TORCH_CHECK(cu.is_cuda() && cu.scalar_type() == torch::kInt32 && cu.is_contiguous(), "cu_seqlens int32 on device");
-  const bool has_sinks = sinks.has_value() && sinks->defined(), has_gate = gate.has_value() && gate->defined();
+  const bool has_sinks = sinks.has_value() && sinks->defined();
   if (has_sinks) TORCH_CHECK(sinks->is_cuda() && sinks->scalar_type() == st && sinks->is_contiguous() && sinks->numel() == q.size(1), "sinks [Hq]");
-  if (has_gate) TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == st && gate->dim() == 2 && gate->size(0) == q.size(0) && gate->size(1) == q.size(1) && gate->stride(1) == 1, "gate [T, Hq]");
+  const OutGate g = out_gate(gate, q.size(0), q.size(1), v.size(2), st);
+  const ScoreTerms terms = score_terms(cap, temp, slope, rate, table, bucket, q.size(1), st);
   c10::cuda::CUDAGuard guard(q.device());
   const int hq = q.size(1), hkv = k.size(1), D = q.size(2), E = v.size(2), nseq = cu.numel() - 1;
   auto out = torch::empty({q.size(0), hq, E}, q.options());
@@ -131,8 +146,8 @@ torch::Tensor attention_packed(const torch::Tensor& q, const torch::Tensor& k, c
     TK_CUDA_CHECK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)));
     kern<<<grid, 256, smem, stream>>>(reinterpret_cast<const T*>(q.data_ptr()), reinterpret_cast<const T*>(k.data_ptr()), reinterpret_cast<const T*>(v.data_ptr()),
                                       reinterpret_cast<T*>(out.data_ptr()), cu.data_ptr<int>(), hq, hkv, D, E, static_cast<float>(scale * 1.4426950408889634),
-                                      has_sinks ? reinterpret_cast<const T*>(sinks->data_ptr()) : nullptr, has_gate ? reinterpret_cast<const T*>(gate->data_ptr()) : nullptr,
-                                      has_gate ? gate->stride(0) : 0L, static_cast<int>(window), static_cast<int>(chunk));
+                                      has_sinks ? reinterpret_cast<const T*>(sinks->data_ptr()) : nullptr, g, static_cast<int>(window),
+                                      static_cast<int>(chunk), terms);
   };
   if (st == torch::kBFloat16) {
     if (E <= 64) go(attention_packed_kernel<bf16, 8>, bf16{});

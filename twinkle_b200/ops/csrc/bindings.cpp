@@ -10,11 +10,11 @@ torch::Tensor gemm(const torch::Tensor&, const torch::Tensor&, const std::string
                    c10::optional<torch::ScalarType>);
 std::vector<torch::Tensor> flash_attn_fwd(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t,
                                           bool, double, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&,
-                                          const c10::optional<torch::Tensor>&, int64_t, int64_t, const c10::optional<torch::Tensor>&);
+                                          const c10::optional<torch::Tensor>&, int64_t, int64_t, const c10::optional<torch::Tensor>&, double, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
 torch::Tensor attention_packed(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t, double,
-                               const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, int64_t, int64_t);
+                               const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, int64_t, int64_t, double, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
 torch::Tensor paged_attn_decode(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, double, int64_t, int64_t,
-                                const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
+                                const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, double, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
 std::vector<torch::Tensor> sample_tokens(const torch::Tensor&, double, int64_t, double, const torch::Tensor&);
 std::vector<torch::Tensor> conv_heads(const torch::Tensor&, const c10::optional<torch::Tensor>&, const torch::Tensor&, int64_t, int64_t, int64_t, int64_t,
                                       double, double, int64_t, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, bool,
@@ -49,7 +49,22 @@ torch::Tensor head_gemm(const torch::Tensor&, const torch::Tensor&, bool, const 
 torch::Tensor grouped_gemm(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const std::string&, const c10::optional<torch::Tensor>&,
                            const c10::optional<torch::Tensor>&, bool, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&,
                            const c10::optional<std::string>&);
-torch::Tensor glu_columns(const torch::Tensor&, int64_t, int64_t, int64_t, double);
+torch::Tensor glu_columns(const torch::Tensor&, int64_t, int64_t, int64_t, double, bool);
+torch::Tensor stream_normed(torch::Tensor, const c10::optional<torch::Tensor>&, double, const torch::Tensor&, const c10::optional<torch::Tensor>&, const torch::Tensor&, const c10::optional<torch::Tensor>&,
+                            const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
+torch::Tensor embed_positions(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&);
+std::vector<torch::Tensor> plain_heads(const torch::Tensor&, int64_t, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, bool, bool, int64_t,
+                                       int64_t, int64_t, int64_t, double, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&, bool);
+torch::Tensor conv_silu(const torch::Tensor&, int64_t, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, bool, const c10::optional<torch::Tensor>&,
+                        const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
+torch::Tensor selective_prefill(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t, int64_t, const torch::Tensor&,
+                                const torch::Tensor&, int64_t, const torch::Tensor&, int64_t, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
+torch::Tensor selective_step(const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, const torch::Tensor&, int64_t, int64_t, const torch::Tensor&,
+                             const torch::Tensor&, int64_t, const torch::Tensor&, const torch::Tensor&);
+torch::Tensor mlstm_prefill(const torch::Tensor&, int64_t, int64_t, int64_t, int64_t, const torch::Tensor&, const torch::Tensor&, double, const torch::Tensor&, double,
+                            const torch::Tensor&, int64_t, const c10::optional<torch::Tensor>&, const c10::optional<torch::Tensor>&);
+torch::Tensor mlstm_step(const torch::Tensor&, int64_t, int64_t, int64_t, int64_t, const torch::Tensor&, const torch::Tensor&, double, const torch::Tensor&, double,
+                         const torch::Tensor&, const torch::Tensor&);
 void set_gemm_pair(int64_t);
 void set_gemm_staged(int64_t);
 #ifndef TK_SERVING_ONLY
@@ -108,9 +123,11 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("accumulate") = false, py::arg("out_dtype") = py::none());
   m.def("flash_attn_fwd", &tk::flash_attn_fwd, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("cu"), py::arg("max_seqlen"), py::arg("causal"),
         py::arg("scale"), py::arg("cu_k") = py::none(), py::arg("sinks") = py::none(), py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("chunk") = 0,
-        py::arg("key_tail") = py::none());
+        py::arg("key_tail") = py::none(), py::arg("cap") = 0.0, py::arg("temp") = py::none(), py::arg("slope") = py::none(),
+        py::arg("rate") = py::none(), py::arg("table") = py::none(), py::arg("bucket") = py::none());
   m.def("paged_attn_decode", &tk::paged_attn_decode, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("tables"), py::arg("seq_lens"), py::arg("scale"),
-        py::arg("window") = 0, py::arg("chunk") = 0, py::arg("sinks") = py::none(), py::arg("gate") = py::none());
+        py::arg("window") = 0, py::arg("chunk") = 0, py::arg("sinks") = py::none(), py::arg("gate") = py::none(), py::arg("cap") = 0.0, py::arg("temp") = py::none(), py::arg("slope") = py::none(),
+        py::arg("rate") = py::none(), py::arg("table") = py::none(), py::arg("bucket") = py::none());
   m.def("sample_tokens", &tk::sample_tokens);
   m.def("set_gemm_pair", &tk::set_gemm_pair);
   m.def("set_gemm_staged", &tk::set_gemm_staged);
@@ -118,12 +135,25 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("num_sms", &tk::num_sms);
   m.def("launch_count", &tk::launch_count, "Number of kernels launched by this extension so far.");
   m.def("attention_packed", &tk::attention_packed, py::arg("q"), py::arg("k"), py::arg("v"), py::arg("cu"), py::arg("max_seqlen"), py::arg("scale"),
-        py::arg("sinks") = py::none(), py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("chunk") = 0);
+        py::arg("sinks") = py::none(), py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("chunk") = 0, py::arg("cap") = 0.0, py::arg("temp") = py::none(), py::arg("slope") = py::none(),
+        py::arg("rate") = py::none(), py::arg("table") = py::none(), py::arg("bucket") = py::none());
 #ifdef TK_WITH_CONVOLUTION
   m.def("conv_heads", &tk::conv_heads, py::arg("proj"), py::arg("weight"), py::arg("pos"), py::arg("hq"), py::arg("hkv"), py::arg("d"), py::arg("e"), py::arg("eps"),
         py::arg("coef") = 0.0, py::arg("every") = 0, py::arg("v_first") = py::none(), py::arg("lam") = py::none(), py::arg("step") = false,
         py::arg("hist") = py::none(), py::arg("slot") = py::none(), py::arg("left") = py::none(), py::arg("pool_row") = py::none(),
         py::arg("k_pool") = py::none(), py::arg("v_pool") = py::none(), py::arg("want_k") = true);
+#endif
+#ifdef TK_WITH_HEADS
+  m.def("plain_heads", &tk::plain_heads);
+#endif
+#ifdef TK_WITH_SELECTIVE
+  m.def("conv_silu", &tk::conv_silu);
+  m.def("selective_prefill", &tk::selective_prefill);
+  m.def("selective_step", &tk::selective_step);
+#endif
+#ifdef TK_WITH_MEMORY
+  m.def("mlstm_prefill", &tk::mlstm_prefill);
+  m.def("mlstm_step", &tk::mlstm_step);
 #endif
 #ifdef TK_WITH_ROTARY
   m.def("rotary_table", &tk::rotary_table);
@@ -133,6 +163,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("stream_rmsnorm", &tk::stream_rmsnorm, py::arg("x"), py::arg("w"), py::arg("eps"), py::arg("y1") = py::none(), py::arg("s1") = py::none(),
         py::arg("y2") = py::none(), py::arg("s2") = py::none(), py::arg("mult") = 1.0, py::arg("offset") = 0.0);
   m.def("stream_gated_rmsnorm", &tk::stream_gated_rmsnorm);
+  m.def("stream_normed", &tk::stream_normed);
+  m.def("embed_positions", &tk::embed_positions);
   m.def("stream_joined_rmsnorm", &tk::stream_joined_rmsnorm, py::arg("x"), py::arg("w"), py::arg("eps"), py::arg("offset"), py::arg("y"), py::arg("row_of") = py::none(),
         py::arg("share") = py::none(), py::arg("beside") = py::none(), py::arg("open") = py::none());
 #ifdef TK_WITH_LATENT
@@ -153,7 +185,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("head_gemm", &tk::head_gemm, py::arg("x"), py::arg("w"), py::arg("nn"), py::arg("out") = py::none());
   m.def("grouped_gemm", &tk::grouped_gemm, py::arg("x"), py::arg("w"), py::arg("offsets"), py::arg("layout") = "nt", py::arg("group_map") = py::none(),
         py::arg("out") = py::none(), py::arg("accumulate") = false, py::arg("x2") = py::none(), py::arg("w2") = py::none(), py::arg("act") = py::none());
-  m.def("glu_columns", &tk::glu_columns, py::arg("p"), py::arg("gate"), py::arg("up"), py::arg("width"), py::arg("limit") = 0.0);
+  m.def("glu_columns", &tk::glu_columns, py::arg("p"), py::arg("gate"), py::arg("up"), py::arg("width"), py::arg("limit") = 0.0, py::arg("gelu") = false);
 #ifndef TK_SERVING_ONLY
   m.def("grouped_gemm_wgrad", &tk::grouped_gemm_wgrad);
   m.def("rmsnorm_fwd", &tk::rmsnorm_fwd, py::arg("x"), py::arg("w"), py::arg("eps"), py::arg("offset"), py::arg("residual") = py::none());

@@ -8,6 +8,7 @@
 
 #include "common.cuh"
 #include "host.h"
+#include "scores.cuh"
 
 namespace tk {
 
@@ -19,11 +20,12 @@ using bf16 = __nv_bfloat16;
 // of up to 256 bytes: 32 token rows per CTA in flight).  Every lane group keeps an online-softmax state per query head;
 // lane groups and warps are merged at the end.  Key and value rows are `d` and `e` elements wide, whole 16-byte vectors.
 // Optional: only the last `window` keys or the query's block of `chunk` positions, a sink logit per head in the denominator, a
-// sigmoid gate per head on the result.
+// sigmoid gate per head or element on the result; TERMS: scores go through ScoreTerms, the lanes of a group taking a head each.
 struct PagedExtras {
-  const void *sinks, *gate;   // [hq], [B, hq] with row stride ldg (nullptr: none)
-  long ldg;
+  const void* sinks;          // [hq] (nullptr: none)
+  OutGate gate;
   int window, chunk;
+  ScoreTerms terms;
 };
 __device__ __forceinline__ void unpack_vec(const uint4& u, float (&x)[8], const bf16*) {
   const uint32_t w[4] = {u.x, u.y, u.z, u.w};
@@ -41,7 +43,7 @@ __device__ __forceinline__ float to_float(float v) { return v; }
 __device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v); }
 __device__ __forceinline__ void put(float* p, float v) { *p = v; }
 
-template <typename T, int GH, int NC, int U>
+template <typename T, int GH, int NC, int U, bool TERMS>
 __global__ void __launch_bounds__(128) paged_decode_kernel(const T* __restrict__ q, const T* __restrict__ kc, const T* __restrict__ vc,
                                                             const int* __restrict__ tables, const int* __restrict__ seq_lens, T* __restrict__ out,
                                                             int hq, int hkv, int d, int e, int block_size, int max_blocks, float scale_log2, int G, const PagedExtras x) {
@@ -53,8 +55,11 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const T* __restrict__
   __shared__ __align__(16) float s_q[GH][D];
   for (int i = threadIdx.x; i < GH * D; i += blockDim.x) {
     const int g = i / D, c = i % D;
-    s_q[g][c] = (g0 + g < G && c < d) ? to_float(q[(static_cast<size_t>(b) * hq + h0 + g) * d + c]) * scale_log2 : 0.f;
+    float scale = scale_log2;
+    if constexpr (TERMS) scale *= 0.6931471805599453f * score_temp<T>(x.terms, min(h0 + g, hq - 1));
+    s_q[g][c] = (g0 + g < G && c < d) ? to_float(q[(static_cast<size_t>(b) * hq + h0 + g) * d + c]) * scale : 0.f;
   }
+  const DistanceNumber<T> number(x.terms, TERMS ? min(h0 + sub % GH, hq - 1) : 0);
   __syncthreads();
   float m[GH], l[GH], acc[GH][NC * V];
 #pragma unroll
@@ -96,6 +101,7 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const T* __restrict__
         unpack_vec(kr[u][c], kf[c], kc);
         unpack_vec(vr[u][c], vf[c], vc);
       }
+      float sc[GH];
 #pragma unroll
       for (int g = 0; g < GH; ++g) {
         float s = 0.f;
@@ -112,6 +118,20 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const T* __restrict__
         s += __shfl_xor_sync(0xffffffffu, s, 1);
         s += __shfl_xor_sync(0xffffffffu, s, 2);
         s += __shfl_xor_sync(0xffffffffu, s, 4);
+        sc[g] = s;
+      }
+      if constexpr (TERMS) {   // lane `sub` of a group finishes the score of head sub % GH
+        float mine = sc[0];
+#pragma unroll
+        for (int g = 1; g < GH; ++g) mine = sub % GH == g ? sc[g] : mine;
+        if (x.terms.cap > 0.f) mine = x.terms.cap * tanh_any(mine * x.terms.inv_cap);
+        mine = (mine + number.at(max(n - 1 - (base + grp + u * 16), 0))) * 1.4426950408889634f;
+#pragma unroll
+        for (int g = 0; g < GH; ++g) sc[g] = GH == 1 ? mine : __shfl_sync(0xffffffffu, mine, (lane & 24) + g);
+      }
+#pragma unroll
+      for (int g = 0; g < GH; ++g) {
+        const float s = sc[g];
         if (live) {  // uniform inside an 8-lane group
           const float mn = fmaxf(m[g], s);
           const float corr = exp2f(m[g] - mn), p = exp2f(s - mn);
@@ -169,13 +189,14 @@ __global__ void __launch_bounds__(128) paged_decode_kernel(const T* __restrict__
         ll += s_l[w][g] * c;
         o += s_acc[w][g][i] * c;
       }
-      if (x.gate != nullptr) ll *= 1.f + __expf(-to_float(reinterpret_cast<const T*>(x.gate)[b * x.ldg + h0 + g]));
+      if (x.gate.p != nullptr && i < max(x.gate.e, e * (x.gate.e == 0)))
+        o *= sigmoid_of(to_float(reinterpret_cast<const T*>(x.gate.p)[b * x.gate.ld + (x.gate.e == 0 ? h0 + g : (h0 + g) * x.gate.e + i)]));
       put(out + (static_cast<size_t>(b) * hq + h0 + g) * e + i, ll > 0.f ? o / ll : 0.f);
     }
   }
 }
 
-template <typename T>
+template <typename T, bool TERMS>
 static void launch_paged_decode(const torch::Tensor& q, const torch::Tensor& kc, const torch::Tensor& vc, const torch::Tensor& tables,
                                 const torch::Tensor& seq_lens, torch::Tensor& out, float sl2, const PagedExtras& extras, cudaStream_t stream) {
   constexpr int V = 16 / sizeof(T);
@@ -188,19 +209,19 @@ static void launch_paged_decode(const torch::Tensor& q, const torch::Tensor& kc,
   };
   const int vectors = (std::max(d, e) + 8 * V - 1) / (8 * V);   // per lane
   if (vectors <= 1) {
-    if (G == 1) go(paged_decode_kernel<T, 1, 1, 2>, 1); else if (G == 2) go(paged_decode_kernel<T, 2, 1, 2>, 2); else go(paged_decode_kernel<T, 4, 1, 2>, 4);
+    if (G == 1) go(paged_decode_kernel<T, 1, 1, 2, TERMS>, 1); else if (G == 2) go(paged_decode_kernel<T, 2, 1, 2, TERMS>, 2); else go(paged_decode_kernel<T, 4, 1, 2, TERMS>, 4);
   } else if (vectors <= 2) {
-    if (G == 1) go(paged_decode_kernel<T, 1, 2, 2>, 1); else if (G == 2) go(paged_decode_kernel<T, 2, 2, 2>, 2); else go(paged_decode_kernel<T, 4, 2, 2>, 4);
+    if (G == 1) go(paged_decode_kernel<T, 1, 2, 2, TERMS>, 1); else if (G == 2) go(paged_decode_kernel<T, 2, 2, 2, TERMS>, 2); else go(paged_decode_kernel<T, 4, 2, 2, TERMS>, 4);
   } else if (vectors <= 4) {
-    if (G == 1) go(paged_decode_kernel<T, 1, 4, 1>, 1); else go(paged_decode_kernel<T, 2, 4, 1>, 2);
+    if (G == 1) go(paged_decode_kernel<T, 1, 4, 1, TERMS>, 1); else go(paged_decode_kernel<T, 2, 4, 1, TERMS>, 2);
   } else if constexpr (sizeof(T) == 4) {   // 16-bit rows of up to 256 elements are four vectors per lane
-    go(paged_decode_kernel<T, 1, 8, 1>, 1);
+    go(paged_decode_kernel<T, 1, 8, 1, TERMS>, 1);
   }
 }
 
 torch::Tensor paged_attn_decode(const torch::Tensor& q, const torch::Tensor& kc, const torch::Tensor& vc, const torch::Tensor& tables,
                                 const torch::Tensor& seq_lens, double scale, int64_t window, int64_t chunk, const c10::optional<torch::Tensor>& sinks,
-                                const c10::optional<torch::Tensor>& gate) {
+                                const c10::optional<torch::Tensor>& gate, double cap, const c10::optional<torch::Tensor>& temp, const c10::optional<torch::Tensor>& slope, const c10::optional<torch::Tensor>& rate, const c10::optional<torch::Tensor>& table, const c10::optional<torch::Tensor>& bucket) {
   const auto st = q.scalar_type();
   TORCH_CHECK(q.is_cuda() && (st == torch::kBFloat16 || st == torch::kFloat32) && q.is_contiguous() && q.dim() == 3, "q [B,Hq,D] bf16 or fp32");
   TORCH_CHECK(kc.is_contiguous() && vc.is_contiguous() && kc.dim() == 4 && vc.dim() == 4 && kc.scalar_type() == st && vc.scalar_type() == st, "caches [blocks,bs,Hkv,·] in q's dtype");
@@ -215,17 +236,19 @@ torch::Tensor paged_attn_decode(const torch::Tensor& q, const torch::Tensor& kc,
     TORCH_CHECK(sinks->is_cuda() && sinks->scalar_type() == st && sinks->is_contiguous() && sinks->numel() == q.size(1), "sinks [Hq] in q's dtype");
     x.sinks = sinks->data_ptr();
   }
-  if (gate.has_value() && gate->defined()) {
-    TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == st && gate->dim() == 2 && gate->size(0) == q.size(0) && gate->size(1) == q.size(1) && gate->stride(1) == 1, "gate [B, Hq]");
-    x.gate = gate->data_ptr(); x.ldg = gate->stride(0);
-  }
+  x.gate = out_gate(gate, q.size(0), q.size(1), vc.size(3), st);
+  x.terms = score_terms(cap, temp, slope, rate, table, bucket, q.size(1), st);
   c10::cuda::CUDAGuard guard(q.device());
   auto out = torch::empty({q.size(0), q.size(1), vc.size(3)}, q.options());
   if (q.size(0) == 0) return out;
   const float sl2 = static_cast<float>(scale * 1.4426950408889634);
   auto stream = at::cuda::getCurrentCUDAStream();
-  if (st == torch::kBFloat16) launch_paged_decode<bf16>(q, kc, vc, tables, seq_lens, out, sl2, x, stream);
-  else launch_paged_decode<float>(q, kc, vc, tables, seq_lens, out, sl2, x, stream);
+  auto run = [&](auto tag, auto terms) { launch_paged_decode<decltype(tag), decltype(terms)::value>(q, kc, vc, tables, seq_lens, out, sl2, x, stream); };
+  if (st == torch::kBFloat16) {
+    if (x.terms.used) run(bf16{}, std::true_type{}); else run(bf16{}, std::false_type{});
+  } else {
+    if (x.terms.used) run(0.f, std::true_type{}); else run(0.f, std::false_type{});
+  }
   count_launch();
   TK_CUDA_CHECK(cudaGetLastError());
   return out;

@@ -1,0 +1,483 @@
+// Selective scan (Mamba) between its projections.
+//   conv_silu          causal depth-wise convolution, bias and silu on columns of a projection; the last inputs of a sequence stay in a ring
+//                      over positions, from which single steps take their past
+//   selective_prefill  packed prompts.  Per channel c and state n, in fp32:
+//                          δ = softplus(dt + b),  S ← e^{−δ e^{A}} S + δ u B,  y = (Σ_n S C + D u) silu(z)
+//                      LN neighbouring lanes share a channel, NS states each in registers; tokens pass through shared memory sixteen (with many states, eight) at a
+//                      time, the next ones on their way while these are worked on.  When sequences × channels do not fill the device,
+//                      sequences are cut into time segments: a first pass forms what each segment builds up from nothing and its sum of
+//                      steps (decays multiply, so the steps add up), and the second starts every segment from those before it.
+//   selective_step     one token of every sequence: the state passes once through the block, 16 bytes per access.
+#include <ATen/cuda/CUDAContext.h>
+#include <c10/cuda/CUDAGuard.h>
+#include <torch/types.h>
+
+#include "common.cuh"
+#include "host.h"
+#include "vec.cuh"
+
+namespace tk {
+
+// ------------------------------------------------------------------- conv_silu
+template <typename T>
+struct ConvSilu {
+  const T* x; long ld;
+  const T *w, *bias;                   // [C, taps], [C]
+  T* out;                              // [rows, C]
+  const int64_t* pos;
+  T* hist; const int *slot, *left;     // [slots, taps − 1, C] (null: not kept)
+  int C, taps, rows, tile;
+  bool step;
+};
+
+__device__ __forceinline__ float silu_of(float z) { return __fdividef(z, 1.f + __expf(-z)); }
+
+// A thread owns eight channels of `tile` consecutive rows and keeps the last TAPS − 1 inputs in registers.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) conv_silu_kernel(const ConvSilu<T> p) {
+  constexpr int N = TAPS > 1 ? TAPS - 1 : 1;      // rows of the ring
+  const int c = (blockIdx.x * 128 + threadIdx.x) * 8;
+  if (c >= p.C) return;
+  const int t0 = blockIdx.y * p.tile, t1 = min(p.rows, t0 + p.tile);
+  float w[TAPS][8], b[8], past[N][8];
+  Raw8<T> r;
+  r.load(p.bias + c);
+  r.get(b);
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+    for (int i = 0; i < 8; ++i) w[j][i] = to_f(p.w[static_cast<size_t>(c + i) * TAPS + j]);
+  auto load = [&](const T* src, float (&y)[8]) {
+    r.load(src);
+    r.get(y);
+  };
+  const int first = static_cast<int>(min(p.pos[t0], static_cast<int64_t>(TAPS)));      // inputs of the same sequence before the tile's first row
+#pragma unroll
+  for (int j = 1; j < TAPS; ++j) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) past[j - 1][i] = 0.f;
+    if (!p.step && j <= first) load(p.x + static_cast<size_t>(t0 - j) * p.ld + c, past[j - 1]);
+  }
+  for (int t = t0; t < t1; ++t) {
+    const int64_t pos = p.pos[t];
+    const int slot = p.hist != nullptr ? p.slot[t] : 0;
+    T* ring = p.hist != nullptr ? p.hist + static_cast<size_t>(slot) * (TAPS - 1) * p.C + c : nullptr;
+    float x[8], y[8];
+    load(p.x + static_cast<size_t>(t) * p.ld + c, x);
+    const Raw8<T> raw = r;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) y[i] = fmaf(w[TAPS - 1][i], x[i], b[i]);
+#pragma unroll
+    for (int j = 1; j < TAPS; ++j) {
+      if (pos < j) continue;
+      if (p.step) load(ring + static_cast<size_t>((pos - j) % N) * p.C, past[j - 1]);
+#pragma unroll
+      for (int i = 0; i < 8; ++i) y[i] = fmaf(w[TAPS - 1 - j][i], past[j - 1][i], y[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) y[i] = silu_of(y[i]);
+    r.set(y);
+    r.store(p.out + static_cast<size_t>(t) * p.C + c);
+    if constexpr (TAPS > 1) {
+      if (ring != nullptr && slot > 0 && p.left[t] < TAPS - 1) raw.store(ring + static_cast<size_t>(pos % N) * p.C);
+#pragma unroll
+      for (int j = TAPS - 2; j > 0; --j)
+#pragma unroll
+        for (int i = 0; i < 8; ++i) past[j][i] = past[j - 1][i];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) past[0][i] = x[i];
+    }
+  }
+}
+
+// Any sizes: one thread per element.
+template <typename T>
+__global__ void __launch_bounds__(256) conv_silu_any_kernel(const ConvSilu<T> p) {
+  const long i = blockIdx.x * 256L + threadIdx.x;
+  if (i >= static_cast<long>(p.rows) * p.C) return;
+  const int t = static_cast<int>(i / p.C), c = static_cast<int>(i - static_cast<long>(t) * p.C), n = p.taps - 1;
+  const int64_t pos = p.pos[t];
+  const int slot = p.hist != nullptr ? p.slot[t] : 0;
+  T* ring = p.hist != nullptr ? p.hist + static_cast<size_t>(slot) * n * p.C + c : nullptr;
+  const T own = p.x[static_cast<size_t>(t) * p.ld + c];
+  float y = to_f(p.bias[c]) + to_f(p.w[static_cast<size_t>(c) * p.taps + n]) * to_f(own);
+  for (int j = 1; j <= n && j <= pos; ++j)
+    y += to_f(p.w[static_cast<size_t>(c) * p.taps + n - j]) * to_f(p.step ? ring[static_cast<size_t>((pos - j) % n) * p.C] : p.x[static_cast<size_t>(t - j) * p.ld + c]);
+  p.out[i] = from_f<T>(silu_of(y));
+  if (ring != nullptr && slot > 0 && p.left[t] < n) ring[static_cast<size_t>(pos % n) * p.C] = own;
+}
+
+// Columns first … first + C of proj [rows, N]; pos [rows] counts from each sequence's start.  hist [slots, taps − 1, C]: kept inputs.
+torch::Tensor conv_silu(const torch::Tensor& proj, int64_t first, const torch::Tensor& w, const torch::Tensor& bias, const torch::Tensor& pos, bool step, const OptT& hist,
+                        const OptT& slot, const OptT& left) {
+  const auto st = proj.scalar_type();
+  TORCH_CHECK(proj.is_cuda() && proj.dim() == 2 && proj.stride(1) == 1 && (st == torch::kBFloat16 || st == torch::kFloat32), "proj [rows, N] bf16 or fp32");
+  TORCH_CHECK(w.dim() == 2 && w.scalar_type() == st && w.is_contiguous() && bias.scalar_type() == st && bias.is_contiguous() && bias.numel() == w.size(0), "filters [C, taps], bias [C]");
+  const int64_t rows = proj.size(0), C = w.size(0), taps = w.size(1);
+  TORCH_CHECK(taps >= 1 && taps <= 1024 && first >= 0 && first + C <= proj.size(1), "columns outside the projection, or no taps");
+  TORCH_CHECK(pos.is_cuda() && pos.scalar_type() == torch::kInt64 && pos.is_contiguous() && pos.numel() == rows, "positions int64 [rows]");
+  if (has(hist)) {
+    TORCH_CHECK(hist->is_cuda() && hist->scalar_type() == st && hist->is_contiguous() && hist->dim() == 3 && hist->size(1) == taps - 1 && hist->size(2) == C, "history [slots, taps - 1, C]");
+    TORCH_CHECK(has(slot) && has(left) && slot->scalar_type() == torch::kInt32 && left->scalar_type() == torch::kInt32 && slot->is_contiguous() && left->is_contiguous() &&
+                    slot->numel() == rows && left->numel() == rows, "slots and rows left int32 [rows]");
+  }
+  TORCH_CHECK(!step || taps == 1 || has(hist), "single steps take their past from the history");
+  c10::cuda::CUDAGuard guard(proj.device());
+  auto out = torch::empty({rows, C}, proj.options());
+  if (rows == 0) return out;
+  auto stream = at::cuda::getCurrentCUDAStream();
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    ConvSilu<T> p{};
+    p.x = reinterpret_cast<const T*>(proj.data_ptr()) + first; p.ld = proj.stride(0);
+    p.w = reinterpret_cast<const T*>(w.data_ptr()); p.bias = reinterpret_cast<const T*>(bias.data_ptr()); p.out = reinterpret_cast<T*>(out.data_ptr());
+    p.pos = pos.data_ptr<int64_t>();
+    if (has(hist)) { p.hist = reinterpret_cast<T*>(hist->data_ptr()); p.slot = slot->data_ptr<int>(); p.left = left->data_ptr<int>(); }
+    p.C = C; p.taps = taps; p.rows = rows; p.step = step;
+    const bool vec = C % 8 == 0 && p.ld % 8 == 0 && aligned16(p.x) && aligned16(p.bias) && aligned16(p.out) && aligned16(p.hist) && taps <= 5;
+    if (!vec) {
+      conv_silu_any_kernel<T><<<static_cast<unsigned>((rows * C + 255) / 256), 256, 0, stream>>>(p);
+      return;
+    }
+    const int across = static_cast<int>((C / 8 + 127) / 128);
+    // sixteen rows per thread once that leaves blocks enough; single steps have nothing to share between rows
+    p.tile = step ? 1 : static_cast<int>(std::min<int64_t>(16, std::max<int64_t>(1, rows * across / (num_sms() * 8))));
+    const dim3 grid(across, static_cast<unsigned>((rows + p.tile - 1) / p.tile));
+    TORCH_CHECK(grid.y <= 65535, "too many rows in one call");
+    if (taps == 1) conv_silu_kernel<T, 1><<<grid, 128, 0, stream>>>(p);
+    else if (taps == 2) conv_silu_kernel<T, 2><<<grid, 128, 0, stream>>>(p);
+    else if (taps == 3) conv_silu_kernel<T, 3><<<grid, 128, 0, stream>>>(p);
+    else if (taps == 4) conv_silu_kernel<T, 4><<<grid, 128, 0, stream>>>(p);
+    else conv_silu_kernel<T, 5><<<grid, 128, 0, stream>>>(p);
+  };
+  if (st == torch::kBFloat16) run(bf16{}); else run(float{});
+  count_launch();
+  TK_CUDA_CHECK(cudaGetLastError());
+  return out;
+}
+
+// -------------------------------------------------------------- selective scan
+template <typename T>
+struct Selective {
+  const T *u, *dt, *z; long ldd, ldz;            // [rows, C] with row strides C, ldd, ldz
+  const T *B, *Cm; long ldb;                     // [rows, N]
+  const T *dt_bias, *A_log, *D;                  // [C], [C, N], [C]
+  T* y;                                          // [rows, C]
+  const int* cu;
+  float* pool; const int* slot;                  // [slots, C, N] (null: last states are not kept)
+  float *part, *steps;                           // [n, segments − 1, C, N], [n, segments − 1, C]
+  int C, N, seg_len, segments;
+};
+
+__device__ __forceinline__ float softplus_of(float x) { return x > 15.f ? x : log1pf(__expf(x)); }
+
+namespace sel {
+constexpr int THREADS = 128;
+constexpr int tokens(int states) { return states > 128 ? 8 : 16; }      // per round
+}
+
+// NS states per lane, LN lanes per channel.  PART: only the state a segment builds up from nothing and its sum of steps.
+template <typename T, int NS, int LN, bool PART>
+__global__ void __launch_bounds__(sel::THREADS) selective_prefill_kernel(const Selective<T> p) {
+  using namespace sel;
+  constexpr int CH = THREADS / LN, NP = NS * LN, TOK = tokens(NP), PER = (TOK * CH + THREADS - 1) / THREADS;   // channels of a block, states filled up, staged elements per thread
+  __shared__ float s_d[2][TOK][CH], s_u[2][TOK][CH], s_y[TOK][CH + 1];
+  __shared__ __align__(16) float s_b[2][TOK][NP], s_c[2][TOK][NP];
+  const int seg = blockIdx.y, seq = blockIdx.z, c0 = blockIdx.x * CH;
+  const int s0 = p.cu[seq], len = p.cu[seq + 1] - s0, a = seg * p.seg_len, b = min(len, a + p.seg_len);
+  if (a >= len || (PART && b >= len)) return;         // the last segment of a sequence is nobody's past
+  const int tid = threadIdx.x, sub = tid % LN, ch = tid / LN, c = c0 + ch;
+  const bool mine = c < p.C;
+  // A in log2 units; states that fill up the lanes neither decay nor take anything in
+  float A[NS], S[NS];
+#pragma unroll
+  for (int i = 0; i < NS; ++i) {
+    const int n = sub * NS + i;
+    A[i] = mine && n < p.N ? -__expf(to_f(p.A_log[static_cast<size_t>(c) * p.N + n])) * 1.4426950408889634f : 0.f;
+    S[i] = 0.f;
+  }
+  if constexpr (!PART) {
+    // what the segments before this one leave behind
+    for (int k = 0; k < seg; ++k) {
+      const size_t at = (static_cast<size_t>(seq) * (p.segments - 1) + k) * p.C + c;
+      if (mine) {
+        const float d = p.steps[at];
+#pragma unroll
+        for (int i = 0; i < NS; ++i) {
+          const int n = sub * NS + i;
+          if (n < p.N) S[i] = fmaf(fast_exp2(d * A[i]), S[i], p.part[at * p.N + n]);
+        }
+      }
+    }
+  }
+  // staging: a thread brings in the same channel column for PER rows, and its share of B and C
+  const int sc = tid % CH, sr = tid / CH, gc = c0 + sc;
+  const float dt_bias = gc < p.C ? to_f(p.dt_bias[gc]) : 0.f, skip = !PART && gc < p.C ? to_f(p.D[gc]) : 0.f;
+  constexpr int BC = (2 * TOK * NP + THREADS - 1) / THREADS;
+  T r_u[PER], r_d[PER], r_z[PER], r_b[BC];
+  auto fetch = [&](int t0) {
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int r = sr + i * (THREADS / CH), t = t0 + r;
+      const bool in = r < TOK && t < b && gc < p.C;
+      const size_t row = static_cast<size_t>(s0 + t);
+      r_u[i] = in ? p.u[row * p.C + gc] : from_f<T>(0.f);
+      r_d[i] = in ? p.dt[row * p.ldd + gc] : from_f<T>(0.f);
+      if constexpr (!PART) r_z[i] = in ? p.z[row * p.ldz + gc] : from_f<T>(0.f);
+    }
+#pragma unroll
+    for (int i = 0; i < BC; ++i) {
+      const int e = tid + i * THREADS, t = e / (2 * NP), n = e % (2 * NP);
+      const bool second = n >= NP;
+      const int nn = second ? n - NP : n;
+      r_b[i] = t < TOK && t0 + t < b && nn < p.N ? (second ? p.Cm : p.B)[static_cast<size_t>(s0 + t0 + t) * p.ldb + nn] : from_f<T>(0.f);
+    }
+  };
+  float total = 0.f;
+  float z_now[PER], u_now[PER];
+  auto stage = [&](int buf, int t0) {
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+      const int r = sr + i * (THREADS / CH);
+      const float u = to_f(r_u[i]), d = t0 + r < b ? softplus_of(to_f(r_d[i]) + dt_bias) : 0.f;      // rows past the end change nothing
+      if (r < TOK) {
+        s_d[buf][r][sc] = d;
+        s_u[buf][r][sc] = d * u;
+      }
+      u_now[i] = u;
+      if constexpr (!PART) z_now[i] = to_f(r_z[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < BC; ++i) {
+      const int e = tid + i * THREADS, t = e / (2 * NP), n = e % (2 * NP);
+      if (t < TOK) (n >= NP ? s_c[buf][t][n - NP] : s_b[buf][t][n]) = to_f(r_b[i]);
+    }
+  };
+  fetch(a);
+  int buf = 0;
+  for (int t0 = a; t0 < b; t0 += TOK, buf ^= 1) {
+    stage(buf, t0);
+    __syncthreads();
+    if (t0 + TOK < b) fetch(t0 + TOK);
+#pragma unroll 1
+    for (int t = 0; t < TOK; t += 4) {
+      float y[4];
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        const float d = s_d[buf][t + k][ch], du = s_u[buf][t + k][ch];
+        y[k] = 0.f;
+        if constexpr (PART) total += d;
+#pragma unroll
+        for (int i = 0; i < NS; i += 4) {
+          const float4 b4 = *reinterpret_cast<const float4*>(&s_b[buf][t + k][sub * NS + i]);
+          S[i] = fmaf(fast_exp2(d * A[i]), S[i], du * b4.x);
+          S[i + 1] = fmaf(fast_exp2(d * A[i + 1]), S[i + 1], du * b4.y);
+          S[i + 2] = fmaf(fast_exp2(d * A[i + 2]), S[i + 2], du * b4.z);
+          S[i + 3] = fmaf(fast_exp2(d * A[i + 3]), S[i + 3], du * b4.w);
+          if constexpr (!PART) {
+            const float4 c4 = *reinterpret_cast<const float4*>(&s_c[buf][t + k][sub * NS + i]);
+            y[k] = fmaf(S[i], c4.x, fmaf(S[i + 1], c4.y, fmaf(S[i + 2], c4.z, fmaf(S[i + 3], c4.w, y[k]))));
+          }
+        }
+      }
+      if constexpr (!PART) {
+        // sums over the lanes of a channel: with four of them or more, each of the first four steps halves what is left to add
+        if constexpr (LN >= 4) {
+          const bool o1 = sub & 1, o2 = sub & 2;
+          float v0 = (o1 ? y[1] : y[0]) + __shfl_xor_sync(0xffffffffu, o1 ? y[0] : y[1], 1);
+          float v1 = (o1 ? y[3] : y[2]) + __shfl_xor_sync(0xffffffffu, o1 ? y[2] : y[3], 1);
+          float v = (o2 ? v1 : v0) + __shfl_xor_sync(0xffffffffu, o2 ? v0 : v1, 2);
+#pragma unroll
+          for (int o = 4; o < LN; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+          if (sub < 4) s_y[t + sub][ch] = v;          // lane's token: bit 0 from the first step, bit 1 from the second
+        } else {
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+#pragma unroll
+            for (int o = 1; o < LN; o <<= 1) y[k] += __shfl_xor_sync(0xffffffffu, y[k], o);
+            if (sub == 0) s_y[t + k][ch] = y[k];
+          }
+        }
+      }
+    }
+    if constexpr (!PART) {
+      __syncthreads();
+#pragma unroll
+      for (int i = 0; i < PER; ++i) {
+        const int r = sr + i * (THREADS / CH);
+        if (r < TOK && t0 + r < b && gc < p.C)
+          p.y[static_cast<size_t>(s0 + t0 + r) * p.C + gc] = from_f<T>((s_y[r][sc] + skip * u_now[i]) * silu_of(z_now[i]));
+      }
+    }
+  }
+  float* out = nullptr;
+  if constexpr (PART) {
+    const size_t at = (static_cast<size_t>(seq) * (p.segments - 1) + seg) * p.C + c;
+    out = p.part + at * p.N;
+    if (mine && sub == 0) p.steps[at] = total;
+  } else if (p.pool != nullptr && b == len) {
+    const int sl = p.slot[s0];
+    if (sl > 0) out = p.pool + (static_cast<size_t>(sl) * p.C + c) * p.N;
+  }
+  if (out != nullptr && mine) {
+#pragma unroll
+    for (int i = 0; i < NS; ++i) {
+      const int n = sub * NS + i;
+      if (n < p.N) out[n] = S[i];
+    }
+  }
+}
+
+// One token per sequence.  NS states per lane, LN lanes per channel; VEC: states in 16-byte accesses.
+template <typename T, int NS, int LN, bool VEC>
+__global__ void __launch_bounds__(128) selective_step_kernel(const Selective<T> p) {
+  constexpr int CH = 128 / LN;
+  const int row = blockIdx.y, sub = threadIdx.x % LN, c = blockIdx.x * CH + threadIdx.x / LN, slot = p.slot[row];
+  const bool mine = c < p.C;
+  float y = 0.f, u = 0.f;
+  if (mine) {
+    u = to_f(p.u[static_cast<size_t>(row) * p.C + c]);
+    const float d = softplus_of(to_f(p.dt[static_cast<size_t>(row) * p.ldd + c]) + to_f(p.dt_bias[c])), du = d * u;
+    float* S = p.pool + (static_cast<size_t>(slot) * p.C + c) * p.N;
+    const T *B = p.B + static_cast<size_t>(row) * p.ldb, *Cm = p.Cm + static_cast<size_t>(row) * p.ldb, *A = p.A_log + static_cast<size_t>(c) * p.N;
+    auto advance = [&](float s, int n) {
+      s = fmaf(fast_exp2(-d * 1.4426950408889634f * __expf(to_f(A[n]))), s, du * to_f(B[n]));
+      y = fmaf(s, to_f(Cm[n]), y);
+      return s;
+    };
+#pragma unroll
+    for (int i = 0; i < NS; i += VEC ? 4 : 1) {
+      // neighbouring lanes take neighbouring vectors
+      const int n = VEC ? (i / 4 * LN + sub) * 4 : i * LN + sub;
+      if (n < p.N) {
+        if constexpr (VEC) {
+          float4 s = *reinterpret_cast<const float4*>(S + n);
+          s.x = advance(s.x, n); s.y = advance(s.y, n + 1); s.z = advance(s.z, n + 2); s.w = advance(s.w, n + 3);
+          if (slot > 0) *reinterpret_cast<float4*>(S + n) = s;
+        } else {
+          const float s = advance(S[n], n);
+          if (slot > 0) S[n] = s;
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int o = 1; o < LN; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+  if (mine && sub == 0)
+    p.y[static_cast<size_t>(row) * p.C + c] = from_f<T>((y + to_f(p.D[c]) * u) * silu_of(to_f(p.z[static_cast<size_t>(row) * p.ldz + c])));
+}
+
+template <typename T>
+static Selective<T> selective_params(const torch::Tensor& u, const torch::Tensor& dt, const torch::Tensor& dt_bias, const torch::Tensor& A_log, const torch::Tensor& proj,
+                                     int64_t b0, int64_t c0, const torch::Tensor& D, const torch::Tensor& gate, int64_t z0, torch::Tensor& y) {
+  Selective<T> p{};
+  p.u = reinterpret_cast<const T*>(u.data_ptr());
+  p.dt = reinterpret_cast<const T*>(dt.data_ptr()); p.ldd = dt.stride(0);
+  p.z = reinterpret_cast<const T*>(gate.data_ptr()) + z0; p.ldz = gate.stride(0);
+  p.B = reinterpret_cast<const T*>(proj.data_ptr()) + b0; p.Cm = reinterpret_cast<const T*>(proj.data_ptr()) + c0; p.ldb = proj.stride(0);
+  p.dt_bias = reinterpret_cast<const T*>(dt_bias.data_ptr()); p.A_log = reinterpret_cast<const T*>(A_log.data_ptr()); p.D = reinterpret_cast<const T*>(D.data_ptr());
+  p.y = reinterpret_cast<T*>(y.data_ptr());
+  p.C = A_log.size(0); p.N = A_log.size(1);
+  return p;
+}
+
+static void selective_check(const torch::Tensor& u, const torch::Tensor& dt, const torch::Tensor& dt_bias, const torch::Tensor& A_log, const torch::Tensor& proj, int64_t b0,
+                            int64_t c0, const torch::Tensor& D, const torch::Tensor& gate, int64_t z0) {
+  const auto st = u.scalar_type();
+  TORCH_CHECK(u.is_cuda() && u.dim() == 2 && u.is_contiguous() && (st == torch::kBFloat16 || st == torch::kFloat32), "inputs [rows, channels] bf16 or fp32");
+  const int64_t rows = u.size(0), C = u.size(1);
+  TORCH_CHECK(A_log.scalar_type() == st && A_log.is_contiguous() && A_log.dim() == 2 && A_log.size(0) == C && A_log.size(1) >= 1 && A_log.size(1) <= 256, "A_log [channels, up to 256 states]");
+  const int64_t N = A_log.size(1);
+  for (const auto* t : {&dt_bias, &D}) TORCH_CHECK(t->scalar_type() == st && t->is_contiguous() && t->numel() == C, "step bias and skip [channels]");
+  for (const auto* t : {&dt, &proj, &gate}) TORCH_CHECK(t->scalar_type() == st && t->dim() == 2 && t->stride(1) == 1 && t->size(0) == rows, "projections [rows, .]");
+  TORCH_CHECK(dt.size(1) == C && b0 >= 0 && c0 >= 0 && z0 >= 0 && b0 + N <= proj.size(1) && c0 + N <= proj.size(1) && z0 + C <= gate.size(1), "columns outside the projections");
+}
+
+// Calls f(NS, LN) as integral constants for a number of states.
+template <typename F>
+static void selective_lanes(int64_t N, F f) {
+  auto go = [&](auto ns, auto ln) { f(ns, ln); };
+  using std::integral_constant;
+  if (N <= 4) go(integral_constant<int, 4>{}, integral_constant<int, 1>{});
+  else if (N <= 8) go(integral_constant<int, 4>{}, integral_constant<int, 2>{});
+  else if (N <= 16) go(integral_constant<int, 4>{}, integral_constant<int, 4>{});
+  else if (N <= 32) go(integral_constant<int, 8>{}, integral_constant<int, 4>{});
+  else if (N <= 64) go(integral_constant<int, 8>{}, integral_constant<int, 8>{});
+  else if (N <= 128) go(integral_constant<int, 8>{}, integral_constant<int, 16>{});
+  else go(integral_constant<int, 8>{}, integral_constant<int, 32>{});
+}
+
+torch::Tensor selective_prefill(const torch::Tensor& u, const torch::Tensor& dt, const torch::Tensor& dt_bias, const torch::Tensor& A_log, const torch::Tensor& proj, int64_t b0,
+                                int64_t c0, const torch::Tensor& D, const torch::Tensor& gate, int64_t z0, const torch::Tensor& cu, int64_t max_seqlen, const OptT& pool,
+                                const OptT& slot) {
+  selective_check(u, dt, dt_bias, A_log, proj, b0, c0, D, gate, z0);
+  TORCH_CHECK(cu.is_cuda() && cu.scalar_type() == torch::kInt32 && cu.is_contiguous() && cu.numel() >= 1, "cu_seqlens int32 on device");
+  const int64_t rows = u.size(0), C = u.size(1), N = A_log.size(1), n = cu.numel() - 1;
+  if (has(pool)) {
+    TORCH_CHECK(pool->is_cuda() && pool->scalar_type() == torch::kFloat32 && pool->is_contiguous() && pool->dim() == 3 && pool->size(1) == C && pool->size(2) == N, "states [slots, channels, N] fp32");
+    TORCH_CHECK(has(slot) && slot->scalar_type() == torch::kInt32 && slot->is_contiguous() && slot->numel() == rows, "slots int32 [rows]");
+  }
+  c10::cuda::CUDAGuard guard(u.device());
+  auto y = torch::empty_like(u);
+  if (rows == 0 || n == 0 || max_seqlen <= 0) return y;
+  auto stream = at::cuda::getCurrentCUDAStream();
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    auto p = selective_params<T>(u, dt, dt_bias, A_log, proj, b0, c0, D, gate, z0, y);
+    p.cu = cu.data_ptr<int>();
+    if (has(pool)) { p.pool = pool->data_ptr<float>(); p.slot = slot->data_ptr<int>(); }
+    selective_lanes(N, [&](auto ns, auto ln) {
+      constexpr int NS = decltype(ns)::value, LN = decltype(ln)::value, CH = sel::THREADS / LN, TOK = sel::tokens(NS * LN);
+      const int64_t across = (C + CH - 1) / CH, blocks = across * n, fill = num_sms() * 8L;
+      // segments of at least 64 tokens, as many as fill the device (the work of all but the last is done twice)
+      int64_t segments = blocks * 2 > fill ? 1 : std::min<int64_t>({fill / blocks, (max_seqlen + 63) / 64, 32});
+      const int64_t seg_len = ((max_seqlen + segments - 1) / segments + TOK - 1) / TOK * TOK;
+      segments = (max_seqlen + seg_len - 1) / seg_len;
+      p.segments = static_cast<int>(segments);
+      p.seg_len = static_cast<int>(seg_len);
+      torch::Tensor part, steps;
+      if (segments > 1) {
+        part = torch::empty({n * (segments - 1) * C * N}, u.options().dtype(torch::kFloat32));
+        steps = torch::empty({n * (segments - 1) * C}, part.options());
+        p.part = part.data_ptr<float>();
+        p.steps = steps.data_ptr<float>();
+        selective_prefill_kernel<T, NS, LN, true><<<dim3(across, segments - 1, n), sel::THREADS, 0, stream>>>(p);
+        count_launch();
+      }
+      selective_prefill_kernel<T, NS, LN, false><<<dim3(across, segments, n), sel::THREADS, 0, stream>>>(p);
+      count_launch();
+    });
+  };
+  if (u.scalar_type() == torch::kBFloat16) run(bf16{}); else run(float{});
+  TK_CUDA_CHECK(cudaGetLastError());
+  return y;
+}
+
+torch::Tensor selective_step(const torch::Tensor& u, const torch::Tensor& dt, const torch::Tensor& dt_bias, const torch::Tensor& A_log, const torch::Tensor& proj, int64_t b0,
+                             int64_t c0, const torch::Tensor& D, const torch::Tensor& gate, int64_t z0, const torch::Tensor& pool, const torch::Tensor& slot) {
+  selective_check(u, dt, dt_bias, A_log, proj, b0, c0, D, gate, z0);
+  const int64_t rows = u.size(0), C = u.size(1), N = A_log.size(1);
+  TORCH_CHECK(pool.is_cuda() && pool.scalar_type() == torch::kFloat32 && pool.is_contiguous() && pool.dim() == 3 && pool.size(1) == C && pool.size(2) == N, "states [slots, channels, N] fp32");
+  TORCH_CHECK(slot.scalar_type() == torch::kInt32 && slot.is_contiguous() && slot.numel() == rows && rows <= 65535, "slots int32 [rows]");
+  c10::cuda::CUDAGuard guard(u.device());
+  auto y = torch::empty_like(u);
+  if (rows == 0) return y;
+  auto stream = at::cuda::getCurrentCUDAStream();
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    auto p = selective_params<T>(u, dt, dt_bias, A_log, proj, b0, c0, D, gate, z0, y);
+    p.pool = pool.data_ptr<float>(); p.slot = slot.data_ptr<int>();
+    selective_lanes(N, [&](auto ns, auto ln) {
+      constexpr int NS = decltype(ns)::value, LN = decltype(ln)::value, CH = 128 / LN;
+      const dim3 grid(static_cast<unsigned>((C + CH - 1) / CH), static_cast<unsigned>(rows));
+      if (N % 4 == 0) selective_step_kernel<T, NS, LN, true><<<grid, 128, 0, stream>>>(p);
+      else selective_step_kernel<T, NS, LN, false><<<grid, 128, 0, stream>>>(p);
+    });
+  };
+  if (u.scalar_type() == torch::kBFloat16) run(bf16{}); else run(float{});
+  count_launch();
+  TK_CUDA_CHECK(cudaGetLastError());
+  return y;
+}
+
+}  // namespace tk

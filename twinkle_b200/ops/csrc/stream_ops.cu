@@ -4,7 +4,10 @@
 //                   weighted sum of a token's expert rows, beside a shared expert's row with a weight per token
 //   stream_gated_rmsnorm  x += norm(σ(gate + bias) ⊙ y) in fp32 and the RMS norm of the sum — one pass; y is a row of its own or
 //                   the weighted sum of a token's expert rows
-//   glu_columns     silu(gate) · up, or its clamped form, on two column ranges of a projection
+//   stream_normed_add  x += norm(y + bias) in fp32, or the norm of half the sum of two normed results, and the sum or its RMS norm in the
+//                   compute dtype — one pass
+//   embed_positions an embedding's row plus sines and cosines of the position, fp32
+//   glu_columns     silu(gate) · up, gelu(gate) · up (tanh form) or the clamped form, on two column ranges of a projection
 // All are templated on the compute dtype (bf16 or fp32) and work for any width: vector kernels where rows are made of
 // whole vectors, plain ones otherwise.
 #include <ATen/cuda/CUDAContext.h>
@@ -391,11 +394,200 @@ torch::Tensor stream_joined_rmsnorm(torch::Tensor x, const torch::Tensor& w, dou
   return h;
 }
 
+// ----------------------------------------------------------- stream_normed_add
+// One block per row, as above.
+struct NormedAdd {
+  float* x;
+  const void *y, *bias, *post, *inner, *beside, *beside_inner, *next;     // bias, beside (with the inner norms) and next may be null
+  void* h;
+  int W;
+  float eps;
+};
+
+template <typename T, int VPT>
+__global__ void stream_normed_add_kernel(const NormedAdd p) {
+  __shared__ float sh[32], sh2[32];
+  const int W = p.W, t = blockIdx.x;
+  const size_t base = static_cast<size_t>(t) * W;
+  const T *y = reinterpret_cast<const T*>(p.y) + base, *bias = reinterpret_cast<const T*>(p.bias), *post = reinterpret_cast<const T*>(p.post);
+  const T *inner = reinterpret_cast<const T*>(p.inner), *beside = p.beside != nullptr ? reinterpret_cast<const T*>(p.beside) + base : nullptr;
+  const T *beside_inner = reinterpret_cast<const T*>(p.beside_inner), *next = reinterpret_cast<const T*>(p.next);
+  float* x = p.x + base;
+  T* h = reinterpret_cast<T*>(p.h) + base;
+  const float inv_w = 1.f / W;
+  if constexpr (VPT > 0) {
+    float4 z[VPT], v[VPT], b[VPT];
+    float ss = 0.f, sb = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * 4;
+      z[i] = v[i] = b[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < W) {
+        z[i] = load4(y + c);
+        v[i] = load4(x + c);
+        if (beside != nullptr) b[i] = load4(beside + c);
+        if (bias != nullptr) {
+          const float4 a = load4(bias + c);
+          z[i].x += a.x; z[i].y += a.y; z[i].z += a.z; z[i].w += a.w;
+        }
+      }
+      ss += z[i].x * z[i].x + z[i].y * z[i].y + z[i].z * z[i].z + z[i].w * z[i].w;
+      sb += b[i].x * b[i].x + b[i].y * b[i].y + b[i].z * b[i].z + b[i].w * b[i].w;
+    }
+    float r = rsqrtf(block_sum(ss, sh) * inv_w + p.eps);
+    if (beside != nullptr) {
+      const float rb = 0.5f * rsqrtf(block_sum(sb, sh2) * inv_w + p.eps);
+      r *= 0.5f;
+      ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < VPT; ++i) {
+        const int c = (i * blockDim.x + threadIdx.x) * 4;
+        if (c < W) {
+          const float4 w = load4(inner + c), u = load4(beside_inner + c);
+          z[i].x = z[i].x * r * w.x + b[i].x * rb * u.x; z[i].y = z[i].y * r * w.y + b[i].y * rb * u.y;
+          z[i].z = z[i].z * r * w.z + b[i].z * rb * u.z; z[i].w = z[i].w * r * w.w + b[i].w * rb * u.w;
+        }
+        ss += z[i].x * z[i].x + z[i].y * z[i].y + z[i].z * z[i].z + z[i].w * z[i].w;
+      }
+      r = rsqrtf(block_sum(ss, sh) * inv_w + p.eps);
+    }
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * 4;
+      if (c < W) {
+        const float4 w = load4(post + c);
+        v[i].x += z[i].x * r * w.x; v[i].y += z[i].y * r * w.y; v[i].z += z[i].z * r * w.z; v[i].w += z[i].w * r * w.w;
+        store4(x + c, v[i]);
+        if (next == nullptr) store4(h + c, v[i]);
+      }
+      ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    }
+    if (next == nullptr) return;
+    r = rsqrtf(block_sum(ss, sh2) * inv_w + p.eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (i * blockDim.x + threadIdx.x) * 4;
+      if (c < W) {
+        const float4 w = load4(next + c);
+        store4(h + c, make_float4(v[i].x * r * w.x, v[i].y * r * w.y, v[i].z * r * w.z, v[i].w * r * w.w));
+      }
+    }
+  } else {                                   // any width: results are read once per pass
+    auto own = [&](int c) { return to_f(y[c]) + (bias != nullptr ? to_f(bias[c]) : 0.f); };
+    float ss = 0.f, sb = 0.f;
+    for (int c = threadIdx.x; c < W; c += blockDim.x) {
+      const float a = own(c), b = beside != nullptr ? to_f(beside[c]) : 0.f;
+      ss += a * a;
+      sb += b * b;
+    }
+    float r = rsqrtf(block_sum(ss, sh) * inv_w + p.eps);
+    const float ra = 0.5f * r, rb = 0.5f * rsqrtf(block_sum(sb, sh2) * inv_w + p.eps);
+    auto joined = [&](int c) { return beside != nullptr ? own(c) * ra * to_f(inner[c]) + to_f(beside[c]) * rb * to_f(beside_inner[c]) : own(c); };
+    if (beside != nullptr) {
+      ss = 0.f;
+      for (int c = threadIdx.x; c < W; c += blockDim.x) { const float z = joined(c); ss += z * z; }
+      r = rsqrtf(block_sum(ss, sh) * inv_w + p.eps);
+    }
+    ss = 0.f;
+    for (int c = threadIdx.x; c < W; c += blockDim.x) {
+      const float v = x[c] + joined(c) * r * to_f(post[c]);
+      x[c] = v;
+      if (next == nullptr) h[c] = from_f<T>(v);
+      ss += v * v;
+    }
+    if (next == nullptr) return;
+    r = rsqrtf(block_sum(ss, sh2) * inv_w + p.eps);
+    for (int c = threadIdx.x; c < W; c += blockDim.x) h[c] = from_f<T>(x[c] * r * to_f(next[c]));
+  }
+}
+
+// x [rows, W] fp32 is updated in place; returns the sum (or, with w, its norm) in y's dtype.
+torch::Tensor stream_normed(torch::Tensor x, const OptT& w, double eps, const torch::Tensor& y, const OptT& bias, const torch::Tensor& post, const OptT& inner, const OptT& beside,
+                            const OptT& beside_inner) {
+  const auto st = y.scalar_type();
+  TORCH_CHECK(x.is_cuda() && x.scalar_type() == torch::kFloat32 && x.is_contiguous() && x.dim() == 2, "stream [rows, W] fp32 contiguous");
+  TORCH_CHECK(st == torch::kBFloat16 || st == torch::kFloat32, "bf16 or fp32");
+  const int rows = x.size(0), W = x.size(1);
+  bool vec = W % 4 == 0 && W <= 8192;
+  auto check = [&](const OptT& t, int64_t n, const char* what) -> const void* {
+    if (!has(t)) return nullptr;
+    TORCH_CHECK(t->is_cuda() && t->scalar_type() == st && t->is_contiguous() && t->numel() == n, what);
+    vec = vec && aligned16(t->data_ptr());
+    return t->data_ptr();
+  };
+  TORCH_CHECK(has(beside) == has(inner) && has(beside) == has(beside_inner), "two results come with a norm each");
+  NormedAdd p{};
+  p.x = x.data_ptr<float>(); p.W = W; p.eps = eps;
+  p.y = check(y, x.numel(), "result [rows, W]"); p.beside = check(beside, x.numel(), "second result [rows, W]");
+  p.bias = check(bias, W, "bias [W]"); p.post = check(post, W, "norm weight [W]"); p.next = check(w, W, "norm weight [W]");
+  p.inner = check(inner, W, "norm weight [W]"); p.beside_inner = check(beside_inner, W, "norm weight [W]");
+  c10::cuda::CUDAGuard guard(x.device());
+  auto h = torch::empty(x.sizes(), y.options());
+  if (rows == 0) return h;
+  p.h = h.data_ptr();
+  const int nvec = (W + 3) / 4, vpt = nvec <= 512 ? 1 : (nvec <= 1024 ? 2 : 4);
+  auto stream = at::cuda::getCurrentCUDAStream();
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    const int threads = std::min(512, ((nvec + vpt - 1) / vpt + 31) / 32 * 32);
+    if (!vec) stream_normed_add_kernel<T, 0><<<rows, std::min(512, (W + 31) / 32 * 32), 0, stream>>>(p);
+    else if (vpt == 1) stream_normed_add_kernel<T, 1><<<rows, threads, 0, stream>>>(p);
+    else if (vpt == 2) stream_normed_add_kernel<T, 2><<<rows, threads, 0, stream>>>(p);
+    else stream_normed_add_kernel<T, 4><<<rows, threads, 0, stream>>>(p);
+  };
+  if (st == torch::kBFloat16) run(bf16{}); else run(float{});
+  count_launch();
+  TK_CUDA_CHECK(cudaGetLastError());
+  return h;
+}
+
+// ------------------------------------------------------------- embed_positions
+// A thread forms one pair.  The angle is reduced to half turns in fp64, so that far positions keep their digits.
+template <typename T>
+__global__ void __launch_bounds__(256) embed_positions_kernel(const int64_t* __restrict__ ids, const T* __restrict__ weight, const int64_t* __restrict__ pos,
+                                                              const double* __restrict__ freq, float* __restrict__ out, long total, int pairs, int W) {
+  const long i = blockIdx.x * 256L + threadIdx.x;
+  if (i >= total) return;
+  const long t = i / pairs;
+  const int k = static_cast<int>(i - t * pairs);
+  const double half_turns = static_cast<double>(pos[t]) * (freq[k] * 0.31830988618379067154);
+  float s, c;
+  sincospif(static_cast<float>(half_turns - 2.0 * rint(0.5 * half_turns)), &s, &c);
+  const T* w = weight + static_cast<size_t>(ids[t]) * W + 2 * k;
+  float* o = out + static_cast<size_t>(t) * W + 2 * k;
+  o[0] = to_f(w[0]) + s;
+  if (2 * k + 1 < W) o[1] = to_f(w[1]) + c;
+}
+
+torch::Tensor embed_positions(const torch::Tensor& ids, const torch::Tensor& weight, const torch::Tensor& pos, const torch::Tensor& freq) {
+  const auto st = weight.scalar_type();
+  TORCH_CHECK(weight.is_cuda() && weight.dim() == 2 && weight.is_contiguous() && (st == torch::kBFloat16 || st == torch::kFloat32), "embedding [vocab, W] bf16 or fp32");
+  TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == torch::kInt64 && ids.is_contiguous() && pos.is_cuda() && pos.scalar_type() == torch::kInt64 && pos.is_contiguous() &&
+                  ids.dim() == 1 && ids.numel() == pos.numel(), "token ids and positions int64 [rows]");
+  const int W = weight.size(1), pairs = (W + 1) / 2;
+  TORCH_CHECK(freq.is_cuda() && freq.scalar_type() == torch::kFloat64 && freq.is_contiguous() && freq.numel() == pairs, "frequencies fp64 [pairs]");
+  c10::cuda::CUDAGuard guard(weight.device());
+  auto out = torch::empty({ids.numel(), W}, weight.options().dtype(torch::kFloat32));
+  const long total = ids.numel() * pairs;
+  if (total == 0) return out;
+  auto run = [&](auto tag) {
+    using T = decltype(tag);
+    embed_positions_kernel<T><<<static_cast<unsigned>((total + 255) / 256), 256, 0, at::cuda::getCurrentCUDAStream()>>>(
+        ids.data_ptr<int64_t>(), reinterpret_cast<const T*>(weight.data_ptr()), pos.data_ptr<int64_t>(), freq.data_ptr<double>(), out.data_ptr<float>(), total, pairs, W);
+  };
+  if (st == torch::kBFloat16) run(bf16{}); else run(float{});
+  count_launch();
+  TK_CUDA_CHECK(cudaGetLastError());
+  return out;
+}
+
 // ----------------------------------------------------------------- glu_columns
-// limit 0: silu(g) · u; otherwise g σ(1.702 g) (u + 1) on g ≤ limit, |u| ≤ limit.
-template <bool CLAMP>
+// ACT 0: silu(g) · u; 1: g σ(1.702 g) (u + 1) on g ≤ limit, |u| ≤ limit; 2: gelu in its tanh form times u (½ (1 + tanh a) = σ(2a)).
+template <int ACT>
 __device__ __forceinline__ float glu(float g, float u, float limit) {
-  if constexpr (CLAMP) {
+  if constexpr (ACT == 2) return g / (1.f + __expf(-1.5957691216057308f * fmaf(0.044715f * g * g, g, g))) * u;
+  if constexpr (ACT == 1) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);
@@ -403,7 +595,7 @@ __device__ __forceinline__ float glu(float g, float u, float limit) {
   return g / (1.f + __expf(-g)) * u;
 }
 
-template <typename T, int V, bool CLAMP>
+template <typename T, int V, int ACT>
 __global__ void __launch_bounds__(256) glu_columns_kernel(const T* __restrict__ p, long ld, int gate, int up, T* __restrict__ out, long rows, int I, float limit) {
   const int per_row = I / V;
   const long total = rows * per_row;
@@ -420,17 +612,17 @@ __global__ void __launch_bounds__(256) glu_columns_kernel(const T* __restrict__ 
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         const float2 x = unpack_bf16(pa[k]), y = unpack_bf16(pb[k]);
-        po[k] = pack_bf16(glu<CLAMP>(x.x, y.x, limit), glu<CLAMP>(x.y, y.y, limit));
+        po[k] = pack_bf16(glu<ACT>(x.x, y.x, limit), glu<ACT>(x.y, y.y, limit));
       }
       *reinterpret_cast<uint4*>(o) = make_uint4(po[0], po[1], po[2], po[3]);
     } else {
 #pragma unroll
-      for (int k = 0; k < V; ++k) o[k] = from_f<T>(glu<CLAMP>(to_f(g[k]), to_f(u[k]), limit));
+      for (int k = 0; k < V; ++k) o[k] = from_f<T>(glu<ACT>(to_f(g[k]), to_f(u[k]), limit));
     }
   }
 }
 
-torch::Tensor glu_columns(const torch::Tensor& p, int64_t gate, int64_t up, int64_t I, double limit) {
+torch::Tensor glu_columns(const torch::Tensor& p, int64_t gate, int64_t up, int64_t I, double limit, bool gelu) {
   const auto st = p.scalar_type();
   TORCH_CHECK(p.is_cuda() && p.dim() == 2 && p.stride(1) == 1 && (st == torch::kBFloat16 || st == torch::kFloat32), "projection [rows, N] bf16 or fp32");
   TORCH_CHECK(I > 0 && gate >= 0 && up >= 0 && gate + I <= p.size(1) && up + I <= p.size(1) && limit >= 0, "gate / up columns outside the projection, or a negative limit");
@@ -447,8 +639,9 @@ torch::Tensor glu_columns(const torch::Tensor& p, int64_t gate, int64_t up, int6
     constexpr int V = decltype(width)::value;
     const T* in = reinterpret_cast<const T*>(p.data_ptr());
     T* o = reinterpret_cast<T*>(out.data_ptr());
-    if (limit > 0) glu_columns_kernel<T, V, true><<<blocks, 256, 0, stream>>>(in, ld, gate, up, o, rows, I, static_cast<float>(limit));
-    else glu_columns_kernel<T, V, false><<<blocks, 256, 0, stream>>>(in, ld, gate, up, o, rows, I, 0.f);
+    if (gelu) glu_columns_kernel<T, V, 2><<<blocks, 256, 0, stream>>>(in, ld, gate, up, o, rows, I, 0.f);
+    else if (limit > 0) glu_columns_kernel<T, V, 1><<<blocks, 256, 0, stream>>>(in, ld, gate, up, o, rows, I, static_cast<float>(limit));
+    else glu_columns_kernel<T, V, 0><<<blocks, 256, 0, stream>>>(in, ld, gate, up, o, rows, I, 0.f);
   };
   if (vec) go(bf16{}, std::integral_constant<int, 8>{});
   else if (st == torch::kBFloat16) go(bf16{}, std::integral_constant<int, 1>{});

@@ -263,6 +263,104 @@ def latent_rotary(proj: torch.Tensor, q0: int, heads: int, d: int, r: int, c0: i
     return q, kept
 
 
+# ------------------------------------------- layers with norms on their results
+def position_waves(positions: torch.Tensor, frequencies: torch.Tensor, width: int) -> torch.Tensor:
+    """``[T, width]`` fp32: sine and cosine of position times frequency side by side (angles in fp64)."""
+    a = positions.double()[:, None] * frequencies
+    return torch.stack([a.sin(), a.cos()], -1).flatten(1)[:, :width].float()
+
+
+def stream_normed(x: torch.Tensor, weight: Optional[torch.Tensor], eps: float, out_dtype: torch.dtype, y: torch.Tensor, bias: Optional[torch.Tensor], post: torch.Tensor,
+                  inner: Optional[torch.Tensor] = None, beside: Optional[torch.Tensor] = None, beside_inner: Optional[torch.Tensor] = None):
+    unit = lambda t: t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps)  # noqa: E731
+    z = y.float() if bias is None else y.float() + bias.float()
+    if beside is not None:
+        z = 0.5 * (unit(z) * inner.float() + unit(beside.float()) * beside_inner.float())
+    x = x + unit(z) * post.float()
+    return (x if weight is None else unit(x) * weight.float()).to(out_dtype), x
+
+
+def plain_heads(proj: torch.Tensor, first: int, bias: Optional[torch.Tensor], q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], value_norm: bool,
+                values_are_keys: bool, hq: int, hkv: int, d: int, e: int, eps: float):
+    T, sizes = proj.shape[0], (hq * d, hkv * d, 0 if values_are_keys else hkv * e)
+    y = proj[:, first:first + sum(sizes)].float()
+    q, k, v = (y if bias is None else y + bias.float()).split(sizes, -1)
+    v = (k if values_are_keys else v).reshape(T, hkv, e)
+
+    def normed(t, w, h):
+        whole = w is not None and w.numel() == h * d and h > 1         # one head: the same thing
+        t = t if whole else t.reshape(T, h, d)
+        if w is not None:
+            t = t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+        return t.reshape(T, h, d)
+    if value_norm:
+        v = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)
+    return tuple(t.to(proj.dtype) for t in (normed(q, q_weight, hq), normed(k, k_weight, hkv), v))
+
+
+# ------------------------------------------- selective scan, matrix memory
+def conv_silu(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, positions: torch.Tensor, history: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None):
+    return F.silu(short_conv(x, weight, positions, history, slots) + bias.float()).to(x.dtype)
+
+
+def selective_scan(u: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor, B: torch.Tensor, C: torch.Tensor, D: torch.Tensor, z: torch.Tensor,
+                   bounds, states=None):
+    """Sequences ``bounds`` of rows, from ``states`` (None: empty ones) → ``(y [T, inner], last states)``; token by token."""
+    dtype, (u, B, C) = u.dtype, (t.float() for t in (u, B, C))
+    step = F.softplus(dt.float() + dt_bias.float())
+    A, du = -torch.exp(A_log.float()), step * u
+    rows, last = [], []
+    for n, (a, b) in enumerate(zip(bounds[:-1], bounds[1:])):
+        S = A.new_zeros(A.shape) if states is None else states[n]
+        for t in range(a, b):
+            S = torch.exp(step[t][:, None] * A) * S + du[t][:, None] * B[t]
+            rows.append(S @ C[t])
+        last.append(S)
+    y = torch.stack(rows) if rows else torch.zeros_like(u)
+    return ((y + D.float() * u) * F.silu(z.float())).to(dtype), last
+
+
+def matrix_memory_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, i: torch.Tensor, f: torch.Tensor, state, chunk: int = 32):
+    """One sequence ``q, k [T, H, d]``, ``v [T, H, e]``, log gates ``[T, H]``, from ``(S, n, m)`` → ``(o [T, H, e], last (S, n, m))``, in chunks: a token's
+    weight on an earlier one is the exponential of summed log gates, taken relative to the running maximum."""
+    S, n, m = state
+    out = []
+    for a in range(0, q.shape[0], chunk):
+        qc, kc, vc, ic, fc = (t[a:a + chunk].transpose(0, 1) for t in (q, k, v, i, f))         # [H, L, ·], [H, L]
+        F_ = fc.cumsum(-1)
+        g = ic - F_                                                                              # what a token is worth at the chunk's start
+        top = torch.maximum(m[:, None], g.cummax(-1).values) + F_                               # running maximum
+        start = torch.exp(F_ + m[:, None] - top)                                                # weight of the state at the chunk's start
+        w = torch.exp((F_ - top)[:, :, None] + g[:, None, :]).tril()                            # [H, L, L]
+        A = (qc @ kc.transpose(1, 2)) * w
+        num = A @ vc + start[..., None] * (qc @ S)
+        den = A.sum(-1) + start * (qc @ n[..., None])[..., 0]
+        out.append((num / (torch.maximum(den.abs(), torch.exp(-top)) + 1e-6)[..., None]).transpose(0, 1))
+        end = w[:, -1, :, None] * kc
+        S = start[:, -1, None, None] * S + end.transpose(1, 2) @ vc
+        n = start[:, -1, None] * n + end.sum(1)
+        m = top[:, -1]
+    return (torch.cat(out) if out else torch.zeros_like(v)), (S, n, m)
+
+
+def matrix_memory(proj: torch.Tensor, first: int, heads: int, dim: int, vdim: int, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, weight: torch.Tensor, eps: float,
+                  bounds, states=None):
+    """Columns ``[q | k | v | gate | i | f]`` from ``first`` on → ``(o [T, heads · vdim], last states)``; a state is ``(S, n, m)``."""
+    T, nd, ne = proj.shape[0], heads * dim, heads * vdim
+    q, k, v, g, i, f = proj[:, first:first + 2 * nd + 2 * ne + 2 * heads].float().split([nd, nd, ne, ne, heads, heads], -1)
+    q, k, v = q.reshape(T, heads, dim) * dim**-0.5, k.reshape(T, heads, dim), v.reshape(T, heads, vdim)
+    i, f = cap * torch.tanh((i + i_bias.float()) / cap), F.logsigmoid(cap * torch.tanh((f + f_bias.float()) / cap))
+    out, last = [], []
+    for n, (a, b) in enumerate(zip(bounds[:-1], bounds[1:])):
+        s = (q.new_zeros(heads, dim, vdim), q.new_zeros(heads, dim), q.new_zeros(heads)) if states is None else states[n]
+        o, s = matrix_memory_scan(q[a:b], k[a:b], v[a:b], i[a:b], f[a:b], s)
+        out.append(o)
+        last.append(s)
+    o = torch.cat(out)
+    o = (o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)).reshape(T, ne) * weight.float() * torch.sigmoid(g)
+    return o.to(proj.dtype), last
+
+
 # ------------------------------------------- latent attention, HGRN2
 def latent_norms(proj: torch.Tensor, q0: int, nq: int, wq: torch.Tensor, c0: int, nc: int, wc: Optional[torch.Tensor], eps: float):
     """RMS norms of the query-bottleneck and latent column ranges of a projection (``nc`` 0: no latent)."""
@@ -340,7 +438,7 @@ def relu2(x: torch.Tensor) -> torch.Tensor:
 # ----------------------------------------------------------------- attention
 def attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqlens: torch.Tensor, causal: bool = True,
                      scale: Optional[float] = None, return_lse: bool = False, cu_seqlens_k: Optional[torch.Tensor] = None,
-                     window: Optional[int] = None, softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0):
+                     window: Optional[int] = None, softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0, terms=None):
     """Packed attention.  ``q [T,Hq,D]``, ``k,v [Tk,Hkv,D]``, ``cu_seqlens`` int
     ``[n+1]``; tokens of different segments never attend to each other; GQA by
     repeating each kv head ``Hq/Hkv`` times.  With ``cu_seqlens_k`` the keys of a segment may be longer than its
@@ -348,7 +446,8 @@ def attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqle
     ``window``: a query sees only the last ``window`` keys up to and including its own position (sliding-window
     checkpoints); ``softcap``: scores pass through ``cap · tanh(s / cap)`` before the softmax (Gemma-2); ``sinks [Hq]``: a
     learned logit per head that takes part in the softmax and carries no value (GPT-OSS), i.e. it only enlarges the
-    denominator; ``chunk``: a query sees only the keys of its own block of that many positions, counted from the sequence's start."""
+    denominator; ``chunk``: a query sees only the keys of its own block of that many positions, counted from the sequence's start; ``terms``
+    (an ``ops.ScoreTerms``): what else happens to a score."""
     T, Hq, D = q.shape
     Hkv = k.shape[1]
     rep = Hq // Hkv
@@ -366,6 +465,8 @@ def attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqle
         s = qs @ ks.transpose(1, 2) * scale
         if softcap:
             s = torch.tanh(s / softcap) * softcap
+        if terms is not None:
+            s = terms.apply(s, torch.arange(b - a, device=q.device)[:, None] + (kbnd - ka - b + a) - torch.arange(kbnd - ka, device=q.device))
         if causal:
             L, Lk = b - a, kbnd - ka
             s = s.masked_fill(torch.ones(L, Lk, dtype=torch.bool, device=q.device).triu(1 + Lk - L), float('-inf'))
@@ -385,7 +486,7 @@ def attention_varlen(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_seqle
 
 def paged_attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_tables: torch.Tensor,
                            seq_lens: torch.Tensor, scale: Optional[float] = None, window: Optional[int] = None,
-                           softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0) -> torch.Tensor:
+                           softcap: Optional[float] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0, terms=None) -> torch.Tensor:
     """One query token per sequence against a paged KV cache.
     ``q [B,Hq,D]``; caches ``[num_blocks, block_size, Hkv, D]`` (values may have a width of their own); ``block_tables
     [B, max_blocks]`` int; ``seq_lens [B]`` (including the current token)."""
@@ -406,6 +507,8 @@ def paged_attention_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
         s = torch.einsum('hd,nhd->hn', q[b].float(), kk) * scale
         if softcap:
             s = torch.tanh(s / softcap) * softcap
+        if terms is not None:
+            s = terms.apply(s[:, None], n - 1 - torch.arange(n, device=q.device)[None])[:, 0]
         if window and n > window:
             s[:, :n - window] = float('-inf')
         if chunk:
