@@ -224,3 +224,102 @@ def forward(cfg, weights, tokens, dtype=torch.float64):
             x = x + norm(feed_forward(x, part(W, p + 'mlp.')), W[p + 'norm2'], eps)
         trail.append(x)
     return norm(x, W['final.norm'], eps) @ W['head'].t(), trail
+
+
+# ---------------------------------------------------------------- models for the tests
+def attention(heads, kv_heads, dim, vdim, scale, size, cap, ff=None):
+    return {'type': 'attention', 'mixer': {'heads': heads, 'kv_heads': kv_heads, 'dim': dim, 'vdim': vdim, 'scale': scale, 'softcap': cap, 'mask': {'size': size}}, 'mlp': dense(ff)}
+
+
+def mamba1(inner, state, dt_rank, conv, ff=None):
+    return {'type': 'mamba1', 'mixer': {'inner': inner, 'state': state, 'dt_rank': dt_rank, 'conv': conv}, 'mlp': dense(ff)}
+
+
+def parallel(left, right, ff=None):
+    """``left``: heads, kv_heads, dim, scale, window, softcap, rows of the distance table, its last distance; ``right``: heads, dim, vdim, gate cap."""
+    heads, kv_heads, dim, scale, size, cap, rows, far = left
+    h, d, e, gate_cap = right
+    return {'type': 'parallel', 'mlp': dense(ff),
+            'mixer': {'left': {'heads': heads, 'kv_heads': kv_heads, 'dim': dim, 'vdim': dim, 'scale': scale, 'softcap': cap, 'bias_max': far, 'mask': {'size': size}},
+                      'right': {'heads': h, 'dim': d, 'vdim': e, 'gate_cap': gate_cap}}, 'rows': rows}
+
+
+def dense(ff):
+    return None if ff is None else {'kind': 'dense', 'ff': ff}
+
+
+CONFIGS = {
+    # every kind of layer twice, of unequal sizes, with and without a feed-forward block
+    'mixed': dict(vocab=120, width=96, norm={'eps': 1e-4},
+                  layers=[parallel((6, 2, 24, 0.25, 19, 6.0, 10, 37), (3, 16, 40, 4.0), 128), mamba1(80, 12, 8, 3, 72), attention(6, 3, 24, 40, 0.3, 23, 5.0),
+                          mamba1(64, 16, 24, 4), parallel((4, 4, 40, 0.2, 70, 20.0, 32, 128), (2, 24, 32, 9.0)), attention(8, 2, 16, 16, 0.4, 33, 3.0, 96)]),
+    # sizes that are no whole vectors, one head, windows of one, a table of two rows, filters of one and of six taps, odd numbers of states
+    'odd': dict(vocab=97, width=52, norm={'eps': 1e-3},
+                layers=[mamba1(30, 5, 3, 2, 18), parallel((3, 1, 11, 0.3, 13, 2.5, 7, 20), (1, 10, 7, 3.0), 20), attention(5, 1, 10, 7, 0.35, 1, 4.0, 9), mamba1(21, 1, 1, 1),
+                        attention(1, 1, 14, 5, 0.3, 17, 8.0), mamba1(12, 9, 5, 6, 33), parallel((2, 2, 9, 0.3, 30, 30.0, 2, 4), (5, 3, 9, 1.5)), parallel((1, 1, 6, 0.4, 1, 1.0, 5, 3), (2, 5, 12, 6.0), 11)]),
+    # head widths on both sides of 64 and 128, values in several blocks, many states, windows around a tile of 128
+    'wide': dict(vocab=64, width=72, norm={'eps': 1e-6},
+                 layers=[attention(8, 1, 128, 72, 0.06, 129, 30.0, 40), parallel((4, 2, 160, 0.05, 128, 15.0, 16, 100), (2, 128, 136, 15.0)), mamba1(136, 64, 8, 4),
+                         parallel((4, 4, 128, 0.07, 250, 50.0, 64, 333), (1, 256, 64, 7.0), 48), attention(3, 3, 200, 136, 0.06, 127, 10.0), mamba1(64, 130, 16, 5, 24)]),
+}
+_ROWS = {}
+for _n, _c in CONFIGS.items():
+    _c['architecture'] = 'Puzonex'
+    _ROWS[_n] = [layer.pop('rows', 0) for layer in _c['layers']]
+
+
+def random_weights(cfg, seed=0, rows=None):
+    """Weights under their checkpoint names, every value representable in bfloat16.  Sinks weigh as much as a few keys, distances shift scores by
+    about one, forget gates are mostly open, and a scan's steps reach from a few tokens to hundreds."""
+    rows = rows if rows is not None else next((_ROWS[n] for n, c in CONFIGS.items() if c is cfg), None)
+    g = torch.Generator().manual_seed(seed)
+    rnd = lambda *s: torch.randn(*s, generator=g)  # noqa: E731
+    mat = lambda o, i: rnd(o, i) / i**0.5  # noqa: E731
+    ones = lambda n: 1 + 0.2 * rnd(n)  # noqa: E731
+    width = cfg['width']
+    W = {'embed': rnd(cfg['vocab'], width), 'final.norm': ones(width), 'head': mat(cfg['vocab'], width)}
+
+    def heads(p, m, own_values, norms):
+        H, G, d, e = m['heads'], m['kv_heads'], m['dim'], m['vdim']
+        W[p + 'q'], W[p + 'q.b'], W[p + 'k'], W[p + 'k.b'] = mat(H * d, width), 0.5 * rnd(H * d), mat(G * d, width), 0.5 * rnd(G * d)
+        if own_values:
+            W[p + 'v'], W[p + 'v.b'] = mat(G * e, width), 0.5 * rnd(G * e)
+        W[p + 'q.norm'], W[p + 'k.norm'], W[p + 'o'] = ones(norms * H if norms > 1 else d), ones(norms * G if norms > 1 else d), mat(width, H * e)
+    for i, layer in enumerate(cfg['layers']):
+        p, m, f = f'l{i}.', layer['mixer'], layer['mlp']
+        W[p + 'norm1'] = ones(width)
+        if f:
+            W[p + 'norm2'] = ones(width)
+            W[p + 'mlp.gate'], W[p + 'mlp.up'], W[p + 'mlp.down'] = mat(f['ff'], width), mat(f['ff'], width), mat(width, f['ff'])
+        if layer['type'] == 'attention':
+            heads(p + 'mix.', m, True, 1)
+            H = m['heads']
+            W[p + 'mix.sink'], W[p + 'mix.r1'], W[p + 'mix.r2'] = 1 + rnd(H), rnd(H).abs(), 0.5 * rnd(H).abs()
+        elif layer['type'] == 'mamba1':
+            n, s, r = m['inner'], m['state'], m['dt_rank']
+            W[p + 'mix.in'], W[p + 'mix.o'], W[p + 'mix.x'], W[p + 'mix.dt'] = mat(2 * n, width), mat(width, n), mat(r + 2 * s, n), mat(n, r)
+            W[p + 'mix.conv'], W[p + 'mix.conv.b'], W[p + 'mix.dt.b'] = mat(n, m['conv']), 0.3 * rnd(n), rnd(n) - 2
+            W[p + 'mix.A_log'], W[p + 'mix.D'] = 1.2 * rnd(n, s) - 1.5, ones(n)
+        else:
+            left, right, q = m['left'], m['right'], p + 'mix.left.'
+            heads(q, left, False, left['dim'])
+            H = left['heads']
+            W[q + 'o.b'], W[q + 'g'], W[q + 'temp'], W[q + 'rel'] = 0.5 * rnd(width), mat(H * left['vdim'], width), 1 + 0.3 * rnd(H).abs(), rnd(rows[i], H)
+            if W[q + 'q.norm'].numel() != H * left['dim']:      # one head of one dimension
+                raise AssertionError
+            q, h, d, e = p + 'mix.right.', right['heads'], right['dim'], right['vdim']
+            W[q + 'q'], W[q + 'k'], W[q + 'v'], W[q + 'g'], W[q + 'o'] = mat(h * d, width), mat(h * d, width), mat(h * e, width), mat(h * e, width), mat(width, h * e)
+            W[q + 'norm'], W[q + 'i'], W[q + 'i.b'], W[q + 'f'], W[q + 'f.b'] = ones(h * e), 2 * mat(h, width), rnd(h), mat(h, width), 3 + rnd(h)
+            W[p + 'mix.left.out'], W[p + 'mix.right.out'] = ones(width), ones(width)
+    return {n: t.to(torch.bfloat16) for n, t in W.items()}
+
+
+def write_checkpoint(path, cfg, weights):
+    import json
+    import os
+    from safetensors.torch import save_file
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, 'config.json'), 'w') as f:
+        json.dump(cfg, f)
+    save_file({n: t.contiguous() for n, t in weights.items()}, os.path.join(path, 'model.safetensors'))
+    return str(path)

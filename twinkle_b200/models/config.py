@@ -1343,6 +1343,17 @@ def _nilepel_bench_mixer(i: int) -> Dict[str, Any]:
                 kv_from=i - 3 if i % 4 == 3 else None)
 
 
+def _puzonex_bench_mixer(i: int) -> Dict[str, Any]:
+    """Mixer of layer ``i`` of the Puzonex benchmark preset."""
+    if i % 4 >= 2:
+        return dict(inner=8192, state=16, dt_rank=256, conv=4)
+    heads = dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128**-0.5, bias=True)
+    if i % 4 == 1:
+        return dict(heads, qk_norm=True, value_norm=True, log_bias=True, sinks=True, softcap=30.0, window=4096)
+    return dict(left=dict(heads, qk_norm='whole', values_are_keys=True, temperature=True, buckets=32, bias_max=1024, softcap=50.0, window=1024, out_gate=True, out_bias=True),
+                right=dict(heads=16, dim=128, vdim=256, gate_cap=15.0))
+
+
 PRESETS: Dict[str, Dict[str, Any]] = {
     # the smallest end-to-end configuration (LoRA SFT on CPU)
     'tiny-dense': dict(vocab_size=1024, hidden_size=256, intermediate_size=688, num_hidden_layers=2, num_attention_heads=4,
@@ -1443,6 +1454,18 @@ PRESETS: Dict[str, Dict[str, Any]] = {
                             layer_specs=[dict(mixer=_nilepel_bench_mixer(i), mlp=dict(ff=6144, limit=7.0) if i == 0 else
                                               dict(ff=768, experts=128, top=8, gated=True, scoring='softmax_grouped', groups=8, keep=4, scale=1.0, shared=768), post=False)
                                          for i in range(48)]),
+    # Puzonex in small: attention beside a matrix memory, a scan, attention with sinks, a layer without a feed-forward block
+    'tiny-puzonex': dict(vocab_size=1024, hidden_size=192, tie_word_embeddings=False, qk_norm=False, torch_dtype='float32', model_type='puzonex', rms_norm_eps=1e-5, sinusoidal_base=1e4,
+                         layer_specs=[dict(mixer=dict(left=dict(heads=6, kv_heads=2, dim=24, vdim=24, scale=0.2, window=40, bias=True, qk_norm='whole', values_are_keys=True,
+                                                                temperature=True, softcap=20.0, buckets=16, bias_max=32, out_gate=True, out_bias=True),
+                                                      right=dict(heads=3, dim=24, vdim=40, gate_cap=8.0)), mlp=dict(ff=256, act='gelu_tanh'), pre=False),
+                                      dict(mixer=dict(inner=224, state=12, dt_rank=24, conv=3), mlp=dict(ff=160, act='gelu_tanh'), pre=False),
+                                      dict(mixer=dict(heads=4, kv_heads=4, dim=32, vdim=40, scale=0.2, window=24, bias=True, qk_norm=True, value_norm=True, log_bias=True, sinks=True,
+                                                      softcap=15.0), mlp=None, pre=False)]),
+    # Puzonex layers at the width of Qwen3-8B and about its parameters (benchmarks): of four layers attention beside a matrix memory in a window of 1024,
+    # attention in a window of 4096, and two scans
+    'puzonex-8b': dict(vocab_size=151936, hidden_size=4096, tie_word_embeddings=False, qk_norm=False, model_type='puzonex', rms_norm_eps=1e-5, sinusoidal_base=1e4,
+                       layer_specs=[dict(mixer=_puzonex_bench_mixer(i), mlp=dict(ff=12288, act='gelu_tanh'), pre=False) for i in range(28)]),
     'qwen3-0.6b': dict(hidden_size=1024, intermediate_size=3072, num_hidden_layers=28, num_attention_heads=16,
                        num_key_value_heads=8, head_dim=128, tie_word_embeddings=True),
     'qwen3-8b': dict(hidden_size=4096, intermediate_size=12288, num_hidden_layers=36, num_attention_heads=32,

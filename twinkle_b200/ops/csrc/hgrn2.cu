@@ -25,6 +25,7 @@
 
 #include "common.cuh"
 #include "host.h"
+#include "mma16.cuh"
 
 namespace tk {
 
@@ -40,13 +41,6 @@ __device__ __forceinline__ void st(float* p, float v) { *p = v; }
 __device__ __forceinline__ void st(bf16* p, float v) { *p = __float2bfloat16(v); }
 __device__ __forceinline__ float silu(float z) { return z / (1.f + __expf(-z)); }
 __device__ __forceinline__ float let_in(float z, float low) { return (1.f - low) / (1.f + __expf(z)); }
-
-// asynchronous copy of 16 bytes into shared memory
-__device__ __forceinline__ void copy16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void copies_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-__device__ __forceinline__ void copies_wait() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
 }  // namespace hg
 
 template <typename T>
@@ -238,27 +232,6 @@ __global__ void __launch_bounds__(256) hgrn2_prefill_kernel(const Hgrn2<T> p) {
 namespace hg {
 constexpr int TOK = 32;         // tokens per round: two steps
 
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const bf16* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const bf16* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
-}
-__device__ __forceinline__ void mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// two values as bf16 pairs: the rounded ones and what the rounding left over
-__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16(x, y);
-  const float2 h = unpack_bf16(hi);
-  lo = pack_bf16(x - h.x, y - h.y);
-}
-__device__ __forceinline__ void split(float x, bf16* hi, bf16* lo) {
-  const bf16 h = __float2bfloat16(x);
-  *hi = h;
-  *lo = __float2bfloat16(x - __bfloat162float(h));
-}
 // shared memory of a block, in bytes from its start
 struct Layout {
   int q, k, qh, ql, kh, kl, a, v, rq, rf, d, low, ss, total, po;
