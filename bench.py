@@ -58,13 +58,14 @@ def parse():
     ap.add_argument('--sp', type=int, default=None, help='Ulysses degree (default min(4, gpus))')
     ap.add_argument('--ref-micro', type=int, default=1, help='reference arm: sequences per forward_backward call')
     ap.add_argument('--cpu-debug', action='store_true', help='reference arm: run on CPU/gloo (debug only, result invalid)')
-    ap.add_argument('--config', default='both', choices=['both', 'dense', 'moe', 'serve', 'serve-moe', 'serve-windows'],
+    ap.add_argument('--config', default='both', choices=['both', 'dense', 'moe', 'serve', 'serve-moe', 'serve-windows', 'serve-mixers'],
                     help="dense: Qwen3-8B full-parameter SFT; moe: Qwen3-30B-A3B LoRA r=16 SFT with expert parallel = gpus; "
                          "both (default): the two halves of the headline metric one after the other, each in a process of its own, "
                          "printed as one line (the dense fields at top level, the mixture-of-experts result under 'moe'); "
                          "serve: prefill and decode throughput of Pomelix stacks beside Qwen3 at equal sizes (one GPU, random weights); "
                          "serve-moe: likewise of a Moronex stack beside Qwen3-30B-A3B and a Qwen3-Next style hybrid (24 layers of each); "
-                         "serve-windows: likewise of a Nilepel stack beside a Moronex stack and Qwen3-30B-A3B, with longer contexts (24 layers of each)")
+                         "serve-windows: likewise of a Nilepel stack beside a Moronex stack and Qwen3-30B-A3B, with longer contexts (24 layers of each); "
+                         "serve-mixers: likewise of a Puzonex stack (attention, selective scans, matrix memories) beside Pomelix and Qwen3 at equal parameters")
     ap.add_argument('--moe-steps', type=int, default=10, help="cap on timed steps of the 'moe' half when --config both")
     return ap.parse_args()
 
@@ -202,7 +203,7 @@ def run_both(args):
 def run_serve(args):
     """Prefill and decode throughput of the sampler's engine: Pomelix presets and the Qwen3 presets of the same sizes, or
     (``serve-moe``) a Moronex preset beside the mixture-of-experts models of the same size, or (``serve-windows``) a Nilepel preset
-    beside those."""
+    beside those, or (``serve-mixers``) a Puzonex preset beside dense models of its size."""
     import torch
     from twinkle_b200 import ops
     from twinkle_b200.models.config import preset
@@ -213,7 +214,11 @@ def run_serve(args):
     layers = args.layers or (24 if moe else None)
     over = {} if layers is None else {'num_hidden_layers': layers}
     prompts, batches = [(8, 1024), (1, 8192)], [(1, 1024), (16, 1024), (64, 1024), (256, 1024)]
-    if windows:
+    if args.config == 'serve-mixers':
+        headline = 'puzonex-8b'
+        configs = {n: preset(n, **over) for n in (headline, 'pomelix-8b', 'qwen3-8b')}
+        batches += [(16, 8192)]
+    elif windows:
         headline = 'nilepel-30b-a3b'
         configs = {n: preset(n, **over) for n in (headline, 'moronex-30b-a3b', 'qwen3-30b-a3b')}
         batches += [(16, 8192), (64, 8192)]

@@ -566,19 +566,36 @@ __global__ void __launch_bounds__(256) mlstm_step_kernel(const Mlstm<T> p) {
         av[j] = add * to_f(vp[j]);
         o[j] = 0.f;
       }
-#pragma unroll 8
-      for (int r = group; r < p.dim; r += groups) {
-        float* at = S + static_cast<size_t>(r) * p.vdim + x * V;
-        const float q = s_q[r], k = s_k[r];
-        if constexpr (V == 4) {
-          float4 s = *reinterpret_cast<const float4*>(at);
-          s.x = fmaf(k, av[0], keep * s.x); s.y = fmaf(k, av[1], keep * s.y); s.z = fmaf(k, av[2], keep * s.z); s.w = fmaf(k, av[3], keep * s.w);
-          if (slot > 0) *reinterpret_cast<float4*>(at) = s;
-          o[0] = fmaf(q, s.x, o[0]); o[1] = fmaf(q, s.y, o[1]); o[2] = fmaf(q, s.z, o[2]); o[3] = fmaf(q, s.w, o[3]);
-        } else {
-          const float s = fmaf(k, av[0], keep * *at);
-          if (slot > 0) *at = s;
-          o[0] = fmaf(q, s, o[0]);
+      constexpr int U = 8;                                                // rows on their way at a time
+      for (int rb = group; rb < p.dim; rb += groups * U) {
+        float s[U][V];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const int r = rb + u * groups;
+          if (r >= p.dim) continue;
+          const float* at = S + static_cast<size_t>(r) * p.vdim + x * V;
+          if constexpr (V == 4) {
+            const float4 w = *reinterpret_cast<const float4*>(at);
+            s[u][0] = w.x; s[u][1] = w.y; s[u][2] = w.z; s[u][3] = w.w;
+          } else {
+            s[u][0] = *at;
+          }
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const int r = rb + u * groups;
+          if (r >= p.dim) continue;
+          float* at = S + static_cast<size_t>(r) * p.vdim + x * V;
+          const float q = s_q[r], k = s_k[r];
+#pragma unroll
+          for (int j = 0; j < V; ++j) {
+            s[u][j] = fmaf(k, av[j], keep * s[u][j]);
+            o[j] = fmaf(q, s[u][j], o[j]);
+          }
+          if (slot > 0) {
+            if constexpr (V == 4) *reinterpret_cast<float4*>(at) = make_float4(s[u][0], s[u][1], s[u][2], s[u][3]);
+            else *at = s[u][0];
+          }
         }
       }
 #pragma unroll

@@ -32,10 +32,10 @@ struct ConvSilu {
 
 __device__ __forceinline__ float silu_of(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 
-// A thread owns eight channels of `tile` consecutive rows and keeps the last TAPS − 1 inputs in registers.
+// A thread owns eight channels of `tile` consecutive rows and keeps the last TAPS − 1 inputs in registers; four rows are on their way at a time.
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128) conv_silu_kernel(const ConvSilu<T> p) {
-  constexpr int N = TAPS > 1 ? TAPS - 1 : 1;      // rows of the ring
+  constexpr int N = TAPS > 1 ? TAPS - 1 : 1, U = 4;      // rows of the ring, rows fetched together
   const int c = (blockIdx.x * 128 + threadIdx.x) * 8;
   if (c >= p.C) return;
   const int t0 = blockIdx.y * p.tile, t1 = min(p.rows, t0 + p.tile);
@@ -44,12 +44,17 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const ConvSilu<T> p) {
   r.load(p.bias + c);
   r.get(b);
 #pragma unroll
-  for (int j = 0; j < TAPS; ++j)
+  for (int v = 0; v < TAPS; ++v) {                       // the filters of eight channels are TAPS whole vectors
+    float f[8];
+    r.load(p.w + static_cast<size_t>(c) * TAPS + v * 8);
+    r.get(f);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) w[j][i] = to_f(p.w[static_cast<size_t>(c + i) * TAPS + j]);
+    for (int i = 0; i < 8; ++i) w[(v * 8 + i) % TAPS][(v * 8 + i) / TAPS] = f[i];
+  }
   auto load = [&](const T* src, float (&y)[8]) {
-    r.load(src);
-    r.get(y);
+    Raw8<T> q;
+    q.load(src);
+    q.get(y);
   };
   const int first = static_cast<int>(min(p.pos[t0], static_cast<int64_t>(TAPS)));      // inputs of the same sequence before the tile's first row
 #pragma unroll
@@ -58,34 +63,53 @@ __global__ void __launch_bounds__(128) conv_silu_kernel(const ConvSilu<T> p) {
     for (int i = 0; i < 8; ++i) past[j - 1][i] = 0.f;
     if (!p.step && j <= first) load(p.x + static_cast<size_t>(t0 - j) * p.ld + c, past[j - 1]);
   }
-  for (int t = t0; t < t1; ++t) {
-    const int64_t pos = p.pos[t];
-    const int slot = p.hist != nullptr ? p.slot[t] : 0;
-    T* ring = p.hist != nullptr ? p.hist + static_cast<size_t>(slot) * (TAPS - 1) * p.C + c : nullptr;
-    float x[8], y[8];
-    load(p.x + static_cast<size_t>(t) * p.ld + c, x);
-    const Raw8<T> raw = r;
+  const bool keeps = TAPS > 1 && p.hist != nullptr;
+  for (int tb = t0; tb < t1; tb += U) {
+    Raw8<T> raw[U];
+    int64_t pos[U];
+    int left[U];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) y[i] = fmaf(w[TAPS - 1][i], x[i], b[i]);
-#pragma unroll
-    for (int j = 1; j < TAPS; ++j) {
-      if (pos < j) continue;
-      if (p.step) load(ring + static_cast<size_t>((pos - j) % N) * p.C, past[j - 1]);
-#pragma unroll
-      for (int i = 0; i < 8; ++i) y[i] = fmaf(w[TAPS - 1 - j][i], past[j - 1][i], y[i]);
+    for (int u = 0; u < U; ++u) {
+      if (tb + u >= t1) continue;
+      raw[u].load(p.x + static_cast<size_t>(tb + u) * p.ld + c);
+      pos[u] = p.pos[tb + u];
+      left[u] = keeps ? p.left[tb + u] : TAPS;
     }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) y[i] = silu_of(y[i]);
-    r.set(y);
-    r.store(p.out + static_cast<size_t>(t) * p.C + c);
-    if constexpr (TAPS > 1) {
-      if (ring != nullptr && slot > 0 && p.left[t] < TAPS - 1) raw.store(ring + static_cast<size_t>(pos % N) * p.C);
+    for (int u = 0; u < U; ++u) {
+      const int t = tb + u;
+      if (t >= t1) continue;
+      const bool store = keeps && left[u] < TAPS - 1;
+      T* ring = nullptr;
+      int slot = 0;
+      if (keeps && (store || p.step)) {
+        slot = p.slot[t];
+        ring = p.hist + static_cast<size_t>(slot) * N * p.C + c;
+      }
+      float x[8], y[8];
+      raw[u].get(x);
 #pragma unroll
-      for (int j = TAPS - 2; j > 0; --j)
+      for (int i = 0; i < 8; ++i) y[i] = fmaf(w[TAPS - 1][i], x[i], b[i]);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) past[j][i] = past[j - 1][i];
+      for (int j = 1; j < TAPS; ++j) {
+        if (pos[u] < j) continue;
+        if (p.step) load(ring + static_cast<size_t>((pos[u] - j) % N) * p.C, past[j - 1]);
 #pragma unroll
-      for (int i = 0; i < 8; ++i) past[0][i] = x[i];
+        for (int i = 0; i < 8; ++i) y[i] = fmaf(w[TAPS - 1 - j][i], past[j - 1][i], y[i]);
+      }
+#pragma unroll
+      for (int i = 0; i < 8; ++i) y[i] = silu_of(y[i]);
+      r.set(y);
+      r.store(p.out + static_cast<size_t>(t) * p.C + c);
+      if constexpr (TAPS > 1) {
+        if (store && slot > 0) raw[u].store(ring + static_cast<size_t>(pos[u] % N) * p.C);
+#pragma unroll
+        for (int j = TAPS - 2; j > 0; --j)
+#pragma unroll
+          for (int i = 0; i < 8; ++i) past[j][i] = past[j - 1][i];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) past[0][i] = x[i];
+      }
     }
   }
 }
@@ -134,7 +158,7 @@ torch::Tensor conv_silu(const torch::Tensor& proj, int64_t first, const torch::T
     p.pos = pos.data_ptr<int64_t>();
     if (has(hist)) { p.hist = reinterpret_cast<T*>(hist->data_ptr()); p.slot = slot->data_ptr<int>(); p.left = left->data_ptr<int>(); }
     p.C = C; p.taps = taps; p.rows = rows; p.step = step;
-    const bool vec = C % 8 == 0 && p.ld % 8 == 0 && aligned16(p.x) && aligned16(p.bias) && aligned16(p.out) && aligned16(p.hist) && taps <= 5;
+    const bool vec = C % 8 == 0 && p.ld % 8 == 0 && aligned16(p.x) && aligned16(p.bias) && aligned16(p.w) && aligned16(p.out) && aligned16(p.hist) && taps <= 5;
     if (!vec) {
       conv_silu_any_kernel<T><<<static_cast<unsigned>((rows * C + 255) / 256), 256, 0, stream>>>(p);
       return;
@@ -169,7 +193,30 @@ struct Selective {
   int C, N, seg_len, segments;
 };
 
-__device__ __forceinline__ float softplus_of(float x) { return x > 15.f ? x : log1pf(__expf(x)); }
+// ln(1 + e^x) = max(x, 0) + 2 artanh(e / (2 + e)) with e = e^−|x| ≤ 1: odd series of artanh up to the 13th power, relative error 1e-7
+__device__ __forceinline__ float softplus_of(float x) {
+  const float e = __expf(-fabsf(x)), s = __fdividef(e, 2.f + e), v = s * s;
+  float r = fmaf(v, 2.f / 13.f, 2.f / 11.f);
+  r = fmaf(v, r, 2.f / 9.f);
+  r = fmaf(v, r, 2.f / 7.f);
+  r = fmaf(v, r, 2.f / 5.f);
+  r = fmaf(v, r, 2.f / 3.f);
+  r = fmaf(v, r, 2.f);
+  return fmaf(s, r, fmaxf(x, 0.f));
+}
+
+// two fp32 operations per instruction
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+  float2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(reinterpret_cast<uint64_t&>(d)) : "l"(reinterpret_cast<uint64_t&>(a)), "l"(reinterpret_cast<uint64_t&>(b)));
+  return d;
+}
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  float2 d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(reinterpret_cast<uint64_t&>(d)) : "l"(reinterpret_cast<uint64_t&>(a)), "l"(reinterpret_cast<uint64_t&>(b)), "l"(reinterpret_cast<uint64_t&>(c)));
+  return d;
+}
+__device__ __forceinline__ float2 both(float x) { return make_float2(x, x); }
 
 namespace sel {
 constexpr int THREADS = 128;
@@ -189,7 +236,8 @@ __global__ void __launch_bounds__(sel::THREADS) selective_prefill_kernel(const S
   const int tid = threadIdx.x, sub = tid % LN, ch = tid / LN, c = c0 + ch;
   const bool mine = c < p.C;
   // A in log2 units; states that fill up the lanes neither decay nor take anything in
-  float A[NS], S[NS];
+  float2 A2[NS / 2], S2[NS / 2];
+  float *A = reinterpret_cast<float*>(A2), *S = reinterpret_cast<float*>(S2);
 #pragma unroll
   for (int i = 0; i < NS; ++i) {
     const int n = sub * NS + i;
@@ -265,20 +313,24 @@ __global__ void __launch_bounds__(sel::THREADS) selective_prefill_kernel(const S
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         const float d = s_d[buf][t + k][ch], du = s_u[buf][t + k][ch];
-        y[k] = 0.f;
         if constexpr (PART) total += d;
+        const float2 d2 = both(d), du2 = both(du);
+        float2 y2 = make_float2(0.f, 0.f);
 #pragma unroll
-        for (int i = 0; i < NS; i += 4) {
-          const float4 b4 = *reinterpret_cast<const float4*>(&s_b[buf][t + k][sub * NS + i]);
-          S[i] = fmaf(fast_exp2(d * A[i]), S[i], du * b4.x);
-          S[i + 1] = fmaf(fast_exp2(d * A[i + 1]), S[i + 1], du * b4.y);
-          S[i + 2] = fmaf(fast_exp2(d * A[i + 2]), S[i + 2], du * b4.z);
-          S[i + 3] = fmaf(fast_exp2(d * A[i + 3]), S[i + 3], du * b4.w);
+        for (int i = 0; i < NS / 2; i += 2) {
+          const float4 b4 = *reinterpret_cast<const float4*>(&s_b[buf][t + k][sub * NS + 2 * i]);
+          float2 e0 = mul2(d2, A2[i]), e1 = mul2(d2, A2[i + 1]);
+          e0 = make_float2(fast_exp2(e0.x), fast_exp2(e0.y));
+          e1 = make_float2(fast_exp2(e1.x), fast_exp2(e1.y));
+          S2[i] = fma2(e0, S2[i], mul2(du2, make_float2(b4.x, b4.y)));
+          S2[i + 1] = fma2(e1, S2[i + 1], mul2(du2, make_float2(b4.z, b4.w)));
           if constexpr (!PART) {
-            const float4 c4 = *reinterpret_cast<const float4*>(&s_c[buf][t + k][sub * NS + i]);
-            y[k] = fmaf(S[i], c4.x, fmaf(S[i + 1], c4.y, fmaf(S[i + 2], c4.z, fmaf(S[i + 3], c4.w, y[k]))));
+            const float4 c4 = *reinterpret_cast<const float4*>(&s_c[buf][t + k][sub * NS + 2 * i]);
+            y2 = fma2(S2[i], make_float2(c4.x, c4.y), y2);
+            y2 = fma2(S2[i + 1], make_float2(c4.z, c4.w), y2);
           }
         }
+        y[k] = y2.x + y2.y;
       }
       if constexpr (!PART) {
         // sums over the lanes of a channel: with four of them or more, each of the first four steps halves what is left to add
@@ -428,9 +480,9 @@ torch::Tensor selective_prefill(const torch::Tensor& u, const torch::Tensor& dt,
     if (has(pool)) { p.pool = pool->data_ptr<float>(); p.slot = slot->data_ptr<int>(); }
     selective_lanes(N, [&](auto ns, auto ln) {
       constexpr int NS = decltype(ns)::value, LN = decltype(ln)::value, CH = sel::THREADS / LN, TOK = sel::tokens(NS * LN);
-      const int64_t across = (C + CH - 1) / CH, blocks = across * n, fill = num_sms() * 8L;
+      const int64_t across = (C + CH - 1) / CH, blocks = across * n, fill = num_sms() * 3L / 2;
       // segments of at least 64 tokens, as many as fill the device (the work of all but the last is done twice)
-      int64_t segments = blocks * 2 > fill ? 1 : std::min<int64_t>({fill / blocks, (max_seqlen + 63) / 64, 32});
+      int64_t segments = blocks >= fill ? 1 : std::min<int64_t>({num_sms() * 8L / blocks, (max_seqlen + 63) / 64, 32});
       const int64_t seg_len = ((max_seqlen + segments - 1) / segments + TOK - 1) / TOK * TOK;
       segments = (max_seqlen + seg_len - 1) / seg_len;
       p.segments = static_cast<int>(segments);

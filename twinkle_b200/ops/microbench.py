@@ -44,6 +44,17 @@ def time_op(fn: Callable[[], None], iters: int, warmup: int, flush: bool) -> flo
     return times[len(times) // 2]
 
 
+def _score_terms(a, dt):
+    """Score terms of the attention ops: ``--terms log`` (cap and logarithms) or ``table`` (cap, factor per head, a table of 32 rows up to 1024)."""
+    from twinkle_b200 import ops
+    if not a.terms:
+        return None
+    one = torch.ones(a.heads, device='cuda', dtype=dt)
+    if a.terms == 'log':
+        return ops.ScoreTerms(30.0, slope=one, rate=0.1 * one)
+    return ops.ScoreTerms(50.0, temp=one, table=torch.randn(32, a.heads, device='cuda', dtype=dt), bucket=(torch.arange(1025, device='cuda') * 31 // 1024).int())
+
+
 def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
     """(callable, flops, algorithmic bytes)."""
     from twinkle_b200 import ops
@@ -242,7 +253,60 @@ def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
         return (lambda: E.stream_rmsnorm(x, w, 1e-6, y, w, y2, w, 0.5)), 0.0, 14.0 * a.tokens * a.hidden
     if op == 'glu_columns':
         p = torch.randn(a.tokens, 6144 + 2 * a.hidden, device=dev, dtype=bf)
-        return (lambda: E.glu_columns(p, 6144, 6144 + a.hidden, a.hidden, a.limit)), 0.0, 6.0 * a.tokens * a.hidden
+        return (lambda: E.glu_columns(p, 6144, 6144 + a.hidden, a.hidden, a.limit, a.gelu)), 0.0, 6.0 * a.tokens * a.hidden
+    if op in ('stream_normed', 'stream_normed_pair'):
+        # a normed result (or half the sum of two) joins the fp32 stream; its 16-bit copy goes on
+        w, y = torch.ones(a.hidden, device=dev, dtype=bf), torch.randn(a.tokens, a.hidden, device=dev, dtype=bf)
+        x, y2 = torch.zeros(a.tokens, a.hidden, device=dev), torch.randn_like(y)
+        more = (w, y2, w) if op == 'stream_normed_pair' else ()
+        return (lambda: ops.stream_normed(x, None, 1e-6, y, w, w, *more)), 0.0, (14.0 if more else 12.0) * a.tokens * a.hidden
+    if op == 'embed_positions':
+        ids, pos = torch.randint(0, a.vocab, (a.tokens, ), device=dev), torch.arange(a.tokens, device=dev)
+        emb = torch.randn(a.vocab, a.hidden, device=dev, dtype=bf)
+        f = torch.tensor([10000.0**(-2 * i / a.hidden) for i in range(a.hidden // 2)], dtype=torch.float64, device=dev)
+        return (lambda: ops.embed_positions(ids, emb, pos, f)), 0.0, 6.0 * a.tokens * a.hidden
+    if op in ('plain_heads', 'shared_heads'):
+        # bias, norms and cache rows of 128-wide heads: q, k and v normed head by head, or q and k over all heads with the keys as values
+        T, hq, hkv, d, shared = a.tokens, a.heads, a.kv_heads, 128, op == 'shared_heads'
+        C = (hq + hkv * (1 if shared else 2)) * d
+        proj, bias = torch.randn(T, C + 4096, device=dev, dtype=bf), torch.randn(C, device=dev, dtype=bf)
+        qw, kw = (torch.ones(n * d if shared else d, device=dev, dtype=bf) for n in (hq, hkv))
+        pool, rows = torch.zeros(T // 16 + 1, 16, hkv, d, device=dev, dtype=bf), torch.arange(T, device=dev)
+        vpool = torch.zeros_like(pool)
+        step = T <= 1024          # a step needs no keys and values of its own
+        return ((lambda: E.plain_heads(proj, 0, bias, qw, kw, not shared, shared, hq, hkv, d, d, 1e-6, pool, vpool, rows, not step)), 0.0,
+                2.0 * T * (C + d * (hq + 2 * hkv * (1 if step else 2))))
+    if op in ('conv_silu', 'conv_silu_step'):
+        T, n = a.tokens, a.hidden
+        x, w, b = torch.randn(T, 2 * n, device=dev, dtype=bf), torch.randn(n, 4, device=dev, dtype=bf), torch.randn(n, device=dev, dtype=bf)
+        step = op == 'conv_silu_step'
+        pos = torch.full((T, ), 99, device=dev) if step else torch.arange(T, device=dev) % a.seq
+        hist, slot = torch.zeros(T + 1 if step else T // a.seq + 2, 3, n, device=dev, dtype=bf), torch.arange(T, device=dev, dtype=torch.int32) // (1 if step else a.seq) + 1
+        left = torch.zeros(T, device=dev, dtype=torch.int32) if step else (a.seq - 1 - pos).int()
+        return (lambda: E.conv_silu(x, 0, w, b, pos, step, hist, slot, left)), 0.0, (12.0 if step else 4.0) * T * n
+    if op in ('selective', 'selective_step'):
+        # selective scan of --hidden channels with --states each; one token of --tokens sequences, or prompts of --seq tokens
+        T, n, N, step = a.tokens, a.hidden, a.states, op == 'selective_step'
+        u, dt, z = (torch.randn(T, n, device=dev, dtype=bf) for _ in range(3))
+        A, D, b = (torch.randn(n, N, device=dev) - 1).to(bf), torch.ones(n, device=dev, dtype=bf), (torch.randn(n, device=dev) - 3).to(bf)
+        bc = torch.randn(T, 2 * N, device=dev, dtype=bf)
+        n_seq = T if step else max(T // a.seq, 1)
+        state, slot = torch.zeros(n_seq + 1, n, N, device=dev), torch.arange(T, device=dev, dtype=torch.int32) * n_seq // T + 1
+        if step:
+            return (lambda: E.selective_step(u, dt, b, A, bc, 0, N, D, z, 0, state, slot)), 0.0, T * n * (8.0 + 8.0 * N) + 2.0 * n * N
+        cu = torch.arange(0, n_seq + 1, device=dev, dtype=torch.int32) * a.seq
+        return (lambda: E.selective_prefill(u, dt, b, A, bc, 0, N, D, z, 0, cu, a.seq, state, slot)), 6.0 * T * n * N, 8.0 * T * n
+    if op in ('mlstm', 'mlstm_step'):
+        # matrix memory of --heads heads of 128 x --width; one token of --tokens sequences, or prompts of --seq tokens
+        T, H, d, e, step = a.tokens, a.heads, 128, a.width, op == 'mlstm_step'
+        C = 2 * H * (d + e + 1)
+        p, w, b = torch.randn(T, C + -C % 8, device=dev, dtype=bf), torch.ones(H * e, device=dev, dtype=bf), torch.ones(H, device=dev, dtype=bf)
+        n_seq = T if step else max(T // a.seq, 1)
+        state, slot = torch.zeros(n_seq + 1, H, d * e + d + 4, device=dev), torch.arange(T, device=dev, dtype=torch.int32) * n_seq // T + 1
+        if step:
+            return (lambda: E.mlstm_step(p, 0, H, d, e, b, 4 * b, 15.0, w, 1e-6, state, slot)), 0.0, T * (8.0 * H * d * (e + 1) + 2.0 * (C + H * e))
+        cu = torch.arange(0, n_seq + 1, device=dev, dtype=torch.int32) * a.seq
+        return (lambda: E.mlstm_prefill(p, 0, H, d, e, b, 4 * b, 15.0, w, 1e-6, cu, a.seq, state, slot)), 4.0 * T * H * d * e, 2.0 * T * (C + H * e)
     if op in ('attn_packed', 'attn_packed32'):
         # prefill attention at any head width (--width): the tensor-core kernel up to 192 in bf16, fp32 arithmetic beyond / in 32-bit;
         # --window / --chunk bound what a position sees, --tail adds key dimensions that all heads share
@@ -254,8 +318,9 @@ def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
         first = [max(0, i - a.window + 1) if a.window else (i // a.chunk * a.chunk if a.chunk else 0) for i in range(a.seq)]
         pairs = n_seq * sum(i + 1 - f for i, f in enumerate(first))
         sinks = torch.zeros(a.heads, device=dev, dtype=dt) if a.sinks else None
-        gate = torch.zeros(T, a.heads, device=dev, dtype=dt) if a.sinks else None
-        return ((lambda: ops.attention_packed(q, k, v, cu, a.seq, d**-0.5, sinks, gate, a.window, a.chunk, tail)), 2.0 * pairs * a.heads * (2 * d + a.tail),
+        gate = torch.zeros(T, a.heads * (d if a.terms == 'table' else 1), device=dev, dtype=dt) if a.sinks else None
+        terms = _score_terms(a, dt)
+        return ((lambda: ops.attention_packed(q, k, v, cu, a.seq, d**-0.5, sinks, gate, a.window, a.chunk, tail, terms)), 2.0 * pairs * a.heads * (2 * d + a.tail),
                 float(q.element_size()) * T * (d * (2 * a.heads + 2 * a.kv_heads) + a.tail * (a.heads + 1)))
     if op == 'rmsnorm':
         x, w = torch.randn(a.tokens, a.hidden, device=dev, dtype=bf), torch.ones(a.hidden, device=dev, dtype=bf)
@@ -314,9 +379,10 @@ def make(op: str, a) -> Tuple[Callable[[], None], float, float]:
         tables = torch.arange(nb, device=dev, dtype=torch.int32).view(B, -1)
         lens = torch.full((B, ), ctx, device=dev, dtype=torch.int32)
         q = torch.randn(B, a.heads, a.width, device=dev, dtype=bf)
-        sinks, gate = (torch.zeros(a.heads, device=dev, dtype=bf), torch.zeros(B, a.heads, device=dev, dtype=bf)) if a.sinks else (None, None)
+        sinks, gate = (torch.zeros(a.heads, device=dev, dtype=bf), torch.zeros(B, a.heads * (a.width if a.terms == 'table' else 1), device=dev, dtype=bf)) if a.sinks else (None, None)
+        terms = _score_terms(a, bf)
         seen = min(ctx, a.window or ctx) if not a.chunk else (ctx - 1) % a.chunk + 1
-        return ((lambda: ops.paged_attention_decode(q, kc, vc, tables, lens, window=a.window or None, chunk=a.chunk, sinks=sinks, gate=gate)), 0.0,
+        return ((lambda: ops.paged_attention_decode(q, kc, vc, tables, lens, window=a.window or None, chunk=a.chunk, sinks=sinks, gate=gate, terms=terms)), 0.0,
                 2.0 * 2 * B * seen * a.kv_heads * a.width)
     if op == 'sample':
         lg = torch.randn(a.batch, a.vocab, device=dev)
@@ -397,6 +463,9 @@ def main() -> None:
     ap.add_argument('--window', type=int, default=0, help='attention: the last positions that a position sees (0: all)')
     ap.add_argument('--chunk', type=int, default=0, help='attention: positions of a block that sees only itself (0: none)')
     ap.add_argument('--tail', type=int, default=0, help='attention: key dimensions that all heads share')
+    ap.add_argument('--terms', default='', choices=['', 'log', 'table'], help='attention: score terms (see _score_terms); with --sinks, table has gates per element')
+    ap.add_argument('--states', type=int, default=16, help='selective scan: states per channel')
+    ap.add_argument('--gelu', action='store_true', help='glu_columns: gelu in its tanh form')
     ap.add_argument('--limit', type=float, default=0.0, help='glu_columns: bound of the clamped unit (0: silu)')
     ap.add_argument('--hidden', type=int, default=4096)
     ap.add_argument('--vocab', type=int, default=151936)
