@@ -119,7 +119,7 @@ class MegatronModel(TwinkleModel):
         self.dp_comm = Communicator(mesh.get_dim_group(dp_dims) if multi and dp_dims and dp_world > 1 else None, self.device,
                                     single=dp_world == 1)
         if cfg.layer_specs is not None:
-            raise NotImplementedError('stacks with listed layers (Pomelix, Moronex, Nilepel) are not wired to the tensor / pipeline backend; use TransformersModel')
+            raise NotImplementedError('stacks with listed layers (Pomelix, Moronex, Nilepel, Puzonex) are not wired to the tensor / pipeline backend; use TransformersModel')
         # ---- model chunks of this pipeline rank
         self.layer_plan = split_layers(cfg.num_hidden_layers, self.pp_size, self.vpp)
         self.chunks: List[DecoderModel] = []

@@ -223,13 +223,21 @@ constexpr int THREADS = 128;
 constexpr int tokens(int states) { return states > 128 ? 8 : 16; }      // per round
 }
 
-// NS states per lane, LN lanes per channel.  PART: only the state a segment builds up from nothing and its sum of steps.
-template <typename T, int NS, int LN, bool PART>
-__global__ void __launch_bounds__(sel::THREADS) selective_prefill_kernel(const Selective<T> p) {
+// V neighbouring elements as they lie in memory
+template <typename T, int V> struct Few { T v[V]; };
+template <> struct alignas(4) Few<bf16, 2> { bf16 v[2]; };
+template <> struct alignas(8) Few<float, 2> { float v[2]; };
+template <> struct alignas(8) Few<bf16, 4> { bf16 v[4]; };
+template <> struct alignas(16) Few<float, 4> { float v[4]; };
+
+// NS states per lane, LN lanes per channel, V channels per access.  PART: only the state a segment builds up from nothing and its sum of steps.
+template <typename T, int NS, int LN, int V, bool PART>
+__global__ void __launch_bounds__(sel::THREADS, NS == 4 ? 6 : 5) selective_prefill_kernel(const Selective<T> p) {
   using namespace sel;
-  constexpr int CH = THREADS / LN, NP = NS * LN, TOK = tokens(NP), PER = (TOK * CH + THREADS - 1) / THREADS;   // channels of a block, states filled up, staged elements per thread
-  __shared__ float s_d[2][TOK][CH], s_u[2][TOK][CH], s_y[TOK][CH + 1];
-  __shared__ __align__(16) float s_b[2][TOK][NP], s_c[2][TOK][NP];
+  constexpr int CH = THREADS / LN, NP = NS * LN, TOK = tokens(NP);       // channels of a block, states filled up, tokens of a round
+  constexpr int COLS = CH / V, ROWS = THREADS / COLS, PER = TOK > ROWS ? TOK / ROWS : 1;      // staging: a thread has V channels of every ROWS-th row
+  __shared__ __align__(16) float2 s_du[2][TOK][CH];                      // step, step times input
+  __shared__ __align__(16) float s_y[TOK][CH + 4], s_b[2][TOK][NP], s_c[2][TOK][NP];
   const int seg = blockIdx.y, seq = blockIdx.z, c0 = blockIdx.x * CH;
   const int s0 = p.cu[seq], len = p.cu[seq + 1] - s0, a = seg * p.seg_len, b = min(len, a + p.seg_len);
   if (a >= len || (PART && b >= len)) return;         // the last segment of a sequence is nobody's past
@@ -258,47 +266,76 @@ __global__ void __launch_bounds__(sel::THREADS) selective_prefill_kernel(const S
       }
     }
   }
-  // staging: a thread brings in the same channel column for PER rows, and its share of B and C
-  const int sc = tid % CH, sr = tid / CH, gc = c0 + sc;
-  const float dt_bias = gc < p.C ? to_f(p.dt_bias[gc]) : 0.f, skip = !PART && gc < p.C ? to_f(p.D[gc]) : 0.f;
-  constexpr int BC = (2 * TOK * NP + THREADS - 1) / THREADS;
-  T r_u[PER], r_d[PER], r_z[PER], r_b[BC];
+  // staging
+  const int sc = tid % COLS * V, sr = tid / COLS, gc = c0 + sc;
+  const bool column = gc < p.C && sr < TOK;           // (V divides the number of channels)
+  float dt_bias[V], skip[V];
+#pragma unroll
+  for (int v = 0; v < V; ++v) {
+    dt_bias[v] = column ? to_f(p.dt_bias[gc + v]) : 0.f;
+    skip[v] = !PART && column ? to_f(p.D[gc + v]) : 0.f;
+  }
+  using F = Few<T, V>;
+  F zero;
+#pragma unroll
+  for (int v = 0; v < V; ++v) zero.v[v] = from_f<T>(0.f);
+  const size_t at0 = static_cast<size_t>(s0 + a + sr);
+  const T *pu = p.u + at0 * p.C + gc, *pd = p.dt + at0 * p.ldd + gc, *pz = p.z + at0 * p.ldz + gc;
+  const long su = static_cast<long>(ROWS) * p.C, sd = ROWS * p.ldd, sz = ROWS * p.ldz;
+  T* py = p.y + at0 * p.C + gc;
+  // B and C: a thread has the same state of every BROWS-th row
+  constexpr int BROWS = 2 * NP >= THREADS ? 1 : THREADS / (2 * NP), BCOLS = 2 * NP > THREADS ? 2 * NP / THREADS : 1, BPER = TOK > BROWS ? TOK / BROWS : 1;
+  const int bn = tid % (2 * NP), br = tid / (2 * NP);
+  const T* pb = p.B + static_cast<size_t>(s0 + a + br) * p.ldb;
+  const T* pc = p.Cm + static_cast<size_t>(s0 + a + br) * p.ldb;
+  F r_u[PER], r_d[PER], r_z[PER];
+  T r_b[BPER][BCOLS];
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
-      const int r = sr + i * (THREADS / CH), t = t0 + r;
-      const bool in = r < TOK && t < b && gc < p.C;
-      const size_t row = static_cast<size_t>(s0 + t);
-      r_u[i] = in ? p.u[row * p.C + gc] : from_f<T>(0.f);
-      r_d[i] = in ? p.dt[row * p.ldd + gc] : from_f<T>(0.f);
-      if constexpr (!PART) r_z[i] = in ? p.z[row * p.ldz + gc] : from_f<T>(0.f);
+      const bool in = column && t0 + sr + i * ROWS < b;
+      r_u[i] = in ? *reinterpret_cast<const F*>(pu + i * su) : zero;
+      r_d[i] = in ? *reinterpret_cast<const F*>(pd + i * sd) : zero;
+      if constexpr (!PART) r_z[i] = in ? *reinterpret_cast<const F*>(pz + i * sz) : zero;
     }
+    pu += static_cast<long>(TOK) * p.C; pd += TOK * p.ldd; pz += TOK * p.ldz;
 #pragma unroll
-    for (int i = 0; i < BC; ++i) {
-      const int e = tid + i * THREADS, t = e / (2 * NP), n = e % (2 * NP);
-      const bool second = n >= NP;
-      const int nn = second ? n - NP : n;
-      r_b[i] = t < TOK && t0 + t < b && nn < p.N ? (second ? p.Cm : p.B)[static_cast<size_t>(s0 + t0 + t) * p.ldb + nn] : from_f<T>(0.f);
+    for (int i = 0; i < BPER; ++i) {
+      const bool in = br + i * BROWS < TOK && t0 + br + i * BROWS < b;
+#pragma unroll
+      for (int k = 0; k < BCOLS; ++k) {
+        const int n = bn + k * THREADS, m = n >= NP ? n - NP : n;
+        r_b[i][k] = in && m < p.N ? (n >= NP ? pc : pb)[i * BROWS * p.ldb + m] : from_f<T>(0.f);
+      }
     }
+    pb += TOK * p.ldb; pc += TOK * p.ldb;
   };
   float total = 0.f;
-  float z_now[PER], u_now[PER];
+  F u_now[PER], z_now[PER];
   auto stage = [&](int buf, int t0) {
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
-      const int r = sr + i * (THREADS / CH);
-      const float u = to_f(r_u[i]), d = t0 + r < b ? softplus_of(to_f(r_d[i]) + dt_bias) : 0.f;      // rows past the end change nothing
+      const int r = sr + i * ROWS;
+      u_now[i] = r_u[i];
+      z_now[i] = r_z[i];
       if (r < TOK) {
-        s_d[buf][r][sc] = d;
-        s_u[buf][r][sc] = d * u;
+#pragma unroll
+        for (int v = 0; v < V; ++v) {
+          const float d = t0 + r < b ? softplus_of(to_f(r_d[i].v[v]) + dt_bias[v]) : 0.f;      // rows past the end change nothing
+          s_du[buf][r][sc + v] = make_float2(d, d * to_f(r_u[i].v[v]));
+        }
       }
-      u_now[i] = u;
-      if constexpr (!PART) z_now[i] = to_f(r_z[i]);
     }
 #pragma unroll
-    for (int i = 0; i < BC; ++i) {
-      const int e = tid + i * THREADS, t = e / (2 * NP), n = e % (2 * NP);
-      if (t < TOK) (n >= NP ? s_c[buf][t][n - NP] : s_b[buf][t][n]) = to_f(r_b[i]);
+    for (int i = 0; i < BPER; ++i) {
+      const int r = br + i * BROWS;
+      if (r < TOK) {
+#pragma unroll
+        for (int k = 0; k < BCOLS; ++k) {
+          const int n = bn + k * THREADS;
+          (n >= NP ? s_c[buf][r] - NP : s_b[buf][r])[n] = to_f(r_b[i][k]);
+        }
+      }
     }
   };
   fetch(a);
@@ -312,9 +349,9 @@ __global__ void __launch_bounds__(sel::THREADS) selective_prefill_kernel(const S
       float y[4];
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
-        const float d = s_d[buf][t + k][ch], du = s_u[buf][t + k][ch];
-        if constexpr (PART) total += d;
-        const float2 d2 = both(d), du2 = both(du);
+        const float2 du = s_du[buf][t + k][ch];
+        if constexpr (PART) total += du.x;
+        const float2 d2 = both(du.x), u2 = both(du.y);
         float2 y2 = make_float2(0.f, 0.f);
 #pragma unroll
         for (int i = 0; i < NS / 2; i += 2) {
@@ -322,8 +359,8 @@ __global__ void __launch_bounds__(sel::THREADS) selective_prefill_kernel(const S
           float2 e0 = mul2(d2, A2[i]), e1 = mul2(d2, A2[i + 1]);
           e0 = make_float2(fast_exp2(e0.x), fast_exp2(e0.y));
           e1 = make_float2(fast_exp2(e1.x), fast_exp2(e1.y));
-          S2[i] = fma2(e0, S2[i], mul2(du2, make_float2(b4.x, b4.y)));
-          S2[i + 1] = fma2(e1, S2[i + 1], mul2(du2, make_float2(b4.z, b4.w)));
+          S2[i] = fma2(e0, S2[i], mul2(u2, make_float2(b4.x, b4.y)));
+          S2[i + 1] = fma2(e1, S2[i + 1], mul2(u2, make_float2(b4.z, b4.w)));
           if constexpr (!PART) {
             const float4 c4 = *reinterpret_cast<const float4*>(&s_c[buf][t + k][sub * NS + 2 * i]);
             y2 = fma2(S2[i], make_float2(c4.x, c4.y), y2);
@@ -333,22 +370,23 @@ __global__ void __launch_bounds__(sel::THREADS) selective_prefill_kernel(const S
         y[k] = y2.x + y2.y;
       }
       if constexpr (!PART) {
-        // sums over the lanes of a channel: with four of them or more, each of the first four steps halves what is left to add
+        // sums over the lanes of a channel: the first two steps leave a lane one of the four tokens
         if constexpr (LN >= 4) {
           const bool o1 = sub & 1, o2 = sub & 2;
-          float v0 = (o1 ? y[1] : y[0]) + __shfl_xor_sync(0xffffffffu, o1 ? y[0] : y[1], 1);
-          float v1 = (o1 ? y[3] : y[2]) + __shfl_xor_sync(0xffffffffu, o1 ? y[2] : y[3], 1);
+          const float v0 = (o1 ? y[1] : y[0]) + __shfl_xor_sync(0xffffffffu, o1 ? y[0] : y[1], 1);
+          const float v1 = (o1 ? y[3] : y[2]) + __shfl_xor_sync(0xffffffffu, o1 ? y[2] : y[3], 1);
           float v = (o2 ? v1 : v0) + __shfl_xor_sync(0xffffffffu, o2 ? v0 : v1, 2);
 #pragma unroll
           for (int o = 4; o < LN; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
           if (sub < 4) s_y[t + sub][ch] = v;          // lane's token: bit 0 from the first step, bit 1 from the second
+        } else if constexpr (LN == 2) {
+          const float v0 = (sub ? y[1] : y[0]) + __shfl_xor_sync(0xffffffffu, sub ? y[0] : y[1], 1);
+          const float v1 = (sub ? y[3] : y[2]) + __shfl_xor_sync(0xffffffffu, sub ? y[2] : y[3], 1);
+          s_y[t + sub][ch] = v0;
+          s_y[t + 2 + sub][ch] = v1;
         } else {
 #pragma unroll
-          for (int k = 0; k < 4; ++k) {
-#pragma unroll
-            for (int o = 1; o < LN; o <<= 1) y[k] += __shfl_xor_sync(0xffffffffu, y[k], o);
-            if (sub == 0) s_y[t + k][ch] = y[k];
-          }
+          for (int k = 0; k < 4; ++k) s_y[t + k][ch] = y[k];
         }
       }
     }
@@ -356,10 +394,15 @@ __global__ void __launch_bounds__(sel::THREADS) selective_prefill_kernel(const S
       __syncthreads();
 #pragma unroll
       for (int i = 0; i < PER; ++i) {
-        const int r = sr + i * (THREADS / CH);
-        if (r < TOK && t0 + r < b && gc < p.C)
-          p.y[static_cast<size_t>(s0 + t0 + r) * p.C + gc] = from_f<T>((s_y[r][sc] + skip * u_now[i]) * silu_of(z_now[i]));
+        const int r = sr + i * ROWS;
+        if (column && r < TOK && t0 + r < b) {
+          F o;
+#pragma unroll
+          for (int v = 0; v < V; ++v) o.v[v] = from_f<T>(fmaf(skip[v], to_f(u_now[i].v[v]), s_y[r][sc + v]) * silu_of(to_f(z_now[i].v[v])));
+          *reinterpret_cast<F*>(py + i * su) = o;
+        }
       }
+      py += static_cast<long>(TOK) * p.C;
     }
   }
   float* out = nullptr;
@@ -380,43 +423,79 @@ __global__ void __launch_bounds__(sel::THREADS) selective_prefill_kernel(const S
   }
 }
 
-// One token per sequence.  NS states per lane, LN lanes per channel; VEC: states in 16-byte accesses.
-template <typename T, int NS, int LN, bool VEC>
-__global__ void __launch_bounds__(128) selective_step_kernel(const Selective<T> p) {
-  constexpr int CH = 128 / LN;
-  const int row = blockIdx.y, sub = threadIdx.x % LN, c = blockIdx.x * CH + threadIdx.x / LN, slot = p.slot[row];
+// One token of RB sequences.  NS states per lane, LN lanes per channel; VEC: states in 16-byte accesses.  All states of a thread are on their way
+// before the first is worked on; the decays' exponents are formed once for all sequences.
+template <typename T, int NS, int LN, int RB, bool VEC>
+__global__ void __launch_bounds__(128, RB == 4 && NS == 4 ? 7 : 4) selective_step_kernel(const Selective<T> p, int rows) {
+  constexpr int CH = 128 / LN, NV = VEC ? 4 : 1;
+  const int row0 = blockIdx.y * RB, sub = threadIdx.x % LN, c = blockIdx.x * CH + threadIdx.x / LN;
   const bool mine = c < p.C;
-  float y = 0.f, u = 0.f;
-  if (mine) {
-    u = to_f(p.u[static_cast<size_t>(row) * p.C + c]);
-    const float d = softplus_of(to_f(p.dt[static_cast<size_t>(row) * p.ldd + c]) + to_f(p.dt_bias[c])), du = d * u;
-    float* S = p.pool + (static_cast<size_t>(slot) * p.C + c) * p.N;
-    const T *B = p.B + static_cast<size_t>(row) * p.ldb, *Cm = p.Cm + static_cast<size_t>(row) * p.ldb, *A = p.A_log + static_cast<size_t>(c) * p.N;
-    auto advance = [&](float s, int n) {
-      s = fmaf(fast_exp2(-d * 1.4426950408889634f * __expf(to_f(A[n]))), s, du * to_f(B[n]));
-      y = fmaf(s, to_f(Cm[n]), y);
-      return s;
-    };
+  // neighbouring lanes take neighbouring vectors
+  auto place = [&](int i) { return (i / NV * LN + sub) * NV + i % NV; };
+  using Raw = Few<T, NV>;                                // kept as they lie in memory until they are used
+  float s[RB][NS], A[NS];
+  Raw bn[RB][NS / NV], cn[RB][NS / NV];
+  T u[RB], d[RB], z[RB];
+  int slot[RB];
 #pragma unroll
-    for (int i = 0; i < NS; i += VEC ? 4 : 1) {
-      // neighbouring lanes take neighbouring vectors
-      const int n = VEC ? (i / 4 * LN + sub) * 4 : i * LN + sub;
+  for (int r = 0; r < RB; ++r) {
+    const int row = min(row0 + r, rows - 1);
+    slot[r] = p.slot[row];
+    const float* S = p.pool + (static_cast<size_t>(slot[r]) * p.C + (mine ? c : 0)) * p.N;
+    const T *B = p.B + static_cast<size_t>(row) * p.ldb, *Cm = p.Cm + static_cast<size_t>(row) * p.ldb;
+#pragma unroll
+    for (int i = 0; i < NS; i += NV) {
+      const int n = min(place(i), p.N - NV);          // places past the last state repeat it: their A is not used
+      if constexpr (VEC) {
+        const float4 w = *reinterpret_cast<const float4*>(S + n);
+        s[r][i] = w.x; s[r][i + 1] = w.y; s[r][i + 2] = w.z; s[r][i + 3] = w.w;
+      } else {
+        s[r][i] = S[n];
+      }
+      bn[r][i / NV] = *reinterpret_cast<const Raw*>(B + n);
+      cn[r][i / NV] = *reinterpret_cast<const Raw*>(Cm + n);
+    }
+    const int own = mine ? c : 0;
+    z[r] = p.z[static_cast<size_t>(row) * p.ldz + own];
+    u[r] = p.u[static_cast<size_t>(row) * p.C + own];
+    d[r] = p.dt[static_cast<size_t>(row) * p.ldd + own];
+  }
+  const float bias = mine ? to_f(p.dt_bias[c]) : 0.f, skip = mine ? to_f(p.D[c]) : 0.f;
+#pragma unroll
+  for (int i = 0; i < NS; ++i) {
+    const int n = place(i);
+    A[i] = mine && n < p.N ? -1.4426950408889634f * __expf(to_f(p.A_log[static_cast<size_t>(c) * p.N + n])) : 0.f;
+  }
+#pragma unroll
+  for (int r = 0; r < RB; ++r) {
+    const int row = row0 + r;
+    if (row >= rows) break;                            // the same for the whole block
+    const float step = softplus_of(to_f(d[r]) + bias), du = step * to_f(u[r]);
+    float y = 0.f;
+#pragma unroll
+    for (int i = 0; i < NS; ++i) {
+      const int n = place(i);
       if (n < p.N) {
-        if constexpr (VEC) {
-          float4 s = *reinterpret_cast<const float4*>(S + n);
-          s.x = advance(s.x, n); s.y = advance(s.y, n + 1); s.z = advance(s.z, n + 2); s.w = advance(s.w, n + 3);
-          if (slot > 0) *reinterpret_cast<float4*>(S + n) = s;
-        } else {
-          const float s = advance(S[n], n);
-          if (slot > 0) S[n] = s;
+        s[r][i] = fmaf(fast_exp2(step * A[i]), s[r][i], du * to_f(bn[r][i / NV].v[i % NV]));
+        y = fmaf(s[r][i], to_f(cn[r][i / NV].v[i % NV]), y);
+      }
+    }
+    if (mine && slot[r] > 0) {
+      float* S = p.pool + (static_cast<size_t>(slot[r]) * p.C + c) * p.N;
+#pragma unroll
+      for (int i = 0; i < NS; i += NV) {
+        const int n = place(i);
+        if (n < p.N) {
+          if constexpr (VEC) *reinterpret_cast<float4*>(S + n) = make_float4(s[r][i], s[r][i + 1], s[r][i + 2], s[r][i + 3]);
+          else S[n] = s[r][i];
         }
       }
     }
-  }
 #pragma unroll
-  for (int o = 1; o < LN; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-  if (mine && sub == 0)
-    p.y[static_cast<size_t>(row) * p.C + c] = from_f<T>((y + to_f(p.D[c]) * u) * silu_of(to_f(p.z[static_cast<size_t>(row) * p.ldz + c])));
+    for (int o = 1; o < LN; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+    if (mine && sub == 0)
+      p.y[static_cast<size_t>(row) * p.C + c] = from_f<T>(fmaf(skip, to_f(u[r]), y) * silu_of(to_f(z[r])));
+  }
 }
 
 template <typename T>
@@ -478,11 +557,12 @@ torch::Tensor selective_prefill(const torch::Tensor& u, const torch::Tensor& dt,
     auto p = selective_params<T>(u, dt, dt_bias, A_log, proj, b0, c0, D, gate, z0, y);
     p.cu = cu.data_ptr<int>();
     if (has(pool)) { p.pool = pool->data_ptr<float>(); p.slot = slot->data_ptr<int>(); }
-    selective_lanes(N, [&](auto ns, auto ln) {
-      constexpr int NS = decltype(ns)::value, LN = decltype(ln)::value, CH = sel::THREADS / LN, TOK = sel::tokens(NS * LN);
-      const int64_t across = (C + CH - 1) / CH, blocks = across * n, fill = num_sms() * 3L / 2;
+    auto pair = [](const T* q, int64_t ld) { return reinterpret_cast<uintptr_t>(q) % (2 * sizeof(T)) == 0 && ld % 2 == 0; };
+    auto go = [&](auto ns, auto ln, auto v) {
+      constexpr int NS = decltype(ns)::value, LN = decltype(ln)::value, V = decltype(v)::value, CH = sel::THREADS / LN, TOK = sel::tokens(NS * LN);
+      const int64_t across = (C + CH - 1) / CH, blocks = across * n, fill = num_sms() * 6L;
       // segments of at least 64 tokens, as many as fill the device (the work of all but the last is done twice)
-      int64_t segments = blocks >= fill ? 1 : std::min<int64_t>({num_sms() * 8L / blocks, (max_seqlen + 63) / 64, 32});
+      int64_t segments = blocks * 2 > fill ? 1 : std::min<int64_t>({fill / blocks, (max_seqlen + 63) / 64, 32});
       const int64_t seg_len = ((max_seqlen + segments - 1) / segments + TOK - 1) / TOK * TOK;
       segments = (max_seqlen + seg_len - 1) / seg_len;
       p.segments = static_cast<int>(segments);
@@ -493,12 +573,16 @@ torch::Tensor selective_prefill(const torch::Tensor& u, const torch::Tensor& dt,
         steps = torch::empty({n * (segments - 1) * C}, part.options());
         p.part = part.data_ptr<float>();
         p.steps = steps.data_ptr<float>();
-        selective_prefill_kernel<T, NS, LN, true><<<dim3(across, segments - 1, n), sel::THREADS, 0, stream>>>(p);
+        selective_prefill_kernel<T, NS, LN, V, true><<<dim3(across, segments - 1, n), sel::THREADS, 0, stream>>>(p);
         count_launch();
       }
-      selective_prefill_kernel<T, NS, LN, false><<<dim3(across, segments, n), sel::THREADS, 0, stream>>>(p);
+      selective_prefill_kernel<T, NS, LN, V, false><<<dim3(across, segments, n), sel::THREADS, 0, stream>>>(p);
       count_launch();
-    });
+    };
+    using std::integral_constant;
+    // odd numbers of channels: one instance for any number of states
+    if (pair(p.u, C) && pair(p.dt, p.ldd) && pair(p.z, p.ldz)) selective_lanes(N, [&](auto ns, auto ln) { go(ns, ln, integral_constant<int, 2>{}); });
+    else go(integral_constant<int, 8>{}, integral_constant<int, 32>{}, integral_constant<int, 1>{});
   };
   if (u.scalar_type() == torch::kBFloat16) run(bf16{}); else run(float{});
   TK_CUDA_CHECK(cudaGetLastError());
@@ -521,9 +605,14 @@ torch::Tensor selective_step(const torch::Tensor& u, const torch::Tensor& dt, co
     p.pool = pool.data_ptr<float>(); p.slot = slot.data_ptr<int>();
     selective_lanes(N, [&](auto ns, auto ln) {
       constexpr int NS = decltype(ns)::value, LN = decltype(ln)::value, CH = 128 / LN;
-      const dim3 grid(static_cast<unsigned>((C + CH - 1) / CH), static_cast<unsigned>(rows));
-      if (N % 4 == 0) selective_step_kernel<T, NS, LN, true><<<grid, 128, 0, stream>>>(p);
-      else selective_step_kernel<T, NS, LN, false><<<grid, 128, 0, stream>>>(p);
+      const int64_t across = (C + CH - 1) / CH;
+      auto go = [&](auto kern, int rb) { kern<<<dim3(static_cast<unsigned>(across), static_cast<unsigned>((rows + rb - 1) / rb)), 128, 0, stream>>>(p, static_cast<int>(rows)); };
+      // four sequences per block once that leaves blocks enough
+      const bool vec = N % 4 == 0 && p.ldb % 4 == 0 && reinterpret_cast<uintptr_t>(p.B) % (4 * sizeof(T)) == 0 && reinterpret_cast<uintptr_t>(p.Cm) % (4 * sizeof(T)) == 0;
+      const bool four = across * rows >= 4L * 8 * num_sms();
+      if (!vec) go(selective_step_kernel<T, NS, LN, 1, false>, 1);
+      else if (four) go(selective_step_kernel<T, NS, LN, 4, true>, 4);
+      else go(selective_step_kernel<T, NS, LN, 1, true>, 1);
     });
   };
   if (u.scalar_type() == torch::kBFloat16) run(bf16{}); else run(float{});

@@ -543,21 +543,25 @@ torch::Tensor stream_normed(torch::Tensor x, const OptT& w, double eps, const to
 }
 
 // ------------------------------------------------------------- embed_positions
-// A thread forms one pair.  The angle is reduced to half turns in fp64, so that far positions keep their digits.
+// One block per row, a pair per thread at a time.  The angle is reduced to half turns in fp64, so that far positions keep their digits.
 template <typename T>
 __global__ void __launch_bounds__(256) embed_positions_kernel(const int64_t* __restrict__ ids, const T* __restrict__ weight, const int64_t* __restrict__ pos,
-                                                              const double* __restrict__ freq, float* __restrict__ out, long total, int pairs, int W) {
-  const long i = blockIdx.x * 256L + threadIdx.x;
-  if (i >= total) return;
-  const long t = i / pairs;
-  const int k = static_cast<int>(i - t * pairs);
-  const double half_turns = static_cast<double>(pos[t]) * (freq[k] * 0.31830988618379067154);
-  float s, c;
-  sincospif(static_cast<float>(half_turns - 2.0 * rint(0.5 * half_turns)), &s, &c);
-  const T* w = weight + static_cast<size_t>(ids[t]) * W + 2 * k;
-  float* o = out + static_cast<size_t>(t) * W + 2 * k;
-  o[0] = to_f(w[0]) + s;
-  if (2 * k + 1 < W) o[1] = to_f(w[1]) + c;
+                                                              const double* __restrict__ freq, float* __restrict__ out, int pairs, int W) {
+  const int t = blockIdx.x;
+  const double at = static_cast<double>(pos[t]) * 0.31830988618379067154;
+  const T* w = weight + static_cast<size_t>(ids[t]) * W;
+  float* o = out + static_cast<size_t>(t) * W;
+  for (int k = threadIdx.x; k < pairs; k += 256) {
+    const double half_turns = at * freq[k];
+    float s, c;
+    sincospif(static_cast<float>(half_turns - 2.0 * rint(0.5 * half_turns)), &s, &c);
+    if (W % 2 == 0) {
+      *reinterpret_cast<float2*>(o + 2 * k) = make_float2(to_f(w[2 * k]) + s, to_f(w[2 * k + 1]) + c);
+    } else {
+      o[2 * k] = to_f(w[2 * k]) + s;
+      if (2 * k + 1 < W) o[2 * k + 1] = to_f(w[2 * k + 1]) + c;
+    }
+  }
 }
 
 torch::Tensor embed_positions(const torch::Tensor& ids, const torch::Tensor& weight, const torch::Tensor& pos, const torch::Tensor& freq) {
@@ -569,12 +573,11 @@ torch::Tensor embed_positions(const torch::Tensor& ids, const torch::Tensor& wei
   TORCH_CHECK(freq.is_cuda() && freq.scalar_type() == torch::kFloat64 && freq.is_contiguous() && freq.numel() == pairs, "frequencies fp64 [pairs]");
   c10::cuda::CUDAGuard guard(weight.device());
   auto out = torch::empty({ids.numel(), W}, weight.options().dtype(torch::kFloat32));
-  const long total = ids.numel() * pairs;
-  if (total == 0) return out;
+  if (out.numel() == 0) return out;
   auto run = [&](auto tag) {
     using T = decltype(tag);
-    embed_positions_kernel<T><<<static_cast<unsigned>((total + 255) / 256), 256, 0, at::cuda::getCurrentCUDAStream()>>>(
-        ids.data_ptr<int64_t>(), reinterpret_cast<const T*>(weight.data_ptr()), pos.data_ptr<int64_t>(), freq.data_ptr<double>(), out.data_ptr<float>(), total, pairs, W);
+    embed_positions_kernel<T><<<static_cast<unsigned>(ids.numel()), 256, 0, at::cuda::getCurrentCUDAStream()>>>(
+        ids.data_ptr<int64_t>(), reinterpret_cast<const T*>(weight.data_ptr()), pos.data_ptr<int64_t>(), freq.data_ptr<double>(), out.data_ptr<float>(), pairs, W);
   };
   if (st == torch::kBFloat16) run(bf16{}); else run(float{});
   count_launch();

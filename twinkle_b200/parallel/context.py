@@ -123,7 +123,7 @@ def apply_context_parallel(model, mesh) -> Optional[ContextParallelAttention]:
     if group is None:
         return None
     if getattr(getattr(model, 'cfg', None), 'layer_specs', None) is not None:
-        raise NotImplementedError('stacks with listed layers (Pomelix, Moronex, Nilepel) have no context-parallel split here; shard the data instead')
+        raise NotImplementedError('stacks with listed layers (Pomelix, Moronex, Nilepel, Puzonex) have no context-parallel split here; shard the data instead')
     dev = next(model.parameters()).device
     strat = ContextParallelAttention(Communicator(group, dev))
     for layer in model.layers:

@@ -281,7 +281,7 @@ def apply_tensor_parallel(model, cfg, comm: Communicator, sequence_parallel: boo
         raise NotImplementedError('multi-head latent attention has no tensor-parallel split here; use tp_size=1 '
                                   '(data, sharded-data, expert and pipeline parallelism apply)')
     if getattr(cfg, 'layer_specs', None) is not None:
-        raise NotImplementedError('stacks with listed layers (Pomelix, Moronex, Nilepel) have no tensor-parallel split here; use tp_size=1')
+        raise NotImplementedError('stacks with listed layers (Pomelix, Moronex, Nilepel, Puzonex) have no tensor-parallel split here; use tp_size=1')
     tp = TPContext(comm, sequence_parallel)
     tp.fused = fused
     assert cfg.num_key_value_heads % tp.size == 0 and cfg.num_attention_heads % tp.size == 0, 'heads must divide over tp'

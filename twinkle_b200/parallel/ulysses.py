@@ -326,7 +326,7 @@ def apply_ulysses(model, mesh, cfg, backend: str = 'auto') -> None:
     if comm.world_size <= 1:
         return
     if getattr(cfg, 'layer_specs', None) is not None:
-        raise NotImplementedError('stacks with listed layers (Pomelix, Moronex, Nilepel) have no sequence-parallel split here; shard the data instead')
+        raise NotImplementedError('stacks with listed layers (Pomelix, Moronex, Nilepel, Puzonex) have no sequence-parallel split here; shard the data instead')
     if backend in ('auto', 'symm') and dev.type == 'cuda':
         try:
             from .symm import SymmCommunicator
