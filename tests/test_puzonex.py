@@ -88,7 +88,7 @@ def _prompt_rows(lens, slots):
 
 # ------------------------------------------------------------------------------------------------ mechanisms
 @BACKENDS
-@pytest.mark.parametrize('width', [1, 7, 52, 320, 1024])
+@pytest.mark.parametrize('width', [1, 7, 52, 328, 1024])
 def test_embedding_with_waves_of_near_and_far_positions(where, width):
     from twinkle_b200 import ops
     pos = torch.tensor([0, 1, 2, 17, 1000, 65537, 3_000_001])
